@@ -620,3 +620,115 @@ class DepolixConfig:
                 "logit_scale": self.logit_scale,
                 "layers": [{"type": l.type, "mixer": dict(l.mixer), "mlp": None if l.mlp is None else dict(l.mlp)}
                            for l in self.layers]}
+
+
+# ---------------------------------------------------------------------------------------------------------------
+_LARUZEN_MIXERS = ("gla", "lightning", "parallel")
+
+
+@dataclass(frozen=True)
+class LaruzenLayer:
+    type: str                   # "gla" | "lightning" | "parallel"
+    mixer: dict                 # the mixer's sizes and constants, as config.json gives them
+    mlp: Optional[dict]         # None, {"kind": "dense", "ff"} or {"kind": "moe", "expert": {"ff"}, "router": {...}, "shared": {"ff"}}
+
+
+@dataclass(frozen=True)
+class LaruzenConfig:
+    """Laruzen: a decoder whose layers are listed one by one in config.json, each with an RMS norm (gain stored around zero)
+    before and after both of its sublayers around one float residual stream, and a token shift in front of its mixer.  The
+    embedding adds a row for the pair (token before, token), hashed into `embedding.bigram.buckets`.  The mixer is `gla` (gated
+    linear attention: a decay per head and key channel), `lightning` (linear attention with one fixed `decay` a head) or
+    `parallel`: `left`, windowed attention with biases, normed heads, a partial rotation with stretched frequencies, normed
+    values, a learned sink and an output gate, beside `right`, a gated linear recurrence of `width` channels in `blocks` parts
+    behind a short convolution; each side is normed over the width and the result is half their sum.  The feed-forward is a gated
+    layer (tanh-form gelu), a mixture of gated SiLU experts weighted by the softmax over the chosen logits beside a shared one, or
+    absent.  Keys: `vocab`, `width`, `norm.eps`, `embedding.bigram` {buckets, mul_prev, mul_cur}, `layers[i]` = {type, mixer{...},
+    mlp}.  There is no largest position."""
+    vocab: int
+    width: int
+    eps: float
+    layers: tuple
+    bigram: Optional[tuple] = None      # (buckets, mul_prev, mul_cur)
+    torch_dtype: str = "bfloat16"
+
+    architecture = "Laruzen"
+
+    @staticmethod
+    def _check_left(m: dict, w: str) -> None:
+        for k in ("heads", "kv_heads", "dim", "vdim"):
+            _need(m, k, int, w)
+        if m["heads"] % m["kv_heads"]:
+            raise ConfigError(f"{w}: heads {m['heads']} is not a multiple of kv_heads {m['kv_heads']}")
+        _need(m, "scale", float, w)
+        if m.get("mask") is not None:
+            _count(_sub(m, "mask", w), "size", w + ".mask")
+        if m.get("rot") is not None:
+            rot = _sub(m, "rot", w)
+            dims = rot.get("dims")
+            if isinstance(dims, bool) or not isinstance(dims, int) or dims < 0 or dims % 2 or dims > m["dim"]:
+                raise ConfigError(f"{w}: rot.dims {dims!r} must be even and between 0 and dim {m['dim']}")
+            if dims:
+                _need(rot, "base", float, w + ".rot")
+            if rot.get("scaling") is not None:
+                s = _sub(rot, "scaling", w + ".rot")
+                for k in ("factor", "original", "fast", "slow"):
+                    if _need(s, k, float, w + ".rot.scaling") <= 0:
+                        raise ConfigError(f"{w}: rot.scaling.{k} must be positive")
+
+    @classmethod
+    def from_dict(cls, d: dict, where: str = "config.json") -> "LaruzenConfig":
+        layers = d.get("layers")
+        if not isinstance(layers, list) or not layers:
+            raise ConfigError(f"{where}: 'layers' must be a non-empty list")
+        out = []
+        for i, layer in enumerate(layers):
+            w = f"{where}: layers[{i}]"
+            if not isinstance(layer, dict):
+                raise ConfigError(f"{w} must be an object")
+            kind = layer.get("type")
+            if kind not in _LARUZEN_MIXERS:
+                raise ConfigError(f"{w}: type {kind!r} is not one of {list(_LARUZEN_MIXERS)}")
+            m = _sub(layer, "mixer", w)
+            if kind == "parallel":
+                cls._check_left(_sub(m, "left", w), w + ".left")
+                right = _sub(m, "right", w)
+                for k in ("width", "blocks", "conv"):
+                    _need(right, k, int, w + ".right")
+                if right["width"] % right["blocks"]:
+                    raise ConfigError(f"{w}: right.width {right['width']} does not fall into {right['blocks']} equal blocks")
+            else:
+                for k in ("heads", "dim", "vdim"):
+                    _need(m, k, int, w)
+                if kind == "gla":
+                    if _need(m, "tau", float, w) <= 0:
+                        raise ConfigError(f"{w}: tau must be positive")
+                else:
+                    decay = m.get("decay")
+                    if (not isinstance(decay, list) or len(decay) != m["heads"]
+                            or any(isinstance(x, bool) or not isinstance(x, (int, float)) for x in decay)):
+                        raise ConfigError(f"{w}: decay must be a list of {m['heads']} numbers, one a head")
+            mlp = layer.get("mlp")
+            if mlp is not None:
+                _check_moe(mlp, w)
+                if mlp["kind"] == "moe" and mlp.get("shared") is not None:
+                    _need(_sub(mlp, "shared", w + ".mlp"), "ff", int, w + ".mlp.shared")
+            out.append(LaruzenLayer(kind, dict(m), None if mlp is None else dict(mlp)))
+        bigram = None
+        if isinstance(d.get("embedding"), dict) and d["embedding"].get("bigram") is not None:
+            b, w = _sub(d["embedding"], "bigram", where + ".embedding"), where + ".embedding.bigram"
+            bigram = (_need(b, "buckets", int, w), _count(b, "mul_prev", w), _count(b, "mul_cur", w))
+        dtype = d.get("torch_dtype", d.get("dtype", "bfloat16"))
+        if not isinstance(dtype, str) or dtype not in _DTYPE_NAMES:
+            raise ConfigError(f"{where}: torch_dtype {dtype!r} is not one of {sorted(set(_DTYPE_NAMES))}")
+        return cls(vocab=_need(d, "vocab", int, where), width=_need(d, "width", int, where),
+                   eps=_need(_sub(d, "norm", where), "eps", float, where + ".norm"), layers=tuple(out), bigram=bigram,
+                   torch_dtype=_DTYPE_NAMES[dtype])
+
+    def to_dict(self) -> dict:
+        d = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.eps},
+             "layers": [{"type": l.type, "mixer": dict(l.mixer), "mlp": None if l.mlp is None else dict(l.mlp)}
+                        for l in self.layers]}
+        if self.bigram is not None:
+            d["embedding"] = {"bigram": {"buckets": self.bigram[0], "mul_prev": self.bigram[1], "mul_cur": self.bigram[2]}}
+        return d

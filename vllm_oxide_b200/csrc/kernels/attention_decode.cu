@@ -152,7 +152,7 @@ attention_decode_kernel(const __nv_bfloat16* q, long q_stride, __nv_bfloat16* ou
     const float val = L > 0.f ? O / L : 0.f;
     const int head = kh * G + r;
     if (num_splits == 1) {
-      const float Ls = L + sink_weight(ep, M);
+      const float Ls = L + sink_weight(ep, M, head);
       store_out(out, (size_t)t * nh * HD + (size_t)head * HD + d, Ls > 0.f ? O / Ls * head_gate(ep, t, head) : 0.f, ep);
     } else {
       const size_t p = ((size_t)b * nh + head) * num_splits + split;
@@ -377,7 +377,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
     const float lse = (L > 0.f && !aborted) ? M + log2f(L) : -INFINITY;
     const int head = kh * G + r;
     if (num_splits == 1) {
-      const float Ls = L + sink_weight(ep, M);
+      const float Ls = L + sink_weight(ep, M, head);
       store_out(out, (size_t)t * nh * HD + (size_t)head * HD + d, Ls > 0.f ? O / Ls * head_gate(ep, t, head) : 0.f, ep);
     } else if (cluster) {
       fo[idx] = val;
@@ -424,7 +424,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
         W += w;
         O += w * v[sp];
       }
-      W += sink_weight(ep, M);                // the sink counts once, whatever the number of splits
+      W += sink_weight(ep, M, kh * G + r);    // the sink counts once, whatever the number of splits
       store_out(out, (size_t)t * nh * HD + (size_t)(kh * G) * HD + idx, W > 0.f ? O / W * head_gate(ep, t, kh * G + r) : 0.f, ep);
     }
   }
@@ -679,7 +679,7 @@ attention_decode_tma_items_kernel(const __grid_constant__ CUtensorMap tmK, const
             L += wl[w * 16 + r] * f;
             O += wo[((size_t)w * G + r) * HD + d] * f;
           }
-          L += sink_weight(ep, M);
+          L += sink_weight(ep, M, kh * G + r);
           store_out(out, (size_t)t * nh * HD + (size_t)(kh * G + r) * HD + d, L > 0.f ? O / L * head_gate(ep, t, kh * G + r) : 0.f, ep);
         }
       }
@@ -720,7 +720,7 @@ __global__ void attention_decode_combine_kernel(const float* part_o, const float
       W += w;
       O += w * part_o[(base + s) * HD + d];
     }
-    W += sink_weight(ep, M);
+    W += sink_weight(ep, M, head);
     store_out(out, (size_t)t * nh * HD + (size_t)head * HD + d, W > 0.f ? O / W * head_gate(ep, t, head) : 0.f, ep);
   }
 }
@@ -748,7 +748,7 @@ static int attention_decode_launch(const void* map_k, const void* map_v, const v
                                    const int* cu_q, const int* context_lens, int num_requests, int nh, int kvh,
                                    int block_size, int window, float scale, long num_pages, int num_splits, float* scratch,
                                    unsigned* pairs_counter, int* err, cudaStream_t stream,
-                                   HeadEpilogue ep = head_options(0, nullptr, 0, 0.f, 1.f, 0, 1)) {
+                                   HeadEpilogue ep = head_options(0, nullptr, nullptr, 0, 0.f, 1.f, 0, 1)) {
   if (num_requests <= 0) return 0;
   if (kvh <= 0 || nh % kvh || nh / kvh > 16 || block_size <= 0 || num_splits < 1 || num_splits > 65535) return VOB_UNSUPPORTED;
   static bool configured = false;
@@ -852,7 +852,8 @@ VOB_API int vob_attention_decode_tma(const void* map_k, const void* map_v, const
                                  scratch, pairs_counter, err, stream);
 }
 
-// Both of the above (null maps: cp.async) with what may follow the softmax: `sink` (a silent extra entry of score 0) and
+// Both of the above (null maps: cp.async) with what may follow the softmax: `sink` (a silent extra entry of score 0; `sinks`, float
+// [nh] or null: of the head's own score) and
 // `gate` (bfloat16; head h of token t is multiplied by sigmoid(gate[t * gate_stride + h]); null: none); and with other
 // rules for the scores: `softcap` > 0 (a score becomes softcap * tanh(score / softcap)), `chunk` > 0 (a query sees the
 // keys of its own block of `chunk` positions; `window` is then not looked at), `value_div` > 1 (the value plane has
@@ -863,7 +864,7 @@ VOB_API int vob_attention_decode_ex(const void* map_k, const void* map_v, const 
                                     const void* kcache, const void* vcache, const int* block_tables, int table_stride,
                                     const int* cu_q, const int* context_lens, int num_requests, int nh, int kvh,
                                     int block_size, int window, float scale, long num_pages, int num_splits,
-                                    float* scratch, unsigned* pairs_counter, int sink, const void* gate, long gate_stride,
+                                    float* scratch, unsigned* pairs_counter, int sink, const float* sinks, const void* gate, long gate_stride,
                                     float softcap, int chunk, int value_div, int out_float, int keep_first,
                                     const float* dist_bias, int dist_rows, int* err, cudaStream_t stream) {
   if (value_div > 1 && kvh % value_div) return VOB_BAD_ARGUMENT;
@@ -871,7 +872,7 @@ VOB_API int vob_attention_decode_ex(const void* map_k, const void* map_v, const 
   return attention_decode_launch(map_k, map_v, q, q_stride, out, kcache, vcache, block_tables, table_stride, cu_q,
                                  context_lens, num_requests, nh, kvh, block_size, window, scale, num_pages, num_splits,
                                  scratch, pairs_counter, err, stream,
-                                 head_options(sink, gate, gate_stride, softcap, scale, chunk, value_div, out_float, keep_first,
+                                 head_options(sink, sinks, gate, gate_stride, softcap, scale, chunk, value_div, out_float, keep_first,
                                               dist_bias, dist_rows));
 }
 

@@ -75,7 +75,7 @@ paged_attention_generic_kernel(const T* q, long q_stride, T* out,
                                const int* __restrict__ block_tables, int table_stride,
                                const int* __restrict__ token_req, const int* __restrict__ positions,
                                const int* __restrict__ skip_single_cu_q, int nh, int kvh, int hd, int vd, int block_size,
-                               int window, float scale, long num_pages, int sink, const T* gate, long gate_stride,
+                               int window, float scale, long num_pages, int sink, const float* __restrict__ sinks, const T* gate, long gate_stride,
                                int vkvh, int v_row, float softcap, int chunk, int out_float, int keep_first,
                                const float* __restrict__ dist_bias, int dist_rows, int* err) {
   extern __shared__ float smem[];
@@ -153,9 +153,11 @@ paged_attention_generic_kernel(const T* q, long q_stride, T* out,
   float mm = -INFINITY;
 #pragma unroll
   for (int w = 0; w < ATT_WARPS; ++w) mm = fmaxf(mm, ms[w]);
-  // a sink is one more entry of score 0 that has no value: it adds exp(0 - max) to the denominator and nothing else
-  if (sink) mm = fmaxf(mm, 0.f);
-  float f[ATT_WARPS], lt = sink ? expf(-mm) : 0.f;
+  // a sink is one more entry, of score 0 or of the head's own score, that has no value: it adds exp(score - max) to the
+  // denominator and nothing else
+  const float sink_score = sinks ? sinks[h] : 0.f;
+  if (sink || sinks) mm = fmaxf(mm, sink_score);
+  float f[ATT_WARPS], lt = (sink || sinks) ? expf(sink_score - mm) : 0.f;
 #pragma unroll
   for (int w = 0; w < ATT_WARPS; ++w) {
     f[w] = (ms[w] == -INFINITY) ? 0.f : expf(ms[w] - mm);
@@ -181,7 +183,7 @@ using namespace vob;
 // q: rows of q_stride elements, head h at h*hd; out [T, nh*vd]; caches [num_pages, kvh, block_size, hd];
 // block_tables [B, table_stride]; token_req [T] (-1: padding); positions [T].  Of a value row the first vd elements are
 // read (vd = hd: all of it; less when keys and values are one row and the key is the longer one).  `sink`: the softmax
-// has a silent extra entry of score 0 (weights exp(s) / (1 + sum exp(s))); `gate` (rows of gate_stride elements, one
+// has a silent extra entry of score 0, or (`sinks`, float [nh] or null) of the head's own score (weights exp(s) / (1 + sum exp(s))); `gate` (rows of gate_stride elements, one
 // number a head): head h of token t is multiplied by sigmoid(gate[t, h]).
 // vkvh, v_row: heads and head size of the value plane [num_pages, vkvh, block_size, v_row] (0: those of the key plane);
 // softcap, chunk, keep_first, dist_bias: see above (0 / null: off); out_float: out is float whatever `dtype`.
@@ -189,7 +191,7 @@ VOB_API int vob_paged_attention_generic(const void* q, long q_stride, void* out,
                                         const int* block_tables, int table_stride, const int* token_req,
                                         const int* positions, const int* skip_single_cu_q, int T, int nh, int kvh, int hd,
                                         int vd, int block_size,
-                                        int window, float scale, long num_pages, int sink, const void* gate,
+                                        int window, float scale, long num_pages, int sink, const float* sinks, const void* gate,
                                         long gate_stride, int vkvh, int v_row, float softcap, int chunk, int out_float,
                                         int keep_first, const float* dist_bias, int dist_rows,
                                         int dtype, int* err, cudaStream_t stream) {
@@ -204,13 +206,13 @@ VOB_API int vob_paged_attention_generic(const void* q, long q_stride, void* out,
   if (dtype == VOB_F32)
     return launch_kernel(paged_attention_generic_kernel<float>, grid, ATT_WARPS * 32, smem, stream, (const float*)q, q_stride,
                          (float*)out, (const float*)kcache, (const float*)vcache, block_tables, table_stride, token_req,
-                         positions, skip_single_cu_q, nh, kvh, hd, vd, block_size, window, scale, num_pages, sink,
+                         positions, skip_single_cu_q, nh, kvh, hd, vd, block_size, window, scale, num_pages, sink, sinks,
                          (const float*)gate, gate_stride, vkvh, v_row, softcap, chunk, out_float, keep_first, dist_bias, dist_rows, err);
   if (dtype == VOB_BF16)
     return launch_kernel(paged_attention_generic_kernel<__nv_bfloat16>, grid, ATT_WARPS * 32, smem, stream,
                          (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)kcache,
                          (const __nv_bfloat16*)vcache, block_tables, table_stride, token_req, positions, skip_single_cu_q,
-                         nh, kvh, hd, vd, block_size, window, scale, num_pages, sink, (const __nv_bfloat16*)gate,
+                         nh, kvh, hd, vd, block_size, window, scale, num_pages, sink, sinks, (const __nv_bfloat16*)gate,
                          gate_stride, vkvh, v_row, softcap, chunk, out_float, keep_first, dist_bias, dist_rows, err);
   return VOB_BAD_ARGUMENT;
 }

@@ -62,7 +62,8 @@ __device__ __forceinline__ float fast_rcp(float x) {
 
 // What a head's softmax does besides scaling and the causal mask, and what may come after it.  `sink`: the softmax has a
 // silent extra entry of score 0 that has no value; it adds 2^(0 - M) to a denominator that is taken relative to M (scores in
-// the base-2 domain).  `gate`: head h of token t is multiplied by sigmoid(gate[t * gate_stride + h]).  `cap_out` > 0: a
+// the base-2 domain).  `sinks` (float [heads]): the extra entry's score is a number of the head's own instead, as it is (the
+// scale does not touch it).  `gate`: head h of token t is multiplied by sigmoid(gate[t * gate_stride + h]).  `cap_out` > 0: a
 // score becomes cap * tanh(score / cap); the two factors are cap_in = scale / cap * 2 log2(e) (on the raw product) and
 // cap_out = cap * log2(e) (see head_options).  `chunk` > 0: a query sees only the keys of its own block of `chunk`
 // positions, counted from position 0.  `value_div` > 1: the value plane has kv_heads / value_div heads, and key head k
@@ -70,6 +71,7 @@ __device__ __forceinline__ float fast_rcp(float x) {
 // (same shape), for heads that are combined before anything rounds them.  All zero leaves the softmax as it is.
 struct HeadEpilogue {
   int sink;
+  const float* sinks;
   const __nv_bfloat16* gate;
   long gate_stride;
   float cap_in, cap_out;
@@ -81,10 +83,10 @@ struct HeadEpilogue {
   int dist_rows;              // the head's row is added to the scaled score (a learned bias by distance; neighbouring keys
                               // read neighbouring floats)
 };
-__host__ inline HeadEpilogue head_options(int sink, const void* gate, long gate_stride, float softcap, float scale, int chunk,
+__host__ inline HeadEpilogue head_options(int sink, const float* sinks, const void* gate, long gate_stride, float softcap, float scale, int chunk,
                                           int value_div, int out_float = 0, int keep_first = 0, const float* dist_bias = nullptr,
                                           int dist_rows = 0) {
-  HeadEpilogue ep{sink, (const __nv_bfloat16*)gate, gate_stride, 0.f, 0.f, chunk > 0 ? chunk : 0, value_div > 1 ? value_div : 1,
+  HeadEpilogue ep{sink, sinks, (const __nv_bfloat16*)gate, gate_stride, 0.f, 0.f, chunk > 0 ? chunk : 0, value_div > 1 ? value_div : 1,
                   out_float, keep_first > 0 ? keep_first : 0, dist_rows > 0 ? dist_bias : nullptr, dist_rows};
   if (softcap > 0.f) {
     ep.cap_in = scale / softcap * 2.f * 1.4426950408889634f;
@@ -144,7 +146,10 @@ __device__ __forceinline__ void store_out(__nv_bfloat16* out, size_t i, float v,
 __device__ __forceinline__ int value_heads(int kvh, const HeadEpilogue& ep) { return ep.value_div > 1 ? kvh / ep.value_div : kvh; }
 __device__ __forceinline__ int value_head(int kh, const HeadEpilogue& ep) { return ep.value_div > 1 ? kh / ep.value_div : kh; }
 // The sink's share of a denominator relative to M.  A maximum far below zero gives +inf, and the head's output 0: the limit.
-__device__ __forceinline__ float sink_weight(const HeadEpilogue& ep, float M) { return ep.sink ? exp2f(-M) : 0.f; }
+__device__ __forceinline__ float sink_weight(const HeadEpilogue& ep, float M, int head) {
+  if (ep.sinks) return exp2f(fmaf(ep.sinks[head], LOG2E, -M));
+  return ep.sink ? exp2f(-M) : 0.f;
+}
 __device__ __forceinline__ float head_gate(const HeadEpilogue& ep, int t, int head) {
   if (!ep.gate) return 1.f;
   const float g = __bfloat162float(ep.gate[(size_t)t * ep.gate_stride + head]);

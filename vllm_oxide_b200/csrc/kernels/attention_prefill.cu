@@ -145,7 +145,7 @@ attention_prefill_kernel(const __nv_bfloat16* q, long q_stride, __nv_bfloat16* o
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     if (!rvalid[h]) continue;
-    const float lsum = st.l[h] + sink_weight(ep, st.m[h]);
+    const float lsum = st.l[h] + sink_weight(ep, st.m[h], rhead[h]);
     const float inv = lsum > 0.f ? head_gate(ep, t0 + rtok[h], rhead[h]) / lsum : 0.f;
     __nv_bfloat16* orow = out + (size_t)(t0 + rtok[h]) * nh * HD + (size_t)rhead[h] * HD + tq * 2;
     if (ep.out_float) {
@@ -435,7 +435,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gr
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     if (!rvalid[h]) continue;
-    const float lsum = l[h] + sink_weight(ep, m[h]);
+    const float lsum = l[h] + sink_weight(ep, m[h], rhead[h]);
     const float inv = lsum > 0.f ? head_gate(ep, t0 + rtok[h], rhead[h]) / lsum : 0.f;
     __nv_bfloat16* orow = out + (size_t)(t0 + rtok[h]) * nh * HD + (size_t)rhead[h] * HD + tq * 2;
     if (ep.out_float) {
@@ -459,7 +459,7 @@ static int attention_prefill_launch(const void* map_k, const void* map_v, const 
                                     const void* kcache, const void* vcache, const int* block_tables, int table_stride,
                                     const int* cu_q, const int* context_lens, int num_requests, int max_q, int nh, int kvh,
                                     int block_size, int window, float scale, long num_pages, int* err, cudaStream_t stream,
-                                    HeadEpilogue ep = head_options(0, nullptr, 0, 0.f, 1.f, 0, 1)) {
+                                    HeadEpilogue ep = head_options(0, nullptr, nullptr, 0, 0.f, 1.f, 0, 1)) {
   if (num_requests <= 0 || max_q <= 1) return 0;
   if (kvh <= 0 || nh % kvh || block_size <= 0 || kvh > 65535 || num_requests > 65535) return VOB_UNSUPPORTED;
   const long rows = (long)max_q * (nh / kvh);
@@ -512,7 +512,8 @@ VOB_API int vob_attention_prefill_tma(const void* map_k, const void* map_v, cons
                                   context_lens, num_requests, max_q, nh, kvh, block_size, window, scale, num_pages, err, stream);
 }
 
-// Both of the above (null maps: cp.async) with what may follow the softmax: `sink` (a silent extra entry of score 0) and
+// Both of the above (null maps: cp.async) with what may follow the softmax: `sink` (a silent extra entry of score 0; `sinks`, float
+// [nh] or null: of the head's own score) and
 // `gate` (bfloat16; head h of token t is multiplied by sigmoid(gate[t * gate_stride + h]); null: none); and with other
 // rules for the scores: `softcap` > 0 (a score becomes softcap * tanh(score / softcap)), `chunk` > 0 (a query sees the
 // keys of its own block of `chunk` positions; `window` is then not looked at), `value_div` > 1 (the value plane has
@@ -522,13 +523,13 @@ VOB_API int vob_attention_prefill_tma(const void* map_k, const void* map_v, cons
 VOB_API int vob_attention_prefill_ex(const void* map_k, const void* map_v, const void* q, long q_stride, void* out,
                                      const void* kcache, const void* vcache, const int* block_tables, int table_stride,
                                      const int* cu_q, const int* context_lens, int num_requests, int max_q, int nh,
-                                     int kvh, int block_size, int window, float scale, long num_pages, int sink,
+                                     int kvh, int block_size, int window, float scale, long num_pages, int sink, const float* sinks,
                                      const void* gate, long gate_stride, float softcap, int chunk, int value_div, int out_float,
                                      int keep_first, const float* dist_bias, int dist_rows, int* err, cudaStream_t stream) {
   if (value_div > 1 && kvh % value_div) return VOB_BAD_ARGUMENT;
   if (keep_first < 0 || (dist_bias && dist_rows <= 0)) return VOB_BAD_ARGUMENT;
   return attention_prefill_launch(map_k, map_v, q, q_stride, out, kcache, vcache, block_tables, table_stride, cu_q,
                                   context_lens, num_requests, max_q, nh, kvh, block_size, window, scale, num_pages, err, stream,
-                                  head_options(sink, gate, gate_stride, softcap, scale, chunk, value_div, out_float, keep_first,
+                                  head_options(sink, sinks, gate, gate_stride, softcap, scale, chunk, value_div, out_float, keep_first,
                                                dist_bias, dist_rows));
 }

@@ -465,7 +465,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap tmK, const __gr
       ok = __all_sync(0xffffffffu, ok);
       if (ok) {
         t5_fence_after();
-        const float lsum = l + sink_weight(ep, m_ref);       // the sink relative to the row's reference, like every P
+        const float lsum = l + sink_weight(ep, m_ref, min(head, nh - 1));       // the sink relative to the row's reference, like every P
         const float inv = lsum > 0.f ? head_gate(ep, valid ? t0 + tok : t0, head) / lsum : 0.f;
         __nv_bfloat16* orow = out + (size_t)(t0 + tok) * nh * HD + (size_t)head * HD;
         if (o_by_tma && all_rows) {
@@ -563,17 +563,17 @@ VOB_API int vob_attention_prefill_has_tc5() {
 
 // As vob_attention_prefill_tma (same tensor maps: 64-column slices, boxes of vob_attention_decode_box_keys rows), for
 // head sizes 64 and 128.  `query_tiles` is 1 or 2: how many tiles of 128 query rows a block takes.  `sink`: the softmax has a
-// silent extra entry of score 0; `gate` (bfloat16, may be null): head h of token t is multiplied by
+// silent extra entry of score 0, or (`sinks`, float [nh] or null) of the head's own score; `gate` (bfloat16, may be null): head h of token t is multiplied by
 // sigmoid(gate[t * gate_stride + h]).  `softcap`, `chunk`, `value_div`, `out_float`, `keep_first`, `dist_bias`: as for
 // vob_attention_prefill_ex.
 VOB_API int vob_attention_prefill_tc5(const void* map_k, const void* map_v, const void* map_q, const void* map_o, const void* q, long q_stride, void* out,
                                       const int* block_tables, int table_stride, const int* cu_q, const int* context_lens,
                                       int num_requests, int max_q, int nh, int kvh, int block_size, int window, float scale,
-                                      long num_pages, int query_tiles, int sink, const void* gate, long gate_stride,
+                                      long num_pages, int query_tiles, int sink, const float* sinks, const void* gate, long gate_stride,
                                       float softcap, int chunk, int value_div, int out_float, int keep_first,
                                       const float* dist_bias, int dist_rows, int* err, cudaStream_t stream) {
 #if VOB_HD == 64 || VOB_HD == 128
-  const HeadEpilogue ep = head_options(sink, gate, gate_stride, softcap, scale, chunk, value_div, out_float, keep_first, dist_bias,
+  const HeadEpilogue ep = head_options(sink, sinks, gate, gate_stride, softcap, scale, chunk, value_div, out_float, keep_first, dist_bias,
                                        dist_rows);
   if (keep_first < 0 || (dist_bias && dist_rows <= 0)) return VOB_BAD_ARGUMENT;
   if (out_float && map_o) return VOB_BAD_ARGUMENT;           // whole tiles leave by the copy engine as bfloat16 only

@@ -10,7 +10,9 @@
 //
 // Four kernels (short_conv_step is the first two in one, for steps of short portions):
 //   short_conv_silu    out[t, c] = f(sum_j w[c, j] x[t - (taps-1) + j, c]), inputs before the portion's start from the slot;
-//                      f is SiLU or (`act` 0) the identity
+//                      f is SiLU or (`act` 0) the identity.  With `bias_in` the filter's inputs are x + bias_in (zeros stay
+//                      zeros before the sequence's start; the slot keeps the sums), with `bias_out` a number a channel is
+//                      added behind the filter; the output is float or (TO) of the model's type
 //   short_conv_state   the slot's taps - 1 inputs after this portion (run after the first: it overwrites what that one reads)
 //   delta_scan         the recurrence.  A column of S lives in the registers of LANES threads (ROWS rows each, rows
 //                      interleaved so that a warp's loads of the state fill whole sectors); a block takes the columns
@@ -29,11 +31,12 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); 
 
 constexpr int CONV_TOKENS = 8;    // tokens a thread walks in a large step: the filter's window slides through registers
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(128)
-short_conv_silu_kernel(const T* x, long x_stride, const float* __restrict__ w, const float* state, long state_stride,
+short_conv_silu_kernel(const T* x, long x_stride, const float* __restrict__ w, const float* __restrict__ bias_in,
+                       const float* __restrict__ bias_out, const float* state, long state_stride,
                        long conv_off, const int* __restrict__ token_req, const int* __restrict__ cu_q,
-                       const int* __restrict__ state_slots, float* out, int num_tokens, int walk, int C, int taps, long num_slots,
+                       const int* __restrict__ state_slots, TO* out, int num_tokens, int walk, int C, int taps, long num_slots,
                        int act, int* err) {
   pdl_launch_dependents();
   const int t_first = blockIdx.x * walk;
@@ -42,6 +45,7 @@ short_conv_silu_kernel(const T* x, long x_stride, const float* __restrict__ w, c
 #pragma unroll
   for (int s = 0; s < DELTA_MAX_TAPS; ++s) wt[s] = (c < C && s < taps) ? w[(size_t)c * taps + s] : 0.f;
   const float w_now = c < C ? w[(size_t)c * taps + taps - 1] : 0.f;      // the current token's tap
+  const float b_in = bias_in && c < C ? bias_in[c] : 0.f, b_out = bias_out && c < C ? bias_out[c] : 0.f;
   pdl_wait();
   if (c >= C) return;
   float win[DELTA_MAX_TAPS - 1];      // win[s]: the input taps - 1 - s tokens back
@@ -64,18 +68,18 @@ short_conv_silu_kernel(const T* x, long x_stride, const float* __restrict__ w, c
       for (int s = 0; s < DELTA_MAX_TAPS - 1; ++s) {
         if (s < taps - 1) {
           const int rel = j - (taps - 1) + s;      // place within the portion; before its start the slot has the input
-          win[s] = rel >= 0 ? to_f<T>(x[(size_t)(t - (taps - 1) + s) * x_stride + c]) : st[(size_t)(taps - 1 + rel) * C + c];
+          win[s] = rel >= 0 ? to_f<T>(x[(size_t)(t - (taps - 1) + s) * x_stride + c]) + b_in : st[(size_t)(taps - 1 + rel) * C + c];
         }
       }
       have = true;
     }
-    const float cur = to_f<T>(x[(size_t)t * x_stride + c]);
-    float acc = 0.f;
+    const float cur = to_f<T>(x[(size_t)t * x_stride + c]) + b_in;
+    float acc = b_out;
 #pragma unroll
     for (int s = 0; s < DELTA_MAX_TAPS - 1; ++s)
       if (s < taps - 1) acc = fmaf(wt[s], win[s], acc);          // oldest input first
     acc = fmaf(w_now, cur, acc);
-    out[(size_t)t * C + c] = act ? silu_f(acc) : acc;
+    out[(size_t)t * C + c] = from_f<TO>(act ? silu_f(acc) : acc);
 #pragma unroll
     for (int s = 0; s < DELTA_MAX_TAPS - 1; ++s) {
       if (s < taps - 2) win[s] = win[s + 1 < DELTA_MAX_TAPS - 1 ? s + 1 : s];
@@ -86,7 +90,7 @@ short_conv_silu_kernel(const T* x, long x_stride, const float* __restrict__ w, c
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-short_conv_state_kernel(const T* x, long x_stride, float* state, long state_stride, long conv_off,
+short_conv_state_kernel(const T* x, long x_stride, const float* __restrict__ bias_in, float* state, long state_stride, long conv_off,
                         const int* __restrict__ cu_q, const int* __restrict__ state_slots, int C, int taps, long num_slots) {
   pdl_launch_dependents();
   const int b = blockIdx.y;
@@ -95,13 +99,14 @@ short_conv_state_kernel(const T* x, long x_stride, float* state, long state_stri
   const int slot = state_slots[b];
   pdl_wait();
   if (n <= 0 || slot < 0 || slot >= num_slots || c >= C) return;
+  const float b_in = bias_in ? bias_in[c] : 0.f;
   float* st = state + (size_t)slot * state_stride + conv_off;
   float nv[DELTA_MAX_TAPS - 1];
 #pragma unroll
   for (int s = 0; s < DELTA_MAX_TAPS - 1; ++s) {
     if (s < taps - 1) {
       const int rel = n - (taps - 1) + s;     // place within the portion of the input that entry s holds afterwards
-      nv[s] = rel >= 0 ? to_f<T>(x[(size_t)(t0 + rel) * x_stride + c]) : st[(size_t)(s + n) * C + c];
+      nv[s] = rel >= 0 ? to_f<T>(x[(size_t)(t0 + rel) * x_stride + c]) + b_in : st[(size_t)(s + n) * C + c];
     }
   }
 #pragma unroll
@@ -112,10 +117,11 @@ short_conv_state_kernel(const T* x, long x_stride, float* state, long state_stri
 // Both of the above in one launch for steps whose portions are short (decoding): a thread owns one channel of one request,
 // takes its window from the slot, walks the request's few tokens and leaves the window in the slot.  The same sums in the
 // same order as the two kernels.
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(128)
-short_conv_step_kernel(const T* x, long x_stride, const float* __restrict__ w, float* state, long state_stride, long conv_off,
-                       const int* __restrict__ cu_q, const int* __restrict__ state_slots, float* out, int C, int taps,
+short_conv_step_kernel(const T* x, long x_stride, const float* __restrict__ w, const float* __restrict__ bias_in,
+                       const float* __restrict__ bias_out, float* state, long state_stride, long conv_off,
+                       const int* __restrict__ cu_q, const int* __restrict__ state_slots, TO* out, int C, int taps,
                        long num_slots, int act, int* err) {
   pdl_launch_dependents();
   const int b = blockIdx.y;
@@ -126,6 +132,7 @@ short_conv_step_kernel(const T* x, long x_stride, const float* __restrict__ w, f
 #pragma unroll
   for (int s = 0; s < DELTA_MAX_TAPS; ++s) wt[s] = (c < C && s < taps) ? w[(size_t)c * taps + s] : 0.f;
   const float w_now = c < C ? w[(size_t)c * taps + taps - 1] : 0.f;
+  const float b_in = bias_in && c < C ? bias_in[c] : 0.f, b_out = bias_out && c < C ? bias_out[c] : 0.f;
   pdl_wait();
   if (n <= 0) return;
   if (slot < 0 || slot >= num_slots) {
@@ -138,13 +145,13 @@ short_conv_step_kernel(const T* x, long x_stride, const float* __restrict__ w, f
 #pragma unroll
   for (int s = 0; s < DELTA_MAX_TAPS - 1; ++s) win[s] = s < taps - 1 ? st[(size_t)s * C + c] : 0.f;
   for (int i = 0; i < n; ++i) {
-    const float cur = to_f<T>(x[(size_t)(t0 + i) * x_stride + c]);
-    float acc = 0.f;
+    const float cur = to_f<T>(x[(size_t)(t0 + i) * x_stride + c]) + b_in;
+    float acc = b_out;
 #pragma unroll
     for (int s = 0; s < DELTA_MAX_TAPS - 1; ++s)
       if (s < taps - 1) acc = fmaf(wt[s], win[s], acc);
     acc = fmaf(w_now, cur, acc);
-    out[(size_t)(t0 + i) * C + c] = act ? silu_f(acc) : acc;
+    out[(size_t)(t0 + i) * C + c] = from_f<TO>(act ? silu_f(acc) : acc);
 #pragma unroll
     for (int s = 0; s < DELTA_MAX_TAPS - 1; ++s) {
       if (s < taps - 2) win[s] = win[s + 1 < DELTA_MAX_TAPS - 1 ? s + 1 : s];
@@ -369,56 +376,85 @@ delta_out_norm_kernel(const float* raw, const T* gate, long gate_stride, const f
   }
 }
 
+// The same for wide rows (all heads normed as one): a block takes a row.
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_out_norm_wide_kernel(const float* raw, const T* gate, long gate_stride, const float* __restrict__ w, T* out, int heads,
+                           int vdim, float eps, int gate_sigmoid) {
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x / heads, h = blockIdx.x % heads;
+  const float* o = raw + ((size_t)t * heads + h) * vdim;
+  const T* grow = gate + (size_t)t * gate_stride + (size_t)h * vdim;
+  T* orow = out + ((size_t)t * heads + h) * vdim;
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < vdim; d += 256) ss = fmaf(o[d], o[d], ss);
+  const float inv = 1.f / sqrtf(block_sum<256>(ss, scratch) / (float)vdim + eps);
+  for (int d = threadIdx.x; d < vdim; d += 256) {
+    const float gv = to_f<T>(grow[d]);
+    orow[d] = from_f<T>(o[d] * inv * w[d] * (gate_sigmoid ? 1.f / (1.f + expf(-gv)) : silu_f(gv)));
+  }
+}
+
 }  // namespace vob
 
 using namespace vob;
 
-// x: rows of x_stride elements of `dtype`, the C channels first; w float [C, taps]; state float [num_slots, state_stride]
-// with the convolutions' part ((taps - 1) x C) at conv_off; out float [T, C].
-VOB_API int vob_short_conv_silu(const void* x, long x_stride, const float* w, const float* state, long state_stride,
-                                long conv_off, const int* token_req, const int* cu_q, const int* state_slots, float* out,
-                                int T, int C, int taps, long num_slots, int act, int dtype, int* err, cudaStream_t stream) {
+// x: rows of x_stride elements of `dtype`, the C channels first; w float [C, taps]; bias_in, bias_out float [C] or null; state
+// float [num_slots, state_stride] with the convolutions' part ((taps - 1) x C) at conv_off; out [T, C] float, or of `dtype`
+// without `out_float`.
+VOB_API int vob_short_conv_silu(const void* x, long x_stride, const float* w, const float* bias_in, const float* bias_out,
+                                const float* state, long state_stride, long conv_off, const int* token_req, const int* cu_q,
+                                const int* state_slots, void* out, int T, int C, int taps, long num_slots, int act, int out_float,
+                                int dtype, int* err, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (C <= 0 || taps < 1 || taps > DELTA_MAX_TAPS) return VOB_UNSUPPORTED;
   const int walk = T >= 32 * CONV_TOKENS ? CONV_TOKENS : 1;      // few tokens (decoding): one each, nothing to slide
   dim3 grid((T + walk - 1) / walk, (C + 127) / 128);
   if (grid.y > 65535) return VOB_UNSUPPORTED;
-  if (dtype == VOB_F32)
-    return launch_kernel(short_conv_silu_kernel<float>, grid, 128, 0, stream, (const float*)x, x_stride, w, state, state_stride,
-                         conv_off, token_req, cu_q, state_slots, out, T, walk, C, taps, num_slots, act, err);
-  if (dtype == VOB_BF16)
-    return launch_kernel(short_conv_silu_kernel<__nv_bfloat16>, grid, 128, 0, stream, (const __nv_bfloat16*)x, x_stride, w,
-                         state, state_stride, conv_off, token_req, cu_q, state_slots, out, T, walk, C, taps, num_slots, act, err);
+#define VOB_SC(TT, TO)                                                                                                           \
+  return launch_kernel(short_conv_silu_kernel<TT, TO>, grid, 128, 0, stream, (const TT*)x, x_stride, w, bias_in, bias_out, state, \
+                       state_stride, conv_off, token_req, cu_q, state_slots, (TO*)out, T, walk, C, taps, num_slots, act, err)
+  if (dtype == VOB_F32) { VOB_SC(float, float); }
+  if (dtype == VOB_BF16) {
+    if (out_float) { VOB_SC(__nv_bfloat16, float); }
+    VOB_SC(__nv_bfloat16, __nv_bfloat16);
+  }
+#undef VOB_SC
   return VOB_BAD_ARGUMENT;
 }
 
-VOB_API int vob_short_conv_state(const void* x, long x_stride, float* state, long state_stride, long conv_off,
+VOB_API int vob_short_conv_state(const void* x, long x_stride, const float* bias_in, float* state, long state_stride, long conv_off,
                                  const int* cu_q, const int* state_slots, int B, int C, int taps, long num_slots, int dtype,
                                  cudaStream_t stream) {
   if (B <= 0 || taps <= 1) return 0;
   if (C <= 0 || taps > DELTA_MAX_TAPS) return VOB_UNSUPPORTED;
   dim3 grid((C + 127) / 128, B);
   if (dtype == VOB_F32)
-    return launch_kernel(short_conv_state_kernel<float>, grid, 128, 0, stream, (const float*)x, x_stride, state, state_stride,
+    return launch_kernel(short_conv_state_kernel<float>, grid, 128, 0, stream, (const float*)x, x_stride, bias_in, state, state_stride,
                          conv_off, cu_q, state_slots, C, taps, num_slots);
   if (dtype == VOB_BF16)
-    return launch_kernel(short_conv_state_kernel<__nv_bfloat16>, grid, 128, 0, stream, (const __nv_bfloat16*)x, x_stride,
+    return launch_kernel(short_conv_state_kernel<__nv_bfloat16>, grid, 128, 0, stream, (const __nv_bfloat16*)x, x_stride, bias_in,
                          state, state_stride, conv_off, cu_q, state_slots, C, taps, num_slots);
   return VOB_BAD_ARGUMENT;
 }
 
-VOB_API int vob_short_conv_step(const void* x, long x_stride, const float* w, float* state, long state_stride, long conv_off,
-                                const int* cu_q, const int* state_slots, float* out, int B, int C, int taps, long num_slots,
-                                int act, int dtype, int* err, cudaStream_t stream) {
+VOB_API int vob_short_conv_step(const void* x, long x_stride, const float* w, const float* bias_in, const float* bias_out, float* state,
+                                long state_stride, long conv_off, const int* cu_q, const int* state_slots, void* out, int B, int C,
+                                int taps, long num_slots, int act, int out_float, int dtype, int* err, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (C <= 0 || taps < 1 || taps > DELTA_MAX_TAPS || B > 65535) return VOB_UNSUPPORTED;
   dim3 grid((C + 127) / 128, B);
-  if (dtype == VOB_F32)
-    return launch_kernel(short_conv_step_kernel<float>, grid, 128, 0, stream, (const float*)x, x_stride, w, state, state_stride,
-                         conv_off, cu_q, state_slots, out, C, taps, num_slots, act, err);
-  if (dtype == VOB_BF16)
-    return launch_kernel(short_conv_step_kernel<__nv_bfloat16>, grid, 128, 0, stream, (const __nv_bfloat16*)x, x_stride, w,
-                         state, state_stride, conv_off, cu_q, state_slots, out, C, taps, num_slots, act, err);
+#define VOB_SC(TT, TO)                                                                                                           \
+  return launch_kernel(short_conv_step_kernel<TT, TO>, grid, 128, 0, stream, (const TT*)x, x_stride, w, bias_in, bias_out, state, \
+                       state_stride, conv_off, cu_q, state_slots, (TO*)out, C, taps, num_slots, act, err)
+  if (dtype == VOB_F32) { VOB_SC(float, float); }
+  if (dtype == VOB_BF16) {
+    if (out_float) { VOB_SC(__nv_bfloat16, float); }
+    VOB_SC(__nv_bfloat16, __nv_bfloat16);
+  }
+#undef VOB_SC
   return VOB_BAD_ARGUMENT;
 }
 
@@ -471,6 +507,15 @@ VOB_API int vob_delta_out_norm(const float* raw, const void* gate, long gate_str
                                int vdim, float eps, int gate_sigmoid, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   const int total = T * heads;
+  if (vdim > 512) {
+    if (dtype == VOB_F32)
+      return launch_kernel(delta_out_norm_wide_kernel<float>, dim3(total), 256, 0, stream, raw, (const float*)gate, gate_stride, w,
+                           (float*)out, heads, vdim, eps, gate_sigmoid);
+    if (dtype == VOB_BF16)
+      return launch_kernel(delta_out_norm_wide_kernel<__nv_bfloat16>, dim3(total), 256, 0, stream, raw, (const __nv_bfloat16*)gate,
+                           gate_stride, w, (__nv_bfloat16*)out, heads, vdim, eps, gate_sigmoid);
+    return VOB_BAD_ARGUMENT;
+  }
   dim3 grid((total + 3) / 4);
   if (dtype == VOB_F32)
     return launch_kernel(delta_out_norm_kernel<float>, grid, 128, 0, stream, raw, (const float*)gate, gate_stride, w,

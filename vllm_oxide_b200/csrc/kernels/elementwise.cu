@@ -195,11 +195,11 @@ __global__ void __launch_bounds__(NT) add_rmsnorm_kernel(const T* x, T* residual
   }
 }
 
-// ---------------------------------------------------------------- SiLU(gate) * up
+// ---------------------------------------------------------------- SiLU(gate) * up, or gelu(gate) * up
 // gu holds, per token, either I gate values then I up values, or (interleaved) groups of sixteen columns:
 // eight gate values and the eight up values of the same outputs.  VEC: eight outputs per thread with 16-byte
-// accesses (I a multiple of 8, 16-byte aligned rows).
-template <typename T, bool VEC>
+// accesses (I a multiple of 8, 16-byte aligned rows).  GELU: the tanh form of gelu in place of SiLU.
+template <typename T, bool VEC, bool GELU>
 __global__ void silu_mul_kernel(const T* gu, T* out, int I, size_t total, int interleaved) {
   pdl_launch_dependents();
   pdl_wait();
@@ -220,13 +220,13 @@ __global__ void silu_mul_kernel(const T* gu, T* out, int I, size_t total, int in
         load16<T>(gp, reinterpret_cast<float(&)[Vec16<T>::N]>(g));
         load16<T>(up, reinterpret_cast<float(&)[Vec16<T>::N]>(u));
 #pragma unroll
-        for (int j = 0; j < N; ++j) o[j] = round_to<T>(__fdividef(g[j], 1.f + __expf(-g[j]))) * u[j];   // 2 ulp of float: far below bfloat16's step
+        for (int j = 0; j < N; ++j) o[j] = round_to<T>(GELU ? gelu_tanh_f(g[j]) : __fdividef(g[j], 1.f + __expf(-g[j]))) * u[j];   // 2 ulp of float: far below bfloat16's step
         store16<T>(out + gidx * N, reinterpret_cast<float(&)[Vec16<T>::N]>(o));
       } else {
 #pragma unroll
         for (int j = 0; j < N; ++j) {
           const float g = to_f<T>(gp[j]), u = to_f<T>(up[j]);
-          out[gidx * N + j] = from_f<T>(round_to<T>(g / (1.f + expf(-g))) * u);
+          out[gidx * N + j] = from_f<T>(round_to<T>(GELU ? gelu_tanh_f(g) : g / (1.f + expf(-g))) * u);
         }
       }
     }
@@ -239,7 +239,7 @@ __global__ void silu_mul_kernel(const T* gu, T* out, int I, size_t total, int in
     const int ui = interleaved ? gi + 8 : I + i;
     const float g = to_f<T>(gu[t * 2 * I + gi]);
     const float u = to_f<T>(gu[t * 2 * I + ui]);
-    const float s = round_to<T>(g / (1.f + expf(-g)));
+    const float s = round_to<T>(GELU ? gelu_tanh_f(g) : g / (1.f + expf(-g)));
     out[idx] = from_f<T>(s * u);
   }
 }
@@ -621,7 +621,7 @@ VOB_API int vob_add_rmsnorm(const void* x, void* residual, const float* w, void*
   return VOB_BAD_ARGUMENT;
 }
 
-VOB_API int vob_silu_mul(const void* gu, void* out, int T, int I, int interleaved, int dtype, cudaStream_t stream) {
+VOB_API int vob_silu_mul(const void* gu, void* out, int T, int I, int interleaved, int gelu, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (interleaved && I % 8) return VOB_BAD_ARGUMENT;
   const size_t total = (size_t)T * I;
@@ -629,14 +629,20 @@ VOB_API int vob_silu_mul(const void* gu, void* out, int T, int I, int interleave
   const size_t work = vec ? total / 8 : total;
   const size_t cap = (size_t)sm_count() * 16;
   const int blocks = (int)((work + 255) / 256 < cap ? (work + 255) / 256 : cap);
-  if (dtype == VOB_F32)
-    return vec ? launch_kernel(silu_mul_kernel<float, true>, blocks, 256, 0, stream, (const float*)gu, (float*)out, I, total, interleaved)
-               : launch_kernel(silu_mul_kernel<float, false>, blocks, 256, 0, stream, (const float*)gu, (float*)out, I, total, interleaved);
-  if (dtype == VOB_BF16)
-    return vec ? launch_kernel(silu_mul_kernel<__nv_bfloat16, true>, blocks, 256, 0, stream, (const __nv_bfloat16*)gu,
-                               (__nv_bfloat16*)out, I, total, interleaved)
-               : launch_kernel(silu_mul_kernel<__nv_bfloat16, false>, blocks, 256, 0, stream, (const __nv_bfloat16*)gu,
-                               (__nv_bfloat16*)out, I, total, interleaved);
+#define VOB_SM(TT, VV)                                                                                                          \
+  do {                                                                                                                          \
+    if (gelu) return launch_kernel(silu_mul_kernel<TT, VV, true>, blocks, 256, 0, stream, (const TT*)gu, (TT*)out, I, total, interleaved); \
+    return launch_kernel(silu_mul_kernel<TT, VV, false>, blocks, 256, 0, stream, (const TT*)gu, (TT*)out, I, total, interleaved); \
+  } while (0)
+  if (dtype == VOB_F32) {
+    if (vec) VOB_SM(float, true);
+    VOB_SM(float, false);
+  }
+  if (dtype == VOB_BF16) {
+    if (vec) VOB_SM(__nv_bfloat16, true);
+    VOB_SM(__nv_bfloat16, false);
+  }
+#undef VOB_SM
   return VOB_BAD_ARGUMENT;
 }
 

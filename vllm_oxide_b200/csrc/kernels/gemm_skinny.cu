@@ -44,7 +44,7 @@ constexpr int SK_SLICES = SK_KC / TMA_BOX_COLS;   // boxes of 64 columns per sta
 constexpr int SK_CONSUMERS = 4;
 constexpr int SK_THREADS = (SK_CONSUMERS + 1) * 32;
 
-enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_ADD = 3 };
+enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_ADD = 3, EPI_GEGLU = 4 };
 
 __device__ __forceinline__ void sk_ldmatrix_x4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
@@ -267,7 +267,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
       const bool aborted = *abort_flag != 0;
       if (aborted) {
         // nothing is written for a tile that was not finished
-      } else if (EPI == EPI_SWIGLU) {
+      } else if (EPI == EPI_SWIGLU || EPI == EPI_GEGLU) {
         for (int idx = tid; idx < (R / 2) * m_rows; idx += SK_CONSUMERS * 32) {
           const int tok = idx / (R / 2), r = idx % (R / 2);
           const long n = (long)tile * (R / 2) + r;
@@ -284,7 +284,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
           }
           gate = bf16_round(gate);
           up = bf16_round(up);
-          const float act = bf16_round(gate / (1.f + expf(-gate)));
+          const float act = bf16_round(EPI == EPI_GEGLU ? gelu_tanh_f(gate) : gate / (1.f + expf(-gate)));
           reinterpret_cast<__nv_bfloat16*>(out)[(long)tok * ldo + n] = __float2bfloat16_rn(act * up);
         }
       } else {
@@ -370,6 +370,7 @@ static int skinny_dispatch(int epilogue, const CUtensorMap* tw, const CUtensorMa
   if (epilogue == EPI_BF16) return skinny_launch<R, MT, EPI_BF16, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
   if (epilogue == EPI_F32) return skinny_launch<R, MT, EPI_F32, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
   if (epilogue == EPI_SWIGLU) return skinny_launch<R, MT, EPI_SWIGLU, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
+  if (epilogue == EPI_GEGLU) return skinny_launch<R, MT, EPI_GEGLU, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
   if (epilogue == EPI_ADD) return skinny_launch<R, MT, EPI_ADD, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
   return VOB_BAD_ARGUMENT;
 }
@@ -397,7 +398,7 @@ VOB_API int vob_gemm_skinny_token_box(int M) { return M <= 8 ? 8 : 16; }
 // a multiple of 64).
 // epilogue: 0 bfloat16 out [M,N]; 1 float out [M,N] (rounded to bfloat16 first); 2 SiLU(gate)*up over rows that
 // alternate in groups of eight between gate and up, out [M,N/2] bfloat16; 3 out [M,N] bfloat16 += the product rounded to
-// bfloat16 (the residual stream).  norm_w (may be null; epilogues 0 and 2): float [K], the weight of an RMSNorm with
+// bfloat16 (the residual stream); 4 as 2 with the tanh form of gelu in place of SiLU (without a norm).  norm_w (may be null; epilogues 0 and 2): float [K], the weight of an RMSNorm with
 // `eps` that is applied to x on the way.  ss_parts (may be null; instead of norm_w): x is already the tokens times the
 // norm's weight, and ss_parts [ss_count][8 or 16] (the token rows of a box for this M) holds sums of squares of the
 // unscaled tokens that add up to each token's; the product is scaled by 1/rms.  emit_w / emit_xn / emit_ss (all or none;
@@ -408,7 +409,7 @@ VOB_API int vob_gemm_skinny(const void* map_w, const void* map_x, void* out, lon
                             void* emit_xn, float* emit_ss, int* err, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 16 || K <= 0 || K % 64 || !map_w || !map_x) return VOB_UNSUPPORTED;
-  if (epilogue == EPI_SWIGLU && N % 16) return VOB_BAD_ARGUMENT;
+  if ((epilogue == EPI_SWIGLU || epilogue == EPI_GEGLU) && N % 16) return VOB_BAD_ARGUMENT;
   if (norm_w && (uintptr_t)norm_w % 8) return VOB_BAD_ARGUMENT;
   if (ss_parts && (norm_w || ss_count <= 0)) return VOB_BAD_ARGUMENT;
   if ((emit_w != nullptr) != (emit_xn != nullptr) || (emit_w != nullptr) != (emit_ss != nullptr)) return VOB_BAD_ARGUMENT;

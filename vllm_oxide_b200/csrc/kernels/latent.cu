@@ -124,9 +124,9 @@ __global__ void latent_query_rotate_kernel(const T* q, T* qa, const float* __res
 // the order of the warps.  The order of operations of an output depends on I alone, not on the tile it falls into.
 constexpr int HL_TT = 8, HL_WARPS = 8, HL_O = 32;
 
-template <typename T>
+template <typename T, typename TY>
 __global__ void __launch_bounds__(HL_WARPS * 32)
-head_linear_kernel(const T* x, long x_ts, long x_hs, const T* __restrict__ w, T* y, long y_ts, long y_hs, int tokens, int I, int O) {
+head_linear_kernel(const T* x, long x_ts, long x_hs, const T* __restrict__ w, TY* y, long y_ts, long y_hs, int tokens, int I, int O) {
   extern __shared__ float xs[];                 // [HL_TT][I], then the partial sums [HL_WARPS][HL_TT][HL_O]
   float* part = xs + HL_TT * I;
   pdl_launch_dependents();
@@ -159,7 +159,7 @@ head_linear_kernel(const T* x, long x_ts, long x_hs, const T* __restrict__ w, T*
     float s = 0.f;
 #pragma unroll
     for (int k = 0; k < HL_WARPS; ++k) s += part[(k * HL_TT + tt) * HL_O + lane];
-    y[(size_t)(t0 + tt) * y_ts + (size_t)h * y_hs + o] = from_f<T>(s);
+    y[(size_t)(t0 + tt) * y_ts + (size_t)h * y_hs + o] = from_f<TY>(s);
   }
 }
 
@@ -262,19 +262,26 @@ VOB_API int vob_latent_query_rotate(const void* q, void* qa, const float* freq, 
   return VOB_BAD_ARGUMENT;
 }
 
-// x: token stride x_ts, head stride x_hs (elements); w [heads, I, O]; y likewise.
+// x: token stride x_ts, head stride x_hs (elements); w [heads, I, O]; y likewise, of `dtype` or (`y_float`) float.
 VOB_API int vob_head_linear(const void* x, long x_ts, long x_hs, const void* w, void* y, long y_ts, long y_hs, int T, int heads,
-                            int I, int O, int dtype, cudaStream_t stream) {
+                            int I, int O, int y_float, int dtype, cudaStream_t stream) {
   if (T <= 0 || heads <= 0 || O <= 0) return 0;
   if (I <= 0) return VOB_BAD_ARGUMENT;
   const size_t smem = ((size_t)HL_TT * I + (size_t)HL_WARPS * HL_TT * HL_O) * sizeof(float);
   dim3 grid((O + HL_O - 1) / HL_O, heads, (T + HL_TT - 1) / HL_TT);
-  if (smem > 48 * 1024 || grid.y > 65535 || grid.z > 65535) return VOB_UNSUPPORTED;
-  if (dtype == VOB_F32)
-    return launch_kernel(head_linear_kernel<float>, grid, dim3(HL_WARPS * 32), smem, stream, (const float*)x, x_ts, x_hs, (const float*)w,
-                         (float*)y, y_ts, y_hs, T, I, O);
-  if (dtype == VOB_BF16)
-    return launch_kernel(head_linear_kernel<__nv_bfloat16>, grid, dim3(HL_WARPS * 32), smem, stream, (const __nv_bfloat16*)x, x_ts, x_hs,
-                         (const __nv_bfloat16*)w, (__nv_bfloat16*)y, y_ts, y_hs, T, I, O);
+  if (smem > 200 * 1024 || grid.y > 65535 || grid.z > 65535) return VOB_UNSUPPORTED;
+#define VOB_HL(TT, TY)                                                                                                        \
+  do {                                                                                                                        \
+    if (smem > 48 * 1024)                                                                                                     \
+      cudaFuncSetAttribute(head_linear_kernel<TT, TY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
+    return launch_kernel(head_linear_kernel<TT, TY>, grid, dim3(HL_WARPS * 32), smem, stream, (const TT*)x, x_ts, x_hs,       \
+                         (const TT*)w, (TY*)y, y_ts, y_hs, T, I, O);                                                          \
+  } while (0)
+  if (dtype == VOB_F32) VOB_HL(float, float);
+  if (dtype == VOB_BF16) {
+    if (y_float) VOB_HL(__nv_bfloat16, float);
+    VOB_HL(__nv_bfloat16, __nv_bfloat16);
+  }
+#undef VOB_HL
   return VOB_BAD_ARGUMENT;
 }

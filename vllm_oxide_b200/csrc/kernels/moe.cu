@@ -14,7 +14,8 @@
 //                 (rows of W in pairs: gate row, up row) SiLU(gate) * up, which halves the output's width.
 //                 Float accumulation, one chain of fused multiply-adds over k in ascending order for every output element
 //                 (the float path's product, with a tile's expert in front of it).
-//   moe_combine   out[t] = sum_j weight[t, j] * y[row of (t, j)], j in order, in float.
+//   moe_combine   out[t] = sum_j weight[t, j] * y[row of (t, j)], j in order, in float; a row may be added to it (`add`: what
+//                 an expert that every token uses has made of the token).
 //   relu_squared  out = max(x, 0)^2 (the dense feed-forward's activation).
 #include "common.cuh"
 
@@ -303,7 +304,7 @@ moe_gemm_kernel(const TA* A, long lda, const TA* __restrict__ W, TC* C, long ldc
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_combine_kernel(const float* y, const int* slot_of, const float* weights, T* out, int D, int top) {
+moe_combine_kernel(const float* y, const int* slot_of, const float* weights, const T* add, T* out, int D, int top) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -313,6 +314,7 @@ moe_combine_kernel(const float* y, const int* slot_of, const float* weights, T* 
       const int row = slot_of ? slot_of[(size_t)t * top + j] : t * top + j;
       if (row >= 0) acc = fmaf(weights[(size_t)t * top + j], y[(size_t)row * D + d], acc);
     }
+    if (add) acc += to_f<T>(add[(size_t)t * D + d]);
     out[(size_t)t * D + d] = from_f<T>(acc);
   }
 }
@@ -548,13 +550,16 @@ VOB_API int vob_moe_gemv(const void* A, long lda, const void* W, void* C, long l
   return VOB_UNSUPPORTED;
 }
 
-VOB_API int vob_moe_combine(const float* y, const int* slot_of, const float* weights, void* out, int T, int D, int top, int dtype,
-                            cudaStream_t stream) {
+// add [T, D] of `dtype`, or null.
+VOB_API int vob_moe_combine(const float* y, const int* slot_of, const float* weights, const void* add, void* out, int T, int D,
+                            int top, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (dtype == VOB_F32)
-    return launch_kernel(moe_combine_kernel<float>, dim3(T), 256, 0, stream, y, slot_of, weights, (float*)out, D, top);
+    return launch_kernel(moe_combine_kernel<float>, dim3(T), 256, 0, stream, y, slot_of, weights, (const float*)add, (float*)out, D,
+                         top);
   if (dtype == VOB_BF16)
-    return launch_kernel(moe_combine_kernel<__nv_bfloat16>, dim3(T), 256, 0, stream, y, slot_of, weights, (__nv_bfloat16*)out, D, top);
+    return launch_kernel(moe_combine_kernel<__nv_bfloat16>, dim3(T), 256, 0, stream, y, slot_of, weights, (const __nv_bfloat16*)add,
+                         (__nv_bfloat16*)out, D, top);
   return VOB_BAD_ARGUMENT;
 }
 

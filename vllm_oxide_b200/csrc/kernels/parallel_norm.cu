@@ -181,25 +181,26 @@ rms_norm_step_kernel(float* stream, const T* y1, const T* y2, const float* __res
 }
 
 // out = 0.5 * (a / rms(a) * wa + b / rms(b) * wb): two mixers side by side over the same input, each with an RMS norm over
-// the width (plain gains), then their mean.  One block a token; float sums.
+// the width (plain gains), then their mean; `ba` is added to a's rows first (a bias of the product that made them).  One
+// block a token; float sums.
 template <typename T>
 __global__ void __launch_bounds__(PN_NT)
-pair_norm_mean_kernel(const T* a, const T* b, const float* __restrict__ wa, const float* __restrict__ wb, T* out, int D,
-                      float eps) {
+pair_norm_mean_kernel(const T* a, const T* b, const float* __restrict__ ba, const float* __restrict__ wa,
+                      const float* __restrict__ wb, T* out, int D, float eps) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
   const size_t base = (size_t)blockIdx.x * D;
   float sa = 0.f, sb = 0.f;
   for (int d = threadIdx.x; d < D; d += PN_NT) {
-    const float x = to_f<T>(a[base + d]), y = to_f<T>(b[base + d]);
+    const float x = to_f<T>(a[base + d]) + (ba ? ba[d] : 0.f), y = to_f<T>(b[base + d]);
     sa = fmaf(x, x, sa);
     sb = fmaf(y, y, sb);
   }
   const float ia = 1.f / sqrtf(block_sum<PN_NT>(sa, scratch) / (float)D + eps);
   const float ib = 1.f / sqrtf(block_sum<PN_NT>(sb, scratch) / (float)D + eps);
   for (int d = threadIdx.x; d < D; d += PN_NT)
-    out[base + d] = from_f<T>(0.5f * (to_f<T>(a[base + d]) * ia * wa[d] + to_f<T>(b[base + d]) * ib * wb[d]));
+    out[base + d] = from_f<T>(0.5f * ((to_f<T>(a[base + d]) + (ba ? ba[d] : 0.f)) * ia * wa[d] + to_f<T>(b[base + d]) * ib * wb[d]));
 }
 
 }  // namespace vob
@@ -252,14 +253,14 @@ VOB_API int vob_rms_norm_step(float* stream, const void* y1, const void* y2, con
   return VOB_BAD_ARGUMENT;
 }
 
-VOB_API int vob_pair_norm_mean(const void* a, const void* b, const float* wa, const float* wb, void* out, int T, int D, float eps,
+VOB_API int vob_pair_norm_mean(const void* a, const void* b, const float* ba, const float* wa, const float* wb, void* out, int T, int D, float eps,
                                int dtype, cudaStream_t stream) {
   if (T <= 0 || D <= 0) return 0;
   if (dtype == VOB_F32)
-    return launch_kernel(pair_norm_mean_kernel<float>, dim3(T), PN_NT, 0, stream, (const float*)a, (const float*)b, wa, wb,
+    return launch_kernel(pair_norm_mean_kernel<float>, dim3(T), PN_NT, 0, stream, (const float*)a, (const float*)b, ba, wa, wb,
                          (float*)out, D, eps);
   if (dtype == VOB_BF16)
     return launch_kernel(pair_norm_mean_kernel<__nv_bfloat16>, dim3(T), PN_NT, 0, stream, (const __nv_bfloat16*)a,
-                         (const __nv_bfloat16*)b, wa, wb, (__nv_bfloat16*)out, D, eps);
+                         (const __nv_bfloat16*)b, ba, wa, wb, (__nv_bfloat16*)out, D, eps);
   return VOB_BAD_ARGUMENT;
 }

@@ -11,6 +11,11 @@
 //                           place; k goes to the key plane [pages, kvh, block_size, kd] and v, as projected, to the value
 //                           plane [pages, vh, block_size, vd], at the token's slot (-1 writes nothing).  Sums, norms, angles
 //                           and the rotation are float on both paths and spelled out with rounding intrinsics.
+//   headnorm_rope_kv_write  The same row, with biases, norms a head and values that are normed too: every q and k head gets its
+//                           bias and passes an RMS norm over its own elements with a gain shared by the heads (wq, wk [kd]);
+//                           its first rot_dim elements turn, cos and sin times an amplitude; every value head gets its bias
+//                           and (v_norm) is divided by its root mean square, no gain.  q goes back in place, k and v to the
+//                           planes.  A warp takes a head at a time, through shared memory.
 //   diff_heads_combine      o = a1 - lambda * a2 per head (float), o / sqrt(mean(o^2) + eps) * post, times
 //                           sigmoid(gate) element by element where a gate is given.  a holds, per key/value head, the
 //                           first maps of its r query heads and then their second maps (the order in which attention ran
@@ -164,6 +169,103 @@ rownorm_rope_kv_write_kernel(T* qkv, long row_stride, const int* __restrict__ po
     }
 }
 
+// NT threads, a warp a head.  Heads may be padded with zeros behind kd_norm (vd_norm) elements; the biases and gains then have
+// zeros there too.
+constexpr int HP_WARPS = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(HP_WARPS * 32)
+headnorm_rope_kv_write_kernel(T* qkv, long row_stride, const float* __restrict__ bias, const int* __restrict__ positions,
+                              const int* __restrict__ slots, const float* __restrict__ wq, const float* __restrict__ wk,
+                              const float* __restrict__ freq, float amp, T* kcache, T* vcache, int nh, int kvh, int kd, int vh, int vd,
+                              int kd_norm, int vd_norm, int rot_dim, int interleaved, int v_norm, float eps, long num_slots,
+                              int block_size, int write_kv, int wide, int* err) {
+  __shared__ float2 turn[QP_MAX_ROT / 2];               // (cos, sin) of every angle, times the amplitude
+  __shared__ __align__(16) float heads[HP_WARPS][512];
+  constexpr int N = Wide16<T>::N;
+  pdl_launch_dependents();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = positions[t];
+  const int slot = slots ? slots[t] : -1;
+  const int half = rot_dim >> 1;
+  if (pos >= 0)
+    for (int j = threadIdx.x; j < half; j += HP_WARPS * 32) {
+      float sn, cs;
+      sincosf(__fmul_rn((float)pos, freq[j]), &sn, &cs);
+      turn[j] = make_float2(cs * amp, sn * amp);
+    }
+  pdl_wait();
+  if (pos < 0) {
+    if (threadIdx.x == 0) atomicOr(err, VOB_ERR_POSITION);
+    return;
+  }
+  const bool put = write_kv && slot >= 0;
+  if (put && slot >= num_slots) {
+    if (threadIdx.x == 0) atomicOr(err, VOB_ERR_SLOT);
+    return;
+  }
+  __syncthreads();
+  T* row = qkv + (size_t)t * row_stride;
+  const size_t page = put ? (size_t)(slot / block_size) : 0;
+  const int in_page = put ? slot % block_size : 0;
+  float* x = heads[warp];
+  for (int head = warp; head < nh + kvh + vh; head += HP_WARPS) {
+    const bool is_q = head < nh, is_v = head >= nh + kvh;
+    if (!is_q && !put) break;
+    const int size = is_v ? vd : kd;
+    const int off = is_v ? (nh + kvh) * kd + (head - nh - kvh) * vd : head * kd;
+    const T* src = row + off;
+    float ss = 0.f;
+    if (wide) {
+      for (int d = lane * N; d < size; d += 32 * N) {
+        float v[N];
+        Wide16<T>::load(src + d, v);
+#pragma unroll
+        for (int j = 0; j < N; ++j) {
+          if (bias) v[j] += bias[off + d + j];
+          ss = fmaf(v[j], v[j], ss);
+          x[d + j] = v[j];
+        }
+      }
+    } else {
+      for (int d = lane; d < size; d += 32) {
+        const float v = to_f<T>(src[d]) + (bias ? bias[off + d] : 0.f);
+        ss = fmaf(v, v, ss);
+        x[d] = v;
+      }
+    }
+    ss = warp_sum(ss);
+    __syncwarp();
+    const float* w = is_v ? nullptr : (is_q ? wq : wk);
+    const float inv = is_v ? (v_norm ? 1.f / sqrtf(ss / (float)vd_norm + eps) : 1.f) : (w ? 1.f / sqrtf(ss / (float)kd_norm + eps) : 1.f);
+    T* dst = is_q ? row + off
+                  : (is_v ? vcache + ((page * vh + (head - nh - kvh)) * block_size + in_page) * (size_t)vd
+                          : kcache + ((page * kvh + (head - nh)) * block_size + in_page) * (size_t)kd);
+    auto normed = [&](int d) { return w ? x[d] * inv * w[d] : x[d] * inv; };
+    auto value = [&](int d) {
+      if (is_v || d >= rot_dim) return normed(d);
+      int j, other;
+      bool low;                          // the pair's first element
+      if (interleaved) { j = d >> 1; low = !(d & 1); other = d ^ 1; }
+      else { low = d < half; j = low ? d : d - half; other = low ? d + half : d - half; }
+      const float a = normed(d), b = normed(other);
+      const float2 cs = turn[j];
+      return low ? __fsub_rn(__fmul_rn(a, cs.x), __fmul_rn(b, cs.y)) : __fadd_rn(__fmul_rn(a, cs.x), __fmul_rn(b, cs.y));
+    };
+    if (wide) {
+      for (int d = lane * N; d < size; d += 32 * N) {
+        float o[N];
+#pragma unroll
+        for (int j = 0; j < N; ++j) o[j] = value(d + j);
+        Wide16<T>::store(dst + d, o);
+      }
+    } else {
+      for (int d = lane; d < size; d += 32) dst[d] = from_f<T>(value(d));
+    }
+    __syncwarp();
+  }
+}
+
 // One warp a (token, head).  a: [tokens, 2 * heads * vd] of TA; out [tokens, heads * vd] of T; gate rows of gate_stride.
 template <typename T, typename TA>
 __global__ void __launch_bounds__(128)
@@ -212,6 +314,30 @@ VOB_API int vob_rownorm_rope_kv_write(void* qkv, long row_stride, const int* pos
     return launch_kernel(rownorm_rope_kv_write_kernel<__nv_bfloat16>, dim3(T), QP_NT, 0, stream, (__nv_bfloat16*)qkv,
                          row_stride, positions, slots, wq, wk, freq, (__nv_bfloat16*)kcache, (__nv_bfloat16*)vcache, nh, kvh,
                          kd, vh, vd, rot_dim, interleaved, eps, num_slots, block_size, write_kv, err, kd_norm);
+  return VOB_BAD_ARGUMENT;
+}
+
+// qkv: rows of row_stride elements, nh q heads and kvh k heads of kd, vh v heads of vd; bias float (as long as the three) or null;
+// wq, wk float [kd] or null (both or neither); freq float [rot_dim / 2]; the planes as above.
+VOB_API int vob_headnorm_rope_kv_write(void* qkv, long row_stride, const float* bias, const int* positions, const int* slots,
+                                       const float* wq, const float* wk, const float* freq, float amp, void* kcache, void* vcache, int T,
+                                       int nh, int kvh, int kd, int vh, int vd, int kd_norm, int vd_norm, int rot_dim, int interleaved,
+                                       int v_norm, float eps, long num_slots, int block_size, int write_kv, int dtype, int* err,
+                                       cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (kd <= 0 || vd <= 0 || kd > 512 || vd > 512 || nh <= 0 || kvh <= 0 || vh <= 0 || block_size <= 0 || rot_dim < 0 || rot_dim > kd ||
+      rot_dim % 2 || (rot_dim > 0 && !freq) || (wq == nullptr) != (wk == nullptr) || rot_dim > QP_MAX_ROT || kd_norm <= 0 ||
+      kd_norm > kd || vd_norm <= 0 || vd_norm > vd)
+    return VOB_BAD_ARGUMENT;
+  const int n = dtype == VOB_F32 ? 4 : 8;
+  const int wide = kd % n == 0 && vd % n == 0 && row_stride % n == 0 && (((uintptr_t)qkv | (uintptr_t)kcache | (uintptr_t)vcache) & 15) == 0;
+#define VOB_HP(TT)                                                                                                               \
+  return launch_kernel(headnorm_rope_kv_write_kernel<TT>, dim3(T), HP_WARPS * 32, 0, stream, (TT*)qkv, row_stride, bias, positions, \
+                       slots, wq, wk, freq, amp, (TT*)kcache, (TT*)vcache, nh, kvh, kd, vh, vd, kd_norm, vd_norm, rot_dim,       \
+                       interleaved, v_norm, eps, num_slots, block_size, write_kv, wide, err)
+  if (dtype == VOB_F32) { VOB_HP(float); }
+  if (dtype == VOB_BF16) { VOB_HP(__nv_bfloat16); }
+#undef VOB_HP
   return VOB_BAD_ARGUMENT;
 }
 

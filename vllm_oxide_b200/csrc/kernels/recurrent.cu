@@ -88,16 +88,96 @@ mingru_scan_kernel(const T* zxg, const T* __restrict__ bz, const T* __restrict__
   if (ch == NCH - 1 && live) state[(size_t)slot * W + c] = s;
 }
 
-// ---------------------------------------------------------------- HGRN2
-// qfv [tokens, heads*dk | heads*dk | heads*dv]: pre-activations of q and of the forget gate, and the values.
-//   q = silu(q);  f = l + (1 - l) sigmoid(f + bf);  M = diag(f) M + (1 - f) v^T;  o = M^T q;  out = o / rms(o) * w
+// ---------------------------------------------------------------- a gated linear recurrence a channel (RG-LRU)
+// u [tokens, W] of T (the convolution's output), gates float [tokens, blocks, 2, W / blocks] (pre-activations of r and i,
+// block by block), y rows of y_stride elements (the other branch's projection):
+//   r = sigmoid(r + br), i = sigmoid(i + bi), log a = -8 r softplus(lam), S = a S + sqrt(1 - a^2) i u,
+//   out = S * gelu(y + by)                                 (the tanh form of gelu)
+// 1 - a^2 = -expm1(2 log a): the difference would lose what a slow channel (a near 1) writes.  Cut along the tokens as minGRU.
+struct LruStep { float a, b; };
+
+__device__ __forceinline__ LruStep lru_step(float gr, float gi, float u, float rate) {
+  const float log_a = rate * sigmoid_f(gr);
+  return {expf(log_a), sqrtf(-expm1f(2.f * log_a)) * sigmoid_f(gi) * u};
+}
+
+template <typename T, int NCH>
+__global__ void __launch_bounds__(32 * NCH)
+lru_scan_kernel(const T* u, const float* gates, const T* y, long y_stride, const float* __restrict__ br, const float* __restrict__ bi,
+                const float* __restrict__ lam, const float* __restrict__ by, float* state, long state_stride,
+                const int* __restrict__ cu_q, const int* __restrict__ state_slots, T* out, int W, int per_block, int num_slots,
+                int* err) {
+  __shared__ float As[NCH][32], Bs[NCH][32];
+  pdl_launch_dependents();
+  const int b = blockIdx.y, lane = threadIdx.x, ch = threadIdx.y;
+  const int c = min(blockIdx.x * 32 + lane, W - 1);
+  const bool live = blockIdx.x * 32 + lane < W;
+  const int t0 = cu_q[b], t1 = cu_q[b + 1];
+  const int slot = state_slots[b];
+  const float l = lam[c], biasr = br[c], biasi = bi[c], biasy = by[c];
+  const float rate = -8.f * (fmaxf(l, 0.f) + log1pf(expf(-fabsf(l))));
+  const size_t goff = (size_t)(c / per_block) * 2 * per_block + c % per_block;
+  pdl_wait();
+  if (t1 <= t0) return;
+  if (slot < 0 || slot >= num_slots) {
+    if (threadIdx.x == 0 && ch == 0) atomicOr(err, VOB_ERR_SLOT);
+    return;
+  }
+  const int per = (t1 - t0 + NCH - 1) / NCH;
+  const int lo = min(t1, t0 + ch * per), hi = min(t1, lo + per);
+  float s = state[(size_t)slot * state_stride + c];
+  auto step = [&](int t) {
+    const float* g = gates + (size_t)t * 2 * W + goff;
+    return lru_step(g[0] + biasr, g[per_block] + biasi, to_f<T>(u[(size_t)t * W + c]), rate);
+  };
+  if (NCH > 1) {
+    float A = 1.f, B = 0.f;
+#pragma unroll 4
+    for (int t = lo; t < hi; ++t) {
+      const LruStep g = step(t);
+      A *= g.a;
+      B = fmaf(g.a, B, g.b);
+    }
+    As[ch][lane] = A;
+    Bs[ch][lane] = B;
+    __syncthreads();
+    for (int k = 0; k < ch; ++k) s = fmaf(As[k][lane], s, Bs[k][lane]);
+    __syncthreads();
+  }
+  // four tokens at a time: their loads are issued before the first store
+  for (int t = lo; t < hi; t += 4) {
+    LruStep g[4];
+    float yv[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int tk = min(t + k, hi - 1);
+      g[k] = step(tk);
+      yv[k] = to_f<T>(y[(size_t)tk * y_stride + c]) + biasy;
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (t + k < hi) {
+        s = fmaf(g[k].a, s, g[k].b);
+        if (live) out[(size_t)(t + k) * W + c] = from_f<T>(s * gelu_tanh_f(yv[k]));
+      }
+  }
+  if (ch == NCH - 1 && live) state[(size_t)slot * state_stride + c] = s;
+}
+
+// ---------------------------------------------------------------- matrix states with a gate a row
+// One recurrence, three ways to make its numbers.  Per head, with a state M [dk, dv]:
+//     M = diag(f) M + w v^T,   o = M^T q            f: what a row keeps, w: what is written into it, q: the read-out
+// A SOURCE makes q, f, w and v of a token from its projected row:
+//   HgrnSource       qfv [tokens, heads*dk | heads*dk | heads*dv]: q = silu(q), f = l + (1 - l) sigmoid(f + bf), w = 1 - f
+//   GlaSource        q * scale, w = k, f = sigmoid(z + bz)^(1 / tau) = exp(-softplus(-(z + bz)) / tau), a number a head and row
+//   LightningSource  q = silu(q), w = silu(k), v = silu(v), f = a fixed number a head
 // Column j of a head's state M (dk floats) is shared by PARTS neighbouring lanes, R rows each, in registers: a token costs
 // a thread R multiply-adds twice, and the lanes of a column add their parts of o by shuffles.  The gates of HG_TT tokens are
 // made by the whole block at once and parked in shared memory (rows padded so that the PARTS lanes of a column read
-// different banks).  FUSE: the block holds all dv columns of the head and also takes the norm over them (decoding: one
-// launch); otherwise a block holds as many columns as 128 threads cover, so that a long portion of one request spreads
-// over more blocks, o leaves in float and head_gain_norm_kernel follows.  Both give the same numbers: an element's
-// chain of operations depends on (R, PARTS) alone, and those follow from dk.
+// different banks).  FUSE: the block holds all dv columns of the head and also takes the norm over them (and what the source
+// puts behind it), for decoding: one launch; otherwise a block holds as many columns as 128 threads cover, so that a long
+// portion of one request spreads over more blocks, o leaves in float and a norm kernel follows.  Both give the same numbers:
+// an element's chain of operations depends on (R, PARTS) alone, and those follow from dk.
 //
 // A long portion is also cut along the tokens (`chunks` > 1, four launches): MODE 1 walks every range from a zero state
 // and leaves its end state L; hgrn2_range_gates_kernel takes the product F of every range's gates; hgrn2_join_kernel goes
@@ -111,19 +191,99 @@ constexpr int HG_TT = 16;
 // (32 or 64 rows apart) read different banks with 16-byte loads
 __device__ __forceinline__ int hg_pad(int i) { return i + 4 * (i >> 5); }
 
+struct ScanGates { float q, f, w; };
+
+// What a source keeps of a (head, row) over the tokens, what it reads of a token, and what it makes of both.
+template <typename T>
+struct HgrnSource {
+  const T* rows;
+  long width;
+  const T* bf;
+  const float* lower;
+  int heads, dk, dv;
+  struct Fixed { float l, bias; };
+  struct Raw { float q, f; };
+  __device__ __forceinline__ Fixed fixed(int h, int i) const { return {lower[h * dk + i], to_f<T>(bf[h * dk + i])}; }
+  __device__ __forceinline__ Raw load(size_t t, int h, int i) const {
+    const T* row = rows + t * width;
+    return {to_f<T>(row[h * dk + i]), to_f<T>(row[(heads + h) * dk + i])};
+  }
+  __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed& x) const {
+    const float f = forget_gate(x.l, r.f, x.bias);
+    return {r.q * sigmoid_f(r.q), f, 1.f - f};
+  }
+  __device__ __forceinline__ float value(size_t t, int h, int c) const { return to_f<T>(rows[t * width + (size_t)2 * heads * dk + h * dv + c]); }
+  __device__ __forceinline__ float decay(size_t t, int h, int i, const Fixed& x) const {
+    return forget_gate(x.l, to_f<T>(rows[t * width + (size_t)(heads + h) * dk + i]), x.bias);
+  }
+  __device__ __forceinline__ float finish(float o, size_t, int, int) const { return o; }
+};
+
+// rows: q | k | v (heads*dk, heads*dk, heads*dv), the decay's pre-activations at z_off, the output gate at gate_off.
+template <typename T>
+struct GlaSource {
+  const T* rows;
+  long width;
+  const float* bias;       // [heads * dk]
+  int heads, dk, dv, z_off, gate_off;
+  float scale, inv_tau;
+  struct Fixed { float bias; };
+  struct Raw { float q, k, z; };
+  __device__ __forceinline__ Fixed fixed(int h, int i) const { return {bias[h * dk + i]}; }
+  __device__ __forceinline__ Raw load(size_t t, int h, int i) const {
+    const T* row = rows + t * width;
+    return {to_f<T>(row[h * dk + i]), to_f<T>(row[(heads + h) * dk + i]), to_f<T>(row[z_off + h * dk + i])};
+  }
+  // sigmoid(z)^(1/tau) by its logarithm: log sigmoid(z) = -softplus(-z) = min(z, 0) - log(1 + e^-|z|)
+  __device__ __forceinline__ float keep(float z) const { return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau); }
+  __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed& x) const { return {r.q * scale, keep(r.z + x.bias), r.k}; }
+  __device__ __forceinline__ float value(size_t t, int h, int c) const { return to_f<T>(rows[t * width + (size_t)2 * heads * dk + h * dv + c]); }
+  __device__ __forceinline__ float decay(size_t t, int h, int i, const Fixed& x) const {
+    return keep(to_f<T>(rows[t * width + z_off + (size_t)h * dk + i]) + x.bias);
+  }
+  // behind the head's norm: times silu(gate)
+  __device__ __forceinline__ float finish(float o, size_t t, int h, int c) const {
+    const float g = to_f<T>(rows[t * width + gate_off + (size_t)h * dv + c]);
+    return o * (g * sigmoid_f(g));
+  }
+};
+
+// rows: q | k | v (heads*dk, heads*dk, heads*dv).
+template <typename T>
+struct LightningSource {
+  const T* rows;
+  long width;
+  const float* decays;     // [heads]
+  int heads, dk, dv;
+  struct Fixed { float f; };
+  struct Raw { float q, k; };
+  __device__ __forceinline__ Fixed fixed(int h, int) const { return {decays[h]}; }
+  __device__ __forceinline__ Raw load(size_t t, int h, int i) const {
+    const T* row = rows + t * width;
+    return {to_f<T>(row[h * dk + i]), to_f<T>(row[(heads + h) * dk + i])};
+  }
+  __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed& x) const { return {r.q * sigmoid_f(r.q), x.f, r.k * sigmoid_f(r.k)}; }
+  __device__ __forceinline__ float value(size_t t, int h, int c) const {
+    const float v = to_f<T>(rows[t * width + (size_t)2 * heads * dk + h * dv + c]);
+    return v * sigmoid_f(v);
+  }
+  __device__ __forceinline__ float decay(size_t, int, int, const Fixed& x) const { return x.f; }
+  __device__ __forceinline__ float finish(float o, size_t, int, int) const { return o; }
+};
+
 // FULL: dk = R * PARTS, every row a thread holds exists (no test per element: the tests were two of seven instructions).
-template <typename T, int R, int PARTS, bool FUSE, int MODE, bool FULL>
+template <typename T, typename SOURCE, int R, int PARTS, bool FUSE, int MODE, bool FULL>
 __global__ void __launch_bounds__(FUSE ? (R > 32 ? 256 : 512) : 128)
-hgrn2_scan_kernel(const T* qfv, const T* __restrict__ bf, const float* __restrict__ lower, const float* __restrict__ nw,
-                  float* state, const int* __restrict__ cu_q, const int* __restrict__ state_slots, T* out, float* raw,
-                  float* ends, float* gates, int heads, int dk, int dv, int col_blocks, float eps, int num_slots, int* err) {
+hgrn2_scan_kernel(const SOURCE src, const float* __restrict__ nw,
+                  float* state, long state_stride, const int* __restrict__ cu_q, const int* __restrict__ state_slots, T* out, float* raw,
+                  float* ends, int heads, int dk, int dv, int col_blocks, float eps, int num_slots, int* err) {
   extern __shared__ float4 sm4[];
   float* sm = reinterpret_cast<float*>(sm4);
   const int gate_row = hg_pad(R * PARTS);
   const int cols = blockDim.x / PARTS;
   float* qs = sm;                        // [HG_TT][gate_row]
   float* fs = qs + HG_TT * gate_row;     // [HG_TT][gate_row]  f
-  float* gs = fs + HG_TT * gate_row;     // [HG_TT][gate_row]  1 - f
+  float* gs = fs + HG_TT * gate_row;     // [HG_TT][gate_row]  w
   float* vs = gs + HG_TT * gate_row;     // [HG_TT][cols]
   float* os = vs + HG_TT * cols;         // [HG_TT][cols]  (FUSE)
   pdl_launch_dependents();
@@ -140,9 +300,8 @@ hgrn2_scan_kernel(const T* qfv, const T* __restrict__ bf, const float* __restric
   }
   const int per = (q1 - q0 + chunks - 1) / chunks;
   const int t0 = min(q1, q0 + chunk * per), t1 = min(q1, t0 + per);
-  const size_t width = (size_t)heads * (2 * dk + dv);
   const int i0 = part * R;
-  float* mine = MODE == 0 ? state + (((size_t)slot * heads + h) * dk + i0) * dv + j
+  float* mine = MODE == 0 ? state + (size_t)slot * state_stride + ((size_t)h * dk + i0) * dv + j
                           : ends + ((((size_t)b * chunks + chunk) * heads + h) * dk + i0) * dv + j;
   float M[R];
 #pragma unroll
@@ -154,32 +313,27 @@ hgrn2_scan_kernel(const T* qfv, const T* __restrict__ bf, const float* __restric
   for (int ts = t0; ts < t1; ts += HG_TT) {
     const int n = min(HG_TT, t1 - ts);
     for (int i = gate_i; i < dk; i += gate_lanes) {
-      const float l = lower[h * dk + i], bias = to_f<T>(bf[h * dk + i]);
+      const typename SOURCE::Fixed fx = src.fixed(h, i);
       // eight tokens' loads are issued before the first of them is used
       for (int tb = gate_t; tb < n; tb += 8 * gate_step) {
-        float qa[8], fa[8];
+        typename SOURCE::Raw raws[8];
 #pragma unroll
-        for (int k = 0; k < 8; ++k) {
-          const int tt = min(tb + k * gate_step, n - 1);
-          const T* row = qfv + (size_t)(ts + tt) * width;
-          qa[k] = to_f<T>(row[h * dk + i]);
-          fa[k] = to_f<T>(row[(heads + h) * dk + i]);
-        }
+        for (int k = 0; k < 8; ++k) raws[k] = src.load((size_t)(ts + min(tb + k * gate_step, n - 1)), h, i);
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
           const int tt = tb + k * gate_step;
           if (tt < n) {
-            const float f = forget_gate(l, fa[k], bias);
-            if (MODE != 1) qs[tt * gate_row + hg_pad(i)] = qa[k] * sigmoid_f(qa[k]);
-            fs[tt * gate_row + hg_pad(i)] = f;
-            gs[tt * gate_row + hg_pad(i)] = 1.f - f;
+            const ScanGates g = src.make(raws[k], fx);
+            if (MODE != 1) qs[tt * gate_row + hg_pad(i)] = g.q;
+            fs[tt * gate_row + hg_pad(i)] = g.f;
+            gs[tt * gate_row + hg_pad(i)] = g.w;
           }
         }
       }
     }
     for (int idx = threadIdx.x; idx < n * cols; idx += blockDim.x) {
       const int tt = idx / cols, c = idx % cols;
-      vs[idx] = cb * cols + c < dv ? to_f<T>(qfv[(size_t)(ts + tt) * width + (size_t)2 * heads * dk + h * dv + cb * cols + c]) : 0.f;
+      vs[idx] = cb * cols + c < dv ? src.value((size_t)(ts + tt), h, cb * cols + c) : 0.f;
     }
     __syncthreads();
 #pragma unroll 2
@@ -219,7 +373,7 @@ hgrn2_scan_kernel(const T* qfv, const T* __restrict__ bf, const float* __restric
         for (int c = lane; c < dv; c += 32) ss += os[tt * cols + c] * os[tt * cols + c];
         const float denom = sqrtf(warp_sum(ss) / (float)dv + eps);
         for (int c = lane; c < dv; c += 32)
-          out[(size_t)(ts + tt) * heads * dv + h * dv + c] = from_f<T>(os[tt * cols + c] / denom * nw[c]);
+          out[(size_t)(ts + tt) * heads * dv + h * dv + c] = from_f<T>(src.finish(os[tt * cols + c] / denom * nw[c], (size_t)(ts + tt), h, c));
       }
       __syncthreads();
     }
@@ -235,10 +389,9 @@ hgrn2_scan_kernel(const T* qfv, const T* __restrict__ bf, const float* __restric
 // gates[b][c][h][i] = the product of the forget gates of range c of request b: what an end state of that range owes to its start.
 // A block takes 32 gates of one range; its eight warps take every eighth token, and their partial products are multiplied
 // in the order of the warps.
-template <typename T>
+template <typename SOURCE>
 __global__ void __launch_bounds__(256)
-hgrn2_range_gates_kernel(const T* qfv, const T* __restrict__ bf, const float* __restrict__ lower, float* gates,
-                         const int* __restrict__ cu_q, int heads, int dk, int dv) {
+hgrn2_range_gates_kernel(const SOURCE src, float* gates, const int* __restrict__ cu_q, int heads, int dk) {
   __shared__ float part[8][32];
   pdl_launch_dependents();
   pdl_wait();
@@ -249,11 +402,10 @@ hgrn2_range_gates_kernel(const T* qfv, const T* __restrict__ bf, const float* __
   if (q1 <= q0) return;
   const int per = (q1 - q0 + chunks - 1) / chunks;
   const int t0 = min(q1, q0 + chunk * per), t1 = min(q1, t0 + per);
-  const size_t width = (size_t)heads * (2 * dk + dv);
-  const float l = lower[e], bias = to_f<T>(bf[e]);
+  const typename SOURCE::Fixed fx = src.fixed(e / dk, e % dk);
   float F = 1.f;
 #pragma unroll 4
-  for (int t = t0 + warp; t < t1; t += 8) F *= forget_gate(l, to_f<T>(qfv[(size_t)t * width + (size_t)heads * dk + e]), bias);
+  for (int t = t0 + warp; t < t1; t += 8) F *= src.decay((size_t)t, e / dk, e % dk, fx);
   part[warp][lane] = F;
   __syncthreads();
   if (warp == 0 && blockIdx.x * 32 + lane < heads * dk) {
@@ -268,7 +420,7 @@ hgrn2_range_gates_kernel(const T* qfv, const T* __restrict__ bf, const float* __
 // thread's loads are issued before its first store (at most HG_MAX_CHUNKS ranges), or every store would wait for a load.
 constexpr int HG_MAX_CHUNKS = 16;
 
-__global__ void hgrn2_join_kernel(float* state, float* ends, const float* __restrict__ gates, const int* __restrict__ cu_q,
+__global__ void hgrn2_join_kernel(float* state, long state_stride, float* ends, const float* gates, const int* __restrict__ cu_q,
                                   const int* __restrict__ state_slots, int chunks, int heads, int dk, int dv, int num_slots) {
   pdl_launch_dependents();
   pdl_wait();
@@ -284,14 +436,14 @@ __global__ void hgrn2_join_kernel(float* state, float* ends, const float* __rest
       L[c] = ends[((size_t)b * chunks + c) * per + e];
       F[c] = gates[((size_t)b * chunks + c) * heads * dk + row];
     }
-  float M = state[(size_t)slot * per + e];
+  float M = state[(size_t)slot * state_stride + e];
 #pragma unroll
   for (int c = 0; c < HG_MAX_CHUNKS; ++c)
     if (c < chunks) {
       ends[((size_t)b * chunks + c) * per + e] = M;
       M = fmaf(F[c], M, L[c]);
     }
-  state[(size_t)slot * per + e] = M;
+  state[(size_t)slot * state_stride + e] = M;
 }
 
 // out[t, h, :] = raw[t, h, :] / sqrt(mean(raw[t, h, :]^2) + eps) * w; one warp per (token, head).
@@ -308,10 +460,10 @@ __global__ void head_gain_norm_kernel(const float* raw, const float* __restrict_
   for (int c = lane; c < dv; c += 32) out[(size_t)row * dv + c] = from_f<T>(x[c] / denom * w[c]);
 }
 
-template <typename T, int R, int PARTS, int MODE>
-int launch_hgrn2(const void* qfv, const void* bf, const float* lower, const float* nw, float* state, const int* cu_q,
-                 const int* state_slots, void* out, float* raw, float* ends, float* gates, int B, int chunks, int heads, int dk,
-                 int dv, float eps, int num_slots, int fuse, int* err, cudaStream_t stream) {
+template <typename T, typename SOURCE, int R, int PARTS, int MODE>
+int launch_hgrn2(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
+                 void* out, float* raw, float* ends, int B, int chunks, int heads, int dk, int dv, float eps, int num_slots, int fuse,
+                 int* err, cudaStream_t stream) {
   const int gate_row = R * PARTS + 4 * ((R * PARTS) / 32);
   const int threads = fuse ? (dv * PARTS + 31) / 32 * 32 : 128;
   const int cols = threads / PARTS;
@@ -323,22 +475,23 @@ int launch_hgrn2(const void* qfv, const void* bf, const float* lower, const floa
       cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return (int)e;
     }
-    return launch_kernel(kernel, grid, dim3(threads), smem, stream, (const T*)qfv, (const T*)bf, lower, nw, state, cu_q, state_slots,
-                         (T*)out, raw, ends, gates, heads, dk, dv, col_blocks, eps, num_slots, err);
+    return launch_kernel(kernel, grid, dim3(threads), smem, stream, src, nw, state, state_stride, cu_q, state_slots,
+                         (T*)out, raw, ends, heads, dk, dv, col_blocks, eps, num_slots, err);
   };
-  if (fuse) return launch(hgrn2_scan_kernel<T, R, PARTS, true, 0, false>);
-  if (dk == R * PARTS) return launch(hgrn2_scan_kernel<T, R, PARTS, false, MODE, true>);
-  return launch(hgrn2_scan_kernel<T, R, PARTS, false, MODE, false>);
+  if (fuse) return launch(hgrn2_scan_kernel<T, SOURCE, R, PARTS, true, 0, false>);
+  if (dk == R * PARTS) return launch(hgrn2_scan_kernel<T, SOURCE, R, PARTS, false, MODE, true>);
+  return launch(hgrn2_scan_kernel<T, SOURCE, R, PARTS, false, MODE, false>);
 }
 
 // rows of the state a thread keeps, and lanes that share a column: from dk alone
 inline int hgrn2_parts(int dk) { return dk <= 32 ? 1 : dk <= 64 ? 2 : 4; }
+inline bool hgrn2_can_fuse(int dk, int dv) { return dv * hgrn2_parts(dk) <= (dk > 128 ? 256 : 512); }
 
-template <typename T, int MODE>
-int dispatch_hgrn2_mode(const void* qfv, const void* bf, const float* lower, const float* nw, float* state, const int* cu_q,
-                        const int* state_slots, void* out, float* raw, float* ends, float* gates, int B, int chunks, int heads,
-                        int dk, int dv, float eps, int num_slots, int fuse, int* err, cudaStream_t stream) {
-#define VOB_HG(RR, PP) return launch_hgrn2<T, RR, PP, MODE>(qfv, bf, lower, nw, state, cu_q, state_slots, out, raw, ends, gates, B, chunks, heads, dk, dv, eps, num_slots, fuse, err, stream)
+template <typename T, typename SOURCE, int MODE>
+int dispatch_hgrn2_mode(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
+                        void* out, float* raw, float* ends, int B, int chunks, int heads, int dk, int dv, float eps, int num_slots,
+                        int fuse, int* err, cudaStream_t stream) {
+#define VOB_HG(RR, PP) return launch_hgrn2<T, SOURCE, RR, PP, MODE>(src, nw, state, state_stride, cu_q, state_slots, out, raw, ends, B, chunks, heads, dk, dv, eps, num_slots, fuse, err, stream)
   if (dk <= 16) VOB_HG(16, 1);
   if (dk <= 32) VOB_HG(32, 1);
   if (dk <= 64) VOB_HG(32, 2);
@@ -347,31 +500,35 @@ int dispatch_hgrn2_mode(const void* qfv, const void* bf, const float* lower, con
 #undef VOB_HG
 }
 
-template <typename T>
-int dispatch_hgrn2(const void* qfv, const void* bf, const float* lower, const float* nw, float* state, const int* cu_q,
-                   const int* state_slots, void* out, float* raw, float* scratch, int Tn, int B, int chunks, int heads, int dk,
-                   int dv, float eps, int num_slots, int fuse, int* err, cudaStream_t stream) {
+// The recurrence of any source over a step; with `norm` the head norm that follows an unfused walk.
+template <typename T, typename SOURCE>
+int run_matrix_scan(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
+                    void* out, float* raw, float* scratch, int Tn, int B, int chunks, int heads, int dk, int dv, float eps,
+                    int num_slots, int fuse, int norm, int* err, cudaStream_t stream) {
+  if (heads <= 0 || dk <= 0 || dv <= 0 || dk > 256 || B > 65535 || (!fuse && !raw) || (fuse && !hgrn2_can_fuse(dk, dv)) ||
+      chunks < 1 || chunks > HG_MAX_CHUNKS || (chunks > 1 && (fuse || !scratch)) || state_stride < (long)heads * dk * dv)
+    return VOB_UNSUPPORTED;
   int code;
   if (chunks <= 1) {
-    code = dispatch_hgrn2_mode<T, 0>(qfv, bf, lower, nw, state, cu_q, state_slots, out, raw, nullptr, nullptr, B, 1, heads, dk, dv,
-                                     eps, num_slots, fuse, err, stream);
+    code = dispatch_hgrn2_mode<T, SOURCE, 0>(src, nw, state, state_stride, cu_q, state_slots, out, raw, nullptr, B, 1, heads, dk, dv,
+                                             eps, num_slots, fuse, err, stream);
   } else {
     float* ends = scratch;
     float* gates = scratch + (size_t)B * chunks * heads * dk * dv;
-    code = dispatch_hgrn2_mode<T, 1>(qfv, bf, lower, nw, state, cu_q, state_slots, out, raw, ends, gates, B, chunks, heads, dk, dv,
-                                     eps, num_slots, 0, err, stream);
+    code = dispatch_hgrn2_mode<T, SOURCE, 1>(src, nw, state, state_stride, cu_q, state_slots, out, raw, ends, B, chunks, heads, dk, dv,
+                                             eps, num_slots, 0, err, stream);
     if (code != 0) return code;
-    code = launch_kernel(hgrn2_range_gates_kernel<T>, dim3((heads * dk + 31) / 32, B, chunks), dim3(256), 0, stream, (const T*)qfv,
-                         (const T*)bf, lower, gates, cu_q, heads, dk, dv);
+    code = launch_kernel(hgrn2_range_gates_kernel<SOURCE>, dim3((heads * dk + 31) / 32, B, chunks), dim3(256), 0, stream, src, gates,
+                         cu_q, heads, dk);
     if (code != 0) return code;
     const long per = (long)heads * dk * dv;
-    code = launch_kernel(hgrn2_join_kernel, dim3((unsigned)((per + 255) / 256), B), dim3(256), 0, stream, state, ends,
+    code = launch_kernel(hgrn2_join_kernel, dim3((unsigned)((per + 255) / 256), B), dim3(256), 0, stream, state, state_stride, ends,
                          (const float*)gates, cu_q, state_slots, chunks, heads, dk, dv, num_slots);
     if (code != 0) return code;
-    code = dispatch_hgrn2_mode<T, 2>(qfv, bf, lower, nw, state, cu_q, state_slots, out, raw, ends, gates, B, chunks, heads, dk, dv,
-                                     eps, num_slots, 0, err, stream);
+    code = dispatch_hgrn2_mode<T, SOURCE, 2>(src, nw, state, state_stride, cu_q, state_slots, out, raw, ends, B, chunks, heads, dk, dv,
+                                             eps, num_slots, 0, err, stream);
   }
-  if (code != 0 || fuse) return code;
+  if (code != 0 || fuse || !norm) return code;
   const int rows = Tn * heads;
   return launch_kernel(head_gain_norm_kernel<T>, dim3((rows + 3) / 4), dim3(128), 0, stream, (const float*)raw, nw, (T*)out, rows, dv,
                        eps);
@@ -411,20 +568,78 @@ VOB_API int vob_mingru_scan(const void* zxg, const void* bz, const void* bx, flo
 // be able to hold the head: vob_hgrn2_can_fuse); else blocks of 128 threads and raw, float [T, heads*dv], in between.
 // `chunks` > 1 (not with fuse): ranges that a request's tokens are cut into, with scratch of
 // B * chunks * heads * dk * (dv + 1) floats.
-VOB_API int vob_hgrn2_can_fuse(int dk, int dv) { return dv * hgrn2_parts(dk) <= (dk > 128 ? 256 : 512) ? 1 : 0; }
+VOB_API int vob_hgrn2_can_fuse(int dk, int dv) { return hgrn2_can_fuse(dk, dv) ? 1 : 0; }
 
 VOB_API int vob_hgrn2_scan(const void* qfv, const void* bf, const float* lower, const float* nw, float* state, const int* cu_q,
                            const int* state_slots, void* out, float* raw, float* scratch, int T, int B, int chunks, int heads,
                            int dk, int dv, float eps, int num_slots, int fuse, int dtype, int* err, cudaStream_t stream) {
   if (B <= 0 || T <= 0) return 0;
-  if (heads <= 0 || dk <= 0 || dv <= 0 || dk > 256 || B > 65535 || (!fuse && !raw) || (fuse && !vob_hgrn2_can_fuse(dk, dv)) ||
-      chunks < 1 || chunks > HG_MAX_CHUNKS || (chunks > 1 && (fuse || !scratch)))
-    return VOB_UNSUPPORTED;
-  if (dtype == VOB_F32)
-    return dispatch_hgrn2<float>(qfv, bf, lower, nw, state, cu_q, state_slots, out, raw, scratch, T, B, chunks, heads, dk, dv, eps,
-                                 num_slots, fuse, err, stream);
-  if (dtype == VOB_BF16)
-    return dispatch_hgrn2<__nv_bfloat16>(qfv, bf, lower, nw, state, cu_q, state_slots, out, raw, scratch, T, B, chunks, heads, dk,
-                                         dv, eps, num_slots, fuse, err, stream);
+  const long width = (long)heads * (2 * dk + dv), per = (long)heads * dk * dv;
+#define VOB_HS(TT)                                                                                                            \
+  return run_matrix_scan<TT>(HgrnSource<TT>{(const TT*)qfv, width, (const TT*)bf, lower, heads, dk, dv}, nw, state, per, cu_q, \
+                             state_slots, out, raw, scratch, T, B, chunks, heads, dk, dv, eps, num_slots, fuse, 1, err, stream)
+  if (dtype == VOB_F32) { VOB_HS(float); }
+  if (dtype == VOB_BF16) { VOB_HS(__nv_bfloat16); }
+#undef VOB_HS
+  return VOB_BAD_ARGUMENT;
+}
+
+// rows: `width` elements a token, q | k | v first, the decay's pre-activations (heads*dk) at z_off, the output gate (heads*dv)
+// at gate_off; bias float [heads*dk]; nw float [dv]; state float [num_slots, state_stride], the heads' matrices first; out
+// [T, heads*dv] of `dtype` with `fuse` (norm and gate included), else raw float [T, heads*dv] and nothing behind it.
+VOB_API int vob_gla_scan(const void* rows, long width, int z_off, int gate_off, const float* bias, const float* nw, float* state,
+                         long state_stride, const int* cu_q, const int* state_slots, void* out, float* raw, float* scratch, int T,
+                         int B, int chunks, int heads, int dk, int dv, float scale, float inv_tau, float eps, int num_slots,
+                         int fuse, int dtype, int* err, cudaStream_t stream) {
+  if (B <= 0 || T <= 0) return 0;
+#define VOB_GS(TT)                                                                                                             \
+  return run_matrix_scan<TT>(GlaSource<TT>{(const TT*)rows, width, bias, heads, dk, dv, z_off, gate_off, scale, inv_tau}, nw,  \
+                             state, state_stride, cu_q, state_slots, out, raw, scratch, T, B, chunks, heads, dk, dv, eps,      \
+                             num_slots, fuse, 0, err, stream)
+  if (dtype == VOB_F32) { VOB_GS(float); }
+  if (dtype == VOB_BF16) { VOB_GS(__nv_bfloat16); }
+#undef VOB_GS
+  return VOB_BAD_ARGUMENT;
+}
+
+// rows: `width` elements a token, q | k | v first; decays float [heads]; raw float [T, heads*dv].
+VOB_API int vob_lightning_scan(const void* rows, long width, const float* decays, float* state, long state_stride, const int* cu_q,
+                               const int* state_slots, float* raw, float* scratch, int T, int B, int chunks, int heads, int dk,
+                               int dv, int num_slots, int dtype, int* err, cudaStream_t stream) {
+  if (B <= 0 || T <= 0) return 0;
+#define VOB_LS(TT)                                                                                                          \
+  return run_matrix_scan<TT>(LightningSource<TT>{(const TT*)rows, width, decays, heads, dk, dv}, (const float*)nullptr,     \
+                             state, state_stride, cu_q, state_slots, nullptr, raw, scratch, T, B, chunks, heads, dk, dv, 0.f, \
+                             num_slots, 0, 0, err, stream)
+  if (dtype == VOB_F32) { VOB_LS(float); }
+  if (dtype == VOB_BF16) { VOB_LS(__nv_bfloat16); }
+#undef VOB_LS
+  return VOB_BAD_ARGUMENT;
+}
+
+// u and out [T, W] of `dtype`; gates float [T, blocks, 2, W / blocks]; y rows of y_stride elements of `dtype`; br, bi, lam, by
+// float [W]; state float [num_slots, state_stride], the W channels first.  `chunks`: 1, 8 or 32 ranges a request's tokens are
+// cut into.
+VOB_API int vob_lru_scan(const void* u, const float* gates, const void* y, long y_stride, const float* br, const float* bi,
+                         const float* lam, const float* by, float* state, long state_stride, const int* cu_q,
+                         const int* state_slots, void* out, int B, int W, int blocks, int num_slots, int chunks, int dtype, int* err,
+                         cudaStream_t stream) {
+  if (B <= 0 || W <= 0) return 0;
+  if (B > 65535 || blocks <= 0 || W % blocks || state_stride < W || (chunks != 1 && chunks != 8 && chunks != 32)) return VOB_UNSUPPORTED;
+  dim3 grid((W + 31) / 32, B), block(32, chunks);
+#define VOB_LRU(TT, NN)                                                                                                        \
+  return launch_kernel(lru_scan_kernel<TT, NN>, grid, block, 0, stream, (const TT*)u, gates, (const TT*)y, y_stride, br, bi, lam, \
+                       by, state, state_stride, cu_q, state_slots, (TT*)out, W, W / blocks, num_slots, err)
+  if (dtype == VOB_F32) {
+    if (chunks == 1) VOB_LRU(float, 1);
+    if (chunks == 8) VOB_LRU(float, 8);
+    VOB_LRU(float, 32);
+  }
+  if (dtype == VOB_BF16) {
+    if (chunks == 1) VOB_LRU(__nv_bfloat16, 1);
+    if (chunks == 8) VOB_LRU(__nv_bfloat16, 8);
+    VOB_LRU(__nv_bfloat16, 32);
+  }
+#undef VOB_LRU
   return VOB_BAD_ARGUMENT;
 }

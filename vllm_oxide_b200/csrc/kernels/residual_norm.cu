@@ -12,6 +12,14 @@
 // With a list of rows, (5) is computed for those source rows only and nothing is stored (the model's last norm on the
 // rows whose logits are wanted).
 //
+// A second kernel, residual_norm_shift_step, is the same chain (without `inject` and `keep`) followed by a token shift, for
+// layers whose mixer reads a mix of a token's normed row and the row of the token before it:
+//     h_t = RMSNorm(x_t) * w_pre;   out_t = h_t + (h_(t-1) - h_t) * shift          (shift: a number a channel)
+// with h_(-1) of a portion from the request's state slot (zeros for a new request), where the portion's last h is left.
+// A block walks a few tokens and keeps the last h on chip; the h of the token before its first, and (in the block of a
+// portion's first token) the h of the portion's last token, are made again from the rows they come from, so that no block
+// waits for another.  For that the new stream goes to a buffer of its own (stream_out) while all blocks read the old one.
+//
 // The stream, the norms and the sums are float on both paths; y and out are of the model's type T.  A block of fixed
 // size takes a row, so the order of additions in a sum of squares depends on the row's width only.
 #include "common.cuh"
@@ -126,6 +134,100 @@ residual_norm_step_kernel(float* stream, const T* y, const float* __restrict__ w
   }
 }
 
+// The normed row of token t, left in `row` as x (the caller multiplies by the returned 1 / rms); with `put` the new stream
+// row is stored.
+template <typename T, int V>
+__device__ __forceinline__ float shift_row(const float* stream, float* stream_out, const T* y, const float* __restrict__ w_post,
+                                           float* row, int t, bool put, int D, float eps, float* scratch) {
+  const size_t base = (size_t)t * D;
+  float inv_y = 1.f;
+  if (y) {
+    float ss = 0.f;
+    for (int d = threadIdx.x * V; d < D; d += RN_NT * V) {
+      float v[V];
+      RowAccess<T, V>::load(y + base + d, v);
+#pragma unroll
+      for (int j = 0; j < V; ++j) { row[d + j] = v[j]; ss = fmaf(v[j], v[j], ss); }
+    }
+    if (w_post) inv_y = 1.f / sqrtf(block_sum<RN_NT>(ss, scratch) / (float)D + eps);
+  }
+  float ss = 0.f;
+  for (int d = threadIdx.x * V; d < D; d += RN_NT * V) {
+    float x[V];
+    RowAccess<float, V>::load(stream + base + d, x);
+    if (y) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] += w_post ? row[d + j] * inv_y * w_post[d + j] : row[d + j];
+      if (put) RowAccess<float, V>::store(stream_out + base + d, x);
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) { row[d + j] = x[j]; ss = fmaf(x[j], x[j], ss); }
+  }
+  return 1.f / sqrtf(block_sum<RN_NT>(ss, scratch) / (float)D + eps);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(RN_NT)
+residual_norm_shift_kernel(const float* stream, float* stream_out, const T* y, const float* __restrict__ w_post,
+                           const float* __restrict__ w_pre, const float* __restrict__ shift, float* state, long state_stride,
+                           const int* __restrict__ token_req, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
+                           T* out, int num_tokens, int walk, int D, float eps, long num_slots, int* err) {
+  extern __shared__ float4 rn_smem4[];
+  float* row = reinterpret_cast<float*>(rn_smem4);    // [D] the token's stream row
+  float* before = row + D;                             // [D] h of the token before
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  bool have = false;                                   // `before` is that of the token at hand
+  for (int k = 0; k < walk; ++k) {
+    const int t = blockIdx.x * walk + k;
+    if (t >= num_tokens) break;
+    const int req = token_req[t];
+    int slot = -1, first = t, last = t;
+    if (req >= 0) {
+      slot = state_slots[req];
+      first = cu_q[req];
+      last = cu_q[req + 1] - 1;
+      if (slot < 0 || slot >= num_slots) {
+        if (threadIdx.x == 0) atomicOr(err, VOB_ERR_SLOT);
+        slot = -1;
+      }
+    }
+    float* kept = slot >= 0 ? state + (size_t)slot * state_stride : nullptr;
+    // (a thread reads and writes the same elements of `row` and `before` in every pass)
+    if (t == first) {
+      for (int d = threadIdx.x * V; d < D; d += RN_NT * V)
+#pragma unroll
+        for (int j = 0; j < V; ++j) before[d + j] = kept ? kept[d + j] : 0.f;
+    } else if (!have) {
+      const float inv = shift_row<T, V>(stream, stream_out, y, w_post, row, t - 1, false, D, eps, scratch);
+      for (int d = threadIdx.x * V; d < D; d += RN_NT * V)
+#pragma unroll
+        for (int j = 0; j < V; ++j) before[d + j] = row[d + j] * inv * w_pre[d + j];
+    }
+    const float inv = shift_row<T, V>(stream, stream_out, y, w_post, row, t, true, D, eps, scratch);
+    for (int d = threadIdx.x * V; d < D; d += RN_NT * V) {
+      float o[V];
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        const float h = row[d + j] * inv * w_pre[d + j];
+        o[j] = req >= 0 ? fmaf(before[d + j] - h, shift[d + j], h) : h;
+        before[d + j] = h;
+        if (kept && t == last && t == first) kept[d + j] = h;
+      }
+      RowAccess<T, V>::store(out + (size_t)t * D + d, o);
+    }
+    have = true;
+    if (kept && t == first && last > first) {
+      // the portion's last h into the slot: by the block that has just read the slot, so that nothing is overwritten early
+      const float inv_last = shift_row<T, V>(stream, stream_out, y, w_post, row, last, false, D, eps, scratch);
+      for (int d = threadIdx.x * V; d < D; d += RN_NT * V)
+#pragma unroll
+        for (int j = 0; j < V; ++j) kept[d + j] = row[d + j] * inv_last * w_pre[d + j];
+    }
+  }
+}
+
 }  // namespace vob
 
 using namespace vob;
@@ -158,5 +260,40 @@ VOB_API int vob_residual_norm_step(float* stream, const void* y, const float* w_
     VOB_RN_LAUNCH(__nv_bfloat16, 1);
   }
 #undef VOB_RN_LAUNCH
+  return VOB_BAD_ARGUMENT;
+}
+
+// stream [T, D] float, as the sublayer before found it; y [T, D] of `dtype` (null: the stream does not change and stream_out is
+// not written) and w_post as above; stream_out [T, D] float, another buffer than `stream`; w_pre, shift [D] float; state float
+// [num_slots, state_stride]: the last h of every request, D numbers; out [T, D] of `dtype`.
+VOB_API int vob_residual_norm_shift_step(const float* stream, float* stream_out, const void* y, const float* w_post, const float* w_pre,
+                                         const float* shift, float* state, long state_stride, const int* token_req,
+                                         const int* cu_q, const int* state_slots, void* out, int T, int D, float eps,
+                                         long num_slots, int dtype, int* err, cudaStream_t stream_) {
+  if (T <= 0) return 0;
+  if (D <= 0 || !w_pre || !shift || !state || !out || state_stride < D || (y && (!stream_out || stream_out == stream)))
+    return VOB_BAD_ARGUMENT;
+  const size_t smem = (size_t)2 * D * sizeof(float);
+  if (smem > 200 * 1024) return VOB_UNSUPPORTED;
+  const bool vec = D % 4 == 0 && (((uintptr_t)stream | (uintptr_t)stream_out | (uintptr_t)y | (uintptr_t)out) % 16) == 0;
+  // a block makes one row more than it walks: few tokens a block while they fill the device, up to eight beyond
+  const int walk = max(1, min(8, T / (4 * sm_count())));
+#define VOB_RS_LAUNCH(TYPE, V)                                                                                             \
+  do {                                                                                                                     \
+    if (smem > 48 * 1024)                                                                                                  \
+      cudaFuncSetAttribute(residual_norm_shift_kernel<TYPE, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
+    return launch_kernel(residual_norm_shift_kernel<TYPE, V>, dim3((T + walk - 1) / walk), RN_NT, smem, stream_, stream,   \
+                         stream_out, (const TYPE*)y, w_post, w_pre, shift, state, state_stride, token_req, cu_q,           \
+                         state_slots, (TYPE*)out, T, walk, D, eps, num_slots, err);                                        \
+  } while (0)
+  if (dtype == VOB_F32) {
+    if (vec) VOB_RS_LAUNCH(float, 4);
+    VOB_RS_LAUNCH(float, 1);
+  }
+  if (dtype == VOB_BF16) {
+    if (vec) VOB_RS_LAUNCH(__nv_bfloat16, 4);
+    VOB_RS_LAUNCH(__nv_bfloat16, 1);
+  }
+#undef VOB_RS_LAUNCH
   return VOB_BAD_ARGUMENT;
 }

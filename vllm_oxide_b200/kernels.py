@@ -173,12 +173,13 @@ def add_rmsnorm(x, residual, weight, y, eps: float, has_residual: bool, err, row
            "add_rmsnorm")
 
 
-def silu_mul(gate_up, out, num_tokens: int, interleaved: bool = False) -> None:
-    """out = SiLU(gate) * up; gate_up holds [gate | up] per token, or, interleaved, groups of 8 gate + 8 up columns."""
+def silu_mul(gate_up, out, num_tokens: int, interleaved: bool = False, gelu: bool = False) -> None:
+    """out = SiLU(gate) * up; gate_up holds [gate | up] per token, or, interleaved, groups of 8 gate + 8 up columns.  `gelu`:
+    the tanh form of gelu in place of SiLU."""
     _cuda(gate_up, out)
     I = out.shape[-1]
-    _check(lib().vob_silu_mul(_p(gate_up), _p(out), num_tokens, I, int(interleaved), _code(out.dtype), _stream()),
-           "silu_mul")
+    _check(lib().vob_silu_mul(_p(gate_up), _p(out), num_tokens, I, int(interleaved), int(bool(gelu)), _code(out.dtype),
+                              _stream()), "gelu_mul" if gelu else "silu_mul")
 
 
 def qk_norm_rope_kv_write(qkv, bias, positions, slots, wq, wk, rule, kcache, vcache, num_tokens, nh, kvh, hd,
@@ -202,6 +203,15 @@ def qk_norm_rope_kv_write(qkv, bias, positions, slots, wq, wk, rule, kcache, vca
            "qk_norm_rope_kv_write")
 
 
+def _sinks(sink, nh: int):
+    """(flag, pointer) of a softmax's sink: False, True (an entry of score 0) or a float tensor [nh] (a score a head)."""
+    if isinstance(sink, torch.Tensor):
+        _cuda(sink)
+        assert sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh
+        return 0, _p(sink)
+    return int(bool(sink)), _p(None)
+
+
 def paged_attention_generic(q, q_stride, out, kcache, vcache, block_tables, token_req, positions, num_tokens, nh, kvh,
                             hd, window: int, scale: float, err, skip_single_cu_q=None, value_dim: Optional[int] = None,
                             sink: bool = False, gate=None, gate_stride: int = 0, softcap: float = 0.0, chunk: int = 0,
@@ -216,8 +226,9 @@ def paged_attention_generic(q, q_stride, out, kcache, vcache, block_tables, toke
     tanh(score / softcap); `chunk` > 0: a query sees only keys of its own block of `chunk` positions; a float32 `out`
     beside bfloat16 inputs is stored unrounded.  `keep_first` > 0: the keys at positions below it are seen by every later
     query, whatever the window; `dist_bias` (float [nh, rows]): dist_bias[h, min(query position - key position, rows - 1)]
-    is added to head h's scaled score."""
+    is added to head h's scaled score.  `sink` may be a float tensor [nh]: the extra entry's score is then the head's own."""
     _cuda(q, out, kcache, vcache, block_tables, token_req, positions, gate, dist_bias)
+    sink, sinks = _sinks(sink, nh)
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.is_contiguous() and dist_bias.shape[0] == nh)
     assert gate is None or gate.dtype == q.dtype
     own_shape = vcache.shape[1] != kcache.shape[1] or vcache.shape[3] != kcache.shape[3]
@@ -230,7 +241,7 @@ def paged_attention_generic(q, q_stride, out, kcache, vcache, block_tables, toke
                                              _p(block_tables), block_tables.shape[-1], _p(token_req), _p(positions),
                                              _p(skip_single_cu_q), num_tokens, nh, kvh, hd,
                                              hd if value_dim is None else int(value_dim), kcache.shape[2], window,
-                                             ctypes.c_float(scale), ctypes.c_long(kcache.shape[0]), int(bool(sink)), _p(gate),
+                                             ctypes.c_float(scale), ctypes.c_long(kcache.shape[0]), sink, sinks, _p(gate),
                                              ctypes.c_long(gate_stride), vcache.shape[1], vcache.shape[3],
                                              ctypes.c_float(softcap), int(chunk), int(out.dtype != q.dtype), int(keep_first),
                                              _p(dist_bias), 0 if dist_bias is None else dist_bias.shape[1], _code(q.dtype),
@@ -325,12 +336,14 @@ def rms_norm_step(stream, eps: float, err, y1=None, y2=None, w=None, out=None, r
                                    _stream()), "rms_norm_step")
 
 
-def pair_norm_mean(a, b, wa, wb, out, eps: float) -> None:
-    """out = (a / rms(a) * wa + b / rms(b) * wb) / 2, row by row (float sums; a, b, out of one type, wa and wb float)."""
-    _cuda(a, b, wa, wb, out)
+def pair_norm_mean(a, b, wa, wb, out, eps: float, bias_a=None) -> None:
+    """out = (a / rms(a) * wa + b / rms(b) * wb) / 2, row by row (float sums; a, b, out of one type, wa and wb float);
+    `bias_a` (float): added to a's rows first."""
+    _cuda(a, b, wa, wb, out, bias_a)
+    assert bias_a is None or (bias_a.dtype == torch.float32 and bias_a.is_contiguous() and bias_a.numel() == a.shape[1])
     assert a.dtype == b.dtype == out.dtype and a.is_contiguous() and b.is_contiguous() and out.is_contiguous()
     assert a.shape == b.shape == out.shape and wa.dtype == wb.dtype == torch.float32
-    _check(lib().vob_pair_norm_mean(_p(a), _p(b), _p(wa), _p(wb), _p(out), a.shape[0], a.shape[1], ctypes.c_float(eps),
+    _check(lib().vob_pair_norm_mean(_p(a), _p(b), _p(bias_a), _p(wa), _p(wb), _p(out), a.shape[0], a.shape[1], ctypes.c_float(eps),
                                     _code(a.dtype), _stream()), "pair_norm_mean")
 
 
@@ -406,40 +419,48 @@ def residual_norm_step(stream, eps: float, err, y=None, w_post=None, inject=None
 
 
 def short_conv_silu(x, channels: int, taps_w, state, conv_off: int, token_req, cu_q, state_slots, out, num_tokens: int, err,
-                    activation: bool = True) -> None:
-    """out[t, c] = SiLU(sum_j taps_w[c, j] * x[t - (taps - 1) + j, c]) over every request's tokens of this step (float out
-    [tokens, channels]); the inputs before a portion's start come from the request's slot: state [slots, n] float, the
-    last taps - 1 inputs of every channel at conv_off.  x: the first `channels` columns of its rows.  `activation` False:
-    the filter's output as it is.  `state` may be columns of a wider tensor."""
-    _cuda(x, taps_w, state, token_req, cu_q, state_slots, out)
-    assert x.stride(1) == 1 and taps_w.dtype == torch.float32 and taps_w.is_contiguous() and taps_w.shape[0] == channels
-    assert state.dtype == torch.float32 and state.stride(1) == 1 and out.dtype == torch.float32 and out.is_contiguous()
-    _check(lib().vob_short_conv_silu(_p(x), ctypes.c_long(x.stride(0)), _p(taps_w), _p(state), ctypes.c_long(state.stride(0)),
-                                     ctypes.c_long(conv_off), _p(token_req), _p(cu_q), _p(state_slots), _p(out), num_tokens,
-                                     channels, taps_w.shape[1], ctypes.c_long(state.shape[0]), int(bool(activation)),
+                    activation: bool = True, bias_in=None, bias_out=None) -> None:
+    """out[t, c] = SiLU(sum_j taps_w[c, j] * x[t - (taps - 1) + j, c]) over every request's tokens of this step (out
+    [tokens, channels], float or of x's type); the inputs before a portion's start come from the request's slot: state [slots, n]
+    float, the last taps - 1 inputs of every channel at conv_off.  x: the first `channels` columns of its rows.  `activation`
+    False: the filter's output as it is.  `state` may be columns of a wider tensor.  `bias_in` (float [channels]): the filter's
+    inputs are x + bias_in (zeros before the sequence's start stay zeros); `bias_out`: added behind the filter."""
+    _cuda(x, taps_w, state, token_req, cu_q, state_slots, out, bias_in, bias_out)
+    _check_conv(x, channels, taps_w, state, out, bias_in, bias_out)
+    _check(lib().vob_short_conv_silu(_p(x), ctypes.c_long(x.stride(0)), _p(taps_w), _p(bias_in), _p(bias_out), _p(state),
+                                     ctypes.c_long(state.stride(0)), ctypes.c_long(conv_off), _p(token_req), _p(cu_q),
+                                     _p(state_slots), _p(out), num_tokens, channels, taps_w.shape[1],
+                                     ctypes.c_long(state.shape[0]), int(bool(activation)), int(out.dtype == torch.float32),
                                      _code(x.dtype), _p(err), _stream()), "short_conv_silu")
 
 
-def short_conv_state(x, channels: int, taps: int, state, conv_off: int, cu_q, state_slots, num_requests: int) -> None:
+def _check_conv(x, channels, taps_w, state, out, bias_in, bias_out) -> None:
+    assert x.stride(1) == 1 and taps_w.dtype == torch.float32 and taps_w.is_contiguous() and taps_w.shape[0] == channels
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and out.dtype in (torch.float32, x.dtype) and out.is_contiguous()
+    for b in (bias_in, bias_out):
+        assert b is None or (b.dtype == torch.float32 and b.is_contiguous() and b.numel() == channels)
+
+
+def short_conv_state(x, channels: int, taps: int, state, conv_off: int, cu_q, state_slots, num_requests: int, bias_in=None) -> None:
     """Leaves in every request's slot the last taps - 1 inputs of every channel after this step's portion (from the
-    portion, and from what the slot held where the portion is shorter).  Run after short_conv_silu."""
-    _cuda(x, state, cu_q, state_slots)
-    _check(lib().vob_short_conv_state(_p(x), ctypes.c_long(x.stride(0)), _p(state), ctypes.c_long(state.stride(0)),
+    portion, and from what the slot held where the portion is shorter).  Run after short_conv_silu, with its `bias_in`."""
+    _cuda(x, state, cu_q, state_slots, bias_in)
+    _check(lib().vob_short_conv_state(_p(x), ctypes.c_long(x.stride(0)), _p(bias_in), _p(state), ctypes.c_long(state.stride(0)),
                                       ctypes.c_long(conv_off), _p(cu_q), _p(state_slots), num_requests, channels, taps,
                                       ctypes.c_long(state.shape[0]), _code(x.dtype), _stream()), "short_conv_state")
 
 
 def short_conv_step(x, channels: int, taps_w, state, conv_off: int, cu_q, state_slots, out, num_requests: int, err,
-                    activation: bool = True) -> None:
+                    activation: bool = True, bias_in=None, bias_out=None) -> None:
     """short_conv_silu and short_conv_state in one launch, a thread a (request, channel): for steps whose portions are
     short (decoding).  Same numbers."""
-    _cuda(x, taps_w, state, cu_q, state_slots, out)
-    assert x.stride(1) == 1 and taps_w.dtype == torch.float32 and taps_w.is_contiguous() and taps_w.shape[0] == channels
-    assert state.dtype == torch.float32 and state.stride(1) == 1 and out.dtype == torch.float32 and out.is_contiguous()
-    _check(lib().vob_short_conv_step(_p(x), ctypes.c_long(x.stride(0)), _p(taps_w), _p(state), ctypes.c_long(state.stride(0)),
-                                     ctypes.c_long(conv_off), _p(cu_q), _p(state_slots), _p(out), num_requests, channels,
-                                     taps_w.shape[1], ctypes.c_long(state.shape[0]), int(bool(activation)), _code(x.dtype),
-                                     _p(err), _stream()), "short_conv_step")
+    _cuda(x, taps_w, state, cu_q, state_slots, out, bias_in, bias_out)
+    _check_conv(x, channels, taps_w, state, out, bias_in, bias_out)
+    _check(lib().vob_short_conv_step(_p(x), ctypes.c_long(x.stride(0)), _p(taps_w), _p(bias_in), _p(bias_out), _p(state),
+                                     ctypes.c_long(state.stride(0)), ctypes.c_long(conv_off), _p(cu_q), _p(state_slots), _p(out),
+                                     num_requests, channels, taps_w.shape[1], ctypes.c_long(state.shape[0]),
+                                     int(bool(activation)), int(out.dtype == torch.float32), _code(x.dtype), _p(err), _stream()),
+           "short_conv_step")
 
 
 def delta_scan(qkv, ab, b_off: int, a_off: int, A_log, dt_bias, state, cu_q, state_slots, raw, num_requests: int, heads: int,
@@ -575,11 +596,13 @@ def moe_gemv(a, w, c, ids, order, n: int, top: int, relu_squared: bool, silu_pai
                               ctypes.c_float(glu_limit), _stream()), "moe_gemv")
 
 
-def moe_combine(y, slot_of, weights, out, num_tokens: int, top: int) -> None:
-    """out[t] = sum_j weights[t, j] * y[slot_of[t, j]] (float, j in order); slot_of None: pair (t, j) is row t * top + j."""
-    _cuda(y, slot_of, weights, out)
+def moe_combine(y, slot_of, weights, out, num_tokens: int, top: int, add=None) -> None:
+    """out[t] = sum_j weights[t, j] * y[slot_of[t, j]] (float, j in order); slot_of None: pair (t, j) is row t * top + j.
+    `add` (like out): added to the sum before it is rounded."""
+    _cuda(y, slot_of, weights, out, add)
+    assert add is None or (add.dtype == out.dtype and add.shape == out.shape and add.is_contiguous())
     assert y.dtype == torch.float32 and y.is_contiguous() and out.is_contiguous()
-    _check(lib().vob_moe_combine(_p(y), _p(slot_of), _p(weights), _p(out), num_tokens, out.shape[1], top, _code(out.dtype),
+    _check(lib().vob_moe_combine(_p(y), _p(slot_of), _p(weights), _p(add), _p(out), num_tokens, out.shape[1], top, _code(out.dtype),
                                  _stream()), "moe_combine")
 
 
@@ -616,6 +639,122 @@ def stream_sum(streams, sums, num_streams: int, width: int) -> None:
     _cuda(streams, sums)
     assert streams.dtype == sums.dtype == torch.float32 and streams.is_contiguous() and sums.is_contiguous()
     _check(lib().vob_stream_sum(_p(streams), _p(sums), sums.shape[0], num_streams, width, _stream()), "stream_sum")
+
+
+def residual_norm_shift_step(stream, stream_out, eps: float, err, y, w_post, w_pre, shift, state, token_req, cu_q, state_slots,
+                             out) -> None:
+    """residual_norm_step (stream in, stream_out another buffer; y None: the stream stays and stream_out is not written) with a
+    token shift behind its norm: h = RMSNorm(x) * w_pre, out[t] = h[t] + (h[t - 1] - h[t]) * shift, the h before a portion's
+    first token from the request's slot (state float [slots, >= width], rows as wide as they may be), its last h left there."""
+    _cuda(stream, stream_out, y, w_post, w_pre, shift, state, token_req, cu_q, state_slots, out)
+    assert stream.dtype == torch.float32 and stream.is_contiguous() and (y is None or stream_out.is_contiguous())
+    for t in (w_post, w_pre, shift):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == stream.shape[1])
+    for t in (y, out):
+        assert t is None or (t.dtype == out.dtype and t.is_contiguous() and t.shape == stream.shape)
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= stream.shape[1]
+    _check(lib().vob_residual_norm_shift_step(_p(stream), _p(stream_out), _p(y), _p(w_post), _p(w_pre), _p(shift), _p(state),
+                                              ctypes.c_long(state.stride(0)), _p(token_req), _p(cu_q), _p(state_slots), _p(out),
+                                              stream.shape[0], stream.shape[1], ctypes.c_float(eps),
+                                              ctypes.c_long(state.shape[0]), _code(out.dtype), _p(err), _stream()),
+           "residual_norm_shift_step")
+
+
+def pair_embedding(table, pairs, ids, positions, token_req, cu_q, state_slots, state, x, num_tokens: int, buckets: int,
+                   mul_prev: int, mul_cur: int, err) -> None:
+    """x[t] (float) = table[ids[t]] + pairs[(ids[t - 1] * mul_prev + ids[t] * mul_cur) % buckets]; a sequence's first token
+    reads row `buckets`.  The token before a portion comes from the request's slot (state int32 [slots, n]), where the portion's
+    last token is left.  `pairs` None: the token's row alone."""
+    _cuda(table, pairs, ids, positions, token_req, cu_q, state_slots, state, x)
+    assert x.dtype == torch.float32 and x.is_contiguous() and table.is_contiguous() and x.shape[1] == table.shape[1]
+    if pairs is not None:
+        assert pairs.is_contiguous() and pairs.dtype == table.dtype and tuple(pairs.shape) == (buckets + 1, table.shape[1])
+        assert state.dtype == torch.int32 and state.stride(1) == 1
+    _check(lib().vob_pair_embedding(_p(table), _p(pairs), _p(ids), _p(positions), _p(token_req), _p(cu_q), _p(state_slots),
+                                    _p(state), ctypes.c_long(state.stride(0) if state is not None else 0), _p(x), num_tokens,
+                                    table.shape[1], table.shape[0], ctypes.c_long(buckets), ctypes.c_long(mul_prev),
+                                    ctypes.c_long(mul_cur), ctypes.c_long(state.shape[0] if state is not None else 0),
+                                    _code(table.dtype), _p(err), _stream()), "pair_embedding")
+
+
+def headnorm_rope_kv_write(qkv, bias, positions, slots, wq, wk, rule, kcache, vcache, num_tokens: int, nh: int, kvh: int, kd: int,
+                           eps: float, v_norm: bool, write_kv: bool, err, kd_norm: Optional[int] = None,
+                           vd_norm: Optional[int] = None) -> None:
+    """A merged q|k|v row with biases (float, or None), an RMS norm over every q and k head (gains wq, wk float [kd], shared by
+    the heads; both or neither), a rotation of the front of every q and k head by computed angles and the rule's amplitude, and
+    (v_norm) every value head divided by its root mean square: q back in place, k and v to the planes.  `kd_norm`, `vd_norm`: how
+    many elements of a head count in the means (heads padded with zeros)."""
+    _cuda(qkv, bias, positions, slots, wq, wk, rule.frequencies, kcache, vcache)
+    if rule.rotary_dim > 0 and rule.frequencies is None:
+        raise KernelError("headnorm_rope_kv_write turns by computed angles: the rule needs `frequencies`")
+    assert qkv.stride(1) == 1 and kcache.dtype == qkv.dtype == vcache.dtype and tuple(kcache.shape[1::2]) == (kvh, kd)
+    assert kcache.shape[0] == vcache.shape[0] and kcache.shape[2] == vcache.shape[2] and kcache.is_contiguous() and vcache.is_contiguous()
+    vh, vd = vcache.shape[1], vcache.shape[3]
+    for w, n in ((bias, (nh + kvh) * kd + vh * vd), (wq, kd), (wk, kd)):
+        assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == n)
+    _check(lib().vob_headnorm_rope_kv_write(_p(qkv), ctypes.c_long(qkv.stride(0)), _p(bias), _p(positions), _p(slots), _p(wq), _p(wk),
+                                            _p(rule.frequencies), ctypes.c_float(rule.amplitude), _p(kcache), _p(vcache),
+                                            num_tokens, nh, kvh, kd, vh, vd, int(kd_norm or kd), int(vd_norm or vd),
+                                            rule.rotary_dim, int(rule.interleaved), int(bool(v_norm)), ctypes.c_float(eps),
+                                            ctypes.c_long(kcache.shape[0] * kcache.shape[2]), kcache.shape[2], int(write_kv),
+                                            _code(qkv.dtype), _p(err), _stream()), "headnorm_rope_kv_write")
+
+
+def _scan_scratch_ok(chunks: int, raw, scratch, num_requests: int, heads: int, dk: int, dv: int) -> bool:
+    return chunks == 1 or (raw is not None and scratch is not None and scratch.dtype == torch.float32
+                           and scratch.numel() >= num_requests * chunks * heads * dk * (dv + 1))
+
+
+def gla_scan(rows, z_off: int, gate_off: int, bias, norm_weight, state, cu_q, state_slots, num_requests: int, heads: int, dk: int,
+             dv: int, scale: float, tau: float, eps: float, err, out=None, raw=None, chunks: int = 1, scratch=None) -> None:
+    """Gated linear attention, M = diag(f) M + k v^T, o = M^T (scale q), f = sigmoid(z + bias)^(1 / tau), over every request's
+    tokens of this step, from and to its slot (state float [slots, n], the heads' [dk, dv] matrices first).  rows: q | k | v
+    (heads * dk, heads * dk, heads * dv) first, z (heads * dk) at z_off, the output gate (heads * dv) at gate_off.  With `out`
+    one block a (request, head) does it all, the head's RMS norm (norm_weight float [dv]) and the product with SiLU(gate)
+    included (hgrn2_can_fuse); with `raw` (float [tokens, heads * dv]) the bare o.  `chunks`, `scratch`: as hgrn2_scan."""
+    _cuda(rows, bias, norm_weight, state, cu_q, state_slots, out, raw)
+    T = (raw if out is None else out).shape[0]
+    assert rows.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * dk * dv
+    assert bias.dtype == torch.float32 and bias.numel() == heads * dk and norm_weight.dtype == torch.float32
+    assert (out is None) != (raw is None) and (out is None or (out.dtype == rows.dtype and out.is_contiguous()))
+    assert raw is None or (raw.dtype == torch.float32 and raw.is_contiguous())
+    assert _scan_scratch_ok(chunks, raw, scratch, num_requests, heads, dk, dv)
+    _check(lib().vob_gla_scan(_p(rows), ctypes.c_long(rows.stride(0)), z_off, gate_off, _p(bias), _p(norm_weight), _p(state),
+                              ctypes.c_long(state.stride(0)), _p(cu_q), _p(state_slots), _p(out), _p(raw), _p(scratch), T,
+                              num_requests, int(chunks), heads, dk, dv, ctypes.c_float(scale), ctypes.c_float(1.0 / tau),
+                              ctypes.c_float(eps), state.shape[0], int(out is not None), _code(rows.dtype), _p(err), _stream()),
+           "gla_scan")
+
+
+def lightning_scan(rows, decays, state, cu_q, state_slots, raw, num_requests: int, heads: int, dk: int, dv: int, err,
+                   chunks: int = 1, scratch=None) -> None:
+    """M = decay_h M + silu(k) silu(v)^T, o = M^T silu(q) into `raw` (float [tokens, heads * dv]); rows, state, chunks and scratch
+    as gla_scan, decays float [heads]."""
+    _cuda(rows, decays, state, cu_q, state_slots, raw)
+    assert rows.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * dk * dv
+    assert decays.dtype == torch.float32 and decays.numel() == heads and raw.dtype == torch.float32 and raw.is_contiguous()
+    assert _scan_scratch_ok(chunks, raw, scratch, num_requests, heads, dk, dv)
+    _check(lib().vob_lightning_scan(_p(rows), ctypes.c_long(rows.stride(0)), _p(decays), _p(state), ctypes.c_long(state.stride(0)),
+                                    _p(cu_q), _p(state_slots), _p(raw), _p(scratch), raw.shape[0], num_requests, int(chunks), heads,
+                                    dk, dv, state.shape[0], _code(rows.dtype), _p(err), _stream()), "lightning_scan")
+
+
+def lru_scan(u, gates, y, bias_r, bias_i, lam, bias_y, state, cu_q, state_slots, out, num_requests: int, blocks: int, err,
+             chunks: int = 1) -> None:
+    """S = a S + sqrt(1 - a^2) i u, out = S * gelu(y + bias_y), with r = sigmoid(r + bias_r), i = sigmoid(i + bias_i),
+    a = exp(-8 r softplus(lam)), over every request's tokens of this step, from and to its slot (state float [slots, n], the
+    width's channels first).  u, out [tokens, width]; gates float [tokens, blocks, 2, width / blocks] (r, then i, of every block);
+    y: the first `width` columns of its rows.  `chunks`: as mingru_scan."""
+    _cuda(u, gates, y, bias_r, bias_i, lam, bias_y, state, cu_q, state_slots, out)
+    W = out.shape[1]
+    assert u.is_contiguous() and out.is_contiguous() and u.shape == out.shape and u.dtype == y.dtype == out.dtype and y.stride(1) == 1
+    assert gates.dtype == torch.float32 and gates.is_contiguous() and gates.numel() == u.shape[0] * 2 * W
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= W
+    for b in (bias_r, bias_i, lam, bias_y):
+        assert b.dtype == torch.float32 and b.is_contiguous() and b.numel() == W
+    _check(lib().vob_lru_scan(_p(u), _p(gates), _p(y), ctypes.c_long(y.stride(0)), _p(bias_r), _p(bias_i), _p(lam), _p(bias_y),
+                              _p(state), ctypes.c_long(state.stride(0)), _p(cu_q), _p(state_slots), _p(out), num_requests, W, blocks,
+                              state.shape[0], int(chunks), _code(out.dtype), _p(err), _stream()), "lru_scan")
 
 
 def scan_chunks(num_tokens: int, num_requests: int) -> int:
@@ -696,13 +835,13 @@ def latent_query_rotate(q, qa, rule, positions, num_tokens: int, heads: int, dk:
 
 def head_linear(x, x_token_stride: int, x_head_stride: int, w, y, y_token_stride: int, y_head_stride: int, num_tokens: int) -> None:
     """y[t, h, :O] = sum_i w[h, i, :] * x[t, h, i] for per-head matrices w [heads, I, O]; x and y are addressed by token
-    and head strides (elements), so either may be a slice of wider rows."""
+    and head strides (elements), so either may be a slice of wider rows.  A float32 y takes bfloat16 products unrounded."""
     _cuda(x, w, y)
-    assert w.is_contiguous() and w.dim() == 3 and x.dtype == w.dtype == y.dtype
+    assert w.is_contiguous() and w.dim() == 3 and x.dtype == w.dtype and y.dtype in (x.dtype, torch.float32)
     heads, I, O = w.shape
     _check(lib().vob_head_linear(_p(x), ctypes.c_long(x_token_stride), ctypes.c_long(x_head_stride), _p(w), _p(y),
                                  ctypes.c_long(y_token_stride), ctypes.c_long(y_head_stride), num_tokens, heads, I, O,
-                                 _code(x.dtype), _stream()), "head_linear")
+                                 int(y.dtype == torch.float32), _code(x.dtype), _stream()), "head_linear")
 
 
 def attention_decode_scratch_floats(head_dim: int, num_requests: int, nh: int, num_splits: int) -> int:
@@ -719,7 +858,8 @@ def attention_decode(q, q_stride, out, kcache, vcache, block_tables, cu_q, conte
     pair.  Same bits either way.  `sink`, `gate`, `gate_stride`, `softcap`, `chunk`: as for paged_attention_generic.
     `value_div` > 1: `vcache` has kvh // value_div heads, and key head k reads value head k // value_div.  `out` is
     bfloat16 or float32.  `keep_first`, `dist_bias`: as for paged_attention_generic; with either the keys and values come in
-    by cp.async (the TMA kernels walk one range of keys and know no bias)."""
+    by cp.async (the TMA kernels walk one range of keys and know no bias).  A float tensor [nh] as `sink` as there."""
+    sink, sinks = _sinks(sink, nh)
     _cuda(q, out, kcache, vcache, block_tables, cu_q, context_lens, scratch, pairs, gate, dist_bias)
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.is_contiguous() and dist_bias.shape[0] == nh)
     use_tma = use_tma and not keep_first and dist_bias is None
@@ -736,7 +876,7 @@ def attention_decode(q, q_stride, out, kcache, vcache, block_tables, cu_q, conte
         map_k, map_v, _p(q), ctypes.c_long(q_stride), _p(out), _p(kcache), _p(vcache), _p(block_tables),
         block_tables.shape[-1], _p(cu_q), _p(context_lens), num_requests, nh, kvh, kcache.shape[2], window,
         ctypes.c_float(scale), ctypes.c_long(kcache.shape[0]), num_splits, _p(scratch), _p(pairs if map_k is not None else None),
-        int(bool(sink)), _p(gate), ctypes.c_long(gate_stride), ctypes.c_float(softcap), int(chunk), int(value_div), int(out.dtype == torch.float32),
+        sink, sinks, _p(gate), ctypes.c_long(gate_stride), ctypes.c_float(softcap), int(chunk), int(value_div), int(out.dtype == torch.float32),
         int(keep_first), _p(dist_bias), 0 if dist_bias is None else dist_bias.shape[1], _p(err), _stream()),
         "attention_decode_tma" if map_k is not None else
         ("attention_decode_window_bias" if keep_first or dist_bias is not None else "attention_decode"))
@@ -761,7 +901,7 @@ def attention_prefill(q, q_stride, out, kcache, vcache, block_tables, cu_q, cont
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.is_contiguous() and dist_bias.shape[0] == nh)
     assert q.dtype == torch.bfloat16 and kcache.dtype == torch.bfloat16 and (gate is None or gate.dtype == torch.bfloat16)
     L = attention_lib(hd)
-    extras = (int(bool(sink)), _p(gate), ctypes.c_long(gate_stride), ctypes.c_float(softcap), int(chunk), int(value_div),
+    extras = (*_sinks(sink, nh), _p(gate), ctypes.c_long(gate_stride), ctypes.c_float(softcap), int(chunk), int(value_div),
               int(out.dtype == torch.float32))
     map_k = map_v = None
     if use_tma and L.vob_attention_decode_has_tma() and kcache.is_contiguous() and vcache.is_contiguous():
@@ -802,7 +942,7 @@ def gemm_f32(a, w, out, bias=None) -> None:
                               ctypes.c_long(out.stride(0)), _p(bias), M, N, K, _stream()), "gemm_f32")
 
 
-EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_ADD = 0, 1, 2, 3
+EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_ADD, EPI_GEGLU = 0, 1, 2, 3, 4
 _tensor_maps = {}
 
 
@@ -912,7 +1052,8 @@ def gemm_skinny(x, w, out, epilogue: int, err, norm_weight=None, eps: float = 0.
     """out = x @ w^T for at most 16 rows of x (see gemm_skinny_supported); epilogue EPI_BF16 (out bfloat16 [M,N]),
     EPI_F32 (out float32 [M,N], rounded to bfloat16 first), EPI_SWIGLU (the rows of w alternate in groups of
     eight between gate and up; out bfloat16 [M,N/2] = SiLU(gate) * up) or EPI_ADD (out bfloat16 [M,N] += the
-    product rounded to bfloat16: out is the residual stream).  With `norm_weight` (float [K]; EPI_BF16 and EPI_SWIGLU)
+    product rounded to bfloat16: out is the residual stream); EPI_GEGLU is EPI_SWIGLU with the tanh form of gelu (and no norm).
+    With `norm_weight` (float [K]; EPI_BF16 and EPI_SWIGLU)
     the product is that of RMSNorm(x) * norm_weight, the norm computed on the way.
 
     The same norm in two halves, for a chain of products: `emit=(weight, scaled, parts)` (EPI_ADD) makes the product
@@ -925,7 +1066,7 @@ def gemm_skinny(x, w, out, epilogue: int, err, norm_weight=None, eps: float = 0.
     M, K = x.shape
     N = w.shape[0]
     assert w.shape[1] == K and out.stride(1) == 1 and out.shape[0] == M
-    assert out.shape[1] == (N // 2 if epilogue == EPI_SWIGLU else N)
+    assert out.shape[1] == (N // 2 if epilogue in (EPI_SWIGLU, EPI_GEGLU) else N)
     assert out.dtype == (torch.float32 if epilogue == EPI_F32 else torch.bfloat16)
     if norm_weight is not None:
         assert epilogue in (EPI_BF16, EPI_SWIGLU) and norm_weight.dtype == torch.float32 and norm_weight.numel() == K

@@ -9,7 +9,8 @@ the residual stream before the last norm, `compute_logits(hidden, residual, ctx)
 norm and the output product on the wanted rows only and returns float32 logits.
 
 What surrounds the blocks is data of the plan too: a scale on the embedded tokens, position parts that add
-to the embedding (`PositionEncoding.embed`), a soft cap on the logits.  Qwen3 uses none of the three.
+to the embedding (`PositionEncoding.embed`), a soft cap on the logits, an embedding part that takes the lookup's place and
+may keep per-request state.  Qwen3 uses none of them.
 """
 from __future__ import annotations
 
@@ -34,12 +35,17 @@ class CausalLM:
         self.final_norm = build_part("norm", plan.final_norm, **common)
         # a norm of the embedded tokens opens the residual stream; it keeps a copy of its output if a run adds it back later
         self.embedding_norm = build_part("norm", plan.embedding_norm, **common) if plan.embedding_norm is not None else None
+        # an embedding part of the plan's own takes the place of the table lookup; its per-request state lies behind the planes'
+        self.embedding_part = build_part("embedding", plan.embedding, **common) if plan.embedding is not None else None
+        if self.embedding_part is not None and (plan.embedding_norm is not None or not plan.lm_head_name):
+            raise ValueError("an embedding part opens the stream itself and shares no table: no embedding norm, no tied output")
         self._reinjects = any(s.reinject for s in plan.order)
         if self._reinjects and self.embedding_norm is None:
             raise ValueError("a run that adds the embedding's output back needs the plan's embedding norm, which keeps it")
         self.graph_safe = (all(b.graph_safe for b in self.blocks) and self.final_norm.graph_safe
                            and all(p.graph_safe for p in self.positions.values())
-                           and (self.embedding_norm is None or self.embedding_norm.graph_safe))
+                           and (self.embedding_norm is None or self.embedding_norm.graph_safe)
+                           and (self.embedding_part is None or self.embedding_part.graph_safe))
         self.embedding = None
         self.lm_head = None
         self.planes: List[Optional[CachePlane]] = [None] * plan.num_planes()
@@ -52,7 +58,10 @@ class CausalLM:
 
     def tensor_specs(self) -> List[TensorSpec]:
         p = self.plan
-        specs = [TensorSpec(p.embedding_name, (p.vocab_size, p.hidden_size), "embedding")]
+        if self.embedding_part is not None:
+            specs = self.embedding_part.tensor_specs()
+        else:
+            specs = [TensorSpec(p.embedding_name, (p.vocab_size, p.hidden_size), "embedding")]
         if p.lm_head_name:
             specs.append(TensorSpec(p.lm_head_name, (p.vocab_size, p.hidden_size), "matrix", p.hidden_size))
         for part in self.positions.values():
@@ -66,7 +75,10 @@ class CausalLM:
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         p = self.plan
-        self.embedding = tensors[p.embedding_name].contiguous()
+        if self.embedding_part is not None:
+            self.embedding_part.load({s.name: tensors[s.name] for s in self.embedding_part.tensor_specs()})
+        else:
+            self.embedding = tensors[p.embedding_name].contiguous()
         self.lm_head = tensors[p.lm_head_name].contiguous() if p.lm_head_name else self.embedding
         for part in self.positions.values():
             part.load({s.name: tensors[s.name] for s in part.tensor_specs()})
@@ -82,15 +94,15 @@ class CausalLM:
         for s in self.plan.order:
             if s.plane is not None and s.write_cache:
                 out[s.plane] = self.blocks[s.layer].mixer.cache_spec()
-        return out
+        return out + ([None] if self.embedding_part is not None else [])
 
     def state_specs(self) -> List[Optional[StateSpec]]:
-        """Per plane: the fixed-size per-request state of its writer's mixer (None: none)."""
+        """Per plane: the fixed-size per-request state of its writer (None: none); behind the planes, an embedding part's."""
         out: List[Optional[StateSpec]] = [None] * self.plan.num_planes()
         for s in self.plan.order:
             if s.plane is not None and s.write_cache:
-                out[s.plane] = self.blocks[s.layer].mixer.state_spec()
-        return out
+                out[s.plane] = self.blocks[s.layer].state_spec()
+        return out + ([self.embedding_part.state_spec()] if self.embedding_part is not None else [])
 
     def bind(self, planes: List[Optional[CachePlane]], states: List[Optional[torch.Tensor]]) -> None:
         self.planes, self.states = list(planes), list(states)
@@ -101,6 +113,8 @@ class CausalLM:
         tensors = [self.embedding, self.lm_head] + self.final_norm.device_tensors()
         if self.embedding_norm is not None:
             tensors += self.embedding_norm.device_tensors()
+        if self.embedding_part is not None:
+            tensors += self.embedding_part.device_tensors()
         for part in self.positions.values():
             tensors += part.device_tensors()
         for b in self.blocks:
@@ -114,13 +128,16 @@ class CausalLM:
     # ---- one step
     def forward(self, ctx):
         T = ctx.launch_tokens
-        hidden = ctx.ws.get("embedded", T, self.plan.hidden_size, self.dtype)
-        kernels.embedding(self.embedding, ctx.token_ids, hidden, T, ctx.err, self.plan.embedding_scale)
-        for part in self.positions.values():
-            part.embed(hidden, ctx)
-        residual = None
-        if self.embedding_norm is not None:
-            hidden, residual = self.embedding_norm.open_stream(hidden, ctx, keep=self._reinjects)
+        if self.embedding_part is not None:
+            hidden, residual = self.embedding_part.open(ctx, self.states[self.plan.num_planes()])
+        else:
+            hidden = ctx.ws.get("embedded", T, self.plan.hidden_size, self.dtype)
+            kernels.embedding(self.embedding, ctx.token_ids, hidden, T, ctx.err, self.plan.embedding_scale)
+            for part in self.positions.values():
+                part.embed(hidden, ctx)
+            residual = None
+            if self.embedding_norm is not None:
+                hidden, residual = self.embedding_norm.open_stream(hidden, ctx, keep=self._reinjects)
         order = self.plan.order
         ctx.prenormed = ctx.pending_second = None
         for i, s in enumerate(order):

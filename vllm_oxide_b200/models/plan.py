@@ -41,6 +41,7 @@ class ModelPlan:
     default_dtype: str = "bfloat16"
     embedding_scale: float = 1.0           # the embedded tokens are multiplied by it
     logit_softcap: float = 0.0             # > 0: logits = cap * tanh(logits / cap)
+    embedding: Optional[PartSpec] = None   # an embedding part that opens the stream; None: the row of `embedding_name` a token
     embedding_norm: Optional[PartSpec] = None   # a norm of the embedded tokens; it opens the residual stream (`open_stream`)
 
     def num_planes(self) -> int:

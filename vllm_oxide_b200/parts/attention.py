@@ -204,14 +204,15 @@ class SharedKVAttention(Mixer):
 
 
 def paged_attend(q, q_stride, out, keys, values, group: int, ctx, T: int, nh: int, kvh: int, hd: int, window: int,
-                 scale: float, pairs=None, value_dim=None, sink: bool = False, gate=None, gate_stride: int = 0,
+                 scale: float, pairs=None, value_dim=None, sink=False, gate=None, gate_stride: int = 0,
                  softcap: float = 0.0, chunk: int = 0, keep_first: int = 0, dist_bias=None) -> int:
     """Attention of every query of the step over the pages of `keys` / `values`; returns the width of a head in `out`.
     bfloat16: decoding requests (one token) go to the split-key tensor-core kernel, requests with a portion to the
     tensor-core kernel for portions.  The 32-bit path, and sizes those kernels refuse, go to the plain kernel.
     `value_dim` (keys and values are one plane whose rows begin with the value): the plain kernel reads and writes only
     that much of a value row; the tensor-core kernels take whole rows, and the caller uses the first `value_dim`
-    elements of each head of `out`.  `sink`: the softmax has a silent extra entry of score 0.  `gate`: a view whose element
+    elements of each head of `out`.  `sink`: the softmax has a silent extra entry of score 0 (True), or of a score of the head's own
+    (a float tensor [nh]).  `gate`: a view whose element
     [t, h] (rows `gate_stride` apart) is head h's gate of token t; its output is multiplied by the sigmoid of it.
     `softcap` > 0: scores become softcap * tanh(score / softcap); `chunk` > 0: a query sees only keys of its own block of
     `chunk` positions.  `keep_first` > 0: the keys at positions below it are seen by every later query, whatever the window;
@@ -230,7 +231,8 @@ def paged_attend(q, q_stride, out, keys, values, group: int, ctx, T: int, nh: in
     fast = fast and not own_values and (FAST_CAP_AND_CHUNK or not (softcap or chunk))
     fast = fast and (out.dtype == q.dtype or (out.dtype == torch.float32 and FAST_CAP_AND_CHUNK))
     fast = fast and (FAST_KEEP_AND_BIAS or not (keep_first or dist_bias is not None))
-    if not fast or ((sink or gate is not None) and not FAST_SINK_AND_GATE):
+    has_sink = sink if isinstance(sink, bool) else sink is not None
+    if not fast or ((has_sink or gate is not None) and not FAST_SINK_AND_GATE):
         kernels.paged_attention_generic(q, q_stride, out, keys, values, tables, ctx.token_req, ctx.positions, T,
                                         nh, kvh, hd, window, scale, ctx.err, value_dim=value_dim, sink=sink, gate=gate,
                                         gate_stride=gate_stride, softcap=softcap, chunk=chunk, keep_first=keep_first,

@@ -226,18 +226,34 @@ class FeedForward(Part):
         raise NotImplementedError
 
 
+class Embedding(Part):
+    """Opens a step's residual stream from its tokens, in place of the plain table lookup.  It may keep per-request state like a
+    mixer (a plan's embedding gets a state slot of its own behind the planes)."""
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return None
+
+    def open(self, ctx, state: Optional[torch.Tensor]):
+        """(hidden, residual) as the first block takes them."""
+        raise NotImplementedError
+
+
 class Block(Part):
+    def state_spec(self) -> Optional[StateSpec]:
+        """What a run of this block keeps per request: its mixer's state, and what the block itself carries from token to token."""
+        return self.mixer.state_spec()
+
     def forward(self, hidden, residual, ctx, cache, state, write_cache=True):
         raise NotImplementedError
 
 
 # ------------------------------------------------------------------ registries
-_REGISTRIES: Dict[str, Dict[str, Callable]] = {"norm": {}, "position": {}, "mixer": {}, "feed_forward": {}, "block": {}}
+_REGISTRIES: Dict[str, Dict[str, Callable]] = {"norm": {}, "position": {}, "mixer": {}, "feed_forward": {}, "block": {}, "embedding": {}}
 
 
 def register_part(family: str, kind: str, factory: Callable) -> None:
     """Makes `factory(**params, **common)` available under (family, kind).  Families: norm, position,
-    mixer, feed_forward, block.  Registering a kind twice replaces it (tests register toy parts)."""
+    mixer, feed_forward, block, embedding.  Registering a kind twice replaces it (tests register toy parts)."""
     if family not in _REGISTRIES:
         raise KeyError(f"unknown part family {family!r}; families are {sorted(_REGISTRIES)}")
     _REGISTRIES[family][kind] = factory

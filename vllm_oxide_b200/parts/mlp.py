@@ -1,5 +1,6 @@
 """SwiGLU feed-forward: down( silu(gate(x)) * up(x) ) with gate and up merged into one product
-(vllm-oxide, crates/vllm-oxide/src/models/qwen3.rs:60-87, crates/vllm-oxide/src/layers/activation.rs:17-21)."""
+(vllm-oxide, crates/vllm-oxide/src/models/qwen3.rs:60-87, crates/vllm-oxide/src/layers/activation.rs:17-21); other designs gate by the tanh form of
+gelu instead of SiLU.  `ClampedGLU` is a gated feed-forward with clamps and biases."""
 from __future__ import annotations
 
 from typing import Dict, List
@@ -16,9 +17,14 @@ class SwiGLU(FeedForward):
     graph_safe = True
 
     def __init__(self, hidden_size: int, intermediate_size: int, prefix: str,
-                 names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), **_):
-        """`names`: what the checkpoint calls the gate, up and down matrices behind `prefix`."""
-        self.H, self.I, self.prefix = hidden_size, intermediate_size, prefix
+                 names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), activation: str = "silu",
+                 out_name: str = "mlp_out", **_):
+        """`names`: what the checkpoint calls the gate, up and down matrices behind `prefix`; `activation`: "silu" or
+        "gelu_tanh" (the tanh form of gelu) on the gate; `out_name`: the workspace buffer of the output."""
+        self.H, self.I, self.prefix, self.out_name = hidden_size, intermediate_size, prefix, out_name
+        if activation not in ("silu", "gelu_tanh"):
+            raise ValueError(f"a gated feed-forward's activation is 'silu' or 'gelu_tanh', not {activation!r}")
+        self.gelu = activation == "gelu_tanh"
         self.n_gate, self.n_up, self.n_down = (prefix + n for n in names)
         self.wgu = self.wdown = None
         self.interleaved = False
@@ -49,21 +55,21 @@ class SwiGLU(FeedForward):
         act = ctx.ws.get("act", T, self.I, x.dtype)
         if self.interleaved and kernels.gemm_skinny_supported(x, self.wgu):
             # decode-sized steps: the activation is the epilogue of the gate|up product
-            kernels.gemm_skinny(x, self.wgu, act, kernels.EPI_SWIGLU, ctx.err)
-        elif self.interleaved and tc5_product(x, self.wgu, act, kernels.EPI_SWIGLU, ctx):
+            kernels.gemm_skinny(x, self.wgu, act, kernels.EPI_GEGLU if self.gelu else kernels.EPI_SWIGLU, ctx.err)
+        elif self.interleaved and not self.gelu and tc5_product(x, self.wgu, act, kernels.EPI_SWIGLU, ctx):
             pass
         else:
             gu = linear(x, self.wgu, ctx.ws.get("gate_up", T, 2 * self.I, x.dtype), ctx)
-            kernels.silu_mul(gu, act, T, self.interleaved)
+            kernels.silu_mul(gu, act, T, self.interleaved, gelu=self.gelu)
         if add_into is not None:
             linear_into_stream(act, self.wdown, add_into)
             return None
-        return linear(act, self.wdown, ctx.ws.get("mlp_out", T, self.H, x.dtype), ctx)
+        return linear(act, self.wdown, ctx.ws.get(self.out_name, T, self.H, x.dtype), ctx)
 
     # ---- the same with the residual stream kept inside the products (decode-sized steps)
     def can_forward_on_stream(self, stream, ctx) -> bool:
         act = ctx.ws.get("act", stream.shape[0], self.I, stream.dtype)
-        return (self.interleaved and kernels.gemm_skinny_supported(stream, self.wgu)
+        return (self.interleaved and not self.gelu and kernels.gemm_skinny_supported(stream, self.wgu)
                 and kernels.gemm_skinny_supported(act, self.wdown))
 
     def forward_on_stream(self, stream, norm, ctx, prenormed=None, emit_norm=None):

@@ -18,11 +18,12 @@ False has no correction tensor (the choice is by s); `group_top` 2 lets a group 
 scores; `normalise` divides the chosen scores by their sum (+ 1e-20); `weight_scale` multiplies them; `router_bias` adds <prefix>router.b to the logits;
 `activation` "glu_clamped" with `limit` makes an expert down(g * sigmoid(1.702 g) * (u + 1)) with g = min(gate(x), limit),
 u = clamp(up(x), -limit, limit).  The softmax over the chosen logits alone is `scores` "softmax" with `normalise` and no
-correction: the chosen shares of the full softmax, divided by their sum.
+correction: the chosen shares of the full softmax, divided by their sum.  `shared` (a `swiglu` feed-forward's parameters): an
+expert that every token uses, added to the sum of the chosen ones before it is rounded.
 """
 from __future__ import annotations
 
-from typing import Dict, List
+from typing import Dict, List, Optional
 
 import torch
 
@@ -30,6 +31,7 @@ from .. import kernels
 from ..weights.loader import TensorSpec
 from .base import FeedForward, register_part
 from .linear import linear
+from .mlp import SwiGLU
 
 
 # bfloat16 steps with at least this many (token, choice) pairs run the experts' products on the tcgen05 tensor cores (row
@@ -65,7 +67,7 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, expert_size: int, experts: int, top: int, prefix: str, groups: int = 1, keep: int = 1,
                  names=("up", "down", "router", "correction"), activation: str = "relu2", gate_name: str = "gate",
                  scores: str = "softmax", correction: bool = True, group_top: int = 1, normalise: bool = False,
-                 weight_scale: float = 1.0, router_bias: bool = False, limit: float = 0.0, **_):
+                 weight_scale: float = 1.0, router_bias: bool = False, limit: float = 0.0, shared: Optional[dict] = None, **_):
         self.H, self.I, self.E, self.top = int(hidden_size), int(expert_size), int(experts), int(top)
         self.groups, self.keep, self.prefix = int(groups), int(keep), prefix
         if self.E % self.groups or self.keep > self.groups or self.top > (self.E // self.groups) * self.keep:
@@ -80,7 +82,11 @@ class RoutedExperts(FeedForward):
         self.has_router_bias = bool(router_bias)
         self.sigmoid_scores, self.has_correction, self.group_top = scores == "sigmoid", bool(correction), int(group_top)
         self.normalise, self.weight_scale = bool(normalise), float(weight_scale)
+        self.shared = SwiGLU(hidden_size=self.H, out_name="shared_out", **shared) if shared else None
         self.wup = self.wdown = self.router = self.correction = self.router_b = None
+
+    def parts(self):
+        return [self.shared] if self.shared is not None else []
 
     def _expert(self, e: int, name: str) -> str:
         return f"{self.prefix}e{e}.{name}"
@@ -97,7 +103,7 @@ class RoutedExperts(FeedForward):
             specs.append(TensorSpec(self.prefix + self.n_router + ".b", (self.E,), "coefficient", init="small"))
         if self.has_correction:
             specs.append(TensorSpec(self.prefix + self.n_correction, (self.E,), "coefficient", init="small"))
-        return specs
+        return specs + (self.shared.tensor_specs() if self.shared is not None else [])
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         up = torch.stack([tensors[self._expert(e, self.n_up)] for e in range(self.E)])
@@ -110,6 +116,8 @@ class RoutedExperts(FeedForward):
         self.router = tensors[self.prefix + self.n_router].contiguous()
         self.correction = tensors[self.prefix + self.n_correction].contiguous() if self.has_correction else None
         self.router_b = tensors[self.prefix + self.n_router + ".b"].contiguous() if self.has_router_bias else None
+        if self.shared is not None:
+            self.shared.load({s.name: tensors[s.name] for s in self.shared.tensor_specs()})
 
     def _route(self, x, ids, weights, T: int) -> None:
         kernels.moe_route(x, self.router, self.correction, ids, weights, T, self.top, self.groups, self.keep,
@@ -118,6 +126,7 @@ class RoutedExperts(FeedForward):
 
     def forward(self, x, ctx):
         T, top = x.shape[0], self.top
+        shared = self.shared.forward(x, ctx) if self.shared is not None else None
         n = T * top
         # bfloat16 steps of many pairs: the experts' products on the tcgen05 tensor cores, over rows gathered into expert order
         fast = (n >= TC5_MIN_PAIRS and kernels.moe_gemm_tc5_supported(x, self.wup) and self.I % 8 == 0)
@@ -134,7 +143,7 @@ class RoutedExperts(FeedForward):
             y = ctx.ws.get_flat("moe_y", n * self.H, torch.float32).view(n, self.H)
             kernels.moe_gemv(act, self.wdown, y, ids, order, n, top, False)
             out = ctx.ws.get("mlp_out", T, self.H, x.dtype)
-            kernels.moe_combine(y, None, weights, out, T, top)
+            kernels.moe_combine(y, None, weights, out, T, top, add=shared)
             return out
         tile = kernels.moe_tc5_row_tile() if fast else kernels.moe_row_tile()
         # every expert's rows are padded to a row tile: at most tile - 1 rows for each expert that has any
@@ -157,7 +166,7 @@ class RoutedExperts(FeedForward):
                              silu_pairs=self.gated, glu_limit=self.limit)
             kernels.moe_gemm(act, self.wdown, y, row_token, tile_expert, relu_squared=False, gather=False)
         out = ctx.ws.get("mlp_out", T, self.H, x.dtype)
-        kernels.moe_combine(y, slot_of, weights, out, T, top)
+        kernels.moe_combine(y, slot_of, weights, out, T, top, add=shared)
         return out
 
 

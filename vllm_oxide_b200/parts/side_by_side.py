@@ -58,15 +58,18 @@ class SideBySide(Mixer):
 
     def forward(self, x, ctx, cache, state, write_cache: bool = True):
         outs = []
+        # a left mixer that has a bias on its output leaves it to the kernel that norms the pair
+        bias = getattr(self.left, "out_bias", None)
         for m, (off, n) in zip((self.left, self.right), self._states):
             own_cache = cache if m.cache_spec() is not None else None
             own_state = state[:, off:off + n] if n else None
-            outs.append(m.forward(x, ctx, own_cache, own_state, write_cache))
+            later = dict(defer_bias=True) if m is self.left and bias is not None else {}
+            outs.append(m.forward(x, ctx, own_cache, own_state, write_cache, **later))
         a, b = outs
         if a.data_ptr() == b.data_ptr():
             raise RuntimeError("the two mixers wrote their outputs into the same workspace buffer")
         out = ctx.ws.get("side_by_side_out", x.shape[0], self.H, x.dtype)
-        kernels.pair_norm_mean(a, b, self.w_left, self.w_right, out, self.eps)
+        kernels.pair_norm_mean(a, b, self.w_left, self.w_right, out, self.eps, bias_a=bias)
         return out
 
 
