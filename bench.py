@@ -18,7 +18,7 @@ of 8 requests whose context starts at 2,048 tokens, and prints ONE JSON line:
 The cache that the decode steps read was written by a real prefill of random prompts.  Every timed step reads 15 GB of weights, far more than the 126 MB L2, so nothing stays cached
 between iterations.  Peaks come from MEASURED_PEAKS.json beside this file when present.
 
-    python bench.py --workload tofilorn | kesozen | rakizen | depolix [--sizes 2048,4096]
+    python bench.py --workload tofilorn | kesozen | rakizen | depolix | laruzen [--sizes 2048,4096]
 
 measures the Tofilorn design (residual streams, minGRU, HGRN2, latent attention), the Kesozen design (sandwich norms over
 a float stream, attention whose keys are its values, gated delta rule, routed experts) or the Rakizen design (parallel
@@ -39,6 +39,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 import statistics
 import subprocess
@@ -515,6 +516,64 @@ def depolix_kernel_bytes(cfg: dict, T: int) -> dict:
     return b
 
 
+def laruzen_config(width: int, layers: int) -> dict:
+    """Layer sizes of a real model of this width: a block of four layers (gated linear attention, heads of 128, a decay of rank
+    16; lightning attention, heads of 128; two mixers side by side: attention, heads of 128 over 8 key heads, a window of 1,024,
+    and a gated linear recurrence as wide as the model in parts of 256 channels behind filters of 4 taps; gated linear attention
+    again); feed-forwards of 16 gated experts of which a token uses 4 (the four together three times the width) beside a shared
+    one, but for the first layer of each block, whose feed-forward is dense and three times the width."""
+    heads = width // 128
+    gla = dict(heads=heads, dim=128, vdim=128, tau=16.0, rank=16)
+    lightning = dict(heads=heads, dim=128, vdim=128, decay=[math.exp(-2.0 ** (-8.0 * (h + 1) / heads)) for h in range(heads)])
+    sides = {"left": dict(heads=heads, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, mask={"size": 1024},
+                          rot={"dims": 128, "base": 10000.0, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}),
+             "right": dict(width=width, blocks=max(1, width // 256), conv=4)}
+    moe = {"kind": "moe", "expert": {"ff": 3 * width // 4}, "router": {"experts": 16, "top": 4}, "shared": {"ff": 3 * width // 4}}
+    dense = {"kind": "dense", "ff": 3 * width}
+    out = []
+    for _ in range(0, layers, 4):
+        out += [{"type": "gla", "mixer": gla, "mlp": dense}, {"type": "lightning", "mixer": lightning, "mlp": moe},
+                {"type": "parallel", "mixer": sides, "mlp": moe}, {"type": "gla", "mixer": gla, "mlp": moe}]
+    return {"architecture": "Laruzen", "vocab": 32768, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65537, "mul_prev": 31, "mul_cur": 1009}}, "layers": out[:layers]}
+
+
+def laruzen_kernel_bytes(cfg: dict, T: int) -> dict:
+    """Bytes that each of the design's own row-wise kernels must move in a step of T tokens, summed over the layers (weights
+    aside, but for the per-part gate matrices of the recurrence, which a decode step streams): what its time is held against.
+    Attention, the matrix-state scans and the experts' products are held against arithmetic."""
+    D = cfg["width"]
+    b = {"pair_embedding": T * D * (2 + 2 + 4)}
+    add = lambda k, v: b.__setitem__(k, b.get(k, 0) + v)
+    for i, l in enumerate(cfg["layers"]):
+        m, mlp = l["mixer"], l["mlp"]
+        # stream read (and, behind a sublayer, its output read and the new stream written), the mixed normed row out
+        add("residual_norm_shift_step", T * D * (4 + 2 + (2 + 4 if i else 0)))
+        if l["type"] == "parallel":
+            le, ri = m["left"], m["right"]
+            q, k, v, W = le["heads"] * le["dim"], le["kv_heads"] * le["dim"], le["kv_heads"] * le["vdim"], ri["width"]
+            add("headnorm_rope_kv_write", T * (2 * q + 2 * k + 2 * v) * 2)
+            add("sigmoid_gate_mul", T * le["heads"] * le["vdim"] * 3 * 2)
+            add("short_conv_silu", T * W * (2 + 2))
+            add("short_conv_step", T * W * (2 + 2 + 2 * 4 * (ri["conv"] - 1)))
+            add("head_linear", 2 * W * (W // ri["blocks"]) * 2 + T * W * (2 + 8))
+            add("lru_scan", T * W * (2 + 8 + 2 + 2))
+            add("pair_norm_mean", T * 3 * D * 2)
+        else:
+            V = m["heads"] * m["vdim"]
+            add("delta_out_norm", T * V * (4 + 2 + 2))
+        if mlp:
+            add("residual_norm_step", T * D * (2 + 2 * 4 + 2))
+        if mlp and mlp["kind"] == "dense":
+            add("gelu_mul", T * 3 * mlp["ff"] * 2)
+        elif mlp:
+            top = mlp["router"]["top"]
+            add("silu_mul", T * 3 * mlp["shared"]["ff"] * 2)
+            add("moe_gather_rows", T * top * D * 2 * 2)
+            add("moe_combine", T * (top * D * 4 + 2 * D * 2))
+    return b
+
+
 def attention_flops(cfg: dict, T: int) -> float:
     """Multiply-adds x 2 of the score and value products of one prompt of T tokens, every query over the keys it sees."""
     def seen(size, blocks):
@@ -559,7 +618,8 @@ def qwen3_kernel_bytes(cfg: dict, T: int) -> dict:
 
 
 DESIGNS = {"tofilorn": (tofilorn_config, tofilorn_kernel_bytes), "kesozen": (kesozen_config, kesozen_kernel_bytes),
-           "rakizen": (rakizen_config, rakizen_kernel_bytes), "depolix": (depolix_config, depolix_kernel_bytes)}
+           "rakizen": (rakizen_config, rakizen_kernel_bytes), "depolix": (depolix_config, depolix_kernel_bytes),
+           "laruzen": (laruzen_config, laruzen_kernel_bytes)}
 
 
 def float_issue_rate():
@@ -593,6 +653,10 @@ def design_run(design: str, widths, pk=None, layers: int = 16) -> dict:
         if design == "depolix":
             models["kesozen"] = kesozen_config(width, layers)         # the delta rule, the gated heads and the routed experts
             models["tofilorn"] = tofilorn_config(width, layers)       # attention through a latent
+        if design == "laruzen":
+            models["depolix"] = depolix_config(width, layers)         # two mixers side by side, experts by softmax
+            models["tofilorn"] = tofilorn_config(width, layers)       # the matrix-state and the channel recurrence
+            models["kesozen"] = kesozen_config(width, layers)         # norms on both sides of every sublayer
         rec = {}
         for name, cfg in models.items():
             r = {}
@@ -667,7 +731,21 @@ def design_run(design: str, widths, pk=None, layers: int = 16) -> dict:
                         flops = sum(2 * (PROMPT_LEN * (PROMPT_LEN + 1) // 2) * m["heads"] * 2 * row(m) for m in lat)
                         r["prefill_2048"]["latent_attention_ms"] = round(ms, 4)
                         r["prefill_2048"]["latent_attention_frac_of_bf16_peak"] = round(flops / (ms * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
-                if name in ("kesozen", "rakizen", "depolix"):
+                if name == "laruzen":
+                    own, rate = r["prefill_2048"]["own_kernels_ms"], float_issue_rate()
+                    for kind, k in (("gla", "gla_scan"), ("lightning", "lightning_scan")):
+                        # as hgrn2_scan: two walks, five float instructions a lane per state element and token
+                        work = sum(PROMPT_LEN * l["mixer"]["heads"] * l["mixer"]["dim"] * l["mixer"]["vdim"] * 5
+                                   for l in cfg["layers"] if l["type"] == kind)
+                        if rate and own.get(k):
+                            r["prefill_2048"][k + "_frac_of_float_issue_rate"] = round(work / (own[k] * 1e-3) / rate, 4)
+                    le = [l["mixer"]["left"] for l in cfg["layers"] if l["type"] == "parallel"]
+                    seen = sum(min(i, le[0]["mask"]["size"] - 1) + 1 for i in range(PROMPT_LEN)) if le else 0
+                    flops = sum(2 * seen * m["heads"] * (m["dim"] + m["vdim"]) for m in le)
+                    if own.get("attention_prefill_tc5"):
+                        r["prefill_2048"]["window_attention_frac_of_bf16_peak"] = round(
+                            flops / (own["attention_prefill_tc5"] * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
+                if name in ("kesozen", "rakizen", "depolix", "laruzen"):
                     own = r["prefill_2048"]["own_kernels_ms"]
                     if own.get("delta_scan"):
                         # the delta rule is arithmetic too: a multiply and three multiply-adds per state element and token
@@ -675,13 +753,13 @@ def design_run(design: str, widths, pk=None, layers: int = 16) -> dict:
                         work = sum(PROMPT_LEN * l["mixer"]["heads"] * l["mixer"]["dim"] * l["mixer"]["vdim"] * 4
                                    for l in cfg["layers"] if l["type"] == "delta")
                         work += sum(PROMPT_LEN * l["mixer"]["right"]["heads"] * l["mixer"]["right"]["dim"] * l["mixer"]["right"]["vdim"] * 4
-                                    for l in cfg["layers"] if l["type"] == "parallel")
+                                    for l in cfg["layers"] if l["type"] == "parallel" and "dim" in l["mixer"]["right"])
                         if rate:
                             r["prefill_2048"]["delta_scan_frac_of_float_issue_rate"] = round(work / (own["delta_scan"] * 1e-3) / rate, 4)
                     if own.get("moe_gemm_tc5"):
                         # the experts' products against the measured bfloat16 product of the library
                         # (two products an expert; three where it is gated)
-                        flops = sum((6 if name in ("rakizen", "depolix") else 4) * PROMPT_LEN * l["mlp"]["router"]["top"] * cfg["width"] * l["mlp"]["expert"]["ff"]
+                        flops = sum((6 if name in ("rakizen", "depolix", "laruzen") else 4) * PROMPT_LEN * l["mlp"]["router"]["top"] * cfg["width"] * l["mlp"]["expert"]["ff"]
                                     for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe")
                         r["prefill_2048"]["moe_gemm_tc5_frac_of_bf16_peak"] = round(flops / (own["moe_gemm_tc5"] * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
             rec[name] = r
@@ -790,7 +868,7 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--workload", choices=sorted(WORKLOADS) + sorted(DESIGNS), default=None,
                     help="another workload instead of the default run")
-    ap.add_argument("--sizes", default="2048,4096", help="--workload tofilorn | kesozen | rakizen | depolix: the widths to measure")
+    ap.add_argument("--sizes", default="2048,4096", help="--workload tofilorn | kesozen | rakizen | depolix | laruzen: the widths to measure")
     ap.add_argument("--only", choices=["decode", "prefill", "attention"], default=None,
                     help="run one phase and print its time only (for short profiler captures)")
     args = ap.parse_args()

@@ -48,6 +48,47 @@ short_conv_silu_kernel(const T* x, long x_stride, const float* __restrict__ w, c
   const float b_in = bias_in && c < C ? bias_in[c] : 0.f, b_out = bias_out && c < C ? bias_out[c] : 0.f;
   pdl_wait();
   if (c >= C) return;
+  // the usual case of a large step, all of the thread's tokens in one portion: every input is asked for before the first is used
+  if (walk == CONV_TOKENS && t_first + CONV_TOKENS <= num_tokens) {
+    const int req = token_req[t_first];
+    if (req >= 0 && req == token_req[t_first + CONV_TOKENS - 1]) {
+      const int j = t_first - cu_q[req];
+      const int slot = state_slots[req];
+      if (slot < 0 || slot >= num_slots) {
+        atomicOr(err, VOB_ERR_SLOT);
+        return;
+      }
+      const float* st = state + (size_t)slot * state_stride + conv_off;
+      float in[DELTA_MAX_TAPS - 1 + CONV_TOKENS];      // in[s]: input t_first - (DELTA_MAX_TAPS - 1) + s
+#pragma unroll
+      for (int s = 0; s < DELTA_MAX_TAPS - 1; ++s) {
+        const int back = DELTA_MAX_TAPS - 1 - s;        // tokens before the thread's first
+        in[s] = back > taps - 1 ? 0.f
+                                : (j >= back ? to_f<T>(x[(size_t)(t_first - back) * x_stride + c]) + b_in
+                                             : st[(size_t)(taps - 1 + j - back) * C + c]);
+      }
+#pragma unroll
+      for (int k = 0; k < CONV_TOKENS; ++k) in[DELTA_MAX_TAPS - 1 + k] = to_f<T>(x[(size_t)(t_first + k) * x_stride + c]) + b_in;
+      float wr[DELTA_MAX_TAPS];                          // the filter, newest tap last, zeros in front
+#pragma unroll
+      for (int s = 0; s < DELTA_MAX_TAPS; ++s) {
+        wr[s] = 0.f;
+        const int tap = s - (DELTA_MAX_TAPS - taps);
+#pragma unroll
+        for (int q = 0; q < DELTA_MAX_TAPS; ++q)
+          if (q == tap) wr[s] = wt[q];
+      }
+#pragma unroll
+      for (int k = 0; k < CONV_TOKENS; ++k) {
+        float acc = b_out;
+#pragma unroll
+        for (int s = 0; s < DELTA_MAX_TAPS; ++s)
+          if (s >= DELTA_MAX_TAPS - taps) acc = fmaf(wr[s], in[k + s], acc);          // oldest input first
+        out[(size_t)(t_first + k) * C + c] = from_f<TO>(act ? silu_f(acc) : acc);
+      }
+      return;
+    }
+  }
   float win[DELTA_MAX_TAPS - 1];      // win[s]: the input taps - 1 - s tokens back
   bool have = false;
   for (int tt = 0; tt < walk; ++tt) {

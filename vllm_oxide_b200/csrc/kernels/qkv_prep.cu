@@ -266,6 +266,95 @@ headnorm_rope_kv_write_kernel(T* qkv, long row_stride, const float* __restrict__
   }
 }
 
+// The same arithmetic for 16-bit rows whose keys and values have one head size, a multiple of 8, and whose rotated part is whole
+// groups of 8 in halves: LPH lanes (a power of two) hold a head, 8 elements each in registers, so a warp takes 32 / LPH heads at
+// once; a rotation's partner comes by a shuffle.
+template <int LPH>
+__global__ void __launch_bounds__(HP_WARPS * 32)
+headnorm_rope_kv_write_lanes_kernel(__nv_bfloat16* qkv, long row_stride, const float* __restrict__ bias,
+                                    const int* __restrict__ positions, const int* __restrict__ slots, const float* __restrict__ wq,
+                                    const float* __restrict__ wk, const float* __restrict__ freq, float amp, __nv_bfloat16* kcache,
+                                    __nv_bfloat16* vcache, int nh, int kvh, int kd, int vh, int kd_norm, int vd_norm, int rot_dim,
+                                    int v_norm, float eps, long num_slots, int block_size, int write_kv, int* err) {
+  constexpr int HPW = 32 / LPH;                         // heads a warp takes at once
+  __shared__ __align__(16) float cosines[QP_MAX_ROT / 2], sines[QP_MAX_ROT / 2];
+  pdl_launch_dependents();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = positions[t];
+  const int slot = slots ? slots[t] : -1;
+  const int half = rot_dim >> 1;
+  if (pos >= 0)
+    for (int j = threadIdx.x; j < half; j += HP_WARPS * 32) {
+      float sn, cs;
+      sincosf(__fmul_rn((float)pos, freq[j]), &sn, &cs);
+      cosines[j] = cs * amp;
+      sines[j] = sn * amp;
+    }
+  pdl_wait();
+  if (pos < 0) {
+    if (threadIdx.x == 0) atomicOr(err, VOB_ERR_POSITION);
+    return;
+  }
+  const bool put = write_kv && slot >= 0;
+  if (put && slot >= num_slots) {
+    if (threadIdx.x == 0) atomicOr(err, VOB_ERR_SLOT);
+    return;
+  }
+  __syncthreads();
+  __nv_bfloat16* row = qkv + (size_t)t * row_stride;
+  const size_t page = put ? (size_t)(slot / block_size) : 0;
+  const int in_page = put ? slot % block_size : 0;
+  const int total = nh + kvh + vh, sub = lane / LPH, l = lane % LPH, d = l * 8;
+  const bool have = d < kd;
+  const int half_lanes = half >> 3;
+  for (int h0 = warp * HPW; h0 < total; h0 += HP_WARPS * HPW) {
+    const int head = h0 + sub;
+    const bool live = have && head < total && (head < nh || put);
+    const bool is_q = head < nh, is_v = head >= nh + kvh;
+    const int off = head * kd + d;
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = 0.f;
+    if (live) {
+      Wide16<__nv_bfloat16>::load(row + off, v);
+      if (bias) {
+        const float4 b0 = *reinterpret_cast<const float4*>(bias + off), b1 = *reinterpret_cast<const float4*>(bias + off + 4);
+        v[0] += b0.x; v[1] += b0.y; v[2] += b0.z; v[3] += b0.w; v[4] += b1.x; v[5] += b1.y; v[6] += b1.z; v[7] += b1.w;
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float* w = is_v ? nullptr : (is_q ? wq : wk);
+    const float inv = is_v ? (v_norm ? 1.f / sqrtf(ss / (float)vd_norm + eps) : 1.f) : (w ? 1.f / sqrtf(ss / (float)kd_norm + eps) : 1.f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] *= inv;
+    if (w && live) {
+      const float4 g0 = *reinterpret_cast<const float4*>(w + d), g1 = *reinterpret_cast<const float4*>(w + d + 4);
+      v[0] *= g0.x; v[1] *= g0.y; v[2] *= g0.z; v[3] *= g0.w; v[4] *= g1.x; v[5] *= g1.y; v[6] *= g1.z; v[7] *= g1.w;
+    }
+    if (half_lanes > 0) {      // the same for every lane
+      const bool turns = d < rot_dim && !is_v, low = d < half;
+      const int from = lane + (d < rot_dim ? (low ? half_lanes : -half_lanes) : 0);
+      const int a0 = d < rot_dim ? (low ? d : d - half) : 0;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float other = __shfl_sync(0xffffffffu, v[j], from);
+        const float cs = cosines[a0 + j], sn = sines[a0 + j];
+        if (turns) v[j] = low ? __fsub_rn(__fmul_rn(v[j], cs), __fmul_rn(other, sn)) : __fadd_rn(__fmul_rn(v[j], cs), __fmul_rn(other, sn));
+      }
+    }
+    if (live) {
+      __nv_bfloat16* dst = is_q ? row + off
+                                : (is_v ? vcache + ((page * vh + (head - nh - kvh)) * block_size + in_page) * (size_t)kd + d
+                                        : kcache + ((page * kvh + (head - nh)) * block_size + in_page) * (size_t)kd + d);
+      Wide16<__nv_bfloat16>::store(dst, v);
+    }
+  }
+}
+
 // One warp a (token, head).  a: [tokens, 2 * heads * vd] of TA; out [tokens, heads * vd] of T; gate rows of gate_stride.
 template <typename T, typename TA>
 __global__ void __launch_bounds__(128)
@@ -331,6 +420,16 @@ VOB_API int vob_headnorm_rope_kv_write(void* qkv, long row_stride, const float* 
     return VOB_BAD_ARGUMENT;
   const int n = dtype == VOB_F32 ? 4 : 8;
   const int wide = kd % n == 0 && vd % n == 0 && row_stride % n == 0 && (((uintptr_t)qkv | (uintptr_t)kcache | (uintptr_t)vcache) & 15) == 0;
+  if (dtype == VOB_BF16 && wide && kd == vd && kd <= 256 && rot_dim % 16 == 0 && !interleaved &&
+      (((uintptr_t)bias | (uintptr_t)wq | (uintptr_t)wk) & 15) == 0) {
+#define VOB_HPL(L)                                                                                                                 \
+  if (kd <= 8 * L)                                                                                                                 \
+    return launch_kernel(headnorm_rope_kv_write_lanes_kernel<L>, dim3(T), HP_WARPS * 32, 0, stream, (__nv_bfloat16*)qkv, row_stride, \
+                         bias, positions, slots, wq, wk, freq, amp, (__nv_bfloat16*)kcache, (__nv_bfloat16*)vcache, nh, kvh, kd,   \
+                         vh, kd_norm, vd_norm, rot_dim, v_norm, eps, num_slots, block_size, write_kv, err)
+    VOB_HPL(4); VOB_HPL(8); VOB_HPL(16); VOB_HPL(32);
+#undef VOB_HPL
+  }
 #define VOB_HP(TT)                                                                                                               \
   return launch_kernel(headnorm_rope_kv_write_kernel<TT>, dim3(T), HP_WARPS * 32, 0, stream, (TT*)qkv, row_stride, bias, positions, \
                        slots, wq, wk, freq, amp, (TT*)kcache, (TT*)vcache, nh, kvh, kd, vh, vd, kd_norm, vd_norm, rot_dim,       \

@@ -134,6 +134,205 @@ residual_norm_step_kernel(float* stream, const T* y, const float* __restrict__ w
   }
 }
 
+// ---- rows in registers: widths that are a multiple of 4 and fit NV groups of 4 elements a thread.  All loads of a row are issued
+// before its first sum, and (in a walk) the next row's before this row's sums, so a block waits for memory once a row.  The same
+// arithmetic as the kernels that keep the row in shared memory.
+template <typename T, int NT, int NV>
+struct StreamRow {
+  float x[NV][4];      // the stream's row
+  float y[NV][4];      // the sublayer's output
+  __device__ __forceinline__ void load(const float* stream, const T* yin, size_t base, int D, bool init) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (i * NT + threadIdx.x) * 4;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) x[i][j] = y[i][j] = 0.f;
+      if (d < D) {
+        if (!init) RowAccess<float, 4>::load(stream + base + d, x[i]);
+        if (yin) RowAccess<T, 4>::load(yin + base + d, y[i]);
+      }
+    }
+  }
+  // x += RMSNorm(y) * w_post (w_post null: x += y; no y: nothing)
+  __device__ __forceinline__ void add(bool has_y, const float* __restrict__ w_post, int D, float eps, float* scratch) {
+    if (!has_y) return;
+    float inv = 1.f;
+    if (w_post) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss = fmaf(y[i][j], y[i][j], ss);
+      inv = 1.f / sqrtf(block_sum<NT>(ss, scratch) / (float)D + eps);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (i * NT + threadIdx.x) * 4;
+      if (d < D) {
+        float w[4] = {1.f, 1.f, 1.f, 1.f};
+        if (w_post) RowAccess<float, 4>::load(w_post + d, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[i][j] += w_post ? y[i][j] * inv * w[j] : y[i][j];
+      }
+    }
+  }
+  __device__ __forceinline__ float inv_rms(int D, float eps, float* scratch) const {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss = fmaf(x[i][j], x[i][j], ss);
+    return 1.f / sqrtf(block_sum<NT>(ss, scratch) / (float)D + eps);
+  }
+  // x / rms * w_pre into h
+  __device__ __forceinline__ void normed(float inv, const float* __restrict__ w_pre, int D, float (&h)[NV][4]) const {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (i * NT + threadIdx.x) * 4;
+      float w[4] = {1.f, 1.f, 1.f, 1.f};
+      if (w_pre && d < D) RowAccess<float, 4>::load(w_pre + d, w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) h[i][j] = x[i][j] * inv * w[j];
+    }
+  }
+  template <typename TO>
+  static __device__ __forceinline__ void put(TO* p, const float (&v)[NV][4], int D) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (i * NT + threadIdx.x) * 4;
+      if (d < D) RowAccess<TO, 4>::store(p + d, v[i]);
+    }
+  }
+};
+
+template <typename T, int NT, int NV>
+__global__ void __launch_bounds__(NT)
+residual_norm_step_regs_kernel(float* stream, const T* y, const float* __restrict__ w_post, const float* inject, float* keep,
+                               const float* __restrict__ w_pre, T* out, const int* __restrict__ rows, int num_src_rows, int D,
+                               float eps, int init, int* err) {
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x;
+  int src = r;
+  if (rows) {
+    src = rows[r];
+    if (src < 0 || src >= num_src_rows) {
+      if (threadIdx.x == 0) atomicOr(err, VOB_ERR_ROW);
+      return;
+    }
+  }
+  const size_t base = (size_t)src * D;
+  StreamRow<T, NT, NV> row;
+  row.load(stream, y, base, D, init != 0);
+  row.add(y != nullptr, w_post, D, eps, scratch);
+  if (inject) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (i * NT + threadIdx.x) * 4;
+      if (d < D) {
+        float e[4];
+        RowAccess<float, 4>::load(inject + base + d, e);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) row.x[i][j] += e[j];
+      }
+    }
+  }
+  if (!rows) {
+    if (init || y || inject) row.put(stream + base, row.x, D);
+    if (keep) row.put(keep + base, row.x, D);
+  }
+  if (!out) return;
+  float h[NV][4];
+  row.normed(row.inv_rms(D, eps, scratch), w_pre, D, h);
+  row.put(out + (size_t)r * D, h, D);
+}
+
+template <typename T, int NT, int NV>
+__global__ void __launch_bounds__(NT)
+residual_norm_shift_regs_kernel(const float* stream, float* stream_out, const T* y, const float* __restrict__ w_post,
+                                const float* __restrict__ w_pre, const float* __restrict__ shift, float* state, long state_stride,
+                                const int* __restrict__ token_req, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
+                                T* out, int num_tokens, int walk, int D, float eps, long num_slots, int* err) {
+  using Row = StreamRow<T, NT, NV>;
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  const int t0 = blockIdx.x * walk, t1 = min(num_tokens, t0 + walk);
+  int req = token_req[t0];
+  const bool ahead = req >= 0 && t0 > cu_q[req];        // the first token has one before it in its portion
+  pdl_wait();
+  float before[NV][4], h[NV][4];
+  Row next, row;
+  if (ahead) row.load(stream, y, (size_t)(t0 - 1) * D, D, false);
+  next.load(stream, y, (size_t)t0 * D, D, false);
+  if (ahead) {
+    row.add(y != nullptr, w_post, D, eps, scratch);
+    row.normed(row.inv_rms(D, eps, scratch), w_pre, D, before);
+  }
+  for (int t = t0; t < t1; ++t) {
+    row = next;
+    if (t + 1 < t1) next.load(stream, y, (size_t)(t + 1) * D, D, false);
+    req = token_req[t];
+    int slot = -1, first = t, last = t;
+    if (req >= 0) {
+      slot = state_slots[req];
+      first = cu_q[req];
+      last = cu_q[req + 1] - 1;
+      if (slot < 0 || slot >= num_slots) {
+        if (threadIdx.x == 0) atomicOr(err, VOB_ERR_SLOT);
+        slot = -1;
+      }
+    }
+    float* kept = slot >= 0 ? state + (size_t)slot * state_stride : nullptr;
+    if (t == first) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int d = (i * NT + threadIdx.x) * 4;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) before[i][j] = kept && d < D ? kept[d + j] : 0.f;
+      }
+    }
+    row.add(y != nullptr, w_post, D, eps, scratch);
+    if (y) Row::put(stream_out + (size_t)t * D, row.x, D);
+    row.normed(row.inv_rms(D, eps, scratch), w_pre, D, h);
+    if (kept && t == last && t == first) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int d = (i * NT + threadIdx.x) * 4;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (d < D) kept[d + j] = h[i][j];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (i * NT + threadIdx.x) * 4;
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
+      if (req >= 0 && d < D) RowAccess<float, 4>::load(shift + d, s);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float mixed = fmaf(before[i][j] - h[i][j], s[j], h[i][j]);
+        before[i][j] = h[i][j];
+        h[i][j] = req >= 0 ? mixed : h[i][j];
+      }
+    }
+    Row::put(out + (size_t)t * D, h, D);
+    if (kept && t == first && last > first) {
+      // the portion's last h into the slot: by the block that has just read the slot, so that nothing is overwritten early
+      row.load(stream, y, (size_t)last * D, D, false);
+      row.add(y != nullptr, w_post, D, eps, scratch);
+      row.normed(row.inv_rms(D, eps, scratch), w_pre, D, h);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int d = (i * NT + threadIdx.x) * 4;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (d < D) kept[d + j] = h[i][j];
+      }
+    }
+  }
+}
+
 // The normed row of token t, left in `row` as x (the caller multiplies by the returned 1 / rms); with `put` the new stream
 // row is stored.
 template <typename T, int V>
@@ -244,6 +443,23 @@ VOB_API int vob_residual_norm_step(float* stream, const void* y, const float* w_
   if (smem > 200 * 1024) return VOB_UNSUPPORTED;
   const bool vec = D % 4 == 0 && (((uintptr_t)stream | (uintptr_t)y | (uintptr_t)inject | (uintptr_t)keep | (uintptr_t)out |
                                     (uintptr_t)w_post | (uintptr_t)w_pre) % 16) == 0;
+#define VOB_RN_REGS(TYPE, NT, NV)                                                                                           \
+  return launch_kernel(residual_norm_step_regs_kernel<TYPE, NT, NV>, dim3(n_out), NT, 0, stream_, stream, (const TYPE*)y, w_post, \
+                       inject, keep, w_pre, (TYPE*)out, rows, num_src_rows, D, eps, init, err)
+#define VOB_RN_WIDTHS(TYPE)                    \
+  do {                                         \
+    if (D <= 512) VOB_RN_REGS(TYPE, 128, 1);   \
+    if (D <= 1024) VOB_RN_REGS(TYPE, 256, 1);  \
+    if (D <= 2048) VOB_RN_REGS(TYPE, 256, 2);  \
+    if (D <= 4096) VOB_RN_REGS(TYPE, 256, 4);  \
+    VOB_RN_REGS(TYPE, 512, 4);                 \
+  } while (0)
+  if (vec && D <= 8192) {
+    if (dtype == VOB_F32) VOB_RN_WIDTHS(float);
+    if (dtype == VOB_BF16) VOB_RN_WIDTHS(__nv_bfloat16);
+  }
+#undef VOB_RN_WIDTHS
+#undef VOB_RN_REGS
 #define VOB_RN_LAUNCH(TYPE, V)                                                                                            \
   do {                                                                                                                    \
     if (smem > 48 * 1024)                                                                                                 \
@@ -276,8 +492,27 @@ VOB_API int vob_residual_norm_shift_step(const float* stream, float* stream_out,
   const size_t smem = (size_t)2 * D * sizeof(float);
   if (smem > 200 * 1024) return VOB_UNSUPPORTED;
   const bool vec = D % 4 == 0 && (((uintptr_t)stream | (uintptr_t)stream_out | (uintptr_t)y | (uintptr_t)out) % 16) == 0;
+  const bool regs = vec && D <= 8192 && (((uintptr_t)w_post | (uintptr_t)w_pre | (uintptr_t)shift) % 16) == 0;
   // a block makes one row more than it walks: few tokens a block while they fill the device, up to eight beyond
   const int walk = max(1, min(8, T / (4 * sm_count())));
+#define VOB_RS_REGS(TYPE, NT, NV)                                                                                           \
+  return launch_kernel(residual_norm_shift_regs_kernel<TYPE, NT, NV>, dim3((T + walk - 1) / walk), NT, 0, stream_, stream,  \
+                       stream_out, (const TYPE*)y, w_post, w_pre, shift, state, state_stride, token_req, cu_q, state_slots, \
+                       (TYPE*)out, T, walk, D, eps, num_slots, err)
+#define VOB_RS_WIDTHS(TYPE)                    \
+  do {                                         \
+    if (D <= 512) VOB_RS_REGS(TYPE, 128, 1);   \
+    if (D <= 1024) VOB_RS_REGS(TYPE, 256, 1);  \
+    if (D <= 2048) VOB_RS_REGS(TYPE, 256, 2);  \
+    if (D <= 4096) VOB_RS_REGS(TYPE, 256, 4);  \
+    VOB_RS_REGS(TYPE, 512, 4);                 \
+  } while (0)
+  if (regs) {
+    if (dtype == VOB_F32) VOB_RS_WIDTHS(float);
+    if (dtype == VOB_BF16) VOB_RS_WIDTHS(__nv_bfloat16);
+  }
+#undef VOB_RS_WIDTHS
+#undef VOB_RS_REGS
 #define VOB_RS_LAUNCH(TYPE, V)                                                                                             \
   do {                                                                                                                     \
     if (smem > 48 * 1024)                                                                                                  \
