@@ -331,8 +331,9 @@ def test_recurrent_block(D, width, blocks, taps, dt):
              5e-5 if dt == torch.float32 else 0.04)
 
 
-def test_slow_channels_write_what_they_should():
-    """A decay of one minus 1e-6: 1 - a^2 as a difference of floats would be off by percents."""
+@pytest.mark.parametrize("n", [600, 1500])
+def test_slow_channels_write_what_they_should(n):
+    """A decay of one minus 1e-6: 1 - a^2 as a difference of floats would be off by percents.  (1,500 tokens: the most ranges.)"""
     from vllm_oxide_b200.parts import PartSpec, build_part
     D, W = 24, 32
     part = build_part("mixer", PartSpec("recurrent_block", dict(hidden_size=D, width=W, blocks=2, taps=3, prefix="m.")), dtype=torch.float32,
@@ -340,9 +341,9 @@ def test_slow_channels_write_what_they_should():
     w = draw(part, 51)
     w["m.lam"] = torch.linspace(-16.0, 4.0, W, dtype=torch.float64)
     load(part, w, torch.float32)
-    x = held(rand((600, D), 9), torch.float32)
+    x = held(rand((n, D), 9), torch.float32)
     want = P.recurrent_block(x, hold(part, w, torch.float32), "m.", dict(width=W, blocks=2), EPS, torch.float64)
-    run_cuts(part, x, [[600], [100, 1, 7]], want, torch.float32, "slow channels", 5e-5, pages=60)
+    run_cuts(part, x, [[n], [100, 1, 7]], want, torch.float32, "slow channels", 5e-5, pages=100)
 
 
 # ---------------------------------------------------------------- two mixers side by side, pages and slots used again

@@ -209,9 +209,6 @@ constexpr int DS_COMPUTE = 128;   // threads that hold the state
 constexpr int DS_LOADERS = 128;   // threads that prepare the next tokens meanwhile
 constexpr int DS_THREADS = DS_COMPUTE + DS_LOADERS;
 
-__device__ __forceinline__ void named_sync(int id, int count) { asm volatile("bar.sync %0, %1;\n" ::"r"(id), "r"(count) : "memory"); }
-__device__ __forceinline__ void named_arrive(int id, int count) { asm volatile("bar.arrive %0, %1;\n" ::"r"(id), "r"(count) : "memory"); }
-
 // qkv: float [tokens, 2 * kvh * dim + heads * vdim] (q heads, k heads, v heads: the convolutions' output);
 // ab: rows of ab_stride elements of T, beta's pre-activation of head h at b_off + h, the decay's at a_off + h.
 // A column of the state is held by LANES neighbouring threads, ROWS rows each (LANES * ROWS >= dim); 128 such threads

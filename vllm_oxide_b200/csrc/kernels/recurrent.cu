@@ -9,6 +9,10 @@
 namespace vob {
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+// The same for inputs of type T: behind 16-bit inputs the hardware's exponential and division (a few float units, far below
+// the input's own rounding) take a quarter of the instructions.
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float x) { return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-x)) : sigmoid_f(x); }
 // f = l + (1 - l) sigmoid(pre + bias): one spelling for every kernel that needs the gate
 __device__ __forceinline__ float forget_gate(float l, float pre, float bias) { return fmaf(1.f - l, sigmoid_f(pre + bias), l); }
 
@@ -96,22 +100,24 @@ mingru_scan_kernel(const T* zxg, const T* __restrict__ bz, const T* __restrict__
 // 1 - a^2 = -expm1(2 log a): the difference would lose what a slow channel (a near 1) writes.  Cut along the tokens as minGRU.
 struct LruStep { float a, b; };
 
+template <typename T>
 __device__ __forceinline__ LruStep lru_step(float gr, float gi, float u, float rate) {
-  const float log_a = rate * sigmoid_f(gr);
-  return {expf(log_a), sqrtf(-expm1f(2.f * log_a)) * sigmoid_f(gi) * u};
+  const float log_a = rate * sigmoid_t<T>(gr);
+  return {expf(log_a), sqrtf(-expm1f(2.f * log_a)) * sigmoid_t<T>(gi) * u};
 }
 
-template <typename T, int NCH>
-__global__ void __launch_bounds__(32 * NCH)
+// A block owns LANES channels: 32, or 16 with twice the ranges where a long portion would otherwise leave SMs without a block.
+template <typename T, int LANES, int NCH>
+__global__ void __launch_bounds__(LANES * NCH)
 lru_scan_kernel(const T* u, const float* gates, const T* y, long y_stride, const float* __restrict__ br, const float* __restrict__ bi,
                 const float* __restrict__ lam, const float* __restrict__ by, float* state, long state_stride,
                 const int* __restrict__ cu_q, const int* __restrict__ state_slots, T* out, int W, int per_block, int num_slots,
                 int* err) {
-  __shared__ float As[NCH][32], Bs[NCH][32];
+  __shared__ float As[NCH][LANES], Bs[NCH][LANES];
   pdl_launch_dependents();
   const int b = blockIdx.y, lane = threadIdx.x, ch = threadIdx.y;
-  const int c = min(blockIdx.x * 32 + lane, W - 1);
-  const bool live = blockIdx.x * 32 + lane < W;
+  const int c = min(blockIdx.x * LANES + lane, W - 1);
+  const bool live = blockIdx.x * LANES + lane < W;
   const int t0 = cu_q[b], t1 = cu_q[b + 1];
   const int slot = state_slots[b];
   const float l = lam[c], biasr = br[c], biasi = bi[c], biasy = by[c];
@@ -128,7 +134,7 @@ lru_scan_kernel(const T* u, const float* gates, const T* y, long y_stride, const
   float s = state[(size_t)slot * state_stride + c];
   auto step = [&](int t) {
     const float* g = gates + (size_t)t * 2 * W + goff;
-    return lru_step(g[0] + biasr, g[per_block] + biasi, to_f<T>(u[(size_t)t * W + c]), rate);
+    return lru_step<T>(g[0] + biasr, g[per_block] + biasi, to_f<T>(u[(size_t)t * W + c]), rate);
   };
   if (NCH > 1) {
     float A = 1.f, B = 0.f;
@@ -171,19 +177,22 @@ lru_scan_kernel(const T* u, const float* gates, const T* y, long y_stride, const
 //   HgrnSource       qfv [tokens, heads*dk | heads*dk | heads*dv]: q = silu(q), f = l + (1 - l) sigmoid(f + bf), w = 1 - f
 //   GlaSource        q * scale, w = k, f = sigmoid(z + bz)^(1 / tau) = exp(-softplus(-(z + bz)) / tau), a number a head and row
 //   LightningSource  q = silu(q), w = silu(k), v = silu(v), f = a fixed number a head
-// Column j of a head's state M (dk floats) is shared by PARTS neighbouring lanes, R rows each, in registers: a token costs
-// a thread R multiply-adds twice, and the lanes of a column add their parts of o by shuffles.  The gates of HG_TT tokens are
-// made by the whole block at once and parked in shared memory (rows padded so that the PARTS lanes of a column read
-// different banks).  FUSE: the block holds all dv columns of the head and also takes the norm over them (and what the source
-// puts behind it), for decoding: one launch; otherwise a block holds as many columns as 128 threads cover, so that a long
-// portion of one request spreads over more blocks, o leaves in float and a norm kernel follows.  Both give the same numbers:
-// an element's chain of operations depends on (R, PARTS) alone, and those follow from dk.
+// Decoding (matrix_scan_fused): one block a (request, head) that also takes the head's norm and what the source puts behind it.
+// Column j of a head's state M (dk floats) is shared by PARTS neighbouring lanes, R rows each, in registers.  The gates of
+// HG_TT tokens are made by the whole block at once and parked in shared memory (rows padded so that the PARTS lanes of a column
+// read different banks).
+//
+// Portions (matrix_scan_tile): a walker thread holds a tile of 8 rows x 8 columns of M in registers, as pairs of rows, so that
+// every gate it reads from shared memory serves 8 columns and every multiply-add instruction two elements; ceil(dk / 8) lanes
+// (a power of two) share 8 columns and halve their partial sums of o with every exchange.  Up to eight walker warps hold a
+// head; eight loader warps make the gates of the next HG_TT tokens meanwhile, in the other of two buffers (named barriers:
+// "full" when a buffer is ready, "empty" when its tokens have been walked).  o leaves in float and a norm kernel follows.
 //
 // A long portion is also cut along the tokens (`chunks` > 1, four launches): MODE 1 walks every range from a zero state
-// and leaves its end state L; hgrn2_range_gates_kernel takes the product F of every range's gates; hgrn2_join_kernel goes
+// and leaves its end state L; matrix_scan_range_decay takes the product F of every range's decays; matrix_scan_join goes
 // through the ranges in order,
 // M_start(c+1) = diag(F_c) M_start(c) + L_c, leaves every range's start where its L was and the last state in the
-// slot; MODE 2 walks the ranges again from their starts and writes the outputs.  Twice the arithmetic, on as many more
+// slot; MODE 2 walks the ranges again from their starts and writes the outputs.  Nearly twice the arithmetic, on as many more
 // blocks as there are ranges.  MODE 0 is the walk from the slot's state to the slot's state in one launch.
 constexpr int HG_TT = 16;
 
@@ -196,6 +205,7 @@ struct ScanGates { float q, f, w; };
 // What a source keeps of a (head, row) over the tokens, what it reads of a token, and what it makes of both.
 template <typename T>
 struct HgrnSource {
+  static constexpr bool FIXED_DECAY = false;
   const T* rows;
   long width;
   const T* bf;
@@ -210,18 +220,20 @@ struct HgrnSource {
   }
   __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed& x) const {
     const float f = forget_gate(x.l, r.f, x.bias);
-    return {r.q * sigmoid_f(r.q), f, 1.f - f};
+    return {r.q * sigmoid_t<T>(r.q), f, 1.f - f};
   }
   __device__ __forceinline__ float value(size_t t, int h, int c) const { return to_f<T>(rows[t * width + (size_t)2 * heads * dk + h * dv + c]); }
   __device__ __forceinline__ float decay(size_t t, int h, int i, const Fixed& x) const {
     return forget_gate(x.l, to_f<T>(rows[t * width + (size_t)(heads + h) * dk + i]), x.bias);
   }
+  __device__ __forceinline__ float fixed_decay(int) const { return 0.f; }
   __device__ __forceinline__ float finish(float o, size_t, int, int) const { return o; }
 };
 
 // rows: q | k | v (heads*dk, heads*dk, heads*dv), the decay's pre-activations at z_off, the output gate at gate_off.
 template <typename T>
 struct GlaSource {
+  static constexpr bool FIXED_DECAY = false;      // whether a head keeps by one number at every token
   const T* rows;
   long width;
   const float* bias;       // [heads * dk]
@@ -235,13 +247,17 @@ struct GlaSource {
     return {to_f<T>(row[h * dk + i]), to_f<T>(row[(heads + h) * dk + i]), to_f<T>(row[z_off + h * dk + i])};
   }
   // sigmoid(z)^(1/tau) by its logarithm: log sigmoid(z) = -softplus(-z) = min(z, 0) - log(1 + e^-|z|)
-  __device__ __forceinline__ float keep(float z) const { return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau); }
+  __device__ __forceinline__ float keep(float z) const {
+    if (sizeof(T) == 2) return __expf((fminf(z, 0.f) - __logf(1.f + __expf(-fabsf(z)))) * inv_tau);
+    return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
+  }
   __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed& x) const { return {r.q * scale, keep(r.z + x.bias), r.k}; }
   __device__ __forceinline__ float value(size_t t, int h, int c) const { return to_f<T>(rows[t * width + (size_t)2 * heads * dk + h * dv + c]); }
   __device__ __forceinline__ float decay(size_t t, int h, int i, const Fixed& x) const {
     return keep(to_f<T>(rows[t * width + z_off + (size_t)h * dk + i]) + x.bias);
   }
   // behind the head's norm: times silu(gate)
+  __device__ __forceinline__ float fixed_decay(int) const { return 0.f; }
   __device__ __forceinline__ float finish(float o, size_t t, int h, int c) const {
     const float g = to_f<T>(rows[t * width + gate_off + (size_t)h * dv + c]);
     return o * (g * sigmoid_f(g));
@@ -251,6 +267,7 @@ struct GlaSource {
 // rows: q | k | v (heads*dk, heads*dk, heads*dv).
 template <typename T>
 struct LightningSource {
+  static constexpr bool FIXED_DECAY = true;
   const T* rows;
   long width;
   const float* decays;     // [heads]
@@ -258,25 +275,25 @@ struct LightningSource {
   struct Fixed { float f; };
   struct Raw { float q, k; };
   __device__ __forceinline__ Fixed fixed(int h, int) const { return {decays[h]}; }
+  __device__ __forceinline__ float fixed_decay(int h) const { return decays[h]; }
   __device__ __forceinline__ Raw load(size_t t, int h, int i) const {
     const T* row = rows + t * width;
     return {to_f<T>(row[h * dk + i]), to_f<T>(row[(heads + h) * dk + i])};
   }
-  __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed& x) const { return {r.q * sigmoid_f(r.q), x.f, r.k * sigmoid_f(r.k)}; }
+  __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed& x) const { return {r.q * sigmoid_t<T>(r.q), x.f, r.k * sigmoid_t<T>(r.k)}; }
   __device__ __forceinline__ float value(size_t t, int h, int c) const {
     const float v = to_f<T>(rows[t * width + (size_t)2 * heads * dk + h * dv + c]);
-    return v * sigmoid_f(v);
+    return v * sigmoid_t<T>(v);
   }
   __device__ __forceinline__ float decay(size_t, int, int, const Fixed& x) const { return x.f; }
   __device__ __forceinline__ float finish(float o, size_t, int, int) const { return o; }
 };
 
-// FULL: dk = R * PARTS, every row a thread holds exists (no test per element: the tests were two of seven instructions).
-template <typename T, typename SOURCE, int R, int PARTS, bool FUSE, int MODE, bool FULL>
-__global__ void __launch_bounds__(FUSE ? (R > 32 ? 256 : 512) : 128)
-hgrn2_scan_kernel(const SOURCE src, const float* __restrict__ nw,
-                  float* state, long state_stride, const int* __restrict__ cu_q, const int* __restrict__ state_slots, T* out, float* raw,
-                  float* ends, int heads, int dk, int dv, int col_blocks, float eps, int num_slots, int* err) {
+// ---- decoding: a block a (request, head)
+template <typename T, typename SOURCE, int R, int PARTS>
+__global__ void __launch_bounds__(R > 32 ? 256 : 512)
+matrix_scan_fused_kernel(const SOURCE src, const float* __restrict__ nw, float* state, long state_stride, const int* __restrict__ cu_q,
+                         const int* __restrict__ state_slots, T* out, int heads, int dk, int dv, float eps, int num_slots, int* err) {
   extern __shared__ float4 sm4[];
   float* sm = reinterpret_cast<float*>(sm4);
   const int gate_row = hg_pad(R * PARTS);
@@ -285,10 +302,108 @@ hgrn2_scan_kernel(const SOURCE src, const float* __restrict__ nw,
   float* fs = qs + HG_TT * gate_row;     // [HG_TT][gate_row]  f
   float* gs = fs + HG_TT * gate_row;     // [HG_TT][gate_row]  w
   float* vs = gs + HG_TT * gate_row;     // [HG_TT][cols]
-  float* os = vs + HG_TT * cols;         // [HG_TT][cols]  (FUSE)
+  float* os = vs + HG_TT * cols;         // [HG_TT][cols]
   pdl_launch_dependents();
-  const int part = threadIdx.x % PARTS, jj = threadIdx.x / PARTS;
-  const int h = blockIdx.x / col_blocks, cb = blockIdx.x % col_blocks, j = cb * cols + jj;
+  const int part = threadIdx.x % PARTS, j = threadIdx.x / PARTS;
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int t0 = cu_q[b], t1 = cu_q[b + 1];
+  const int slot = state_slots[b];
+  pdl_wait();
+  if (t1 <= t0) return;
+  if (slot < 0 || slot >= num_slots) {
+    if (threadIdx.x == 0) atomicOr(err, VOB_ERR_SLOT);
+    return;
+  }
+  const int i0 = part * R;
+  float* mine = state + (size_t)slot * state_stride + ((size_t)h * dk + i0) * dv + j;
+  float M[R];
+#pragma unroll
+  for (int i = 0; i < R; ++i) M[i] = (i0 + i < dk && j < dv) ? mine[(size_t)i * dv] : 0.f;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+  // the gates of a tile: thread rows over tokens, thread columns over gates (one division, here)
+  const int gate_lanes = min(dk, (int)blockDim.x), gate_step = blockDim.x / gate_lanes;
+  const int gate_i = threadIdx.x % gate_lanes, gate_t = threadIdx.x / gate_lanes < gate_step ? threadIdx.x / gate_lanes : HG_TT;
+  for (int ts = t0; ts < t1; ts += HG_TT) {
+    const int n = min(HG_TT, t1 - ts);
+    for (int i = gate_i; i < dk; i += gate_lanes) {
+      const typename SOURCE::Fixed fx = src.fixed(h, i);
+      for (int tt = gate_t; tt < n; tt += gate_step) {
+        const ScanGates g = src.make(src.load((size_t)(ts + tt), h, i), fx);
+        qs[tt * gate_row + hg_pad(i)] = g.q;
+        fs[tt * gate_row + hg_pad(i)] = g.f;
+        gs[tt * gate_row + hg_pad(i)] = g.w;
+      }
+    }
+    for (int idx = threadIdx.x; idx < n * cols; idx += blockDim.x) {
+      const int tt = idx / cols, c = idx % cols;
+      vs[idx] = c < dv ? src.value((size_t)(ts + tt), h, c) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 2
+    for (int tt = 0; tt < n; ++tt) {
+      float o = 0.f;
+      const float v = vs[tt * cols + j];
+      const float* fr = fs + tt * gate_row + hg_pad(i0);
+      const float* gr = gs + tt * gate_row + hg_pad(i0);
+      const float* qr = qs + tt * gate_row + hg_pad(i0);
+#pragma unroll
+      for (int i = 0; i < R; i += 4) {
+        const float4 f4 = *reinterpret_cast<const float4*>(fr + hg_pad(i));      // hg_pad(i0 + i) = hg_pad(i0) + hg_pad(i)
+        const float4 g4 = *reinterpret_cast<const float4*>(gr + hg_pad(i));
+        const float4 q4 = *reinterpret_cast<const float4*>(qr + hg_pad(i));
+        const float fv[4] = {f4.x, f4.y, f4.z, f4.w}, gv[4] = {g4.x, g4.y, g4.z, g4.w}, qv[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (i0 + i + k < dk) {
+            M[i + k] = fmaf(fv[k], M[i + k], gv[k] * v);
+            o = fmaf(M[i + k], qv[k], o);
+          }
+      }
+#pragma unroll
+      for (int d = 1; d < PARTS; d <<= 1) o += __shfl_xor_sync(0xffffffffu, o, d);
+      if (part == 0) os[tt * cols + j] = o;
+    }
+    __syncthreads();
+    for (int tt = warp; tt < n; tt += nwarps) {
+      float ss = 0.f;
+      for (int c = lane; c < dv; c += 32) ss += os[tt * cols + c] * os[tt * cols + c];
+      const float denom = sqrtf(warp_sum(ss) / (float)dv + eps);
+      for (int c = lane; c < dv; c += 32)
+        out[(size_t)(ts + tt) * heads * dv + h * dv + c] = from_f<T>(src.finish(os[tt * cols + c] / denom * nw[c], (size_t)(ts + tt), h, c));
+    }
+    __syncthreads();
+  }
+  if (j < dv) {
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+      if (i0 + i < dk) mine[(size_t)i * dv] = M[i];
+  }
+}
+
+// ---- portions: walkers and loaders
+constexpr int MS_LOADERS = 256, MS_MAX_WALKERS = 256;
+constexpr int MS_R = 8, MS_C = 8;      // a walker's rows and columns
+
+// Where row i of a head lies among the PARTS * 8 gates of a token in shared memory: the first four rows of every part, then the
+// last four, so that the 16-byte reads of neighbouring parts are neighbours.
+template <int PARTS>
+__device__ __forceinline__ int tile_index(int i) { return (((i & 7) >> 2) * PARTS + (i >> 3)) * 4 + (i & 3); }
+
+// OUT: outputs are made (MODE 0 and 2 above); `mode` says where the walk starts and what it leaves.
+template <typename SOURCE, int PARTS, bool OUT>
+__global__ void __launch_bounds__(MS_LOADERS + MS_MAX_WALKERS, 1)
+matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const int* __restrict__ cu_q,
+                        const int* __restrict__ state_slots, float* raw, float* ends, int heads, int dk, int dv, int col_blocks,
+                        int num_slots, int mode, int* err) {
+  constexpr int W = PARTS * MS_R;              // gates of a token, rows past dk are zeros
+  constexpr bool FIXED = SOURCE::FIXED_DECAY;
+  extern __shared__ float4 sm4[];
+  const int walkers = blockDim.x - MS_LOADERS, threads = blockDim.x;
+  const int cols = walkers / PARTS * MS_C;     // columns of this block
+  const int buffer = HG_TT * ((FIXED ? 2 : 3) * W + cols);
+  float* sm = reinterpret_cast<float*>(sm4);
+  pdl_launch_dependents();
+  const int h = blockIdx.x / col_blocks, c0 = blockIdx.x % col_blocks * cols;
   const int b = blockIdx.y, chunk = blockIdx.z, chunks = gridDim.z;
   const int q0 = cu_q[b], q1 = cu_q[b + 1];
   const int slot = state_slots[b];
@@ -300,89 +415,206 @@ hgrn2_scan_kernel(const SOURCE src, const float* __restrict__ nw,
   }
   const int per = (q1 - q0 + chunks - 1) / chunks;
   const int t0 = min(q1, q0 + chunk * per), t1 = min(q1, t0 + per);
-  const int i0 = part * R;
-  float* mine = MODE == 0 ? state + (size_t)slot * state_stride + ((size_t)h * dk + i0) * dv + j
-                          : ends + ((((size_t)b * chunks + chunk) * heads + h) * dk + i0) * dv + j;
-  float M[R];
+  const int tiles = (t1 - t0 + HG_TT - 1) / HG_TT;
+  if ((int)threadIdx.x >= walkers) {
+    // ------------------------------------------------ loaders
+    const int tid = threadIdx.x - walkers;
+    const int gate_lanes = min(dk, MS_LOADERS), gate_step = MS_LOADERS / gate_lanes;
+    const int gate_i = tid % gate_lanes, gate_t = tid / gate_lanes < gate_step ? tid / gate_lanes : HG_TT;
+    // rows past dk: zeros in both buffers, once
+    for (int k = 0; k < 2; ++k)
+      for (int idx = tid; idx < HG_TT * (W - dk); idx += MS_LOADERS) {
+        float* q = sm + k * buffer + idx / (W - dk) * W + tile_index<PARTS>(dk + idx % (W - dk));
+        q[0] = 0.f;
+        q[HG_TT * W] = 0.f;
+        if (!FIXED) q[2 * HG_TT * W] = 0.f;
+      }
+    for (int k = 0; k < tiles; ++k) {
+      float* qs = sm + (k & 1) * buffer;       // [HG_TT][W] q
+      float* ws = qs + HG_TT * W;              // [HG_TT][W] w
+      float* fs = ws + HG_TT * W;              // [HG_TT][W] f (not where it is one number a head)
+      float* vs = qs + HG_TT * (FIXED ? 2 : 3) * W;      // [HG_TT][cols]
+      const int ts = t0 + k * HG_TT, n = min(HG_TT, t1 - ts);
+      if (k >= 2) named_sync(3 + (k & 1), threads);      // the walkers have left this buffer
+      for (int i = gate_i; i < dk; i += gate_lanes) {
+        const typename SOURCE::Fixed fx = src.fixed(h, i);
+        const int at = tile_index<PARTS>(i);
+        // eight tokens' loads are issued before the first of them is used
+        for (int tb = gate_t; tb < n; tb += 8 * gate_step) {
+          typename SOURCE::Raw raws[8];
 #pragma unroll
-  for (int i = 0; i < R; ++i) M[i] = (MODE != 1 && i0 + i < dk && j < dv) ? mine[(size_t)i * dv] : 0.f;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
-  // the gates of a tile: thread rows over tokens, thread columns over gates (one division, here)
-  const int gate_lanes = min(dk, (int)blockDim.x), gate_step = blockDim.x / gate_lanes;
-  const int gate_i = threadIdx.x % gate_lanes, gate_t = threadIdx.x / gate_lanes < gate_step ? threadIdx.x / gate_lanes : HG_TT;
-  for (int ts = t0; ts < t1; ts += HG_TT) {
-    const int n = min(HG_TT, t1 - ts);
-    for (int i = gate_i; i < dk; i += gate_lanes) {
-      const typename SOURCE::Fixed fx = src.fixed(h, i);
-      // eight tokens' loads are issued before the first of them is used
-      for (int tb = gate_t; tb < n; tb += 8 * gate_step) {
-        typename SOURCE::Raw raws[8];
+          for (int e = 0; e < 8; ++e) raws[e] = src.load((size_t)(ts + min(tb + e * gate_step, n - 1)), h, i);
 #pragma unroll
-        for (int k = 0; k < 8; ++k) raws[k] = src.load((size_t)(ts + min(tb + k * gate_step, n - 1)), h, i);
-#pragma unroll
-        for (int k = 0; k < 8; ++k) {
-          const int tt = tb + k * gate_step;
-          if (tt < n) {
-            const ScanGates g = src.make(raws[k], fx);
-            if (MODE != 1) qs[tt * gate_row + hg_pad(i)] = g.q;
-            fs[tt * gate_row + hg_pad(i)] = g.f;
-            gs[tt * gate_row + hg_pad(i)] = g.w;
+          for (int e = 0; e < 8; ++e) {
+            const int tt = tb + e * gate_step;
+            if (tt < n) {
+              const ScanGates g = src.make(raws[e], fx);
+              if (OUT) qs[tt * W + at] = g.q;
+              ws[tt * W + at] = g.w;
+              if (!FIXED) fs[tt * W + at] = g.f;
+            }
           }
         }
       }
-    }
-    for (int idx = threadIdx.x; idx < n * cols; idx += blockDim.x) {
-      const int tt = idx / cols, c = idx % cols;
-      vs[idx] = cb * cols + c < dv ? src.value((size_t)(ts + tt), h, cb * cols + c) : 0.f;
-    }
-    __syncthreads();
-#pragma unroll 2
-    for (int tt = 0; tt < n; ++tt) {
-      float o = 0.f;
-      const float v = vs[tt * cols + jj];
-      const float* fr = fs + tt * gate_row + hg_pad(i0);
-      const float* gr = gs + tt * gate_row + hg_pad(i0);
-      const float* qr = qs + tt * gate_row + hg_pad(i0);
+      // (a thread keeps its column, eight tokens' loads in flight)
+      const int v_lanes = min(cols, MS_LOADERS), v_step = MS_LOADERS / v_lanes;
+      for (int c = tid % v_lanes; c < cols; c += v_lanes)
+        for (int tb = tid / v_lanes; tb < n; tb += 8 * v_step) {
+          float v[8];
 #pragma unroll
-      for (int i = 0; i < R; i += 4) {
-        const float4 f4 = *reinterpret_cast<const float4*>(fr + hg_pad(i));      // hg_pad(i0 + i) = hg_pad(i0) + hg_pad(i)
-        const float4 g4 = *reinterpret_cast<const float4*>(gr + hg_pad(i));
-        const float4 q4 = MODE == 1 ? f4 : *reinterpret_cast<const float4*>(qr + hg_pad(i));
-        const float fv[4] = {f4.x, f4.y, f4.z, f4.w}, gv[4] = {g4.x, g4.y, g4.z, g4.w}, qv[4] = {q4.x, q4.y, q4.z, q4.w};
+          for (int e = 0; e < 8; ++e) v[e] = c0 + c < dv ? src.value((size_t)(ts + min(tb + e * v_step, n - 1)), h, c0 + c) : 0.f;
 #pragma unroll
-        for (int k = 0; k < 4; ++k)
-          if (FULL || i0 + i + k < dk) {
-            M[i + k] = fmaf(fv[k], M[i + k], gv[k] * v);
-            if (MODE != 1) o = fmaf(M[i + k], qv[k], o);
-          }
-      }
-      if (MODE != 1) {
-#pragma unroll
-        for (int d = 1; d < PARTS; d <<= 1) o += __shfl_xor_sync(0xffffffffu, o, d);
-        if (FUSE) {
-          if (part == 0) os[tt * cols + jj] = o;
-        } else if (part == 0 && j < dv) {
-          raw[(size_t)(ts + tt) * heads * dv + h * dv + j] = o;
+          for (int e = 0; e < 8; ++e)
+            if (tb + e * v_step < n) vs[(tb + e * v_step) * cols + c] = v[e];
         }
-      }
+      __threadfence_block();
+      named_arrive(1 + (k & 1), threads);
     }
-    __syncthreads();
-    if (FUSE && MODE != 1) {
-      for (int tt = warp; tt < n; tt += nwarps) {
-        float ss = 0.f;
-        for (int c = lane; c < dv; c += 32) ss += os[tt * cols + c] * os[tt * cols + c];
-        const float denom = sqrtf(warp_sum(ss) / (float)dv + eps);
-        for (int c = lane; c < dv; c += 32)
-          out[(size_t)(ts + tt) * heads * dv + h * dv + c] = from_f<T>(src.finish(os[tt * cols + c] / denom * nw[c], (size_t)(ts + tt), h, c));
-      }
-      __syncthreads();
-    }
+    return;
   }
-  if (MODE == 2) return;
-  if (j < dv) {
+  // -------------------------------------------------- walkers
+  const int part = threadIdx.x % PARTS, group = threadIdx.x / PARTS;
+  const int j0 = c0 + group * MS_C, i0 = part * MS_R;
+  float* mine = mode == 0 ? state + (size_t)slot * state_stride + (size_t)h * dk * dv
+                          : ends + (((size_t)b * chunks + chunk) * heads + h) * dk * dv;
+  // (a head's matrix starts on a 16-byte boundary where the state's rows do)
+  const bool wide = dv % 4 == 0 && (((uintptr_t)mine) & 15) == 0;
+  f32x2 M[MS_C][MS_R / 2];
 #pragma unroll
-    for (int i = 0; i < R; ++i)
-      if (i0 + i < dk) mine[(size_t)i * dv] = M[i];
+  for (int r = 0; r < MS_R; r += 2) {
+    float a[2][MS_C];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int i = i0 + r + e;
+      const float* row = mine + (size_t)i * dv + j0;
+#pragma unroll
+      for (int c = 0; c < MS_C; c += 4) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (OUT && i < dk) {
+          if (wide) {
+            if (j0 + c < dv) x = *reinterpret_cast<const float4*>(row + c);
+          } else {
+            if (j0 + c < dv) x.x = row[c];
+            if (j0 + c + 1 < dv) x.y = row[c + 1];
+            if (j0 + c + 2 < dv) x.z = row[c + 2];
+            if (j0 + c + 3 < dv) x.w = row[c + 3];
+          }
+        }
+        a[e][c] = x.x; a[e][c + 1] = x.y; a[e][c + 2] = x.z; a[e][c + 3] = x.w;
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < MS_C; ++c) M[c][r / 2] = pack2(a[0][c], a[1][c]);
+  }
+  f32x2 f2[MS_R / 2];
+  if (FIXED) {
+    const float f = src.fixed_decay(h);
+#pragma unroll
+    for (int p = 0; p < MS_R / 2; ++p) f2[p] = pack2(f, f);
+  }
+  // the columns whose sums end in this lane
+  constexpr int HALVINGS = PARTS >= 8 ? 3 : (PARTS >= 4 ? 2 : (PARTS >= 2 ? 1 : 0));
+  constexpr int OWN = MS_C >> HALVINGS;
+  int own = 0;
+#pragma unroll
+  for (int k = 0; k < HALVINGS; ++k)
+    if (part & (1 << k)) own += MS_C >> (k + 1);
+  const bool writes = PARTS <= 8 || part < 8;
+  for (int k = 0; k < tiles; ++k) {
+    const float* qs = sm + (k & 1) * buffer;
+    const float* ws = qs + HG_TT * W;
+    const float* fs = ws + HG_TT * W;
+    const float* vs = qs + HG_TT * (FIXED ? 2 : 3) * W;
+    const int ts = t0 + k * HG_TT, n = min(HG_TT, t1 - ts);
+    named_sync(1 + (k & 1), threads);
+#pragma unroll 1
+    for (int tt = 0; tt < n; ++tt) {
+      f32x2 w2[MS_R / 2], q2[MS_R / 2];
+#pragma unroll
+      for (int p = 0; p < 2; ++p) {
+        const int at = tt * W + (p * PARTS + part) * 4;
+        const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(ws + at);
+        w2[2 * p] = w.x; w2[2 * p + 1] = w.y;
+        if (OUT) {
+          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(qs + at);
+          q2[2 * p] = q.x; q2[2 * p + 1] = q.y;
+        }
+        if (!FIXED) {
+          const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(fs + at);
+          f2[2 * p] = f.x; f2[2 * p + 1] = f.y;
+        }
+      }
+      float v[MS_C], o[MS_C];
+      {
+        const float4* v4 = reinterpret_cast<const float4*>(vs + tt * cols + group * MS_C);
+        const float4 a = v4[0], c = v4[1];
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = c.x; v[5] = c.y; v[6] = c.z; v[7] = c.w;
+      }
+#pragma unroll
+      for (int c = 0; c < MS_C; ++c) {
+        const f32x2 v2 = pack2(v[c], v[c]);
+        f32x2 o2 = 0ull;
+#pragma unroll
+        for (int p = 0; p < MS_R / 2; ++p) {
+          M[c][p] = fma2(f2[p], M[c][p], mul2(w2[p], v2));
+          if (OUT) o2 = p == 0 ? mul2(M[c][p], q2[p]) : fma2(M[c][p], q2[p], o2);
+        }
+        if (OUT) {
+          const float2 s = unpack2(o2);
+          o[c] = s.x + s.y;
+        }
+      }
+      if (OUT) {
+        // every exchange halves the columns a lane still sums, until each has its own
+#pragma unroll
+        for (int e = 0; e < HALVINGS; ++e) {
+          const int half = MS_C >> (e + 1);
+          const bool upper = part & (1 << e);
+#pragma unroll
+          for (int c = 0; c < MS_C / 2; ++c)
+            if (c < half) {
+              const float give = upper ? o[c] : o[c + half], keep = upper ? o[c + half] : o[c];
+              o[c] = keep + __shfl_xor_sync(0xffffffffu, give, 1 << e);
+            }
+        }
+#pragma unroll
+        for (int d = 8; d < PARTS; d <<= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], d);
+        if (writes) {
+          float* dst = raw + (size_t)(ts + tt) * heads * dv + (size_t)h * dv + j0 + own;
+#pragma unroll
+          for (int c = 0; c < OWN; ++c)
+            if (j0 + own + c < dv) dst[c] = o[c];
+        }
+      }
+    }
+    if (k + 2 < tiles) named_arrive(3 + (k & 1), threads);
+  }
+  if (mode == 2) return;
+#pragma unroll
+  for (int r = 0; r < MS_R; r += 2) {
+    float a[2][MS_C];
+#pragma unroll
+    for (int c = 0; c < MS_C; ++c) {
+      const float2 x = unpack2(M[c][r / 2]);
+      a[0][c] = x.x;
+      a[1][c] = x.y;
+    }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int i = i0 + r + e;
+      if (i >= dk) continue;
+      float* row = mine + (size_t)i * dv + j0;
+#pragma unroll
+      for (int c = 0; c < MS_C; c += 4) {
+        if (wide) {
+          if (j0 + c < dv) *reinterpret_cast<float4*>(row + c) = make_float4(a[e][c], a[e][c + 1], a[e][c + 2], a[e][c + 3]);
+        } else {
+#pragma unroll
+          for (int d = 0; d < 4; ++d)
+            if (j0 + c + d < dv) row[c + d] = a[e][c + d];
+        }
+      }
+    }
   }
 }
 
@@ -391,7 +623,7 @@ hgrn2_scan_kernel(const SOURCE src, const float* __restrict__ nw,
 // in the order of the warps.
 template <typename SOURCE>
 __global__ void __launch_bounds__(256)
-hgrn2_range_gates_kernel(const SOURCE src, float* gates, const int* __restrict__ cu_q, int heads, int dk) {
+matrix_scan_range_decay_kernel(const SOURCE src, float* gates, const int* __restrict__ cu_q, int heads, int dk) {
   __shared__ float part[8][32];
   pdl_launch_dependents();
   pdl_wait();
@@ -420,7 +652,7 @@ hgrn2_range_gates_kernel(const SOURCE src, float* gates, const int* __restrict__
 // thread's loads are issued before its first store (at most HG_MAX_CHUNKS ranges), or every store would wait for a load.
 constexpr int HG_MAX_CHUNKS = 16;
 
-__global__ void hgrn2_join_kernel(float* state, long state_stride, float* ends, const float* gates, const int* __restrict__ cu_q,
+__global__ void matrix_scan_join_kernel(float* state, long state_stride, float* ends, const float* gates, const int* __restrict__ cu_q,
                                   const int* __restrict__ state_slots, int chunks, int heads, int dk, int dv, int num_slots) {
   pdl_launch_dependents();
   pdl_wait();
@@ -460,44 +692,69 @@ __global__ void head_gain_norm_kernel(const float* raw, const float* __restrict_
   for (int c = lane; c < dv; c += 32) out[(size_t)row * dv + c] = from_f<T>(x[c] / denom * w[c]);
 }
 
-template <typename T, typename SOURCE, int R, int PARTS, int MODE>
-int launch_hgrn2(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
-                 void* out, float* raw, float* ends, int B, int chunks, int heads, int dk, int dv, float eps, int num_slots, int fuse,
-                 int* err, cudaStream_t stream) {
+// rows of the state a thread of the fused kernel keeps, and lanes that share a column: from dk alone
+inline int fused_parts(int dk) { return dk <= 32 ? 1 : dk <= 64 ? 2 : 4; }
+inline bool scan_can_fuse(int dk, int dv) { return dv * fused_parts(dk) <= (dk > 128 ? 256 : 512); }
+
+template <typename T, typename SOURCE, int R, int PARTS>
+int launch_scan_fused(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
+                      void* out, int B, int heads, int dk, int dv, float eps, int num_slots, int* err, cudaStream_t stream) {
   const int gate_row = R * PARTS + 4 * ((R * PARTS) / 32);
-  const int threads = fuse ? (dv * PARTS + 31) / 32 * 32 : 128;
-  const int cols = threads / PARTS;
-  const int col_blocks = fuse ? 1 : (dv + cols - 1) / cols;
-  const size_t smem = ((size_t)3 * HG_TT * gate_row + (fuse ? 2 : 1) * (size_t)HG_TT * cols) * sizeof(float);
-  dim3 grid(heads * col_blocks, B, chunks);
-  auto launch = [&](auto kernel) -> int {
-    if (smem > 48 * 1024) {      // a head of 256 gates: three rows of gates for 16 tokens pass the default limit
-      cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      if (e != cudaSuccess) return (int)e;
-    }
-    return launch_kernel(kernel, grid, dim3(threads), smem, stream, src, nw, state, state_stride, cu_q, state_slots,
-                         (T*)out, raw, ends, heads, dk, dv, col_blocks, eps, num_slots, err);
-  };
-  if (fuse) return launch(hgrn2_scan_kernel<T, SOURCE, R, PARTS, true, 0, false>);
-  if (dk == R * PARTS) return launch(hgrn2_scan_kernel<T, SOURCE, R, PARTS, false, MODE, true>);
-  return launch(hgrn2_scan_kernel<T, SOURCE, R, PARTS, false, MODE, false>);
+  const int threads = (dv * PARTS + 31) / 32 * 32, cols = threads / PARTS;
+  const size_t smem = ((size_t)3 * HG_TT * gate_row + 2 * (size_t)HG_TT * cols) * sizeof(float);
+  auto kernel = matrix_scan_fused_kernel<T, SOURCE, R, PARTS>;
+  if (smem > 48 * 1024) {      // a head of 256 gates: three rows of gates for 16 tokens pass the default limit
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return launch_kernel(kernel, dim3(heads, B), dim3(threads), smem, stream, src, nw, state, state_stride, cu_q, state_slots, (T*)out,
+                       heads, dk, dv, eps, num_slots, err);
 }
 
-// rows of the state a thread keeps, and lanes that share a column: from dk alone
-inline int hgrn2_parts(int dk) { return dk <= 32 ? 1 : dk <= 64 ? 2 : 4; }
-inline bool hgrn2_can_fuse(int dk, int dv) { return dv * hgrn2_parts(dk) <= (dk > 128 ? 256 : 512); }
+inline int tile_parts(int dk) {
+  int p = 2;
+  while (p * MS_R < dk) p <<= 1;
+  return p;
+}
+// walker threads of a block, and blocks a head
+inline int tile_walkers(int dk, int dv) {
+  const int per_warp = 32 / tile_parts(dk) * MS_C;
+  return min(MS_MAX_WALKERS, (dv + per_warp - 1) / per_warp * 32);
+}
+inline int tile_col_blocks(int dk, int dv) {
+  const int cols = tile_walkers(dk, dv) / tile_parts(dk) * MS_C;
+  return (dv + cols - 1) / cols;
+}
 
-template <typename T, typename SOURCE, int MODE>
-int dispatch_hgrn2_mode(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
-                        void* out, float* raw, float* ends, int B, int chunks, int heads, int dk, int dv, float eps, int num_slots,
-                        int fuse, int* err, cudaStream_t stream) {
-#define VOB_HG(RR, PP) return launch_hgrn2<T, SOURCE, RR, PP, MODE>(src, nw, state, state_stride, cu_q, state_slots, out, raw, ends, B, chunks, heads, dk, dv, eps, num_slots, fuse, err, stream)
-  if (dk <= 16) VOB_HG(16, 1);
-  if (dk <= 32) VOB_HG(32, 1);
-  if (dk <= 64) VOB_HG(32, 2);
-  if (dk <= 128) VOB_HG(32, 4);
-  VOB_HG(64, 4);
-#undef VOB_HG
+template <typename SOURCE, int PARTS, bool OUT>
+int launch_scan_tile(const SOURCE& src, float* state, long state_stride, const int* cu_q, const int* state_slots, float* raw, float* ends,
+                     int B, int chunks, int heads, int dk, int dv, int num_slots, int mode, int* err, cudaStream_t stream) {
+  const int walkers = tile_walkers(dk, dv), cols = walkers / PARTS * MS_C, col_blocks = tile_col_blocks(dk, dv);
+  const size_t smem = (size_t)2 * HG_TT * ((SOURCE::FIXED_DECAY ? 2 : 3) * PARTS * MS_R + cols) * sizeof(float);
+  auto kernel = matrix_scan_tile_kernel<SOURCE, PARTS, OUT>;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return launch_kernel(kernel, dim3(heads * col_blocks, B, chunks), dim3(MS_LOADERS + walkers), smem, stream, src, state, state_stride,
+                       cu_q, state_slots, raw, ends, heads, dk, dv, col_blocks, num_slots, mode, err);
+}
+
+template <typename SOURCE>
+int dispatch_scan_tile(int mode, const SOURCE& src, float* state, long state_stride, const int* cu_q, const int* state_slots, float* raw, float* ends,
+                       int B, int chunks, int heads, int dk, int dv, int num_slots, int* err, cudaStream_t stream) {
+#define VOB_MT(PP)                                                                                                                 \
+  case PP:                                                                                                                         \
+    if (mode == 1)                                                                                                                 \
+      return launch_scan_tile<SOURCE, PP, false>(src, state, state_stride, cu_q, state_slots, raw, ends, B, chunks, heads, dk, dv, \
+                                                 num_slots, mode, err, stream);                                                    \
+    return launch_scan_tile<SOURCE, PP, true>(src, state, state_stride, cu_q, state_slots, raw, ends, B, chunks, heads, dk, dv,    \
+                                              num_slots, mode, err, stream)
+  switch (tile_parts(dk)) {
+    VOB_MT(2); VOB_MT(4); VOB_MT(8); VOB_MT(16); VOB_MT(32);
+  }
+#undef VOB_MT
+  return VOB_UNSUPPORTED;
 }
 
 // The recurrence of any source over a step; with `norm` the head norm that follows an unfused walk.
@@ -505,30 +762,39 @@ template <typename T, typename SOURCE>
 int run_matrix_scan(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
                     void* out, float* raw, float* scratch, int Tn, int B, int chunks, int heads, int dk, int dv, float eps,
                     int num_slots, int fuse, int norm, int* err, cudaStream_t stream) {
-  if (heads <= 0 || dk <= 0 || dv <= 0 || dk > 256 || B > 65535 || (!fuse && !raw) || (fuse && !hgrn2_can_fuse(dk, dv)) ||
+  if (heads <= 0 || dk <= 0 || dv <= 0 || dk > 256 || B > 65535 || (!fuse && !raw) || (fuse && !scan_can_fuse(dk, dv)) ||
       chunks < 1 || chunks > HG_MAX_CHUNKS || (chunks > 1 && (fuse || !scratch)) || state_stride < (long)heads * dk * dv)
     return VOB_UNSUPPORTED;
   int code;
+  if (fuse) {
+#define VOB_SF(RR, PP) return launch_scan_fused<T, SOURCE, RR, PP>(src, nw, state, state_stride, cu_q, state_slots, out, B, heads, dk, dv, eps, num_slots, err, stream)
+    if (dk <= 16) VOB_SF(16, 1);
+    if (dk <= 32) VOB_SF(32, 1);
+    if (dk <= 64) VOB_SF(32, 2);
+    if (dk <= 128) VOB_SF(32, 4);
+    VOB_SF(64, 4);
+#undef VOB_SF
+  }
   if (chunks <= 1) {
-    code = dispatch_hgrn2_mode<T, SOURCE, 0>(src, nw, state, state_stride, cu_q, state_slots, out, raw, nullptr, B, 1, heads, dk, dv,
-                                             eps, num_slots, fuse, err, stream);
+    code = dispatch_scan_tile(0, src, state, state_stride, cu_q, state_slots, raw, nullptr, B, 1, heads, dk, dv, num_slots, err,
+                                         stream);
   } else {
     float* ends = scratch;
     float* gates = scratch + (size_t)B * chunks * heads * dk * dv;
-    code = dispatch_hgrn2_mode<T, SOURCE, 1>(src, nw, state, state_stride, cu_q, state_slots, out, raw, ends, B, chunks, heads, dk, dv,
-                                             eps, num_slots, 0, err, stream);
+    code = dispatch_scan_tile(1, src, state, state_stride, cu_q, state_slots, raw, ends, B, chunks, heads, dk, dv, num_slots, err,
+                                         stream);
     if (code != 0) return code;
-    code = launch_kernel(hgrn2_range_gates_kernel<SOURCE>, dim3((heads * dk + 31) / 32, B, chunks), dim3(256), 0, stream, src, gates,
+    code = launch_kernel(matrix_scan_range_decay_kernel<SOURCE>, dim3((heads * dk + 31) / 32, B, chunks), dim3(256), 0, stream, src, gates,
                          cu_q, heads, dk);
     if (code != 0) return code;
     const long per = (long)heads * dk * dv;
-    code = launch_kernel(hgrn2_join_kernel, dim3((unsigned)((per + 255) / 256), B), dim3(256), 0, stream, state, state_stride, ends,
+    code = launch_kernel(matrix_scan_join_kernel, dim3((unsigned)((per + 255) / 256), B), dim3(256), 0, stream, state, state_stride, ends,
                          (const float*)gates, cu_q, state_slots, chunks, heads, dk, dv, num_slots);
     if (code != 0) return code;
-    code = dispatch_hgrn2_mode<T, SOURCE, 2>(src, nw, state, state_stride, cu_q, state_slots, out, raw, ends, B, chunks, heads, dk, dv,
-                                             eps, num_slots, 0, err, stream);
+    code = dispatch_scan_tile(2, src, state, state_stride, cu_q, state_slots, raw, ends, B, chunks, heads, dk, dv, num_slots, err,
+                                         stream);
   }
-  if (code != 0 || fuse || !norm) return code;
+  if (code != 0 || !norm) return code;
   const int rows = Tn * heads;
   return launch_kernel(head_gain_norm_kernel<T>, dim3((rows + 3) / 4), dim3(128), 0, stream, (const float*)raw, nw, (T*)out, rows, dv,
                        eps);
@@ -568,7 +834,23 @@ VOB_API int vob_mingru_scan(const void* zxg, const void* bz, const void* bx, flo
 // be able to hold the head: vob_hgrn2_can_fuse); else blocks of 128 threads and raw, float [T, heads*dv], in between.
 // `chunks` > 1 (not with fuse): ranges that a request's tokens are cut into, with scratch of
 // B * chunks * heads * dk * (dv + 1) floats.
-VOB_API int vob_hgrn2_can_fuse(int dk, int dv) { return hgrn2_can_fuse(dk, dv) ? 1 : 0; }
+VOB_API int vob_hgrn2_can_fuse(int dk, int dv) { return scan_can_fuse(dk, dv) ? 1 : 0; }
+
+// Ranges that a request's tokens of a step should be cut into (unfused walks): the fewest units of time by a count of float
+// instructions a state element (three a token in one walk, five over the two walks of a cut portion, and what the join and the
+// launches cost in tokens), given how many blocks fit the device at once.
+VOB_API int vob_matrix_scan_chunks(int T, int B, int heads, int dk, int dv) {
+  if (B <= 0 || T <= 0 || heads <= 0 || dk <= 0 || dv <= 0) return 1;
+  const long blocks = (long)heads * tile_col_blocks(dk, dv) * B, sms = sm_count();
+  const double n = (double)T / B;
+  int best = 1;
+  double least = 3.0 * n * ((blocks + sms - 1) / sms);
+  for (int c = 2; c <= HG_MAX_CHUNKS && n / c >= 16; ++c) {
+    const double cost = (5.0 * n / c + 120.0) * ((blocks * c + sms - 1) / sms) + 60.0;
+    if (cost < least) { least = cost; best = c; }
+  }
+  return best;
+}
 
 VOB_API int vob_hgrn2_scan(const void* qfv, const void* bf, const float* lower, const float* nw, float* state, const int* cu_q,
                            const int* state_slots, void* out, float* raw, float* scratch, int T, int B, int chunks, int heads,
@@ -618,28 +900,28 @@ VOB_API int vob_lightning_scan(const void* rows, long width, const float* decays
 }
 
 // u and out [T, W] of `dtype`; gates float [T, blocks, 2, W / blocks]; y rows of y_stride elements of `dtype`; br, bi, lam, by
-// float [W]; state float [num_slots, state_stride], the W channels first.  `chunks`: 1, 8 or 32 ranges a request's tokens are
-// cut into.
+// float [W]; state float [num_slots, state_stride], the W channels first.  `chunks`: 1, 8, 32 or 64 ranges a request's tokens
+// are cut into.
 VOB_API int vob_lru_scan(const void* u, const float* gates, const void* y, long y_stride, const float* br, const float* bi,
                          const float* lam, const float* by, float* state, long state_stride, const int* cu_q,
                          const int* state_slots, void* out, int B, int W, int blocks, int num_slots, int chunks, int dtype, int* err,
                          cudaStream_t stream) {
   if (B <= 0 || W <= 0) return 0;
-  if (B > 65535 || blocks <= 0 || W % blocks || state_stride < W || (chunks != 1 && chunks != 8 && chunks != 32)) return VOB_UNSUPPORTED;
-  dim3 grid((W + 31) / 32, B), block(32, chunks);
-#define VOB_LRU(TT, NN)                                                                                                        \
-  return launch_kernel(lru_scan_kernel<TT, NN>, grid, block, 0, stream, (const TT*)u, gates, (const TT*)y, y_stride, br, bi, lam, \
-                       by, state, state_stride, cu_q, state_slots, (TT*)out, W, W / blocks, num_slots, err)
-  if (dtype == VOB_F32) {
-    if (chunks == 1) VOB_LRU(float, 1);
-    if (chunks == 8) VOB_LRU(float, 8);
-    VOB_LRU(float, 32);
-  }
-  if (dtype == VOB_BF16) {
-    if (chunks == 1) VOB_LRU(__nv_bfloat16, 1);
-    if (chunks == 8) VOB_LRU(__nv_bfloat16, 8);
-    VOB_LRU(__nv_bfloat16, 32);
-  }
+  if (B > 65535 || blocks <= 0 || W % blocks || state_stride < W || (chunks != 1 && chunks != 8 && chunks != 32 && chunks != 64)) return VOB_UNSUPPORTED;
+#define VOB_LRU(TT, LL, NN)                                                                                                     \
+  return launch_kernel(lru_scan_kernel<TT, LL, NN>, dim3((W + LL - 1) / LL, B), dim3(LL, NN), 0, stream, (const TT*)u, gates,   \
+                       (const TT*)y, y_stride, br, bi, lam, by, state, state_stride, cu_q, state_slots, (TT*)out, W, W / blocks, \
+                       num_slots, err)
+#define VOB_LRU_CHUNKS(TT)            \
+  do {                                \
+    if (chunks == 1) VOB_LRU(TT, 32, 1);   \
+    if (chunks == 8) VOB_LRU(TT, 32, 8);   \
+    if (chunks == 32) VOB_LRU(TT, 32, 32); \
+    VOB_LRU(TT, 16, 64);              \
+  } while (0)
+  if (dtype == VOB_F32) VOB_LRU_CHUNKS(float);
+  if (dtype == VOB_BF16) VOB_LRU_CHUNKS(__nv_bfloat16);
+#undef VOB_LRU_CHUNKS
 #undef VOB_LRU
   return VOB_BAD_ARGUMENT;
 }

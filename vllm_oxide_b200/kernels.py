@@ -744,7 +744,7 @@ def lru_scan(u, gates, y, bias_r, bias_i, lam, bias_y, state, cu_q, state_slots,
     """S = a S + sqrt(1 - a^2) i u, out = S * gelu(y + bias_y), with r = sigmoid(r + bias_r), i = sigmoid(i + bias_i),
     a = exp(-8 r softplus(lam)), over every request's tokens of this step, from and to its slot (state float [slots, n], the
     width's channels first).  u, out [tokens, width]; gates float [tokens, blocks, 2, width / blocks] (r, then i, of every block);
-    y: the first `width` columns of its rows.  `chunks`: as mingru_scan."""
+    y: the first `width` columns of its rows.  `chunks`: as mingru_scan, or 64."""
     _cuda(u, gates, y, bias_r, bias_i, lam, bias_y, state, cu_q, state_slots, out)
     W = out.shape[1]
     assert u.is_contiguous() and out.is_contiguous() and u.shape == out.shape and u.dtype == y.dtype == out.dtype and y.stride(1) == 1
@@ -761,6 +761,12 @@ def scan_chunks(num_tokens: int, num_requests: int) -> int:
     """Ranges that a scan cuts a request's tokens of a step into, from the step's mean portion: 1 while decoding."""
     mean = num_tokens / max(1, num_requests)
     return 1 if mean <= 4 else (8 if mean <= 256 else 32)
+
+
+def matrix_scan_chunks(num_tokens: int, num_requests: int, heads: int, dk: int, dv: int) -> int:
+    """Ranges (up to 16) that an unfused matrix-state scan should cut a request's tokens of this step into: more where the heads
+    alone do not fill the device, one where the portions are short."""
+    return int(lib().vob_matrix_scan_chunks(num_tokens, num_requests, heads, dk, dv))
 
 
 def mingru_scan(zxg, bias_z, bias_x, state, cu_q, state_slots, out, num_requests: int, err, chunks: int = 1) -> None:

@@ -73,9 +73,9 @@ class _MatrixState(Mixer):
         return StateSpec((self.nh * self.dk * self.dv,), torch.float32)
 
     def _chunks(self, T: int, ctx):
-        """Ranges a request's tokens are cut into (the mean portion decides, as for every scan), and the scratch they need."""
+        """Ranges a request's tokens are cut into, and the scratch they need."""
         B = ctx.launch_requests
-        chunks = min(kernels.scan_chunks(T, B), 16)
+        chunks = kernels.matrix_scan_chunks(T, B, self.nh, self.dk, self.dv)
         scratch = None if chunks == 1 else ctx.ws.get_flat("matrix_scan_ranges", B * chunks * self.nh * self.dk * (self.dv + 1),
                                                            torch.float32)
         return chunks, scratch

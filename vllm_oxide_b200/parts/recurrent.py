@@ -104,9 +104,9 @@ class HGRN2(Mixer):
         # decoding: one block a (request, head), norm included; portions: a head's columns over several blocks
         fuse = kernels.hgrn2_can_fuse(self.dk, self.dv) and T <= 16 * ctx.launch_requests
         raw = None if fuse else ctx.ws.get("hgrn2_raw", T, self.nh * self.dv, torch.float32)
-        # longer portions are also cut along the tokens (the mean portion decides, as for every scan)
+        # longer portions are also cut along the tokens
         B = ctx.launch_requests
-        chunks = 1 if fuse else min(kernels.scan_chunks(T, B), 16)
+        chunks = 1 if fuse else kernels.matrix_scan_chunks(T, B, self.nh, self.dk, self.dv)
         scratch = None if chunks == 1 else ctx.ws.get_flat("hgrn2_ranges", B * chunks * self.nh * self.dk * (self.dv + 1),
                                                            torch.float32)
         kernels.hgrn2_scan(qfv, self.bf, self.lower, self.norm_weight, state, ctx.cu_q, ctx.state_slots, out,
@@ -170,7 +170,7 @@ class RecurrentBlock(Mixer):
             kernels.head_linear(u, W, part, self.w_gates, gates, 2 * W, 2 * part, T)
         out = ctx.ws.get("recurrent_out", T, W, x.dtype)
         kernels.lru_scan(u, gates, row, self.br, self.bi, self.lam, self.by, state, ctx.cu_q, ctx.state_slots, out, B, self.blocks,
-                         ctx.err, chunks=kernels.scan_chunks(T, B))
+                         ctx.err, chunks=64 if T > 1024 * B else kernels.scan_chunks(T, B))
         return linear(out, self.wo, ctx.ws.get("recurrent_proj", T, self.H, x.dtype), ctx)
 
 
