@@ -26,7 +26,9 @@ layers over a float stream, capped scores, two-map heads over blocks of position
 beside Kesozen, with attention held against arithmetic in prompts and against the keys and values read in decoding) at layer sizes of 1B- and 8B-class
 models beside Qwen3 at the same width, depth and feed-forward size (Kesozen also beside Tofilorn): one 2,048-token prompt in one step, decode at batch 8
 and 64 from a 2,048-token context (CUDA graphs), and, from an eager engine with the per-kernel timers on, the time of each
-of this package's kernels in those steps with the bytes it must move against the copy bandwidth.
+of this package's kernels in those steps with the bytes it must move against the copy bandwidth.  The Laruzen design (token shift,
+gated linear and lightning attention, a gated linear recurrence beside attention with a learned sink, experts beside a shared
+one) is measured beside Depolix, Tofilorn and Kesozen too.
 
     python bench.py --workload serving-0.6b | mixed-32b
 
