@@ -732,3 +732,122 @@ class LaruzenConfig:
         if self.bigram is not None:
             d["embedding"] = {"bigram": {"buckets": self.bigram[0], "mul_prev": self.bigram[1], "mul_cur": self.bigram[2]}}
         return d
+
+
+# ---------------------------------------------------------------------------------------------------------------
+_NESEZEN_MIXERS = ("attention", "mlstm", "latent_attention")
+
+
+@dataclass(frozen=True)
+class NesezenLayer:
+    type: str                   # "attention" | "mlstm" | "latent_attention"
+    mixer: dict                 # the mixer's sizes and constants, as config.json gives them
+    mlp: Optional[dict]         # None, {"kind": "dense", "ff"} or {"kind": "moe", "expert": {"ff"}, "router": {...}, "shared": {"ff"}}
+    weights_of: Optional[int] = None    # the layer whose tensors this one uses
+
+
+@dataclass(frozen=True)
+class NesezenConfig:
+    """Nesezen: a decoder whose layers are listed one by one in config.json, each with the norm tanh(alpha x) * w + b before both of
+    its sublayers around one float residual stream.  The mixer is `attention` (windowed, part of each head rotated with
+    frequencies stretched by wavelength, capped scores), `mlstm` (a matrix state per head with exponential gates, capped at
+    `gate_cap`) or `latent_attention` (low-rank queries, keys and values without positions, a gate a head).  The feed-forward is a
+    gated SiLU layer, a mixture of such experts whose sigmoid scores multiply their inputs, beside a shared one, or absent.  A layer
+    with `weights_of` uses another layer's tensors with a cache or state of its own; the rest of its entry equals that layer's.
+    Keys: `vocab`, `width`, `norm.eps`, `layers[i]` = {type, mixer{...}, mlp, weights_of}.  There is no largest position."""
+    vocab: int
+    width: int
+    eps: float
+    layers: tuple
+    torch_dtype: str = "bfloat16"
+
+    architecture = "Nesezen"
+
+    def owner(self, i: int) -> int:
+        """The layer whose tensors layer i uses: itself, or where its `weights_of` ends."""
+        while self.layers[i].weights_of is not None:
+            i = self.layers[i].weights_of
+        return i
+
+    @staticmethod
+    def _check_attention(m: dict, w: str) -> None:
+        _need(m, "kv_heads", int, w)
+        if m["heads"] % m["kv_heads"]:
+            raise ConfigError(f"{w}: heads {m['heads']} is not a multiple of kv_heads {m['kv_heads']}")
+        _need(m, "scale", float, w)
+        if m.get("softcap") is not None and _need(m, "softcap", float, w) < 0:
+            raise ConfigError(f"{w}: softcap must not be negative")
+        if m.get("mask") is not None:
+            _count(_sub(m, "mask", w), "size", w + ".mask")
+        if m.get("rot") is not None:
+            rot = _sub(m, "rot", w)
+            dims = rot.get("dims")
+            if isinstance(dims, bool) or not isinstance(dims, int) or dims < 0 or dims % 2 or dims > m["dim"]:
+                raise ConfigError(f"{w}: rot.dims {dims!r} must be even and between 0 and dim {m['dim']}")
+            if dims:
+                _need(rot, "base", float, w + ".rot")
+            if rot.get("scaling") is not None:
+                s = _sub(rot, "scaling", w + ".rot")
+                for k in ("factor", "original", "low", "high"):
+                    if _need(s, k, float, w + ".rot.scaling") <= 0:
+                        raise ConfigError(f"{w}: rot.scaling.{k} must be positive")
+                if s["low"] >= s["high"]:
+                    raise ConfigError(f"{w}: rot.scaling.low must lie below rot.scaling.high")
+
+    @classmethod
+    def from_dict(cls, d: dict, where: str = "config.json") -> "NesezenConfig":
+        layers = d.get("layers")
+        if not isinstance(layers, list) or not layers:
+            raise ConfigError(f"{where}: 'layers' must be a non-empty list")
+        out = []
+        for i, layer in enumerate(layers):
+            w = f"{where}: layers[{i}]"
+            if not isinstance(layer, dict):
+                raise ConfigError(f"{w} must be an object")
+            kind = layer.get("type")
+            if kind not in _NESEZEN_MIXERS:
+                raise ConfigError(f"{w}: type {kind!r} is not one of {list(_NESEZEN_MIXERS)}")
+            m = _sub(layer, "mixer", w)
+            for k in ("heads", "dim", "vdim"):
+                _need(m, k, int, w)
+            if kind == "attention":
+                cls._check_attention(m, w)
+            elif kind == "mlstm":
+                if _need(m, "gate_cap", float, w) <= 0:
+                    raise ConfigError(f"{w}: gate_cap must be positive")
+            else:
+                for k in ("q_rank", "kv_rank"):
+                    _need(m, k, int, w)
+                _need(m, "scale", float, w)
+            mlp = layer.get("mlp")
+            if mlp is not None:
+                _check_moe(mlp, w)
+                if mlp["kind"] == "moe" and mlp.get("shared") is not None:
+                    _need(_sub(mlp, "shared", w + ".mlp"), "ff", int, w + ".mlp.shared")
+            src = layer.get("weights_of")
+            if src is not None and (isinstance(src, bool) or not isinstance(src, int) or not 0 <= src < len(layers) or src == i):
+                raise ConfigError(f"{w}: weights_of {src!r} must name another layer")
+            out.append(NesezenLayer(kind, dict(m), None if mlp is None else dict(mlp), src))
+        for i, layer in enumerate(out):
+            j, steps = i, 0
+            while out[j].weights_of is not None:
+                j, steps = out[j].weights_of, steps + 1
+                if steps > len(out):
+                    raise ConfigError(f"{where}: layers[{i}]: weights_of leads round in a circle")
+            if (out[j].type, out[j].mixer, out[j].mlp) != (layer.type, layer.mixer, layer.mlp):
+                raise ConfigError(f"{where}: layers[{i}]: weights_of {layer.weights_of} names a layer of another shape")
+        dtype = d.get("torch_dtype", d.get("dtype", "bfloat16"))
+        if not isinstance(dtype, str) or dtype not in _DTYPE_NAMES:
+            raise ConfigError(f"{where}: torch_dtype {dtype!r} is not one of {sorted(set(_DTYPE_NAMES))}")
+        return cls(vocab=_need(d, "vocab", int, where), width=_need(d, "width", int, where),
+                   eps=_need(_sub(d, "norm", where), "eps", float, where + ".norm"), layers=tuple(out),
+                   torch_dtype=_DTYPE_NAMES[dtype])
+
+    def to_dict(self) -> dict:
+        layers = []
+        for l in self.layers:
+            e = {"type": l.type, "mixer": dict(l.mixer), "mlp": None if l.mlp is None else dict(l.mlp)}
+            if l.weights_of is not None:
+                e["weights_of"] = l.weights_of
+            layers.append(e)
+        return {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.eps}, "layers": layers}

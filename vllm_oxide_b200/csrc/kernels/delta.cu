@@ -18,7 +18,9 @@
 //                      interleaved so that a warp's loads of the state fill whole sectors); a block takes the columns
 //                      c0.. of one (request, head) and walks the request's tokens in order, while half of its warps
 //                      prepare the next tokens in shared memory (unit vectors, decay and beta are made there, in float).
-//   delta_out_norm     o / sqrt(mean(o^2) + eps) * w * SiLU(gate) (or * sigmoid(gate)), per head over vdim
+//   delta_out_norm     o / sqrt(mean(o^2) + eps) * w * SiLU(gate) (or * sigmoid(gate)), per head over vdim; w may be one gain for
+//                      all heads or a gain an element of every head.  With a normaliser (`nq`, `gates`: see recurrent.cu,
+//                      exponential gates) o is first divided by max(|nq|, floor) + 1e-6
 // Everything but the inputs' type T is float on both paths.  The chain of operations of an output depends only on the
 // request's tokens and the state it starts from, not on the cut, the batch or the slot.
 #include "common.cuh"
@@ -391,34 +393,41 @@ delta_scan_kernel(const float* qkv, const T* ab, long ab_stride, int b_off, int 
   }
 }
 
+// What a head's outputs of a token are multiplied by before their norm: 1, or one over its normaliser.
+__device__ __forceinline__ float head_unit(const float* nq, const float4* gates, size_t at) {
+  return nq ? 1.f / (fmaxf(fabsf(nq[at]), gates[at].z) + 1e-6f) : 1.f;
+}
+
 // out[t, h, :] = raw[t, h, :] / sqrt(mean(raw[t, h, :]^2) + eps) * w * SiLU(gate[t, h, :]); one warp a (token, head).
 template <typename T>
 __global__ void __launch_bounds__(128)
-delta_out_norm_kernel(const float* raw, const T* gate, long gate_stride, const float* __restrict__ w, T* out, int heads,
-                      int vdim, float eps, int total, int gate_sigmoid) {
+delta_out_norm_kernel(const float* raw, const T* gate, long gate_stride, const float* __restrict__ w, int w_head, const float* nq,
+                      const float4* gates, T* out, int heads, int vdim, float eps, int total, int gate_sigmoid) {
   pdl_launch_dependents();
   pdl_wait();
   const int idx = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (idx >= total) return;
   const int t = idx / heads, h = idx % heads;
   const float* o = raw + ((size_t)t * heads + h) * vdim;
+  const float unit = head_unit(nq, gates, (size_t)idx);
   float ss = 0.f;
-  for (int d = lane; d < vdim; d += 32) ss = fmaf(o[d], o[d], ss);
+  for (int d = lane; d < vdim; d += 32) { const float x = o[d] * unit; ss = fmaf(x, x, ss); }
   ss = warp_sum(ss);
   const float inv = 1.f / sqrtf(ss / (float)vdim + eps);
+  const float* gain = w + (size_t)h * w_head;
   const T* grow = gate + (size_t)t * gate_stride + (size_t)h * vdim;
   T* orow = out + ((size_t)t * heads + h) * vdim;
   for (int d = lane; d < vdim; d += 32) {
     const float gv = to_f<T>(grow[d]);
-    orow[d] = from_f<T>(o[d] * inv * w[d] * (gate_sigmoid ? 1.f / (1.f + expf(-gv)) : silu_f(gv)));
+    orow[d] = from_f<T>(o[d] * unit * inv * gain[d] * (gate_sigmoid ? 1.f / (1.f + expf(-gv)) : silu_f(gv)));
   }
 }
 
 // The same for wide rows (all heads normed as one): a block takes a row.
 template <typename T>
 __global__ void __launch_bounds__(256)
-delta_out_norm_wide_kernel(const float* raw, const T* gate, long gate_stride, const float* __restrict__ w, T* out, int heads,
-                           int vdim, float eps, int gate_sigmoid) {
+delta_out_norm_wide_kernel(const float* raw, const T* gate, long gate_stride, const float* __restrict__ w, int w_head,
+                           const float* nq, const float4* gates, T* out, int heads, int vdim, float eps, int gate_sigmoid) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
@@ -426,12 +435,14 @@ delta_out_norm_wide_kernel(const float* raw, const T* gate, long gate_stride, co
   const float* o = raw + ((size_t)t * heads + h) * vdim;
   const T* grow = gate + (size_t)t * gate_stride + (size_t)h * vdim;
   T* orow = out + ((size_t)t * heads + h) * vdim;
+  const float unit = head_unit(nq, gates, (size_t)blockIdx.x);
+  const float* gain = w + (size_t)h * w_head;
   float ss = 0.f;
-  for (int d = threadIdx.x; d < vdim; d += 256) ss = fmaf(o[d], o[d], ss);
+  for (int d = threadIdx.x; d < vdim; d += 256) { const float x = o[d] * unit; ss = fmaf(x, x, ss); }
   const float inv = 1.f / sqrtf(block_sum<256>(ss, scratch) / (float)vdim + eps);
   for (int d = threadIdx.x; d < vdim; d += 256) {
     const float gv = to_f<T>(grow[d]);
-    orow[d] = from_f<T>(o[d] * inv * w[d] * (gate_sigmoid ? 1.f / (1.f + expf(-gv)) : silu_f(gv)));
+    orow[d] = from_f<T>(o[d] * unit * inv * gain[d] * (gate_sigmoid ? 1.f / (1.f + expf(-gv)) : silu_f(gv)));
   }
 }
 
@@ -541,25 +552,29 @@ VOB_API int vob_delta_scan(const float* qkv, const void* ab, long ab_stride, int
   return VOB_BAD_ARGUMENT;
 }
 
-VOB_API int vob_delta_out_norm(const float* raw, const void* gate, long gate_stride, const float* w, void* out, int T, int heads,
-                               int vdim, float eps, int gate_sigmoid, int dtype, cudaStream_t stream) {
+// w float [vdim], or [heads * vdim] with w_head = vdim (else 0); nq float [T, heads] and gates float [T, heads, 4], or null.
+VOB_API int vob_delta_out_norm(const float* raw, const void* gate, long gate_stride, const float* w, int w_head, const float* nq,
+                               const float* gates_, void* out, int T, int heads, int vdim, float eps, int gate_sigmoid, int dtype,
+                               cudaStream_t stream) {
   if (T <= 0) return 0;
+  const float4* gates = (const float4*)gates_;
+  if (nq && (!gates || ((uintptr_t)gates & 15))) return VOB_BAD_ARGUMENT;
   const int total = T * heads;
   if (vdim > 512) {
     if (dtype == VOB_F32)
       return launch_kernel(delta_out_norm_wide_kernel<float>, dim3(total), 256, 0, stream, raw, (const float*)gate, gate_stride, w,
-                           (float*)out, heads, vdim, eps, gate_sigmoid);
+                           w_head, nq, gates, (float*)out, heads, vdim, eps, gate_sigmoid);
     if (dtype == VOB_BF16)
       return launch_kernel(delta_out_norm_wide_kernel<__nv_bfloat16>, dim3(total), 256, 0, stream, raw, (const __nv_bfloat16*)gate,
-                           gate_stride, w, (__nv_bfloat16*)out, heads, vdim, eps, gate_sigmoid);
+                           gate_stride, w, w_head, nq, gates, (__nv_bfloat16*)out, heads, vdim, eps, gate_sigmoid);
     return VOB_BAD_ARGUMENT;
   }
   dim3 grid((total + 3) / 4);
   if (dtype == VOB_F32)
     return launch_kernel(delta_out_norm_kernel<float>, grid, 128, 0, stream, raw, (const float*)gate, gate_stride, w,
-                         (float*)out, heads, vdim, eps, total, gate_sigmoid);
+                         w_head, nq, gates, (float*)out, heads, vdim, eps, total, gate_sigmoid);
   if (dtype == VOB_BF16)
     return launch_kernel(delta_out_norm_kernel<__nv_bfloat16>, grid, 128, 0, stream, raw, (const __nv_bfloat16*)gate,
-                         gate_stride, w, (__nv_bfloat16*)out, heads, vdim, eps, total, gate_sigmoid);
+                         gate_stride, w, w_head, nq, gates, (__nv_bfloat16*)out, heads, vdim, eps, total, gate_sigmoid);
   return VOB_BAD_ARGUMENT;
 }

@@ -6,16 +6,22 @@
 //                 as it is (no renormalisation).  Ties go to the lower index.  Options: scores may be sigmoid(z) instead of
 //                 the softmax; there may be no correction; a group may count by the sum of its two best choice scores
 //                 instead of its best; the chosen scores may be divided by their sum (+ 1e-20); and a factor may scale them.
+//                 With `w_shared` (a row like a router's) the sigmoid of its product with h is a number a token beside them:
+//                 the gate of an expert that every token uses.
 //   moe_align     sorts the step's (token, choice) pairs by expert: every expert's rows start on a multiple of the product's
 //                 row tile (padding rows name no token), and each row tile knows its expert.  Everything stays on the
 //                 device: the grid of the products is sized for the worst case and tiles past the end return at once.
+//                 With `weights` a row also gets its pair's weight (row_weight).
 //   moe_gemm      C[row] = f(A[row] W_e^T) for the rows of expert e, W stacked [experts, N, K]; A is either gathered by the
 //                 row's token (the first product) or read in place (the second); f is the identity, the squared relu, or
-//                 (rows of W in pairs: gate row, up row) SiLU(gate) * up, which halves the output's width.
+//                 (rows of W in pairs: gate row, up row) SiLU(gate) * up, which halves the output's width.  With a row's weight
+//                 (`row_weight`; the pair's in moe_gemv) the weight multiplies the expert's INPUT: W (w h) = w (W h), so gate
+//                 and up are multiplied behind the product, in float.
 //                 Float accumulation, one chain of fused multiply-adds over k in ascending order for every output element
 //                 (the float path's product, with a tile's expert in front of it).
 //   moe_combine   out[t] = sum_j weight[t, j] * y[row of (t, j)], j in order, in float; a row may be added to it (`add`: what
-//                 an expert that every token uses has made of the token).
+//                 an expert that every token uses has made of the token), times a number a token (`add_gate`).  No weights:
+//                 all ones (the weights went into the experts).
 //   relu_squared  out = max(x, 0)^2 (the dense feed-forward's activation).
 #include "common.cuh"
 
@@ -54,12 +60,12 @@ constexpr int ROUTE_TOKENS = 4;   // tokens a block: the router's rows are read 
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_NT)
 moe_route_kernel(const T* h, const float* __restrict__ w_router, const float* __restrict__ router_bias,
-                 const float* __restrict__ correction, int* ids, float* weights,
+                 const float* __restrict__ correction, const float* __restrict__ w_shared, float* shared_gate, int* ids, float* weights,
                  int W, int E, int top, int count, int keep, int sigmoid_scores, int group_top, int normalise, float weight_scale,
                  int num_tokens, int per_block) {
   extern __shared__ __align__(16) float route_smem[];
   float* hrows = route_smem;                        // [per_block][W]
-  float* lists = hrows + (size_t)per_block * W;     // per token: [E] scores, [E] choice scores, [count] group scores
+  float* lists = hrows + (size_t)per_block * W;     // per token: [E] scores, [E] choice scores, [count] group scores, [1] shared gate
   pdl_launch_dependents();
   pdl_wait();
   const int t0 = blockIdx.x * per_block, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -68,9 +74,10 @@ moe_route_kernel(const T* h, const float* __restrict__ w_router, const float* __
   __syncthreads();
   // a warp takes experts warp, warp + 8, ...; a lane sums four elements at a time into four chains (one chain where the
   // width is no multiple of 4): the order of a logit's additions depends on the width alone, not on the tokens beside it
-  const bool vec = W % 4 == 0 && ((uintptr_t)w_router % 16) == 0;
-  for (int e = warp; e < E; e += ROUTE_NT / 32) {
-    const float* wr = w_router + (size_t)e * W;
+  const bool vec = W % 4 == 0 && (((uintptr_t)w_router | (uintptr_t)w_shared) % 16) == 0;
+  const int list = 2 * E + count + 1, logits = E + (w_shared ? 1 : 0);
+  for (int e = warp; e < logits; e += ROUTE_NT / 32) {
+    const float* wr = e < E ? w_router + (size_t)e * W : w_shared;
     float z[ROUTE_TOKENS];
     if (vec) {
       float z4[ROUTE_TOKENS][4];
@@ -102,21 +109,25 @@ moe_route_kernel(const T* h, const float* __restrict__ w_router, const float* __
 #pragma unroll
     for (int k = 0; k < ROUTE_TOKENS; ++k) {
       const float sum = warp_sum(z[k]);
-      if (lane == 0 && k < here) lists[(size_t)k * (2 * E + count) + e] = router_bias ? sum + router_bias[e] : sum;
+      if (lane == 0 && k < here) lists[(size_t)k * list + (e < E ? e : list - 1)] = router_bias && e < E ? sum + router_bias[e] : sum;
     }
   }
   __syncthreads();
   // warp k chooses for token k
   if (warp >= here) return;
   const int t = t0 + warp;
-  float* score = lists + (size_t)warp * (2 * E + count);   // [E] softmax or sigmoid
+  float* score = lists + (size_t)warp * list;              // [E] softmax or sigmoid
+  if (w_shared && lane == 0) shared_gate[t] = 1.f / (1.f + expf(-score[list - 1]));
   float* choice = score + E;                               // [E] score + correction, -inf once taken or shut out
   float* gbest = choice + E;                               // [count]
+  // Without a correction the choice is by the logit itself where that gives the same order (it does unless groups count by a sum
+  // of scores): the scores of logits that lie far apart may round to one number (zero or one), and would tie.
+  const bool by_logit = !correction && (keep >= count || group_top < 2);
   if (sigmoid_scores) {
     for (int e = lane; e < E; e += 32) {
-      const float s = 1.f / (1.f + expf(-score[e]));
+      const float z = score[e], s = 1.f / (1.f + expf(-z));
       score[e] = s;
-      choice[e] = correction ? s + correction[e] : s;
+      choice[e] = correction ? s + correction[e] : (by_logit ? z : s);
     }
   } else {
     float m = -INFINITY;
@@ -125,9 +136,6 @@ moe_route_kernel(const T* h, const float* __restrict__ w_router, const float* __
     float sum = 0.f;
     for (int e = lane; e < E; e += 32) sum += expf(score[e] - m);
     sum = warp_sum(sum);
-    // Without a correction the choice is by the logit itself where that gives the same order (it does unless groups count
-    // by a sum of scores): logits far below the largest all become a score of zero, and would tie.
-    const bool by_logit = !correction && (keep >= count || group_top < 2);
     for (int e = lane; e < E; e += 32) {
       const float z = score[e] - m;
       const float s = expf(z) / sum;
@@ -187,7 +195,8 @@ moe_route_kernel(const T* h, const float* __restrict__ w_router, const float* __
 // tile_expert[max_rows / MOE_TM]: the expert of every MOE_TM rows (-1: past the end).  An expert's rows are padded to a
 // multiple of `pad`, itself a multiple of MOE_TM (a product with larger row tiles asks for more).
 __global__ void __launch_bounds__(1024)
-moe_align_kernel(const int* ids, int* slot_of, int* row_token, int* tile_expert, int n, int top, int E, int max_rows, int pad) {
+moe_align_kernel(const int* ids, const float* weights, int* slot_of, int* row_token, float* row_weight, int* tile_expert, int n, int top,
+                 int E, int max_rows, int pad) {
   extern __shared__ int align_smem[];
   int* counts = align_smem;          // [E]
   int* offsets = counts + E;         // [E]
@@ -219,6 +228,7 @@ moe_align_kernel(const int* ids, int* slot_of, int* row_token, int* tile_expert,
     const int row = offsets[e] + atomicAdd(&counts[e], 1);
     slot_of[i] = row;
     row_token[row] = i / top;
+    if (row_weight) row_weight[row] = weights[i];
   }
 }
 
@@ -230,7 +240,7 @@ constexpr int MG_N = 64, MG_K = 16;
 template <typename TA, typename TC, int EPI, bool GATHER>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const TA* A, long lda, const TA* __restrict__ W, TC* C, long ldc, const int* row_token,
-                const int* tile_expert, int N, int K, float glu_limit) {
+                const float* row_weight, const int* tile_expert, int N, int K, float glu_limit) {
   __shared__ float As[MG_K][MOE_TM + 4];
   __shared__ float Ws[MG_K][MG_N + 4];
   __shared__ int src[MOE_TM];
@@ -282,12 +292,12 @@ moe_gemm_kernel(const TA* A, long lda, const TA* __restrict__ W, TC* C, long ldc
     if (src[ty * 4 + i] < 0) continue;
     const int m = m0 + ty * 4 + i;
     if (EPI == 2) {
+      const float rw = row_weight ? row_weight[m] : 1.f;
 #pragma unroll
       for (int j = 0; j < 4; j += 2) {
         const int n = n0 + tx * 4 + j;
         if (n + 1 >= N) continue;
-        const float g = acc[i][j];
-        C[(size_t)m * ldc + n / 2] = from_f<TC>(gated_pair(g, acc[i][j + 1], glu_limit));
+        C[(size_t)m * ldc + n / 2] = from_f<TC>(gated_pair(acc[i][j] * rw, acc[i][j + 1] * rw, glu_limit));
       }
       continue;
     }
@@ -304,17 +314,18 @@ moe_gemm_kernel(const TA* A, long lda, const TA* __restrict__ W, TC* C, long ldc
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_combine_kernel(const float* y, const int* slot_of, const float* weights, const T* add, T* out, int D, int top) {
+moe_combine_kernel(const float* y, const int* slot_of, const float* weights, const T* add, const float* add_gate, T* out, int D, int top) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
+  const float ag = add_gate ? add_gate[t] : 1.f;
   for (int d = threadIdx.x; d < D; d += 256) {
     float acc = 0.f;
     for (int j = 0; j < top; ++j) {
       const int row = slot_of ? slot_of[(size_t)t * top + j] : t * top + j;
-      if (row >= 0) acc = fmaf(weights[(size_t)t * top + j], y[(size_t)row * D + d], acc);
+      if (row >= 0) acc = fmaf(weights ? weights[(size_t)t * top + j] : 1.f, y[(size_t)row * D + d], acc);
     }
-    if (add) acc += to_f<T>(add[(size_t)t * D + d]);
+    if (add) acc = fmaf(ag, to_f<T>(add[(size_t)t * D + d]), acc);
     out[(size_t)t * D + d] = from_f<T>(acc);
   }
 }
@@ -359,7 +370,7 @@ constexpr int MV_ROWS = 64;       // output features a block
 template <int EPI, bool BY_TOKEN>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(const __nv_bfloat16* A, long lda, const __nv_bfloat16* __restrict__ W, void* C, long ldc, const int* ids,
-                const int* order, int top, int N, int K, float glu_limit) {
+                const int* order, const float* weights, int top, int N, int K, float glu_limit) {
   extern __shared__ uint4 gemv_smem[];     // the input row: K bfloat16
   pdl_launch_dependents();
   pdl_wait();
@@ -400,8 +411,9 @@ moe_gemv_kernel(const __nv_bfloat16* A, long lda, const __nv_bfloat16* __restric
     }
     if (EPI == 2) {
       float v[4];
+      const float pw = weights ? weights[pair] : 1.f;
 #pragma unroll
-      for (int r = 0; r < 4; ++r) v[r] = warp_sum(acc[r]);
+      for (int r = 0; r < 4; ++r) v[r] = warp_sum(acc[r]) * pw;
 #pragma unroll
       for (int r = 0; r < 4; r += 2) {
         const int n = n0 + rg * 4 + r;
@@ -460,26 +472,28 @@ using namespace vob;
 VOB_API int vob_moe_row_tile() { return MOE_TM; }
 
 // correction may be null; sigmoid_scores: scores are sigmoid(z), not the softmax; group_top 2: a group counts by its two best;
-// normalise: the chosen scores are divided by their sum; weight_scale: a factor on the weights.
-VOB_API int vob_moe_route(const void* h, const float* w_router, const float* router_bias, const float* correction, int* ids,
-                          float* weights, int T, int W,
+// normalise: the chosen scores are divided by their sum; weight_scale: a factor on the weights.  w_shared float [W] and
+// shared_gate float [T], or null.
+VOB_API int vob_moe_route(const void* h, const float* w_router, const float* router_bias, const float* correction,
+                          const float* w_shared, float* shared_gate, int* ids, float* weights, int T, int W,
                           int E, int top, int count, int keep, int sigmoid_scores, int group_top, int normalise,
                           float weight_scale, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if ((w_shared == nullptr) != (shared_gate == nullptr)) return VOB_BAD_ARGUMENT;
   if (E <= 0 || top <= 0 || top > E || count <= 0 || E % count || keep <= 0 || keep > count || (long)(E / count) * keep < top)
     return VOB_BAD_ARGUMENT;
   // as many tokens a block as 96 KB hold (up to ROUTE_TOKENS) while the blocks still fill the device twice; one where the
   // width is no multiple of 4 (rows stay aligned).  A token's arithmetic does not depend on how many share its block.
   int per_block = (int)std::min<long>(ROUTE_TOKENS, std::max<long>(1, T / (2L * sm_count())));
-  while (per_block > 1 && ((size_t)per_block * (W + 2 * E + count) * sizeof(float) > 96 * 1024 || W % 4)) --per_block;
-  const size_t smem = (size_t)per_block * (W + 2 * E + count) * sizeof(float);
+  while (per_block > 1 && ((size_t)per_block * (W + 2 * E + count + 1) * sizeof(float) > 96 * 1024 || W % 4)) --per_block;
+  const size_t smem = (size_t)per_block * (W + 2 * E + count + 1) * sizeof(float);
   if (smem > 200 * 1024) return VOB_UNSUPPORTED;
 #define VOB_ROUTE(TYPE)                                                                                                  \
   do {                                                                                                                   \
     if (smem > 48 * 1024)                                                                                                \
       cudaFuncSetAttribute(moe_route_kernel<TYPE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);              \
     return launch_kernel(moe_route_kernel<TYPE>, dim3((T + per_block - 1) / per_block), ROUTE_NT, smem, stream,          \
-                         (const TYPE*)h, w_router, router_bias, correction, ids, weights, W, E, top, count, keep, sigmoid_scores,     \
+                         (const TYPE*)h, w_router, router_bias, correction, w_shared, shared_gate, ids, weights, W, E, top, count, keep, sigmoid_scores,     \
                          group_top, normalise, weight_scale, T, per_block);                                              \
   } while (0)
   if (dtype == VOB_F32) VOB_ROUTE(float);
@@ -488,27 +502,29 @@ VOB_API int vob_moe_route(const void* h, const float* w_router, const float* rou
   return VOB_BAD_ARGUMENT;
 }
 
-VOB_API int vob_moe_align(const int* ids, int* slot_of, int* row_token, int* tile_expert, int n, int top, int E, int max_rows,
-                          int pad, cudaStream_t stream) {
+// weights [n] and row_weight [max_rows], or null.
+VOB_API int vob_moe_align(const int* ids, const float* weights, int* slot_of, int* row_token, float* row_weight, int* tile_expert,
+                          int n, int top, int E, int max_rows, int pad, cudaStream_t stream) {
   if (n <= 0) return 0;
+  if (row_weight && !weights) return VOB_BAD_ARGUMENT;
   if (pad <= 0 || pad % MOE_TM || max_rows % pad || E <= 0 || E > 4096) return VOB_BAD_ARGUMENT;
-  return launch_kernel(moe_align_kernel, dim3(1), 1024, (size_t)2 * E * sizeof(int), stream, ids, slot_of, row_token, tile_expert,
-                       n, top, E, max_rows, pad);
+  return launch_kernel(moe_align_kernel, dim3(1), 1024, (size_t)2 * E * sizeof(int), stream, ids, weights, slot_of, row_token,
+                       row_weight, tile_expert, n, top, E, max_rows, pad);
 }
 
 // A: rows of lda elements (`gather`: indexed by the row's token); W [experts, N, K]; C [max_rows, ldc] of `dtype`, or float
 // with `c_float`.  epilogue 0: as it is, 1: squared relu, 2: SiLU(gate) * up over rows of W in (gate, up) pairs: C has N / 2
-// columns.
-VOB_API int vob_moe_gemm(const void* A, long lda, const void* W, void* C, long ldc, const int* row_token, const int* tile_expert,
-                         int max_rows, int N, int K, int epilogue, int gather, int c_float, float glu_limit, int dtype,
+// columns.  row_weight (epilogue 2) or null: a factor on every row's gate and up.
+VOB_API int vob_moe_gemm(const void* A, long lda, const void* W, void* C, long ldc, const int* row_token, const float* row_weight,
+                         const int* tile_expert, int max_rows, int N, int K, int epilogue, int gather, int c_float, float glu_limit, int dtype,
                          cudaStream_t stream) {
   if (max_rows <= 0 || N <= 0) return 0;
-  if (K <= 0 || max_rows % MOE_TM) return VOB_BAD_ARGUMENT;
+  if (K <= 0 || max_rows % MOE_TM || (row_weight && epilogue != 2)) return VOB_BAD_ARGUMENT;
   dim3 grid((N + MG_N - 1) / MG_N, max_rows / MOE_TM);
   if (grid.y > 65535) return VOB_UNSUPPORTED;
 #define VOB_MG(TA, TC, EPI, G)                                                                                       \
   return launch_kernel(moe_gemm_kernel<TA, TC, EPI, G>, grid, 256, 0, stream, (const TA*)A, lda, (const TA*)W, (TC*)C, ldc, \
-                       row_token, tile_expert, N, K, glu_limit)
+                       row_token, row_weight, tile_expert, N, K, glu_limit)
 #define VOB_MG_TYPE(TA)                                                   \
   if (epilogue == 1 && gather && !c_float) VOB_MG(TA, TA, 1, true);       \
   if (epilogue == 2 && gather && !c_float) VOB_MG(TA, TA, 2, true);       \
@@ -529,10 +545,12 @@ VOB_API int vob_moe_order(const int* ids, int* order, int n, int E, cudaStream_t
 
 // A: bfloat16 rows of lda elements, a token's (`by_token`) or a pair's; W bfloat16 [experts, N, K], K a multiple of 8;
 // C [pairs, ldc]: bfloat16 with the squared relu (`epilogue` 1) or with SiLU(gate) * up over rows of W in (gate, up) pairs
-// (2: N / 2 columns), or float (0).  order: the pairs by expert (vob_moe_order).
-VOB_API int vob_moe_gemv(const void* A, long lda, const void* W, void* C, long ldc, const int* ids, const int* order, int n,
-                         int top, int N, int K, int epilogue, int by_token, float glu_limit, cudaStream_t stream) {
+// (2: N / 2 columns), or float (0).  order: the pairs by expert (vob_moe_order).  weights [pairs] (epilogue 2) or null: a factor
+// on every pair's gate and up.
+VOB_API int vob_moe_gemv(const void* A, long lda, const void* W, void* C, long ldc, const int* ids, const int* order,
+                         const float* weights, int n, int top, int N, int K, int epilogue, int by_token, float glu_limit, cudaStream_t stream) {
   if (n <= 0 || N <= 0) return 0;
+  if (weights && epilogue != 2) return VOB_BAD_ARGUMENT;
   if (K <= 0 || K % 8 || (lda * 2) % 16 || ((uintptr_t)A | (uintptr_t)W) % 16 || n > 65535) return VOB_UNSUPPORTED;
   const size_t smem = (size_t)K * 2;
   if (smem > 96 * 1024) return VOB_UNSUPPORTED;
@@ -541,7 +559,7 @@ VOB_API int vob_moe_gemv(const void* A, long lda, const void* W, void* C, long l
   do {                                                                                                                      \
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_gemv_kernel<EPI, BT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     return launch_kernel(moe_gemv_kernel<EPI, BT>, grid, 256, smem, stream, (const __nv_bfloat16*)A, lda,                   \
-                         (const __nv_bfloat16*)W, C, ldc, ids, order, top, N, K, glu_limit);                                       \
+                         (const __nv_bfloat16*)W, C, ldc, ids, order, weights, top, N, K, glu_limit);                                       \
   } while (0)
   if (epilogue == 1 && by_token) VOB_MV(1, true);
   if (epilogue == 2 && by_token && N % 2 == 0) VOB_MV(2, true);
@@ -550,16 +568,16 @@ VOB_API int vob_moe_gemv(const void* A, long lda, const void* W, void* C, long l
   return VOB_UNSUPPORTED;
 }
 
-// add [T, D] of `dtype`, or null.
-VOB_API int vob_moe_combine(const float* y, const int* slot_of, const float* weights, const void* add, void* out, int T, int D,
-                            int top, int dtype, cudaStream_t stream) {
+// add [T, D] of `dtype`, or null; add_gate [T], or null; weights [T, top], or null (ones).
+VOB_API int vob_moe_combine(const float* y, const int* slot_of, const float* weights, const void* add, const float* add_gate, void* out,
+                            int T, int D, int top, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (dtype == VOB_F32)
-    return launch_kernel(moe_combine_kernel<float>, dim3(T), 256, 0, stream, y, slot_of, weights, (const float*)add, (float*)out, D,
-                         top);
+    return launch_kernel(moe_combine_kernel<float>, dim3(T), 256, 0, stream, y, slot_of, weights, (const float*)add, add_gate,
+                         (float*)out, D, top);
   if (dtype == VOB_BF16)
     return launch_kernel(moe_combine_kernel<__nv_bfloat16>, dim3(T), 256, 0, stream, y, slot_of, weights, (const __nv_bfloat16*)add,
-                         (__nv_bfloat16*)out, D, top);
+                         add_gate, (__nv_bfloat16*)out, D, top);
   return VOB_BAD_ARGUMENT;
 }
 

@@ -13,7 +13,8 @@
 //               tcgen05.commit hands a stage back to the producer and, after an item's last, the accumulator to the epilogue;
 //   warps 2-5   epilogue: tcgen05.ld brings the accumulator to registers (a thread owns one output feature for all rows of
 //               the tile), applies f (identity into float, the squared relu into bfloat16, or, rows of W in (gate, up)
-//               pairs, SiLU(gate) * up into bfloat16 feature / 2: the up value comes from the neighbouring lane) and stores
+//               pairs, SiLU(gate) * up into bfloat16 feature / 2: the up value comes from the neighbouring lane; a row's weight,
+//               where the weights multiply the experts' inputs, multiplies both) and stores
 //               the rows that name a token; the next item's MMAs run meanwhile into the other accumulator.
 // Which items exist is only known on the device (the sorting kernel ran just before), so nothing is copied before the wait
 // for the kernels ahead.  Every wait on an mbarrier is bounded; on a timeout the block sets an error bit, stops issuing
@@ -40,7 +41,7 @@ enum { MT_EPI_RELU2_BF16 = 0, MT_EPI_F32 = 1, MT_EPI_SILU_PAIRS_BF16 = 2 };
 template <int EPI>
 __global__ void __launch_bounds__(MT_THREADS, 1)
 moe_tc5_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, void* out, long ldo,
-               const int* row_token, const int* tile_expert, int row_tiles, int N, int K, float glu_limit, int* err) {
+               const int* row_token, const float* row_weight, const int* tile_expert, int row_tiles, int N, int K, float glu_limit, int* err) {
   constexpr int S = MT_S, A_BYTES = MT_ROWS * 128, STAGE_BYTES = MT_STAGE_BYTES;
   constexpr int TMEM_COLS = 2 * MT_NT;
   extern __shared__ __align__(1024) char smem_raw[];
@@ -151,6 +152,7 @@ moe_tc5_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         float v[32];
         t5_ld32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * MT_NT + c0), v);
         const int tok = row_token[mt * MT_NT + c0 + lane];        // lane j's entry belongs to column c0 + j
+        const float rw = EPI == MT_EPI_SILU_PAIRS_BF16 && row_weight && tok >= 0 ? row_weight[mt * MT_NT + c0 + lane] : 1.f;
         if (EPI == MT_EPI_SILU_PAIRS_BF16) {
           // Two lanes hold a (gate, up) pair of features.  They finish two token columns at a time, the even lane column
           // j and the odd lane column j + 1, so every lane takes one exponential for two columns and one exchange
@@ -161,7 +163,8 @@ moe_tc5_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             const bool live0 = __shfl_sync(0xffffffffu, tok, j) >= 0, live1 = __shfl_sync(0xffffffffu, tok, j + 1) >= 0;
             if (!live0 && !live1) continue;                       // the same for every lane of the warp
             const float got = __shfl_xor_sync(0xffffffffu, odd ? v[j] : v[j + 1], 1);
-            const float gate = odd ? got : v[j], up = odd ? v[j + 1] : got;
+            const float wt = row_weight ? __shfl_sync(0xffffffffu, rw, odd ? j + 1 : j) : 1.f;
+            const float gate = (odd ? got : v[j]) * wt, up = (odd ? v[j + 1] : got) * wt;
             if ((odd ? live1 : live0) && (n | 1) < N) {
               const long m = (long)mt * MT_NT + c0 + j + (odd ? 1 : 0);
               reinterpret_cast<__nv_bfloat16*>(out)[m * ldo + (n >> 1)] =
@@ -224,12 +227,13 @@ VOB_API int vob_moe_tc5_row_tile() { return MT_NT; }
 // map_w: tensor map of W [experts * N, K] with box 128 rows; map_x: tensor map of the sorted rows [max_rows, K] with box 128
 // rows (vob_tensor_map_bf16_2d).  out [max_rows, ldo]: bfloat16 with the squared relu (epilogue 0), float (1), or bfloat16
 // SiLU(gate) * up over rows of W in (gate, up) pairs (2: N / 2 columns; with glu_limit > 0 the clamped form
-// min(gate, limit) * sigmoid(1.702 min(gate, limit)) * (clamp(up, -limit, limit) + 1)).
+// min(gate, limit) * sigmoid(1.702 min(gate, limit)) * (clamp(up, -limit, limit) + 1)).  row_weight [max_rows] (epilogue 2) or null:
+// a factor on every row's gate and up.
 VOB_API int vob_moe_gemm_tc5(const void* map_w, const void* map_x, void* out, long ldo, const int* row_token,
-                             const int* tile_expert, int max_rows, int N, int K, int epilogue, float glu_limit, int* err,
+                             const float* row_weight, const int* tile_expert, int max_rows, int N, int K, int epilogue, float glu_limit, int* err,
                              cudaStream_t stream) {
   if (max_rows <= 0 || N <= 0) return 0;
-  if (!map_w || !map_x || K <= 0 || K % 8 || max_rows % MT_NT) return VOB_BAD_ARGUMENT;
+  if (!map_w || !map_x || K <= 0 || K % 8 || max_rows % MT_NT || (row_weight && epilogue != MT_EPI_SILU_PAIRS_BF16)) return VOB_BAD_ARGUMENT;
   const int row_tiles = max_rows / MT_NT;
   const long total = (long)row_tiles * ((N + MT_ROWS - 1) / MT_ROWS);
   const int blocks = (int)(total < sm_count() ? total : sm_count());
@@ -242,7 +246,7 @@ VOB_API int vob_moe_gemm_tc5(const void* map_w, const void* map_x, void* out, lo
       configured[EPI] = true;                                                                                              \
     }                                                                                                                      \
     return launch_kernel(moe_tc5_kernel<EPI>, dim3(blocks), MT_THREADS, MT_SMEM, stream, *(const CUtensorMap*)map_w,       \
-                         *(const CUtensorMap*)map_x, out, ldo, row_token, tile_expert, row_tiles, N, K, glu_limit, err);          \
+                         *(const CUtensorMap*)map_x, out, ldo, row_token, row_weight, tile_expert, row_tiles, N, K, glu_limit, err);          \
   } while (0)
   if (epilogue == MT_EPI_RELU2_BF16) VOB_MT(MT_EPI_RELU2_BF16);
   if (epilogue == MT_EPI_F32) VOB_MT(MT_EPI_F32);

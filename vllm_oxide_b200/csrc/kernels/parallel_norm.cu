@@ -180,6 +180,67 @@ rms_norm_step_kernel(float* stream, const T* y1, const T* y2, const float* __res
     out[(size_t)r * D + d] = from_f<T>(pn_row[d] * inv * (gain_offset + w[d]));
 }
 
+// The same pass with a norm that has no statistics: out = tanh(alpha * x) * w + b, alpha one learned number (Zhu, Chen, He, LeCun
+// and Liu, "Transformers without Normalization").  Every element stands for itself, so a row falls into as many blocks as fill
+// the device.  Behind 16-bit outputs the tanh is 1 - 2 / (1 + e^(2z)) by the hardware's exponential and division (some 1e-7
+// absolute, below the output's own rounding); the 32-bit path takes the accurate function.
+template <typename T>
+__device__ __forceinline__ float norm_tanh(float z) {
+  if (sizeof(T) == 2) return 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(z, 15.f)));
+  return tanhf(z);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(PN_NT)
+tanh_norm_step_kernel(float* stream, const T* y1, const T* y2, const float* __restrict__ alpha, const float* __restrict__ w,
+                      const float* __restrict__ b, T* out, const int* __restrict__ rows, int num_src_rows, int D, int init, int* err,
+                      int wide) {
+  pdl_launch_dependents();
+  const float a = out ? *alpha : 0.f;
+  pdl_wait();
+  const int r = blockIdx.x;
+  int src = r;
+  if (rows) {
+    src = rows[r];
+    if (src < 0 || src >= num_src_rows) {
+      if (threadIdx.x == 0 && blockIdx.y == 0) atomicOr(err, VOB_ERR_ROW);
+      return;
+    }
+  }
+  const size_t base = (size_t)src * D;
+  const bool store = rows == nullptr && (init || y1 || y2);
+  const int step = wide ? 4 : 1, stride = gridDim.y * PN_NT * step;
+  for (int d = (blockIdx.y * PN_NT + threadIdx.x) * step; d < D; d += stride) {
+    float x[4] = {0.f, 0.f, 0.f, 0.f}, u[4] = {0.f, 0.f, 0.f, 0.f}, v[4] = {0.f, 0.f, 0.f, 0.f};
+    float g[4] = {0.f, 0.f, 0.f, 0.f}, c[4] = {0.f, 0.f, 0.f, 0.f}, o[4];
+    if (wide) {
+      if (!init) load4(stream + base + d, x);
+      if (y1) load4(y1 + base + d, u);
+      if (y2) load4(y2 + base + d, v);
+      if (out) load4(w + d, g);
+      if (out && b) load4(b + d, c);
+    } else {
+      if (!init) x[0] = stream[base + d];
+      if (y1) u[0] = to_f<T>(y1[base + d]);
+      if (y2) v[0] = to_f<T>(y2[base + d]);
+      if (out) g[0] = w[d];
+      if (out && b) c[0] = b[d];
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      x[i] += u[i] + v[i];
+      o[i] = fmaf(norm_tanh<T>(a * x[i]), g[i], c[i]);
+    }
+    if (wide) {
+      if (store) store4(stream + base + d, x);
+      if (out) store4(out + (size_t)r * D + d, o);
+    } else {
+      if (store) stream[base + d] = x[0];
+      if (out) out[(size_t)r * D + d] = from_f<T>(o[0]);
+    }
+  }
+}
+
 // out = 0.5 * (a / rms(a) * wa + b / rms(b) * wb): two mixers side by side over the same input, each with an RMS norm over
 // the width (plain gains), then their mean; `ba` is added to a's rows first (a bias of the product that made them).  One
 // block a token; float sums.
@@ -250,6 +311,25 @@ VOB_API int vob_rms_norm_step(float* stream, const void* y1, const void* y2, con
   if (dtype == VOB_F32) VOB_RN_LAUNCH(float);
   if (dtype == VOB_BF16) VOB_RN_LAUNCH(__nv_bfloat16);
 #undef VOB_RN_LAUNCH
+  return VOB_BAD_ARGUMENT;
+}
+
+// As vob_layer_norm_step with the elementwise norm: see tanh_norm_step_kernel.  alpha one float, on the device.
+VOB_API int vob_tanh_norm_step(float* stream, const void* y1, const void* y2, const float* alpha, const float* w, const float* b,
+                               void* out, const int* rows, int n_out, int num_src_rows, int D, int init, int dtype, int* err,
+                               cudaStream_t stream_) {
+  if (n_out <= 0) return 0;
+  if (D <= 0 || (rows && !out) || (out && (!w || !alpha))) return VOB_BAD_ARGUMENT;
+  const int wide = D % 4 == 0 && (((uintptr_t)stream | (uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)w | (uintptr_t)b | (uintptr_t)out) & 15) == 0;
+  // a block for every 256 (x 4) elements of a row: four elements a thread
+  const int per = PN_NT * (wide ? 4 : 1);
+  const dim3 grid(n_out, min(64, (D + per - 1) / per));
+#define VOB_TN_LAUNCH(TYPE)                                                                                            \
+  return launch_kernel(tanh_norm_step_kernel<TYPE>, grid, PN_NT, 0, stream_, stream, (const TYPE*)y1, (const TYPE*)y2, \
+                       alpha, w, b, (TYPE*)out, rows, num_src_rows, D, init, err, wide)
+  if (dtype == VOB_F32) VOB_TN_LAUNCH(float);
+  if (dtype == VOB_BF16) VOB_TN_LAUNCH(__nv_bfloat16);
+#undef VOB_TN_LAUNCH
   return VOB_BAD_ARGUMENT;
 }
 

@@ -177,6 +177,9 @@ lru_scan_kernel(const T* u, const float* gates, const T* y, long y_stride, const
 //   HgrnSource       qfv [tokens, heads*dk | heads*dk | heads*dv]: q = silu(q), f = l + (1 - l) sigmoid(f + bf), w = 1 - f
 //   GlaSource        q * scale, w = k, f = sigmoid(z + bz)^(1 / tau) = exp(-softplus(-(z + bz)) / tau), a number a head and row
 //   LightningSource  q = silu(q), w = silu(k), v = silu(v), f = a fixed number a head
+//   MlstmSource      q * scale, w = put * k, f = keep: two numbers a head and token (exponential gates, mlstm_gates below)
+// A source with a NORMALISER carries one more column beside the head's dv, whose value is 1 at every token: n = diag(f) n + w.
+// Its read-out n . q divides the head's outputs.  The column lies behind all heads' matrices, [heads, dk].
 // Decoding (matrix_scan_fused): one block a (request, head) that also takes the head's norm and what the source puts behind it.
 // Column j of a head's state M (dk floats) is shared by PARTS neighbouring lanes, R rows each, in registers.  The gates of
 // HG_TT tokens are made by the whole block at once and parked in shared memory (rows padded so that the PARTS lanes of a column
@@ -202,10 +205,14 @@ __device__ __forceinline__ int hg_pad(int i) { return i + 4 * (i >> 5); }
 
 struct ScanGates { float q, f, w; };
 
+// What a head keeps by: a number a row and token, one number for all of a head's tokens, or a number a token for all its rows.
+enum { DECAY_ROW = 0, DECAY_FIXED = 1, DECAY_TOKEN = 2 };
+
 // What a source keeps of a (head, row) over the tokens, what it reads of a token, and what it makes of both.
 template <typename T>
 struct HgrnSource {
-  static constexpr bool FIXED_DECAY = false;
+  static constexpr int DECAY = DECAY_ROW;
+  static constexpr bool NORMALISER = false, HEAD_GATES = false;
   const T* rows;
   long width;
   const T* bf;
@@ -233,7 +240,8 @@ struct HgrnSource {
 // rows: q | k | v (heads*dk, heads*dk, heads*dv), the decay's pre-activations at z_off, the output gate at gate_off.
 template <typename T>
 struct GlaSource {
-  static constexpr bool FIXED_DECAY = false;      // whether a head keeps by one number at every token
+  static constexpr int DECAY = DECAY_ROW;
+  static constexpr bool NORMALISER = false, HEAD_GATES = false;
   const T* rows;
   long width;
   const float* bias;       // [heads * dk]
@@ -267,7 +275,8 @@ struct GlaSource {
 // rows: q | k | v (heads*dk, heads*dk, heads*dv).
 template <typename T>
 struct LightningSource {
-  static constexpr bool FIXED_DECAY = true;
+  static constexpr int DECAY = DECAY_FIXED;
+  static constexpr bool NORMALISER = false, HEAD_GATES = false;
   const T* rows;
   long width;
   const float* decays;     // [heads]
@@ -289,6 +298,113 @@ struct LightningSource {
   __device__ __forceinline__ float finish(float o, size_t, int, int) const { return o; }
 };
 
+// ---- exponential gates
+// Per head the pre-activations zi, zf (with biases) become log gates i = cap tanh(zi / cap), f = log sigmoid(cap tanh(zf / cap));
+// with the running maximum m_t = max(f + m_{t-1}, i) a token keeps by exp(f + m_{t-1} - m_t) and writes by exp(i - m_t).  `floor`
+// is exp(-m_t), the least that the normaliser's read-out counts as.
+struct LogGates { float i, f; };
+__device__ __forceinline__ LogGates log_gates(float zi, float zf, float cap) {
+  const float x = cap * tanhf(zf / cap);
+  return {cap * tanhf(zi / cap), fminf(x, 0.f) - log1pf(expf(-fabsf(x)))};
+}
+constexpr float MLSTM_EPS = 1e-6f;      // added to the normaliser
+
+// rows: q | k | v (heads*dk, heads*dk, heads*dv), the pre-activations of i and f (heads each) at i_off and f_off, the output gate
+// (heads*dv) at gate_off.  gates: float4 [tokens, heads] of (keep, put, floor, -), made by mlstm_gates_kernel for portions
+// (GLOBAL), in the kernel itself for decoding.  A request's running maximum lies behind the normalisers, [heads].
+template <typename T, bool GLOBAL>
+struct MlstmSource {
+  static constexpr int DECAY = DECAY_TOKEN;
+  static constexpr bool NORMALISER = true, HEAD_GATES = !GLOBAL;
+  const T* rows;
+  long width;
+  const float* bi;         // [heads]
+  const float* bf;         // [heads]
+  const float4* gates;
+  float* nq;               // [tokens, heads] the normaliser's read-out
+  int heads, dk, dv, i_off, f_off, gate_off;
+  float scale, cap;
+  struct Fixed {};
+  struct Raw { float q, k; float2 g; };
+  __device__ __forceinline__ Fixed fixed(int, int) const { return {}; }
+  __device__ __forceinline__ float fixed_decay(int) const { return 0.f; }
+  __device__ __forceinline__ Raw load(size_t t, int h, int i) const {
+    const T* row = rows + t * width;
+    return {to_f<T>(row[h * dk + i]), to_f<T>(row[(heads + h) * dk + i]),
+            GLOBAL ? *reinterpret_cast<const float2*>(gates + t * heads + h) : make_float2(1.f, 1.f)};
+  }
+  __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed&) const { return {r.q * scale, r.g.x, r.k * r.g.y}; }
+  __device__ __forceinline__ float token_decay(size_t t, int h) const { return gates[t * heads + h].x; }
+  __device__ __forceinline__ float value(size_t t, int h, int c) const { return to_f<T>(rows[t * width + (size_t)2 * heads * dk + h * dv + c]); }
+  __device__ __forceinline__ float decay(size_t t, int h, int, const Fixed&) const { return token_decay(t, h); }
+  __device__ __forceinline__ LogGates pre(size_t t, int h) const {
+    const T* row = rows + t * width;
+    return log_gates(to_f<T>(row[i_off + h]) + bi[h], to_f<T>(row[f_off + h]) + bf[h], cap);
+  }
+  // behind the head's norm: times sigmoid(gate)
+  __device__ __forceinline__ float finish(float o, size_t t, int h, int c) const {
+    return o * sigmoid_f(to_f<T>(rows[t * width + gate_off + (size_t)h * dv + c]));
+  }
+};
+
+// The gates of a step's portions, one block a (request, head).  m over a range of tokens is max(a + m, b) with a the sum of its f:
+// every thread folds its own range, the block scans the folds, and every thread walks its range again from its start.  A
+// range's last maximum is the next range's start by construction, so what a token keeps and writes refers to one and the same m.
+constexpr int MG_NT = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(MG_NT)
+mlstm_gates_kernel(const MlstmSource<T, true> src, float4* gates, float* state, long state_stride, const int* __restrict__ cu_q,
+                   const int* __restrict__ state_slots, int num_slots, int* err) {
+  __shared__ float wa[MG_NT / 32], wb[MG_NT / 32], starts[MG_NT + 1];
+  pdl_launch_dependents();
+  const int h = blockIdx.x, b = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t0 = cu_q[b], t1 = cu_q[b + 1], slot = state_slots[b];
+  pdl_wait();
+  if (t1 <= t0) return;
+  if (slot < 0 || slot >= num_slots) {
+    if (threadIdx.x == 0) atomicOr(err, VOB_ERR_SLOT);
+    return;
+  }
+  float* kept = state + (size_t)slot * state_stride + (size_t)src.heads * src.dk * (src.dv + 1) + h;
+  const float first = *kept;
+  const int per = (t1 - t0 + MG_NT - 1) / MG_NT;
+  const int lo = min(t1, t0 + (int)threadIdx.x * per), hi = min(t1, lo + per);
+  float a = 0.f, m = -INFINITY;
+#pragma unroll 4
+  for (int t = lo; t < hi; ++t) {
+    const LogGates g = src.pre((size_t)t, h);
+    a += g.f;
+    m = fmaxf(g.f + m, g.i);
+  }
+  // inclusive scan over the threads: what a fold (a, m) makes of a fold (a', m') before it
+#pragma unroll
+  for (int d = 1; d < 32; d <<= 1) {
+    const float pa = __shfl_up_sync(0xffffffffu, a, d), pm = __shfl_up_sync(0xffffffffu, m, d);
+    if (lane >= d) {
+      m = fmaxf(a + pm, m);
+      a += pa;
+    }
+  }
+  if (lane == 31) { wa[warp] = a; wb[warp] = m; }
+  __syncthreads();
+  float start = first;
+  for (int w = 0; w < warp; ++w) start = fmaxf(wa[w] + start, wb[w]);
+  starts[threadIdx.x + 1] = fmaxf(a + start, m);
+  if (threadIdx.x == 0) starts[0] = first;
+  __syncthreads();
+  m = starts[threadIdx.x];
+  const float last = starts[threadIdx.x + 1];
+#pragma unroll 2
+  for (int t = lo; t < hi; ++t) {
+    const LogGates g = src.pre((size_t)t, h);
+    const float next = t + 1 < hi ? fmaxf(g.f + m, g.i) : last;
+    gates[(size_t)t * src.heads + h] = make_float4(expf(g.f + m - next), expf(g.i - next), expf(-next), 0.f);
+    m = next;
+  }
+  if (hi == t1 && lo < hi) *kept = m;
+}
+
 // ---- decoding: a block a (request, head)
 template <typename T, typename SOURCE, int R, int PARTS>
 __global__ void __launch_bounds__(R > 32 ? 256 : 512)
@@ -303,6 +419,8 @@ matrix_scan_fused_kernel(const SOURCE src, const float* __restrict__ nw, float* 
   float* gs = fs + HG_TT * gate_row;     // [HG_TT][gate_row]  w
   float* vs = gs + HG_TT * gate_row;     // [HG_TT][cols]
   float* os = vs + HG_TT * cols;         // [HG_TT][cols]
+  __shared__ float keeps[SOURCE::HEAD_GATES ? HG_TT : 1], puts[SOURCE::HEAD_GATES ? HG_TT : 1], floors[SOURCE::HEAD_GATES ? HG_TT : 1];
+  __shared__ float norms[SOURCE::HEAD_GATES ? R * PARTS : 1];      // the head's normaliser: warp 0 walks it, a lane its own rows
   pdl_launch_dependents();
   const int part = threadIdx.x % PARTS, j = threadIdx.x / PARTS;
   const int h = blockIdx.x, b = blockIdx.y;
@@ -319,16 +437,48 @@ matrix_scan_fused_kernel(const SOURCE src, const float* __restrict__ nw, float* 
   float M[R];
 #pragma unroll
   for (int i = 0; i < R; ++i) M[i] = (i0 + i < dk && j < dv) ? mine[(size_t)i * dv] : 0.f;
+  float* norm = nullptr;                   // in the slot: the head's normaliser, the running maximum of its gates
+  float* kept = nullptr;
+  float run = 0.f;
+  if constexpr (SOURCE::HEAD_GATES) {
+    norm = state + (size_t)slot * state_stride + (size_t)heads * dk * dv + (size_t)h * dk;
+    kept = state + (size_t)slot * state_stride + (size_t)heads * dk * (dv + 1) + h;
+    run = *kept;
+    if (threadIdx.x < 32)
+      for (int i = threadIdx.x; i < dk; i += 32) norms[i] = norm[i];
+  }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
   // the gates of a tile: thread rows over tokens, thread columns over gates (one division, here)
   const int gate_lanes = min(dk, (int)blockDim.x), gate_step = blockDim.x / gate_lanes;
   const int gate_i = threadIdx.x % gate_lanes, gate_t = threadIdx.x / gate_lanes < gate_step ? threadIdx.x / gate_lanes : HG_TT;
   for (int ts = t0; ts < t1; ts += HG_TT) {
     const int n = min(HG_TT, t1 - ts);
+    if constexpr (SOURCE::HEAD_GATES) {
+      // warp 0: a lane makes a token's log gates, the maxima go from lane to lane, a lane makes its token's factors
+      if (warp == 0) {
+        const LogGates lg = src.pre((size_t)(ts + min(lane, n - 1)), h);
+        float before = run, now = run;
+        for (int tt = 0; tt < n; ++tt) {
+          const float next = fmaxf(__shfl_sync(0xffffffffu, lg.f, tt) + run, __shfl_sync(0xffffffffu, lg.i, tt));
+          if (lane == tt) { before = run; now = next; }
+          run = next;
+        }
+        if (lane < n) {
+          keeps[lane] = expf(lg.f + before - now);
+          puts[lane] = expf(lg.i - now);
+          floors[lane] = expf(-now);
+        }
+      }
+      __syncthreads();
+    }
     for (int i = gate_i; i < dk; i += gate_lanes) {
       const typename SOURCE::Fixed fx = src.fixed(h, i);
       for (int tt = gate_t; tt < n; tt += gate_step) {
-        const ScanGates g = src.make(src.load((size_t)(ts + tt), h, i), fx);
+        ScanGates g = src.make(src.load((size_t)(ts + tt), h, i), fx);
+        if constexpr (SOURCE::HEAD_GATES) {
+          g.f = keeps[tt];
+          g.w *= puts[tt];
+        }
         qs[tt * gate_row + hg_pad(i)] = g.q;
         fs[tt * gate_row + hg_pad(i)] = g.f;
         gs[tt * gate_row + hg_pad(i)] = g.w;
@@ -339,6 +489,22 @@ matrix_scan_fused_kernel(const SOURCE src, const float* __restrict__ nw, float* 
       vs[idx] = c < dv ? src.value((size_t)(ts + tt), h, c) : 0.f;
     }
     __syncthreads();
+    if constexpr (SOURCE::HEAD_GATES) {
+      // what a token's outputs are divided by takes its floor's place
+      if (warp == 0)
+        for (int tt = 0; tt < n; ++tt) {
+          float s = 0.f;
+          for (int i = lane; i < dk; i += 32) {
+            const int at = tt * gate_row + hg_pad(i);
+            const float x = fmaf(fs[at], norms[i], gs[at]);
+            norms[i] = x;
+            s = fmaf(x, qs[at], s);
+          }
+          s = warp_sum(s);
+          if (lane == 0) floors[tt] = fmaxf(fabsf(s), floors[tt]) + MLSTM_EPS;
+          __syncwarp();
+        }
+    }
 #pragma unroll 2
     for (int tt = 0; tt < n; ++tt) {
       float o = 0.f;
@@ -365,11 +531,17 @@ matrix_scan_fused_kernel(const SOURCE src, const float* __restrict__ nw, float* 
     }
     __syncthreads();
     for (int tt = warp; tt < n; tt += nwarps) {
-      float ss = 0.f;
-      for (int c = lane; c < dv; c += 32) ss += os[tt * cols + c] * os[tt * cols + c];
+      float ss = 0.f, unit = 1.f;
+      if constexpr (SOURCE::HEAD_GATES) unit = 1.f / floors[tt];
+      for (int c = lane; c < dv; c += 32) {
+        const float o = os[tt * cols + c] * unit;
+        ss += o * o;
+      }
       const float denom = sqrtf(warp_sum(ss) / (float)dv + eps);
+      const float* gain = SOURCE::HEAD_GATES ? nw + (size_t)h * dv : nw;      // a gain for all heads' elements, or one head's
       for (int c = lane; c < dv; c += 32)
-        out[(size_t)(ts + tt) * heads * dv + h * dv + c] = from_f<T>(src.finish(os[tt * cols + c] / denom * nw[c], (size_t)(ts + tt), h, c));
+        out[(size_t)(ts + tt) * heads * dv + h * dv + c] =
+            from_f<T>(src.finish(os[tt * cols + c] * unit / denom * gain[c], (size_t)(ts + tt), h, c));
     }
     __syncthreads();
   }
@@ -377,6 +549,11 @@ matrix_scan_fused_kernel(const SOURCE src, const float* __restrict__ nw, float* 
 #pragma unroll
     for (int i = 0; i < R; ++i)
       if (i0 + i < dk) mine[(size_t)i * dv] = M[i];
+  }
+  if constexpr (SOURCE::HEAD_GATES) {
+    if (threadIdx.x < 32)
+      for (int i = threadIdx.x; i < dk; i += 32) norm[i] = norms[i];
+    if (threadIdx.x == 0) *kept = run;
   }
 }
 
@@ -396,11 +573,12 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
                         const int* __restrict__ state_slots, float* raw, float* ends, int heads, int dk, int dv, int col_blocks,
                         int num_slots, int mode, int* err) {
   constexpr int W = PARTS * MS_R;              // gates of a token, rows past dk are zeros
-  constexpr bool FIXED = SOURCE::FIXED_DECAY;
+  constexpr bool ROWS = SOURCE::DECAY == DECAY_ROW;      // a gate f a row lies in shared memory
+  constexpr int KINDS = ROWS ? 3 : 2;                    // rows of gates a token
   extern __shared__ float4 sm4[];
   const int walkers = blockDim.x - MS_LOADERS, threads = blockDim.x;
   const int cols = walkers / PARTS * MS_C;     // columns of this block
-  const int buffer = HG_TT * ((FIXED ? 2 : 3) * W + cols);
+  const int buffer = HG_TT * (KINDS * W + cols + (SOURCE::DECAY == DECAY_TOKEN ? 1 : 0));
   float* sm = reinterpret_cast<float*>(sm4);
   pdl_launch_dependents();
   const int h = blockIdx.x / col_blocks, c0 = blockIdx.x % col_blocks * cols;
@@ -427,13 +605,13 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
         float* q = sm + k * buffer + idx / (W - dk) * W + tile_index<PARTS>(dk + idx % (W - dk));
         q[0] = 0.f;
         q[HG_TT * W] = 0.f;
-        if (!FIXED) q[2 * HG_TT * W] = 0.f;
+        if (ROWS) q[2 * HG_TT * W] = 0.f;
       }
     for (int k = 0; k < tiles; ++k) {
       float* qs = sm + (k & 1) * buffer;       // [HG_TT][W] q
       float* ws = qs + HG_TT * W;              // [HG_TT][W] w
-      float* fs = ws + HG_TT * W;              // [HG_TT][W] f (not where it is one number a head)
-      float* vs = qs + HG_TT * (FIXED ? 2 : 3) * W;      // [HG_TT][cols]
+      float* fs = ws + HG_TT * W;              // [HG_TT][W] f (not where a head's rows share it)
+      float* vs = qs + HG_TT * KINDS * W;      // [HG_TT][cols], behind it [HG_TT] f where it is a number a token
       const int ts = t0 + k * HG_TT, n = min(HG_TT, t1 - ts);
       if (k >= 2) named_sync(3 + (k & 1), threads);      // the walkers have left this buffer
       for (int i = gate_i; i < dk; i += gate_lanes) {
@@ -451,10 +629,13 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
               const ScanGates g = src.make(raws[e], fx);
               if (OUT) qs[tt * W + at] = g.q;
               ws[tt * W + at] = g.w;
-              if (!FIXED) fs[tt * W + at] = g.f;
+              if (ROWS) fs[tt * W + at] = g.f;
             }
           }
         }
+      }
+      if constexpr (SOURCE::DECAY == DECAY_TOKEN) {
+        if (tid < n) vs[HG_TT * cols + tid] = src.token_decay((size_t)(ts + tid), h);
       }
       // (a thread keeps its column, eight tokens' loads in flight)
       const int v_lanes = min(cols, MS_LOADERS), v_step = MS_LOADERS / v_lanes;
@@ -475,8 +656,9 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
   // -------------------------------------------------- walkers
   const int part = threadIdx.x % PARTS, group = threadIdx.x / PARTS;
   const int j0 = c0 + group * MS_C, i0 = part * MS_R;
-  float* mine = mode == 0 ? state + (size_t)slot * state_stride + (size_t)h * dk * dv
-                          : ends + (((size_t)b * chunks + chunk) * heads + h) * dk * dv;
+  float* whole = mode == 0 ? state + (size_t)slot * state_stride
+                           : ends + ((size_t)b * chunks + chunk) * ((size_t)heads * dk * (dv + (SOURCE::NORMALISER ? 1 : 0)));
+  float* mine = whole + (size_t)h * dk * dv;
   // (a head's matrix starts on a 16-byte boundary where the state's rows do)
   const bool wide = dv % 4 == 0 && (((uintptr_t)mine) & 15) == 0;
   f32x2 M[MS_C][MS_R / 2];
@@ -506,11 +688,20 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
 #pragma unroll
     for (int c = 0; c < MS_C; ++c) M[c][r / 2] = pack2(a[0][c], a[1][c]);
   }
-  f32x2 f2[MS_R / 2];
-  if (FIXED) {
+  // the head's normaliser waits in shared memory: the first walker warp walks it tile by tile, behind the tile's matrices
+  __shared__ __align__(16) float norms[SOURCE::NORMALISER ? W : 4];
+  const bool norm_warp = SOURCE::NORMALISER && c0 == 0 && threadIdx.x < 32;
+  float* norm = whole + (size_t)heads * dk * dv + (size_t)h * dk;
+  if constexpr (SOURCE::NORMALISER) {
+    if (norm_warp) {
+      for (int i = threadIdx.x; i < W; i += 32) norms[tile_index<PARTS>(i)] = OUT && i < dk ? norm[i] : 0.f;
+      __syncwarp();
+    }
+  }
+  f32x2 f2[ROWS ? MS_R / 2 : 1];
+  if (SOURCE::DECAY == DECAY_FIXED) {
     const float f = src.fixed_decay(h);
-#pragma unroll
-    for (int p = 0; p < MS_R / 2; ++p) f2[p] = pack2(f, f);
+    f2[0] = pack2(f, f);
   }
   // the columns whose sums end in this lane
   constexpr int HALVINGS = PARTS >= 8 ? 3 : (PARTS >= 4 ? 2 : (PARTS >= 2 ? 1 : 0));
@@ -524,7 +715,7 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
     const float* qs = sm + (k & 1) * buffer;
     const float* ws = qs + HG_TT * W;
     const float* fs = ws + HG_TT * W;
-    const float* vs = qs + HG_TT * (FIXED ? 2 : 3) * W;
+    const float* vs = qs + HG_TT * KINDS * W;
     const int ts = t0 + k * HG_TT, n = min(HG_TT, t1 - ts);
     named_sync(1 + (k & 1), threads);
 #pragma unroll 1
@@ -539,10 +730,14 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
           const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(qs + at);
           q2[2 * p] = q.x; q2[2 * p + 1] = q.y;
         }
-        if (!FIXED) {
+        if (ROWS) {
           const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(fs + at);
-          f2[2 * p] = f.x; f2[2 * p + 1] = f.y;
+          f2[ROWS ? 2 * p : 0] = f.x; f2[ROWS ? 2 * p + 1 : 0] = f.y;
         }
+      }
+      if (SOURCE::DECAY == DECAY_TOKEN) {
+        const float f = vs[HG_TT * cols + tt];
+        f2[0] = pack2(f, f);
       }
       float v[MS_C], o[MS_C];
       {
@@ -556,7 +751,7 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
         f32x2 o2 = 0ull;
 #pragma unroll
         for (int p = 0; p < MS_R / 2; ++p) {
-          M[c][p] = fma2(f2[p], M[c][p], mul2(w2[p], v2));
+          M[c][p] = fma2(f2[ROWS ? p : 0], M[c][p], mul2(w2[p], v2));
           if (OUT) o2 = p == 0 ? mul2(M[c][p], q2[p]) : fma2(M[c][p], q2[p], o2);
         }
         if (OUT) {
@@ -587,9 +782,58 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
         }
       }
     }
+    if constexpr (SOURCE::NORMALISER) {
+      if (norm_warp) {      // the same for every lane of the warp; its groups hold copies
+        f32x2 n2[MS_R / 2];
+#pragma unroll
+        for (int p = 0; p < 2; ++p) {
+          const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(norms + (p * PARTS + part) * 4);
+          n2[2 * p] = x.x; n2[2 * p + 1] = x.y;
+        }
+#pragma unroll 1
+        for (int tt = 0; tt < n; ++tt) {
+          const float f = vs[HG_TT * cols + tt];
+          const f32x2 keep = pack2(f, f);
+          f32x2 s2 = 0ull;
+#pragma unroll
+          for (int p = 0; p < 2; ++p) {
+            const int at = tt * W + (p * PARTS + part) * 4;
+            const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(ws + at);
+            n2[2 * p] = fma2(keep, n2[2 * p], w.x);
+            n2[2 * p + 1] = fma2(keep, n2[2 * p + 1], w.y);
+            if (OUT) {
+              const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(qs + at);
+              s2 = fma2(n2[2 * p], q.x, s2);
+              s2 = fma2(n2[2 * p + 1], q.y, s2);
+            }
+          }
+          if (OUT) {
+            const float2 s = unpack2(s2);
+            float sum = s.x + s.y;
+#pragma unroll
+            for (int d = 1; d < PARTS; d <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+            if (threadIdx.x == 0) src.nq[(size_t)(ts + tt) * heads + h] = sum;
+          }
+        }
+        __syncwarp();
+        if (group == 0) {
+#pragma unroll
+          for (int p = 0; p < 2; ++p) {
+            ulonglong2 x;
+            x.x = n2[2 * p]; x.y = n2[2 * p + 1];
+            *reinterpret_cast<ulonglong2*>(norms + (p * PARTS + part) * 4) = x;
+          }
+        }
+        __syncwarp();
+      }
+    }
     if (k + 2 < tiles) named_arrive(3 + (k & 1), threads);
   }
   if (mode == 2) return;
+  if constexpr (SOURCE::NORMALISER) {
+    if (norm_warp)
+      for (int i = threadIdx.x; i < dk; i += 32) norm[i] = norms[tile_index<PARTS>(i)];
+  }
 #pragma unroll
   for (int r = 0; r < MS_R; r += 2) {
     float a[2][MS_C];
@@ -653,14 +897,15 @@ matrix_scan_range_decay_kernel(const SOURCE src, float* gates, const int* __rest
 constexpr int HG_MAX_CHUNKS = 16;
 
 __global__ void matrix_scan_join_kernel(float* state, long state_stride, float* ends, const float* gates, const int* __restrict__ cu_q,
-                                  const int* __restrict__ state_slots, int chunks, int heads, int dk, int dv, int num_slots) {
+                                  const int* __restrict__ state_slots, int chunks, int heads, int dk, int dv, long per,
+                                  int num_slots) {
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.y;
-  const long e = (long)blockIdx.x * blockDim.x + threadIdx.x, per = (long)heads * dk * dv;
+  const long e = (long)blockIdx.x * blockDim.x + threadIdx.x, matrices = (long)heads * dk * dv;
   const int slot = state_slots[b];
   if (e >= per || cu_q[b + 1] <= cu_q[b] || slot < 0 || slot >= num_slots) return;
-  const long row = e / dv;      // (head, i)
+  const long row = e < matrices ? e / dv : e - matrices;      // (head, i); behind the matrices a column of normalisers
   float L[HG_MAX_CHUNKS], F[HG_MAX_CHUNKS];
 #pragma unroll
   for (int c = 0; c < HG_MAX_CHUNKS; ++c)
@@ -730,7 +975,8 @@ template <typename SOURCE, int PARTS, bool OUT>
 int launch_scan_tile(const SOURCE& src, float* state, long state_stride, const int* cu_q, const int* state_slots, float* raw, float* ends,
                      int B, int chunks, int heads, int dk, int dv, int num_slots, int mode, int* err, cudaStream_t stream) {
   const int walkers = tile_walkers(dk, dv), cols = walkers / PARTS * MS_C, col_blocks = tile_col_blocks(dk, dv);
-  const size_t smem = (size_t)2 * HG_TT * ((SOURCE::FIXED_DECAY ? 2 : 3) * PARTS * MS_R + cols) * sizeof(float);
+  const size_t smem = (size_t)2 * HG_TT * ((SOURCE::DECAY == DECAY_ROW ? 3 : 2) * PARTS * MS_R + cols + (SOURCE::DECAY == DECAY_TOKEN ? 1 : 0)) *
+                      sizeof(float);
   auto kernel = matrix_scan_tile_kernel<SOURCE, PARTS, OUT>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -762,34 +1008,38 @@ template <typename T, typename SOURCE>
 int run_matrix_scan(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
                     void* out, float* raw, float* scratch, int Tn, int B, int chunks, int heads, int dk, int dv, float eps,
                     int num_slots, int fuse, int norm, int* err, cudaStream_t stream) {
+  const long per = (long)heads * dk * (dv + (SOURCE::NORMALISER ? 1 : 0));
   if (heads <= 0 || dk <= 0 || dv <= 0 || dk > 256 || B > 65535 || (!fuse && !raw) || (fuse && !scan_can_fuse(dk, dv)) ||
-      chunks < 1 || chunks > HG_MAX_CHUNKS || (chunks > 1 && (fuse || !scratch)) || state_stride < (long)heads * dk * dv)
+      chunks < 1 || chunks > HG_MAX_CHUNKS || (chunks > 1 && (fuse || !scratch)) || state_stride < per + (SOURCE::NORMALISER ? heads : 0))
     return VOB_UNSUPPORTED;
-  int code;
-  if (fuse) {
+  int code = 0;
+  // (a source that makes its head gates itself walks fused only, one whose gates are ready never)
+  if constexpr (SOURCE::HEAD_GATES || !SOURCE::NORMALISER) {
+    if (fuse) {
 #define VOB_SF(RR, PP) return launch_scan_fused<T, SOURCE, RR, PP>(src, nw, state, state_stride, cu_q, state_slots, out, B, heads, dk, dv, eps, num_slots, err, stream)
-    if (dk <= 16) VOB_SF(16, 1);
-    if (dk <= 32) VOB_SF(32, 1);
-    if (dk <= 64) VOB_SF(32, 2);
-    if (dk <= 128) VOB_SF(32, 4);
-    VOB_SF(64, 4);
+      if (dk <= 16) VOB_SF(16, 1);
+      if (dk <= 32) VOB_SF(32, 1);
+      if (dk <= 64) VOB_SF(32, 2);
+      if (dk <= 128) VOB_SF(32, 4);
+      VOB_SF(64, 4);
 #undef VOB_SF
+    }
   }
-  if (chunks <= 1) {
+  if constexpr (SOURCE::HEAD_GATES) return VOB_UNSUPPORTED;
+  else if (chunks <= 1) {
     code = dispatch_scan_tile(0, src, state, state_stride, cu_q, state_slots, raw, nullptr, B, 1, heads, dk, dv, num_slots, err,
                                          stream);
   } else {
     float* ends = scratch;
-    float* gates = scratch + (size_t)B * chunks * heads * dk * dv;
+    float* gates = scratch + (size_t)B * chunks * per;
     code = dispatch_scan_tile(1, src, state, state_stride, cu_q, state_slots, raw, ends, B, chunks, heads, dk, dv, num_slots, err,
                                          stream);
     if (code != 0) return code;
     code = launch_kernel(matrix_scan_range_decay_kernel<SOURCE>, dim3((heads * dk + 31) / 32, B, chunks), dim3(256), 0, stream, src, gates,
                          cu_q, heads, dk);
     if (code != 0) return code;
-    const long per = (long)heads * dk * dv;
     code = launch_kernel(matrix_scan_join_kernel, dim3((unsigned)((per + 255) / 256), B), dim3(256), 0, stream, state, state_stride, ends,
-                         (const float*)gates, cu_q, state_slots, chunks, heads, dk, dv, num_slots);
+                         (const float*)gates, cu_q, state_slots, chunks, heads, dk, dv, per, num_slots);
     if (code != 0) return code;
     code = dispatch_scan_tile(2, src, state, state_stride, cu_q, state_slots, raw, ends, B, chunks, heads, dk, dv, num_slots, err,
                                          stream);
@@ -923,5 +1173,40 @@ VOB_API int vob_lru_scan(const void* u, const float* gates, const void* y, long 
   if (dtype == VOB_BF16) VOB_LRU_CHUNKS(__nv_bfloat16);
 #undef VOB_LRU_CHUNKS
 #undef VOB_LRU
+  return VOB_BAD_ARGUMENT;
+}
+
+// rows: `width` elements a token, q | k | v first, the pre-activations of the input and forget gates (heads each) at i_off and
+// f_off, the output gate (heads*dv) at gate_off; bi, bf float [heads]; nw float [heads*dv]; gates float [T, heads, 4]; state float
+// [num_slots, state_stride]: the heads' matrices, their normalisers (heads*dk), their running maxima (heads).  With `fuse`, out
+// [T, heads*dv] of `dtype`: gates, recurrence, normaliser, head norm, gain and output gate in one launch.  Else raw float
+// [T, heads*dv] and nq float [T, heads], and vob_delta_out_norm makes the rest of them and of `gates`.  scratch: B * chunks *
+// heads * dk * (dv + 2) floats.
+VOB_API int vob_mlstm_scan(const void* rows, long width, int i_off, int f_off, int gate_off, const float* bi, const float* bf,
+                           const float* nw, float* gates, float* state, long state_stride, const int* cu_q, const int* state_slots,
+                           void* out, float* raw, float* nq, float* scratch, int T, int B, int chunks, int heads, int dk, int dv,
+                           float scale, float cap, float eps, int num_slots, int fuse, int dtype, int* err, cudaStream_t stream) {
+  if (B <= 0 || T <= 0) return 0;
+  if (!(cap > 0.f) || (!fuse && (!nq || !gates || ((uintptr_t)gates & 15)))) return VOB_BAD_ARGUMENT;
+  if (heads <= 0 || B > 65535) return VOB_UNSUPPORTED;
+#define VOB_ML(TT, GG)                                                                                                          \
+  const MlstmSource<TT, GG> src{(const TT*)rows, width, bi, bf, (const float4*)gates, nq, heads, dk, dv, i_off, f_off, gate_off, \
+                                scale, cap};                                                                                    \
+  if constexpr (GG) {                                                                                                           \
+    const int code = launch_kernel(mlstm_gates_kernel<TT>, dim3(heads, B), dim3(MG_NT), 0, stream, src, (float4*)gates, state,  \
+                                   state_stride, cu_q, state_slots, num_slots, err);                                            \
+    if (code != 0) return code;                                                                                                 \
+  }                                                                                                                             \
+  return run_matrix_scan<TT>(src, nw, state, state_stride, cu_q, state_slots, out, raw, scratch, T, B, chunks, heads, dk, dv,   \
+                             eps, num_slots, fuse, 0, err, stream)
+  if (dtype == VOB_F32) {
+    if (fuse) { VOB_ML(float, false); }
+    VOB_ML(float, true);
+  }
+  if (dtype == VOB_BF16) {
+    if (fuse) { VOB_ML(__nv_bfloat16, false); }
+    VOB_ML(__nv_bfloat16, true);
+  }
+#undef VOB_ML
   return VOB_BAD_ARGUMENT;
 }

@@ -336,6 +336,23 @@ def rms_norm_step(stream, eps: float, err, y1=None, y2=None, w=None, out=None, r
                                    _stream()), "rms_norm_step")
 
 
+def tanh_norm_step(stream, err, y1=None, y2=None, alpha=None, w=None, b=None, out=None, rows=None, n_out: Optional[int] = None,
+                   init: bool = False) -> None:
+    """layer_norm_step with a norm that has no statistics: out = tanh(alpha * x) * w + b, `alpha` one float on the device."""
+    _cuda(stream, y1, y2, alpha, w, b, out, rows)
+    assert stream.dtype == torch.float32 and stream.is_contiguous() and (alpha is None or alpha.numel() == 1)
+    for t in (alpha, w, b):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    act = next((t for t in (out, y1, y2) if t is not None), None)
+    for t in (y1, y2, out):
+        assert t is None or (t.dtype == act.dtype and t.is_contiguous() and t.shape[1] == stream.shape[1])
+    n_src = stream.shape[0]
+    n = n_src if rows is None else int(n_out)
+    _check(lib().vob_tanh_norm_step(_p(stream), _p(y1), _p(y2), _p(alpha), _p(w), _p(b), _p(out), _p(rows), n, n_src, stream.shape[1],
+                                    int(bool(init)), _code(act.dtype if act is not None else torch.float32), _p(err), _stream()),
+           "tanh_norm_step")
+
+
 def pair_norm_mean(a, b, wa, wb, out, eps: float, bias_a=None) -> None:
     """out = (a / rms(a) * wa + b / rms(b) * wb) / 2, row by row (float sums; a, b, out of one type, wa and wb float);
     `bias_a` (float): added to a's rows first."""
@@ -481,13 +498,20 @@ def delta_scan(qkv, ab, b_off: int, a_off: int, A_log, dt_bias, state, cu_q, sta
                                 _stream()), "delta_scan")
 
 
-def delta_out_norm(raw, gate, weight, out, num_tokens: int, heads: int, vdim: int, eps: float, gate_sigmoid: bool = False) -> None:
+def delta_out_norm(raw, gate, weight, out, num_tokens: int, heads: int, vdim: int, eps: float, gate_sigmoid: bool = False, nq=None,
+                   gates=None) -> None:
     """out[t, h] = raw[t, h] / sqrt(mean(raw[t, h]^2) + eps) * weight * SiLU(gate[t, h]) per head over vdim; gate: the
-    first heads * vdim columns of its rows.  `gate_sigmoid`: times sigmoid(gate) instead of SiLU(gate)."""
-    _cuda(raw, gate, weight, out)
+    first heads * vdim columns of its rows.  `gate_sigmoid`: times sigmoid(gate) instead of SiLU(gate).  weight: vdim gains
+    shared by the heads, or heads * vdim.  `nq` [tokens, heads] and `gates` [tokens, heads, 4] (float, of mlstm_scan): raw[t, h] is
+    first divided by max(|nq|, gates[..., 2]) + 1e-6."""
+    _cuda(raw, gate, weight, out, nq, gates)
+    assert weight.is_contiguous() and weight.numel() in (vdim, heads * vdim)
+    assert (nq is None) == (gates is None) and (nq is None or (nq.dtype == gates.dtype == torch.float32 and nq.is_contiguous()
+                                                               and gates.is_contiguous()))
     assert raw.dtype == torch.float32 and raw.is_contiguous() and out.is_contiguous() and gate.stride(1) == 1
     assert weight.dtype == torch.float32 and gate.dtype == out.dtype
-    _check(lib().vob_delta_out_norm(_p(raw), _p(gate), ctypes.c_long(gate.stride(0)), _p(weight), _p(out), num_tokens, heads,
+    _check(lib().vob_delta_out_norm(_p(raw), _p(gate), ctypes.c_long(gate.stride(0)), _p(weight),
+                                    0 if weight.numel() == vdim else vdim, _p(nq), _p(gates), _p(out), num_tokens, heads,
                                     vdim, ctypes.c_float(eps), int(bool(gate_sigmoid)), _code(out.dtype), _stream()), "delta_out_norm")
 
 
@@ -498,29 +522,36 @@ def moe_row_tile() -> int:
 
 def moe_route(h, w_router, correction, ids, weights, num_tokens: int, top: int, groups: int, keep: int,
               sigmoid_scores: bool = False, group_top: int = 1, normalise: bool = False, weight_scale: float = 1.0,
-              router_bias=None) -> None:
+              router_bias=None, w_shared=None, shared_gate=None) -> None:
     """ids, weights [tokens, top]: the experts a token uses and their scores (see csrc/kernels/moe.cu): the softmax over
     all experts or (`sigmoid_scores`) a sigmoid each, chosen by score + `correction` (None: by the score) among the `keep`
     groups that count most, a group by its best choice score or (`group_top` 2) by the sum of its two best; the weights
     are the chosen scores, divided by their sum with `normalise`, times `weight_scale`.  `router_bias` (float [experts]) is
-    added to the logits."""
-    _cuda(h, w_router, correction, ids, weights, router_bias)
+    added to the logits.  `w_shared` (float [width]) and `shared_gate` (float [tokens]): the sigmoid of w_shared . h, a number a
+    token, goes to shared_gate."""
+    _cuda(h, w_router, correction, ids, weights, router_bias, w_shared, shared_gate)
+    for t in (w_shared, shared_gate):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    assert w_shared is None or w_shared.numel() == w_router.shape[1]
     assert router_bias is None or (router_bias.dtype == torch.float32 and router_bias.is_contiguous())
     E, W = w_router.shape
     assert h.is_contiguous() and h.shape[1] == W and w_router.dtype == torch.float32
     assert correction is None or (correction.dtype == torch.float32 and correction.is_contiguous())
     assert w_router.is_contiguous() and ids.dtype == torch.int32 and weights.dtype == torch.float32 and group_top in (1, 2)
-    _check(lib().vob_moe_route(_p(h), _p(w_router), _p(router_bias), _p(correction), _p(ids), _p(weights), num_tokens, W, E, top, groups, keep,
+    _check(lib().vob_moe_route(_p(h), _p(w_router), _p(router_bias), _p(correction), _p(w_shared), _p(shared_gate), _p(ids),
+                               _p(weights), num_tokens, W, E, top, groups, keep,
                                int(bool(sigmoid_scores)), int(group_top), int(bool(normalise)), ctypes.c_float(weight_scale),
                                _code(h.dtype), _stream()), "moe_route")
 
 
-def moe_align(ids, slot_of, row_token, tile_expert, n: int, top: int, experts: int, pad: Optional[int] = None) -> None:
+def moe_align(ids, slot_of, row_token, tile_expert, n: int, top: int, experts: int, pad: Optional[int] = None, weights=None,
+              row_weight=None) -> None:
     """Sorts n (token, choice) pairs by expert: slot_of[n] a pair's row, row_token[rows] a row's token or -1, tile_expert
     [rows / moe_row_tile()] the expert of every moe_row_tile() rows or -1.  An expert's rows are padded to `pad` rows (a
-    multiple of moe_row_tile(), which is the default)."""
-    _cuda(ids, slot_of, row_token, tile_expert)
-    _check(lib().vob_moe_align(_p(ids), _p(slot_of), _p(row_token), _p(tile_expert), n, top, experts, row_token.numel(),
+    multiple of moe_row_tile(), which is the default).  `weights` [n], `row_weight` [rows]: a row also gets its pair's weight."""
+    _cuda(ids, slot_of, row_token, tile_expert, weights, row_weight)
+    assert row_weight is None or (row_weight.dtype == weights.dtype == torch.float32 and row_weight.numel() == row_token.numel())
+    _check(lib().vob_moe_align(_p(ids), _p(weights), _p(slot_of), _p(row_token), _p(row_weight), _p(tile_expert), n, top, experts, row_token.numel(),
                                int(pad or moe_row_tile()), _stream()), "moe_align")
 
 
@@ -534,16 +565,20 @@ def moe_gemm_tc5_supported(a, w) -> bool:
             and w.is_contiguous() and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def moe_gemm_tc5(a, w, c, row_token, tile_expert, relu_squared: bool, err, silu_pairs: bool = False, glu_limit: float = 0.0) -> None:
+def moe_gemm_tc5(a, w, c, row_token, tile_expert, relu_squared: bool, err, silu_pairs: bool = False, glu_limit: float = 0.0,
+                 row_weight=None) -> None:
     """c[row] = f(a[row] @ w[expert of the row]^T) on the tcgen05 tensor cores: a [rows, K] bfloat16 already sorted by
     expert in row tiles of moe_tc5_row_tile(), w [experts, N, K]; c bfloat16 with the squared relu, bfloat16 [rows, N / 2]
-    with `silu_pairs` (rows of w in (gate, up) pairs: SiLU(gate) * up), or float."""
-    _cuda(a, w, c, row_token, tile_expert)
+    with `silu_pairs` (rows of w in (gate, up) pairs: SiLU(gate) * up), or float.  `row_weight` (float [rows], with silu_pairs; also
+    in moe_gemm): a factor on a row's gate and up, as if it had multiplied the row."""
+    _cuda(a, w, c, row_token, tile_expert, row_weight)
+    assert row_weight is None or (silu_pairs and row_weight.dtype == torch.float32 and row_weight.numel() == row_token.numel())
     E, N, K = w.shape
     assert moe_gemm_tc5_supported(a, w) and a.shape[0] == row_token.numel() and c.stride(1) == 1
     assert c.dtype == (torch.bfloat16 if relu_squared or silu_pairs else torch.float32) and not (relu_squared and silu_pairs)
     map_w, map_x = tensor_map_2d(w.view(E * N, K), 128), tensor_map_2d(a, 128)
-    _check(lib().vob_moe_gemm_tc5(map_w, map_x, _p(c), ctypes.c_long(c.stride(0)), _p(row_token), _p(tile_expert), a.shape[0], N, K,
+    _check(lib().vob_moe_gemm_tc5(map_w, map_x, _p(c), ctypes.c_long(c.stride(0)), _p(row_token), _p(row_weight), _p(tile_expert),
+                                  a.shape[0], N, K,
                                   2 if silu_pairs else (0 if relu_squared else 1), ctypes.c_float(glu_limit), _p(err), _stream()),
            "moe_gemm_tc5")
 
@@ -557,17 +592,18 @@ def moe_gather_rows(x, xs, row_token) -> None:
 
 
 def moe_gemm(a, w, c, row_token, tile_expert, relu_squared: bool, gather: bool, silu_pairs: bool = False,
-             glu_limit: float = 0.0) -> None:
+             glu_limit: float = 0.0, row_weight=None) -> None:
     """c[row] = f(a[row or its token] @ w[expert of the row]^T), w [experts, N, K]; float accumulation in one chain.  f: the
     squared relu, or (`silu_pairs`: rows of w in (gate, up) pairs, c [rows, N / 2]) SiLU(gate) * up, both with `gather`
     into a's type; or the identity into float.  `glu_limit` > 0 with `silu_pairs`: the clamped form min(gate, limit) *
     sigmoid(1.702 min(gate, limit)) * (clamp(up, -limit, limit) + 1) (also in moe_gemv and moe_gemm_tc5)."""
-    _cuda(a, w, c, row_token, tile_expert)
+    _cuda(a, w, c, row_token, tile_expert, row_weight)
+    assert row_weight is None or (silu_pairs and row_weight.dtype == torch.float32 and row_weight.numel() == row_token.numel())
     assert a.stride(1) == 1 and w.is_contiguous() and c.stride(1) == 1 and a.dtype == w.dtype
     first = relu_squared or silu_pairs
     assert c.dtype == (a.dtype if first else torch.float32) and first == gather and not (relu_squared and silu_pairs)
     _check(lib().vob_moe_gemm(_p(a), ctypes.c_long(a.stride(0)), _p(w), _p(c), ctypes.c_long(c.stride(0)), _p(row_token),
-                              _p(tile_expert), row_token.numel(), w.shape[1], w.shape[2], 2 if silu_pairs else int(relu_squared),
+                              _p(row_weight), _p(tile_expert), row_token.numel(), w.shape[1], w.shape[2], 2 if silu_pairs else int(relu_squared),
                               int(gather), int(not first), ctypes.c_float(glu_limit),
                               _code(a.dtype), _stream()), "moe_gemm")
 
@@ -584,25 +620,28 @@ def moe_gemv_supported(a, w, n: int) -> bool:
             and w.is_contiguous() and n <= 65535)
 
 
-def moe_gemv(a, w, c, ids, order, n: int, top: int, relu_squared: bool, silu_pairs: bool = False, glu_limit: float = 0.0) -> None:
+def moe_gemv(a, w, c, ids, order, n: int, top: int, relu_squared: bool, silu_pairs: bool = False, glu_limit: float = 0.0,
+             weights=None) -> None:
     """c[pair] = f(a[pair or its token] @ w[expert of the pair]^T) for the step's pairs, few of them (decoding): bfloat16,
     bound by the experts' rows, which a warp streams with 16-byte loads.  relu_squared: the first product (a by token, c
-    bfloat16); else the second (a by pair, c float)."""
-    _cuda(a, w, c, ids, order)
+    bfloat16); else the second (a by pair, c float).  `weights` (float [n], with silu_pairs): a factor on a pair's gate and up."""
+    _cuda(a, w, c, ids, order, weights)
+    assert weights is None or (silu_pairs and weights.dtype == torch.float32 and weights.numel() == n)
     first = relu_squared or silu_pairs          # silu_pairs: rows of w in (gate, up) pairs, c bfloat16 [pairs, N / 2]
     assert moe_gemv_supported(a, w, n) and c.stride(1) == 1 and c.dtype == (torch.bfloat16 if first else torch.float32)
-    _check(lib().vob_moe_gemv(_p(a), ctypes.c_long(a.stride(0)), _p(w), _p(c), ctypes.c_long(c.stride(0)), _p(ids), _p(order), n,
-                              top, w.shape[1], w.shape[2], 2 if silu_pairs else int(relu_squared), int(first),
+    _check(lib().vob_moe_gemv(_p(a), ctypes.c_long(a.stride(0)), _p(w), _p(c), ctypes.c_long(c.stride(0)), _p(ids), _p(order),
+                              _p(weights), n, top, w.shape[1], w.shape[2], 2 if silu_pairs else int(relu_squared), int(first),
                               ctypes.c_float(glu_limit), _stream()), "moe_gemv")
 
 
-def moe_combine(y, slot_of, weights, out, num_tokens: int, top: int, add=None) -> None:
+def moe_combine(y, slot_of, weights, out, num_tokens: int, top: int, add=None, add_gate=None) -> None:
     """out[t] = sum_j weights[t, j] * y[slot_of[t, j]] (float, j in order); slot_of None: pair (t, j) is row t * top + j.
-    `add` (like out): added to the sum before it is rounded."""
-    _cuda(y, slot_of, weights, out, add)
+    `add` (like out): added to the sum before it is rounded, times `add_gate` (float [tokens]) if given.  `weights` None: ones."""
+    _cuda(y, slot_of, weights, out, add, add_gate)
+    assert add_gate is None or (add is not None and add_gate.dtype == torch.float32 and add_gate.is_contiguous())
     assert add is None or (add.dtype == out.dtype and add.shape == out.shape and add.is_contiguous())
     assert y.dtype == torch.float32 and y.is_contiguous() and out.is_contiguous()
-    _check(lib().vob_moe_combine(_p(y), _p(slot_of), _p(weights), _p(add), _p(out), num_tokens, out.shape[1], top, _code(out.dtype),
+    _check(lib().vob_moe_combine(_p(y), _p(slot_of), _p(weights), _p(add), _p(add_gate), _p(out), num_tokens, out.shape[1], top, _code(out.dtype),
                                  _stream()), "moe_combine")
 
 
@@ -737,6 +776,34 @@ def lightning_scan(rows, decays, state, cu_q, state_slots, raw, num_requests: in
     _check(lib().vob_lightning_scan(_p(rows), ctypes.c_long(rows.stride(0)), _p(decays), _p(state), ctypes.c_long(state.stride(0)),
                                     _p(cu_q), _p(state_slots), _p(raw), _p(scratch), raw.shape[0], num_requests, int(chunks), heads,
                                     dk, dv, state.shape[0], _code(rows.dtype), _p(err), _stream()), "lightning_scan")
+
+
+def mlstm_scan(rows, i_off: int, f_off: int, gate_off: int, bias_i, bias_f, norm_weight, state, cu_q, state_slots, num_requests: int,
+               heads: int, dk: int, dv: int, scale: float, cap: float, eps: float, err, out=None, gates=None, raw=None, nq=None,
+               chunks: int = 1, scratch=None) -> None:
+    """A matrix memory with exponential gates over every request's tokens of this step, from and to its slot: log gates
+    i = cap tanh((zi + bias_i) / cap), f = log sigmoid(cap tanh((zf + bias_f) / cap)), m = max(f + m', i) (m' the token before's),
+    M = exp(f + m' - m) M + exp(i - m) k v^T, n likewise with k alone, o = M^T (scale q) / (max(|n . scale q|, exp(-m)) + 1e-6).
+    rows: q | k | v (heads * dk, heads * dk, heads * dv) first, zi, zf (heads each) at i_off, f_off, the output gate (heads * dv) at
+    gate_off.  state float [slots, >= heads * (dk * (dv + 1) + 1)]: matrices, n, m.  With `out` one block a (request, head) does it
+    all, the head's RMS norm, the gain (norm_weight float [heads * dv]) and the product with sigmoid(gate) included
+    (hgrn2_can_fuse).  Else `gates` [tokens, heads, 4], `raw` [tokens, heads * dv] and `nq` [tokens, heads] (float) receive the
+    factors, M^T (scale q) and n . scale q, and delta_out_norm makes the rest of them.  `chunks`, `scratch`: as hgrn2_scan, with
+    dv + 2 in the place of dv + 1."""
+    _cuda(rows, bias_i, bias_f, norm_weight, state, cu_q, state_slots, out, gates, raw, nq)
+    T = (raw if out is None else out).shape[0]
+    assert rows.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * (dk * (dv + 1) + 1)
+    for t, n in ((bias_i, heads), (bias_f, heads), (norm_weight, heads * dv)):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n
+    assert (out is None) != (raw is None) and (out is None or (out.dtype == rows.dtype and out.is_contiguous()))
+    for t, n in ((gates, heads * 4), (raw, heads * dv), (nq, heads)):
+        assert out is not None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == T * n)
+    assert _scan_scratch_ok(chunks, raw, scratch, num_requests, heads, dk, dv + 1)
+    _check(lib().vob_mlstm_scan(_p(rows), ctypes.c_long(rows.stride(0)), i_off, f_off, gate_off, _p(bias_i), _p(bias_f), _p(norm_weight),
+                                _p(gates), _p(state), ctypes.c_long(state.stride(0)), _p(cu_q), _p(state_slots), _p(out), _p(raw),
+                                _p(nq), _p(scratch), T, num_requests, int(chunks), heads, dk, dv, ctypes.c_float(scale),
+                                ctypes.c_float(cap), ctypes.c_float(eps), state.shape[0], int(out is not None), _code(rows.dtype),
+                                _p(err), _stream()), "mlstm_scan")
 
 
 def lru_scan(u, gates, y, bias_r, bias_i, lam, bias_y, state, cu_q, state_slots, out, num_requests: int, blocks: int, err,

@@ -7,10 +7,11 @@ from __future__ import annotations
 
 from typing import Callable, Dict, Tuple
 
-from ..config.model_config import ConfigError, DepolixConfig, KesozenConfig, LaruzenConfig, Qwen3Config, RakizenConfig, TofilornConfig
+from ..config.model_config import ConfigError, DepolixConfig, KesozenConfig, LaruzenConfig, NesezenConfig, Qwen3Config, RakizenConfig, TofilornConfig
 from .depolix import depolix_plan
 from .kesozen import kesozen_plan
 from .laruzen import laruzen_plan
+from .nesezen import nesezen_plan
 from .plan import ModelPlan
 from .qwen3 import qwen3_plan
 from .rakizen import rakizen_plan
@@ -49,3 +50,4 @@ register_architecture("Kesozen", KesozenConfig.from_dict, kesozen_plan)
 register_architecture("Rakizen", RakizenConfig.from_dict, rakizen_plan)
 register_architecture("Depolix", DepolixConfig.from_dict, depolix_plan)
 register_architecture("Laruzen", LaruzenConfig.from_dict, laruzen_plan)
+register_architecture("Nesezen", NesezenConfig.from_dict, nesezen_plan)

@@ -23,8 +23,10 @@ largest window of its writer and readers (`cache_window`).
 
 The rotation pairs neighbouring elements, or halves (element i with i + rotary_dim / 2) if the position rule says so, and
 computes its angles from frequencies (a position rule made with `table=False`, see parts/rope.py), so there is no largest
-position.  `gate`: the heads side by side are multiplied element by element by sigmoid(W_g h) (<prefix>g, one more block of
-rows in the down product) before the output product.
+position.  Without a position rule (and rot_dim 0) nothing is rotated.  `gate`: the heads side by side are multiplied by
+sigmoid(W_g h) (<prefix>g, one more block of rows in the down product) before the output product, element by element (`gate`
+True or "element") or with one number a head ("head": the attention kernels multiply a head's sum of latents by it, which W_uv,h
+carries on).
 """
 from __future__ import annotations
 
@@ -62,7 +64,7 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int,
                  scale: float, eps: float, window: Optional[int], position: Optional[str], prefix: str, positions: dict,
-                 dtype, device, borrow: bool = False, cache_window: Optional[int] = None, gate: bool = False, **_):
+                 dtype, device, borrow: bool = False, cache_window: Optional[int] = None, gate=False, **_):
         self.H, self.nh, self.dk, self.dr, self.dv = int(hidden_size), int(num_heads), int(dim), int(rot_dim), int(vdim)
         self.q_rank, self.kv_rank, self.scale, self.eps = int(q_rank), int(kv_rank), float(scale), float(eps)
         self.window = int(window or 0)
@@ -70,7 +72,9 @@ class LatentAttention(Mixer):
         if self.cache_window and (not self.window or self.window > self.cache_window):
             raise ValueError("a plane must keep at least the keys that its own layer reads")
         self.borrow, self.prefix, self.dtype, self.device = bool(borrow), prefix, dtype, device
-        self.gate, self.gate_off = bool(gate), 0
+        if gate not in (False, None, True, "element", "head"):
+            raise ValueError(f"the output gate is 'element' or 'head', or there is none, not {gate!r}")
+        self.gate, self.gate_off, self.head_gate = bool(gate), 0, gate == "head"
         if position is not None and position not in positions:
             raise KeyError(f"the plan names position encoding {position!r}, but has only {sorted(positions)}")
         self.rotation = positions[position].rotation_rule() if position is not None else NO_ROTATION
@@ -94,11 +98,11 @@ class LatentAttention(Mixer):
                   TensorSpec(p + "uv", (nh * self.dv, self.kv_rank), "matrix", self.kv_rank),
                   TensorSpec(p + "o", (H, nh * self.dv), "matrix", nh * self.dv)]
         if self.gate:
-            specs.append(TensorSpec(p + "g", (nh * self.dv, H), "matrix", H))
+            specs.append(TensorSpec(p + "g", (nh if self.head_gate else nh * self.dv, H), "matrix", H))
         return specs
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
-        p = self.prefix
+        p, nh = self.prefix, self.nh
         # rows of the query latent, then (a layer with a plane of its own) of the key/value latent and the shared key part
         rows = [tensors[p + "dq"]] + ([] if self.borrow else [tensors[p + "dkv"]])
         # the gate's rows follow, from a column that is a multiple of 8 (its reader takes 16-byte pieces where it can)
@@ -106,6 +110,8 @@ class LatentAttention(Mixer):
         if self.gate:
             pad = self.gate_off - sum(r.shape[0] for r in rows)
             rows += ([rows[0].new_zeros((pad, self.H))] if pad else []) + [tensors[p + "g"]]
+        if self.head_gate and nh % 8:
+            rows.append(rows[0].new_zeros((8 - nh % 8, self.H)))        # rows of the product stay 16-byte aligned
         self.wdown = torch.cat(rows, dim=0).contiguous()
         self.wq_norm = tensors[p + "dq.norm"].contiguous()
         self.wkv_norm = None if self.borrow else tensors[p + "dkv.norm"].contiguous()
@@ -144,13 +150,14 @@ class LatentAttention(Mixer):
         for k, h0 in enumerate(range(0, nh, step)):
             n = min(step, nh - h0)
             mixed = ctx.ws.get(f"latent_mixed{k}", T, n * self.row, x.dtype)
+            gate = dict(gate=down[:, self.gate_off + h0:], gate_stride=down.shape[1]) if self.head_gate else {}
             w = paged_attend(qa[:, h0 * self.row:(h0 + n) * self.row], nh * self.row, mixed, cache.k, cache.k, cache.group, ctx, T,
                              n, 1, self.row, self.window, self.scale, self._pairs[k] if self._pairs else None,
-                             value_dim=self.kv_rank)
+                             value_dim=self.kv_rank, **gate)
             # the plain kernel packs rows of n * w elements into the buffer, the tensor-core kernels fill its rows
             packed = mixed if w == self.row else mixed.reshape(-1)[:T * n * w].view(T, n * w)
             head_product(packed, w, self.kv_rank, self.wuv[h0:h0 + n], heads[:, h0 * self.dv:(h0 + n) * self.dv], self.dv, T)
-        if self.gate:
+        if self.gate and not self.head_gate:
             kernels.sigmoid_gate_mul(heads, down[:, self.gate_off:], nh * self.dv)
         return linear(heads, self.wo, ctx.ws.get("mixer_proj", T, self.H, x.dtype), ctx)
 

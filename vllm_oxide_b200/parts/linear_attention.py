@@ -14,6 +14,18 @@
     q = SiLU(W_q x),  k = SiLU(W_k x),  v = SiLU(W_v x);   S <- decay_h S + k v^T,   o = S^T q
     out = W_o [ RMSNorm(o over all heads) * norm * sigmoid(W_g x) ]
 
+`MLSTM`, a matrix memory with exponential gates held in range by a running maximum (Beck, Poeppel, Spanring and others, "xLSTM:
+Extended Long Short-Term Memory"), its log gates soft-capped:
+
+    q = W_q x * dim^(-1/2),  k = W_k x  [heads, dim],   v = W_v x  [heads, vdim]
+    i = cap * tanh((W_i x + b_i) / cap),   f = log sigmoid(cap * tanh((W_f x + b_f) / cap))        one of each a head
+    m <- max(f + m, i);   S <- exp(f + m' - m) S + exp(i - m) k v^T,   n likewise with k alone     (m' the maximum before; all 0 first)
+    o = S^T q / (max(|n . q|, exp(-m)) + 1e-6)
+    out = W_o [ RMSNorm_vdim(o) * norm * sigmoid(W_g x) ]                                          norm: a gain an element of every head
+
+Its state is the matrices, behind them n [heads, dim] and m [heads]; the gates of a portion are made ahead of its walk, from a scan of
+the maxima over the tokens.
+
 All projections of x are one product.  The state, [heads, dim, vdim] floats a request, lives in the cache manager's state slots;
 decays, their logarithms, the recurrence and the norms are float on both paths.  The walks are those of the package's other
 matrix states with a gate a row (csrc/kernels/recurrent.cu): one block a (request, head) while decoding, columns over blocks
@@ -72,11 +84,11 @@ class _MatrixState(Mixer):
     def state_spec(self) -> StateSpec:
         return StateSpec((self.nh * self.dk * self.dv,), torch.float32)
 
-    def _chunks(self, T: int, ctx):
-        """Ranges a request's tokens are cut into, and the scratch they need."""
+    def _chunks(self, T: int, ctx, extra: int = 0):
+        """Ranges a request's tokens are cut into, and the scratch they need (`extra`: columns beside a head's dv)."""
         B = ctx.launch_requests
         chunks = kernels.matrix_scan_chunks(T, B, self.nh, self.dk, self.dv)
-        scratch = None if chunks == 1 else ctx.ws.get_flat("matrix_scan_ranges", B * chunks * self.nh * self.dk * (self.dv + 1),
+        scratch = None if chunks == 1 else ctx.ws.get_flat("matrix_scan_ranges", B * chunks * self.nh * self.dk * (self.dv + 1 + extra),
                                                            torch.float32)
         return chunks, scratch
 
@@ -160,5 +172,53 @@ class LightningAttention(_MatrixState):
         return linear(out, self.wo, ctx.ws.get("mixer_proj", T, self.H, x.dtype), ctx)
 
 
+class MLSTM(_MatrixState):
+    def __init__(self, hidden_size: int, num_heads: int, dim: int, vdim: int, gate_cap: float, eps: float, prefix: str, dtype=None,
+                 device=None, **_):
+        super().__init__(hidden_size, num_heads, dim, vdim, eps, prefix)
+        self.cap = float(gate_cap)
+        if not self.cap > 0.0:
+            raise ValueError(f"the cap of the gates must be positive, not {gate_cap}")
+        self.bias_i = self.bias_f = None
+        self.i_off = self.f_off = 0
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        p, H, nh = self.prefix, self.H, self.nh
+        return self._projections() + [TensorSpec(p + "i", (nh, H), "matrix", H), TensorSpec(p + "i.b", (nh,), "coefficient", init="small"),
+                                      TensorSpec(p + "f", (nh, H), "matrix", H), TensorSpec(p + "f.b", (nh,), "coefficient", init="open"),
+                                      TensorSpec(p + "norm", (nh * self.dv,), "norm")]
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        p = self.prefix
+        gates = torch.cat([tensors[p + "i"], tensors[p + "f"]], dim=0)
+        self.w_in, (_, self.gate_off, self.i_off) = merged_rows([self._qkv(tensors), tensors[p + "g"], gates])
+        self.f_off = self.i_off + self.nh
+        self.bias_i, self.bias_f = tensors[p + "i.b"].contiguous(), tensors[p + "f.b"].contiguous()
+        self.norm_weight, self.wo = tensors[p + "norm"].contiguous(), tensors[p + "o"].contiguous()
+
+    def state_spec(self) -> StateSpec:
+        n = self.nh * (self.dk * (self.dv + 1) + 1)
+        return StateSpec(((n + 3) // 4 * 4,), torch.float32)      # rows stay 16-byte aligned
+
+    def forward(self, x, ctx, cache, state, write_cache: bool = True):
+        T, B, nh, dk, dv = x.shape[0], ctx.launch_requests, self.nh, self.dk, self.dv
+        row = linear(x, self.w_in, ctx.ws.get("mlstm_in", T, self.w_in.shape[0], x.dtype), ctx)
+        out = ctx.ws.get("mlstm_out", T, nh * dv, x.dtype)
+        common = (row, self.i_off, self.f_off, self.gate_off, self.bias_i, self.bias_f, self.norm_weight, state, ctx.cu_q,
+                  ctx.state_slots, B, nh, dk, dv, dk ** -0.5, self.cap, self.eps, ctx.err)
+        if kernels.hgrn2_can_fuse(dk, dv) and T <= 16 * B:
+            kernels.mlstm_scan(*common, out=out)
+        else:
+            gates = ctx.ws.get("mlstm_gates", T, nh * 4, torch.float32)
+            raw = ctx.ws.get("matrix_scan_raw", T, nh * dv, torch.float32)
+            nq = ctx.ws.get("mlstm_normaliser", T, nh, torch.float32)
+            chunks, scratch = self._chunks(T, ctx, extra=1)
+            kernels.mlstm_scan(*common, gates=gates, raw=raw, nq=nq, chunks=chunks, scratch=scratch)
+            kernels.delta_out_norm(raw, row[:, self.gate_off:], self.norm_weight, out, T, nh, dv, self.eps, gate_sigmoid=True, nq=nq,
+                                   gates=gates)
+        return linear(out, self.wo, ctx.ws.get("mixer_proj", T, self.H, x.dtype), ctx)
+
+
+register_part("mixer", "mlstm", MLSTM)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "lightning_attention", LightningAttention)

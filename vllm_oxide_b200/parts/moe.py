@@ -18,8 +18,11 @@ False has no correction tensor (the choice is by s); `group_top` 2 lets a group 
 scores; `normalise` divides the chosen scores by their sum (+ 1e-20); `weight_scale` multiplies them; `router_bias` adds <prefix>router.b to the logits;
 `activation` "glu_clamped" with `limit` makes an expert down(g * sigmoid(1.702 g) * (u + 1)) with g = min(gate(x), limit),
 u = clamp(up(x), -limit, limit).  The softmax over the chosen logits alone is `scores` "softmax" with `normalise` and no
-correction: the chosen shares of the full softmax, divided by their sum.  `shared` (a `swiglu` feed-forward's parameters): an
-expert that every token uses, added to the sum of the chosen ones before it is rounded.
+correction: the chosen shares of the full softmax, divided by their sum.  `weight_input`: a weight multiplies its expert's input
+instead of its output, sum_j expert_j(w_j x) (gated experts; by linearity of the first product, gate and up are multiplied behind
+it, in float).  `shared` (a `swiglu` feed-forward's parameters): an expert that every token uses, added to the sum of the chosen
+ones before it is rounded; `shared_gate` names a row (behind <prefix>) whose product with x, through a sigmoid, multiplies what
+the shared expert adds (made by the routing kernel).
 """
 from __future__ import annotations
 
@@ -67,7 +70,8 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, expert_size: int, experts: int, top: int, prefix: str, groups: int = 1, keep: int = 1,
                  names=("up", "down", "router", "correction"), activation: str = "relu2", gate_name: str = "gate",
                  scores: str = "softmax", correction: bool = True, group_top: int = 1, normalise: bool = False,
-                 weight_scale: float = 1.0, router_bias: bool = False, limit: float = 0.0, shared: Optional[dict] = None, **_):
+                 weight_scale: float = 1.0, router_bias: bool = False, limit: float = 0.0, shared: Optional[dict] = None,
+                 weight_input: bool = False, shared_gate: Optional[str] = None, **_):
         self.H, self.I, self.E, self.top = int(hidden_size), int(expert_size), int(experts), int(top)
         self.groups, self.keep, self.prefix = int(groups), int(keep), prefix
         if self.E % self.groups or self.keep > self.groups or self.top > (self.E // self.groups) * self.keep:
@@ -82,7 +86,12 @@ class RoutedExperts(FeedForward):
         self.has_router_bias = bool(router_bias)
         self.sigmoid_scores, self.has_correction, self.group_top = scores == "sigmoid", bool(correction), int(group_top)
         self.normalise, self.weight_scale = bool(normalise), float(weight_scale)
+        self.weight_input = bool(weight_input)
+        if self.weight_input and not self.gated:
+            raise ValueError("weights on the experts' inputs need gated experts")
         self.shared = SwiGLU(hidden_size=self.H, out_name="shared_out", **shared) if shared else None
+        self.n_shared_gate = self.prefix + shared_gate if shared_gate and self.shared is not None else None
+        self.w_shared = None
         self.wup = self.wdown = self.router = self.correction = self.router_b = None
 
     def parts(self):
@@ -103,6 +112,8 @@ class RoutedExperts(FeedForward):
             specs.append(TensorSpec(self.prefix + self.n_router + ".b", (self.E,), "coefficient", init="small"))
         if self.has_correction:
             specs.append(TensorSpec(self.prefix + self.n_correction, (self.E,), "coefficient", init="small"))
+        if self.n_shared_gate:
+            specs.append(TensorSpec(self.n_shared_gate, (1, self.H), "coefficient", self.H, init="normal"))
         return specs + (self.shared.tensor_specs() if self.shared is not None else [])
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -116,13 +127,15 @@ class RoutedExperts(FeedForward):
         self.router = tensors[self.prefix + self.n_router].contiguous()
         self.correction = tensors[self.prefix + self.n_correction].contiguous() if self.has_correction else None
         self.router_b = tensors[self.prefix + self.n_router + ".b"].contiguous() if self.has_router_bias else None
+        self.w_shared = tensors[self.n_shared_gate].reshape(self.H).contiguous() if self.n_shared_gate else None
         if self.shared is not None:
             self.shared.load({s.name: tensors[s.name] for s in self.shared.tensor_specs()})
 
-    def _route(self, x, ids, weights, T: int) -> None:
+    def _route(self, x, ids, weights, T: int, shared_gate=None) -> None:
         kernels.moe_route(x, self.router, self.correction, ids, weights, T, self.top, self.groups, self.keep,
                           sigmoid_scores=self.sigmoid_scores, group_top=self.group_top, normalise=self.normalise,
-                          weight_scale=self.weight_scale, router_bias=self.router_b)
+                          weight_scale=self.weight_scale, router_bias=self.router_b, w_shared=self.w_shared,
+                          shared_gate=shared_gate)
 
     def forward(self, x, ctx):
         T, top = x.shape[0], self.top
@@ -132,18 +145,22 @@ class RoutedExperts(FeedForward):
         fast = (n >= TC5_MIN_PAIRS and kernels.moe_gemm_tc5_supported(x, self.wup) and self.I % 8 == 0)
         ids = ctx.ws.get_flat("moe_ids", n, torch.int32)
         weights = ctx.ws.get_flat("moe_weights", n, torch.float32)
+        sg = ctx.ws.get_flat("moe_shared_gate", T, torch.float32) if self.w_shared is not None else None
+        # where the weights enter: the first product's epilogue, or the sum of the experts' rows
+        in_w, out_w = (weights, None) if self.weight_input else (None, weights)
         if (not fast and x.dtype == torch.bfloat16 and self.I % 8 == 0 and kernels.moe_gemv_supported(x, self.wup, n)):
             # bfloat16 steps of few pairs (decoding): nothing is sorted into tiles; the pairs are listed by expert and each
             # streams its expert's rows
             order = ctx.ws.get_flat("moe_order", n, torch.int32)
-            self._route(x, ids, weights, T)
+            self._route(x, ids, weights, T, sg)
             kernels.moe_order(ids, order, n, self.E)
             act = ctx.ws.get_flat("moe_act", n * self.I, x.dtype).view(n, self.I)
-            kernels.moe_gemv(x, self.wup, act, ids, order, n, top, not self.gated, silu_pairs=self.gated, glu_limit=self.limit)
+            kernels.moe_gemv(x, self.wup, act, ids, order, n, top, not self.gated, silu_pairs=self.gated, glu_limit=self.limit,
+                             weights=in_w)
             y = ctx.ws.get_flat("moe_y", n * self.H, torch.float32).view(n, self.H)
             kernels.moe_gemv(act, self.wdown, y, ids, order, n, top, False)
             out = ctx.ws.get("mlp_out", T, self.H, x.dtype)
-            kernels.moe_combine(y, None, weights, out, T, top, add=shared)
+            kernels.moe_combine(y, None, out_w, out, T, top, add=shared, add_gate=sg)
             return out
         tile = kernels.moe_tc5_row_tile() if fast else kernels.moe_row_tile()
         # every expert's rows are padded to a row tile: at most tile - 1 rows for each expert that has any
@@ -151,22 +168,23 @@ class RoutedExperts(FeedForward):
         slot_of = ctx.ws.get_flat("moe_slot_of", n, torch.int32)
         row_token = ctx.ws.get_flat("moe_row_token", max_rows, torch.int32)
         tile_expert = ctx.ws.get_flat("moe_tile_expert", max_rows // kernels.moe_row_tile(), torch.int32)
-        self._route(x, ids, weights, T)
-        kernels.moe_align(ids, slot_of, row_token, tile_expert, n, top, self.E, pad=tile)
+        row_weight = ctx.ws.get_flat("moe_row_weight", max_rows, torch.float32) if self.weight_input else None
+        self._route(x, ids, weights, T, sg)
+        kernels.moe_align(ids, slot_of, row_token, tile_expert, n, top, self.E, pad=tile, weights=in_w, row_weight=row_weight)
         act = ctx.ws.get_flat("moe_act", max_rows * self.I, x.dtype).view(max_rows, self.I)
         y = ctx.ws.get_flat("moe_y", max_rows * self.H, torch.float32).view(max_rows, self.H)
         if fast:
             rows = ctx.ws.get_flat("moe_rows", max_rows * self.H, x.dtype).view(max_rows, self.H)
             kernels.moe_gather_rows(x, rows, row_token)
             kernels.moe_gemm_tc5(rows, self.wup, act, row_token, tile_expert, not self.gated, ctx.err, silu_pairs=self.gated,
-                                 glu_limit=self.limit)
+                                 glu_limit=self.limit, row_weight=row_weight)
             kernels.moe_gemm_tc5(act, self.wdown, y, row_token, tile_expert, False, ctx.err)
         else:
             kernels.moe_gemm(x, self.wup, act, row_token, tile_expert, relu_squared=not self.gated, gather=True,
-                             silu_pairs=self.gated, glu_limit=self.limit)
+                             silu_pairs=self.gated, glu_limit=self.limit, row_weight=row_weight)
             kernels.moe_gemm(act, self.wdown, y, row_token, tile_expert, relu_squared=False, gather=False)
         out = ctx.ws.get("mlp_out", T, self.H, x.dtype)
-        kernels.moe_combine(y, slot_of, weights, out, T, top, add=shared)
+        kernels.moe_combine(y, slot_of, out_w, out, T, top, add=shared, add_gate=sg)
         return out
 
 

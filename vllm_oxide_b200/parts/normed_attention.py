@@ -7,6 +7,8 @@ frequencies, values divided by their own root mean square, a learned sink a head
     weights = exp(s) / (exp(sink_h) + sum exp(s)),  s = (q . k) * scale       (`sink`; else the plain softmax)
     out     = W_o [ heads * sigmoid(W_g x) ] + b_o                  (`gate`: element by element)
 
+`softcap` > 0: s becomes softcap * tanh(s / softcap).
+
 Every option is a parameter.  q, k, v and the gate are one product; biases, norms, rotation and the cache write are one kernel
 (`kernels.headnorm_rope_kv_write`).  A window lets the cache manager give back the pages behind it.  `out_bias` can be left to
 the kernel that reads the output (`defer_bias`), as the pair of mixers side by side does.
@@ -39,13 +41,15 @@ class NormedAttention(Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float, eps: float, prefix: str,
                  positions: dict, dtype, device, window: Optional[int] = None, position: Optional[str] = None, bias: bool = True,
-                 qk_norm: bool = True, value_norm: bool = True, sink: bool = True, gate: bool = True, **_):
+                 qk_norm: bool = True, value_norm: bool = True, sink: bool = True, gate: bool = True,
+                 softcap: float = 0.0, **_):
         if num_heads % num_kv_heads:
             raise ValueError(f"num_heads {num_heads} is not a multiple of num_kv_heads {num_kv_heads}")
         if not 0 < dim <= 512 or not 0 < vdim <= 512:
             raise ValueError(f"head sizes dim {dim} / vdim {vdim} are not supported by the attention kernels (up to 512)")
         self.H, self.nh, self.kvh, self.kd, self.vd = int(hidden_size), int(num_heads), int(num_kv_heads), int(dim), int(vdim)
         self.scale, self.eps, self.prefix, self.window = float(scale), float(eps), prefix, int(window or 0)
+        self.softcap = float(softcap or 0.0)
         self.bias, self.qk_norm, self.value_norm, self.sink, self.gate = bool(bias), bool(qk_norm), bool(value_norm), bool(sink), bool(gate)
         if position is not None and position not in positions:
             raise KeyError(f"the plan names position encoding {position!r}, but has only {sorted(positions)}")
@@ -104,7 +108,7 @@ class NormedAttention(Mixer):
                                        write_cache, ctx.err, kd_norm=self.kd, vd_norm=self.vd)
         heads = ctx.ws.get("normed_attn_heads", T, self.nh * self.vp, x.dtype)
         paged_attend(row, self.width, heads, cache.k, cache.v, cache.group, ctx, T, self.nh, self.kvh, self.kp, self.window,
-                     self.scale, self._pairs, sink=self.sinks if self.sink else False)
+                     self.scale, self._pairs, sink=self.sinks if self.sink else False, softcap=self.softcap)
         if self.gate:
             kernels.sigmoid_gate_mul(heads, row[:, self.gate_off:], self.nh * self.vp)
         out = linear(heads, self.wo, ctx.ws.get("normed_attn_proj", T, self.H, x.dtype), ctx)

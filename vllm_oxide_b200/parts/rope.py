@@ -13,7 +13,10 @@ slow} slows the long waves down and leaves the short ones alone: with d(t) = rot
 / (2 ln theta), the index whose wave makes t turns over `original` positions, a ramp r_i rises from 0 at
 lo = max(floor(d(fast)), 0) to 1 at hi = min(ceil(d(slow)), rotary_dim - 1) (its width at least 0.001);
 inv_freq[i] becomes inv_freq[i] / factor * r_i + inv_freq[i] * (1 - r_i), and cos and sin are both multiplied by
-0.1 ln(factor) + 1 (the "YaRN" interpolation of Peng, Quesnelle, Fan and Shippole).  `table=False` makes no table:
+0.1 ln(factor) + 1 (the "YaRN" interpolation of Peng, Quesnelle, Fan and Shippole).  `scaling` = {factor, original, low, high}
+goes by wavelength instead, w = 2 pi / inv_freq: inv_freq[i] / factor where w > original / low, inv_freq[i] where
+w < original / high, and between the two (1 - s) inv_freq[i] / factor + s inv_freq[i] with s = (original / w - low) / (high - low);
+cos and sin stay as they are (the scaling of the Llama 3.1 models).  `table=False` makes no table:
 the rule then carries the frequencies and the amplitude, the kernels compute float32(p) * inv_freq[i] where they
 rotate, and `max_position` bounds nothing.
 """
@@ -39,6 +42,14 @@ def scaled_frequencies(rotary_dim: int, theta: float, scaling: Optional[dict], p
     factor, original = float(scaling["factor"]), float(scaling["original"])
     if factor <= 0 or original <= 0:
         raise ValueError(f"rotary scaling needs a positive factor and original length, got {scaling!r}")
+
+    if "low" in scaling:
+        low, high = float(scaling["low"]), float(scaling["high"])
+        if not 0 < low < high:
+            raise ValueError(f"rotary scaling by wavelength needs 0 < low < high, got {scaling!r}")
+        turns = original * inv_freq / (2.0 * math.pi)              # how often a wave turns over the original length
+        share = ((turns - low) / (high - low)).clamp(0.0, 1.0)
+        return ((1.0 - share) * inv_freq / factor + share * inv_freq).to(torch.float32), 1.0
 
     def index_of(turns: float) -> float:
         return rotary_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(float(theta)))

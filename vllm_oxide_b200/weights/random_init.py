@@ -42,6 +42,8 @@ def random_tensor(spec: TensorSpec, seed: int, scheme: str, device, dtype: torch
             x = torch.sigmoid(x)
         elif spec.init == "normal":        # float matrices and vectors that are not near one: routers, filters, rates
             x = x / (float(spec.fan_in) ** 0.5) if spec.fan_in else x
+        elif spec.init == "open":          # pre-activations of gates that keep most of what they see
+            x = 4.0 + x
         elif spec.init == "small":
             x = 0.1 * x
         else:
