@@ -125,29 +125,34 @@ def mlstm_recurrence(q, k, v, i, f):
     """q, k [n, H, dk], v [n, H, dv], log gates i, f [n, H]: o [n, H, dv], from a state of zeros (the running maximum, too,
     starts at 0)."""
     n, H, dk = q.shape
-    S, z, m = q.new_zeros((H, dk, v.shape[2])), q.new_zeros((H, dk)), q.new_zeros(H)
-    out = q.new_zeros((n, H, v.shape[2]))
+    m, maxima = q.new_zeros(H), []
     for t in range(n):
-        new = torch.maximum(f[t] + m, i[t])
-        keep, put = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
-        m = new
-        S = keep[:, None, None] * S + put[:, None, None] * k[t][:, :, None] * v[t][:, None, :]
-        z = keep[:, None] * z + put[:, None] * k[t]
-        floor = torch.maximum((z * q[t]).sum(-1).abs(), torch.exp(-m))
-        out[t] = torch.einsum("hdv,hd->hv", S, q[t]) / (floor + 1e-6)[:, None]
-    return out
+        m = torch.maximum(f[t] + m, i[t])
+        maxima.append(m)
+    m = torch.stack(maxima)
+    before = torch.cat([torch.zeros_like(m[:1]), m[:-1]])
+    keep, put = torch.exp(f + before - m), torch.exp(i - m)
+    # the normaliser is one more value column that holds ones
+    S, w, v1 = q.new_zeros((H, dk, v.shape[2] + 1)), put[:, :, None] * k, torch.cat([v, torch.ones_like(v[:, :, :1])], dim=-1)
+    out = []
+    for t in range(n):
+        S = keep[t][:, None, None] * S + w[t][:, :, None] * v1[t][:, None, :]
+        out.append((q[t][:, None, :] @ S)[:, 0])
+    out = torch.stack(out)
+    floor = torch.maximum(out[..., -1].abs(), torch.exp(-m))
+    return out[..., :-1] / (floor + 1e-6)[..., None]
 
 
-def mlstm(h, W, p, m, eps, dt):
+def mlstm(h, W, p, m, eps, dt, noise=None):
+    """`noise` (a function) is applied to the projections."""
     n = h.shape[0]
     H, dk, dv = int(m["heads"]), int(m["dim"]), int(m["vdim"])
     g = lambda name: W[p + name].to(dt)
-    q = (h @ g("q").T).reshape(n, H, dk) * dk ** -0.5
-    k = (h @ g("k").T).reshape(n, H, dk)
-    v = (h @ g("v").T).reshape(n, H, dv)
-    i, f = mlstm_gates(h @ g("i").T + g("i.b"), h @ g("f").T + g("f.b"), float(m["gate_cap"]))
+    made = lambda name: (noise or (lambda t: t))(h @ g(name).T)
+    q, k, v = made("q").reshape(n, H, dk) * dk ** -0.5, made("k").reshape(n, H, dk), made("v").reshape(n, H, dv)
+    i, f = mlstm_gates(made("i") + g("i.b"), made("f") + g("f.b"), float(m["gate_cap"]))
     o = rms(mlstm_recurrence(q, k, v, i, f), eps).reshape(n, H * dv)
-    return (o * g("norm") * sigmoid(h @ g("g").T)) @ g("o").T
+    return (o * g("norm") * sigmoid(made("g"))) @ g("o").T
 
 
 # ---------------------------------------------------------------- attention through a latent, without positions
