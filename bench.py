@@ -18,7 +18,7 @@ of 8 requests whose context starts at 2,048 tokens, and prints ONE JSON line:
 The cache that the decode steps read was written by a real prefill of random prompts.  Every timed step reads 15 GB of weights, far more than the 126 MB L2, so nothing stays cached
 between iterations.  Peaks come from MEASURED_PEAKS.json beside this file when present.
 
-    python bench.py --workload tofilorn | kesozen | rakizen | depolix | laruzen [--sizes 2048,4096]
+    python bench.py --workload tofilorn | kesozen | rakizen | depolix | laruzen | nesezen [--sizes 2048,4096]
 
 measures the Tofilorn design (residual streams, minGRU, HGRN2, latent attention), the Kesozen design (sandwich norms over
 a float stream, attention whose keys are its values, gated delta rule, routed experts) or the Rakizen design (parallel
@@ -28,7 +28,9 @@ models beside Qwen3 at the same width, depth and feed-forward size (Kesozen also
 and 64 from a 2,048-token context (CUDA graphs), and, from an eager engine with the per-kernel timers on, the time of each
 of this package's kernels in those steps with the bytes it must move against the copy bandwidth.  The Laruzen design (token shift,
 gated linear and lightning attention, a gated linear recurrence beside attention with a learned sink, experts beside a shared
-one) is measured beside Depolix, Tofilorn and Kesozen too.
+one) is measured beside Depolix, Tofilorn and Kesozen too; the Nesezen design (an elementwise norm, matrix memories with exponential
+gates, windowed attention with capped scores, latent attention with a gate a head, experts weighted at their inputs) beside Laruzen,
+Rakizen and Depolix.
 
     python bench.py --workload serving-0.6b | mixed-32b
 
@@ -576,6 +578,51 @@ def laruzen_kernel_bytes(cfg: dict, T: int) -> dict:
     return b
 
 
+def nesezen_config(width: int, layers: int) -> dict:
+    """Layer sizes of a real model of this width: a block of four layers (attention, heads of 128 over 8 key heads, a window of
+    1,024, scores capped at 30; a matrix memory, heads of 128; attention through a latent of 256, heads of 128; a matrix memory
+    again); feed-forwards of 16 gated experts of which a token uses 4 (the four together three times the width) beside a shared one,
+    but for the first layer of each block, whose feed-forward is dense and three times the width."""
+    heads = width // 128
+    window = dict(heads=heads, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask={"size": 1024},
+                  rot={"dims": 128, "base": 10000.0, "scaling": {"factor": 8.0, "original": 2048, "low": 1.0, "high": 4.0}})
+    memory = dict(heads=heads, dim=128, vdim=128, gate_cap=15.0)
+    latent = dict(heads=heads, dim=128, vdim=128, q_rank=3 * width // 8, kv_rank=256, scale=128 ** -0.5)
+    moe = {"kind": "moe", "expert": {"ff": 3 * width // 4}, "router": {"experts": 16, "top": 4}, "shared": {"ff": 3 * width // 4}}
+    dense = {"kind": "dense", "ff": 3 * width}
+    out = []
+    for _ in range(0, layers, 4):
+        out += [{"type": "attention", "mixer": window, "mlp": dense}, {"type": "mlstm", "mixer": memory, "mlp": moe},
+                {"type": "latent_attention", "mixer": latent, "mlp": moe}, {"type": "mlstm", "mixer": memory, "mlp": moe}]
+    return {"architecture": "Nesezen", "vocab": 32768, "width": width, "norm": {"eps": 1e-6}, "layers": out[:layers]}
+
+
+def nesezen_kernel_bytes(cfg: dict, T: int) -> dict:
+    """Bytes that each of the design's own row-wise kernels must move in a step of T tokens, summed over the layers (weights
+    aside): what its time is held against.  Attention, the scans and the experts' products are held against arithmetic."""
+    D = cfg["width"]
+    b = {"tanh_norm_step": T * D * (2 + 4 + 2) - T * D * (2 + 2 * 4 + 2)}         # the stream begins: it is not read, and one output is less
+    add = lambda k, v: b.__setitem__(k, b.get(k, 0) + v)
+    for l in cfg["layers"]:
+        m, mlp = l["mixer"], l["mlp"]
+        add("tanh_norm_step", (2 if mlp else 1) * T * D * (2 + 2 * 4 + 2))
+        if l["type"] == "mlstm":
+            add("delta_out_norm", T * m["heads"] * m["vdim"] * (4 + 2 + 2))
+        elif l["type"] == "attention":
+            add("headnorm_rope_kv_write", T * 2 * ((m["heads"] + m["kv_heads"]) * m["dim"] + m["kv_heads"] * m["vdim"]) * 2)
+        else:
+            row = (m["kv_rank"] + 15) // 16 * 16
+            add("latent_prep", T * (m["q_rank"] + m["kv_rank"] + m["q_rank"] + row) * 2)
+        if mlp and mlp["kind"] == "dense":
+            add("silu_mul", T * 3 * mlp["ff"] * 2)
+        elif mlp:
+            top = mlp["router"]["top"]
+            add("silu_mul", T * 3 * mlp["shared"]["ff"] * 2)
+            add("moe_gather_rows", T * top * D * 2 * 2)
+            add("moe_combine", T * (top * D * 4 + 2 * D * 2))
+    return b
+
+
 def attention_flops(cfg: dict, T: int) -> float:
     """Multiply-adds x 2 of the score and value products of one prompt of T tokens, every query over the keys it sees."""
     def seen(size, blocks):
@@ -621,7 +668,7 @@ def qwen3_kernel_bytes(cfg: dict, T: int) -> dict:
 
 DESIGNS = {"tofilorn": (tofilorn_config, tofilorn_kernel_bytes), "kesozen": (kesozen_config, kesozen_kernel_bytes),
            "rakizen": (rakizen_config, rakizen_kernel_bytes), "depolix": (depolix_config, depolix_kernel_bytes),
-           "laruzen": (laruzen_config, laruzen_kernel_bytes)}
+           "laruzen": (laruzen_config, laruzen_kernel_bytes), "nesezen": (nesezen_config, nesezen_kernel_bytes)}
 
 
 def float_issue_rate():
@@ -659,6 +706,10 @@ def design_run(design: str, widths, pk=None, layers: int = 16) -> dict:
             models["depolix"] = depolix_config(width, layers)         # two mixers side by side, experts by softmax
             models["tofilorn"] = tofilorn_config(width, layers)       # the matrix-state and the channel recurrence
             models["kesozen"] = kesozen_config(width, layers)         # norms on both sides of every sublayer
+        if design == "nesezen":
+            models["laruzen"] = laruzen_config(width, layers)         # matrix states, windows, experts beside a shared one
+            models["rakizen"] = rakizen_config(width, layers)         # capped scores, a norm with a bias on a float stream
+            models["depolix"] = depolix_config(width, layers)         # attention through a latent
         rec = {}
         for name, cfg in models.items():
             r = {}
@@ -747,7 +798,37 @@ def design_run(design: str, widths, pk=None, layers: int = 16) -> dict:
                     if own.get("attention_prefill_tc5"):
                         r["prefill_2048"]["window_attention_frac_of_bf16_peak"] = round(
                             flops / (own["attention_prefill_tc5"] * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
-                if name in ("kesozen", "rakizen", "depolix", "laruzen"):
+                if design == "nesezen" and name in ("nesezen", "laruzen", "rakizen"):
+                    own, rate = r["prefill_2048"]["own_kernels_ms"], float_issue_rate()
+                    if name == "nesezen":
+                        # as hgrn2_scan: two walks, five float instructions a lane per state element and token
+                        memories = [l["mixer"] for l in cfg["layers"] if l["type"] == "mlstm"]
+                        work = sum(PROMPT_LEN * m["heads"] * m["dim"] * m["vdim"] * 5 for m in memories)
+                        if rate and own.get("mlstm_scan"):
+                            r["prefill_2048"]["mlstm_scan_frac_of_float_issue_rate"] = round(work / (own["mlstm_scan"] * 1e-3) / rate, 4)
+                        lat = [l["mixer"] for l in cfg["layers"] if l["type"] == "latent_attention"]
+                        flops = sum(2 * (PROMPT_LEN * (PROMPT_LEN + 1) // 2) * m["heads"] * 2 * ((m["kv_rank"] + 15) // 16 * 16) for m in lat)
+                        ms = own.get("attention_prefill_tma")
+                        if ms:
+                            r["prefill_2048"]["latent_attention_ms"] = ms
+                            r["prefill_2048"]["latent_attention_frac_of_bf16_peak"] = round(flops / (ms * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
+                    # a matrix state is read and written once a decode step
+                    states = [l["mixer"] for l in cfg["layers"] if l["type"] in ("mlstm", "gla")]
+                    ms = r["decode_batch8"]["own_kernels_ms"].get("mlstm_scan" if name == "nesezen" else "gla_scan")
+                    if ms and states:
+                        by = sum(8 * m["heads"] * m["dim"] * (m["vdim"] + (1 if name == "nesezen" else 0)) * 4 * 2 for m in states)
+                        r["decode_batch8"]["state_scan_frac_of_copy"] = round(by / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
+                    # windowed attention, with capped scores but for laruzen
+                    if name == "rakizen":
+                        flops = attention_flops(cfg, PROMPT_LEN)
+                    else:
+                        win = [l["mixer"] if name == "nesezen" else l["mixer"]["left"] for l in cfg["layers"]
+                               if l["type"] == ("attention" if name == "nesezen" else "parallel")]
+                        flops = sum(2 * sum(min(i, m["mask"]["size"] - 1) + 1 for i in range(PROMPT_LEN)) * m["heads"] * (m["dim"] + m["vdim"]) for m in win)
+                    if own.get("attention_prefill_tc5") and flops:
+                        r["prefill_2048"]["window_attention_frac_of_bf16_peak"] = round(
+                            flops / (own["attention_prefill_tc5"] * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
+                if name in ("kesozen", "rakizen", "depolix", "laruzen", "nesezen"):
                     own = r["prefill_2048"]["own_kernels_ms"]
                     if own.get("delta_scan"):
                         # the delta rule is arithmetic too: a multiply and three multiply-adds per state element and token
@@ -761,7 +842,7 @@ def design_run(design: str, widths, pk=None, layers: int = 16) -> dict:
                     if own.get("moe_gemm_tc5"):
                         # the experts' products against the measured bfloat16 product of the library
                         # (two products an expert; three where it is gated)
-                        flops = sum((6 if name in ("rakizen", "depolix", "laruzen") else 4) * PROMPT_LEN * l["mlp"]["router"]["top"] * cfg["width"] * l["mlp"]["expert"]["ff"]
+                        flops = sum((6 if name in ("rakizen", "depolix", "laruzen", "nesezen") else 4) * PROMPT_LEN * l["mlp"]["router"]["top"] * cfg["width"] * l["mlp"]["expert"]["ff"]
                                     for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe")
                         r["prefill_2048"]["moe_gemm_tc5_frac_of_bf16_peak"] = round(flops / (own["moe_gemm_tc5"] * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
             rec[name] = r
@@ -870,7 +951,7 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--workload", choices=sorted(WORKLOADS) + sorted(DESIGNS), default=None,
                     help="another workload instead of the default run")
-    ap.add_argument("--sizes", default="2048,4096", help="--workload tofilorn | kesozen | rakizen | depolix | laruzen: the widths to measure")
+    ap.add_argument("--sizes", default="2048,4096", help="--workload tofilorn | kesozen | rakizen | depolix | laruzen | nesezen: the widths to measure")
     ap.add_argument("--only", choices=["decode", "prefill", "attention"], default=None,
                     help="run one phase and print its time only (for short profiler captures)")
     args = ap.parse_args()

@@ -437,3 +437,54 @@ def test_scores_that_round_to_one_are_told_apart():
     ids, weights = torch.empty((n, 3), dtype=torch.int32, device=DEV), torch.empty((n, 3), device=DEV)
     kernels.moe_route(x, r, None, ids, weights, n, 3, 1, 1, sigmoid_scores=True)
     assert ids[0].tolist() == [2, 4, 6] and bool((weights == 1.0).all())
+
+
+# ---------------------------------------------------------------- sublayers that end in the stream
+@pytest.mark.parametrize("M", [1, 5, 8, 9, 16])
+@pytest.mark.parametrize("N, K", [(64, 128), (100, 320), (4800, 64), (33, 256)])
+def test_a_product_that_ends_in_the_stream(M, N, K):
+    """The weight-streaming product added into a float stream, unrounded, with the norm that follows beside it, or without."""
+    from vllm_oxide_b200 import kernels
+    bf, f32 = torch.bfloat16, torch.float32
+    err = torch.zeros(1, dtype=torch.int32, device=DEV)
+    x, w = rand((M, K), 1).to(bf).to(DEV), rand((N, K), 2, K ** -0.5).to(bf).to(DEV)
+    s0, g, b = rand((M, N), 3, 2.0).float(), (1.0 + 0.3 * rand((N,), 4)).float(), rand((N,), 5, 0.3).float()
+    alpha = torch.tensor([0.6])
+    want = s0.double() + x.double().cpu() @ w.double().cpu().T
+    for bias in (b, None):
+        stream, normed = s0.to(DEV), torch.empty((M, N), dtype=bf, device=DEV)
+        kernels.gemm_skinny(x, w, stream, kernels.EPI_STREAM, err, emit_tanh=(alpha.to(DEV), g.to(DEV), None if bias is None else b.to(DEV), normed))
+        assert_close(stream, want, f32, "stream", 1e-5)
+        assert_close(normed, P.tanh_norm(want, alpha.double(), g.double(), b.double() if bias is not None else 0.0), bf, "normed", 0.005)
+    stream = s0.to(DEV)
+    kernels.gemm_skinny(x, w, stream, kernels.EPI_STREAM, err)
+    assert_close(stream, want, f32, "stream, no norm", 1e-5)
+    assert int(err.item()) == 0
+
+
+@pytest.mark.parametrize("dt", DTYPES)
+@pytest.mark.parametrize("T, D, top", [(3, 64, 4), (7, 30, 2), (5, 1028, 1), (2, 4100, 9), (300, 128, 3)])
+def test_a_sum_of_experts_that_ends_in_the_stream(T, D, top, dt):
+    from vllm_oxide_b200 import kernels
+    f32 = torch.float32
+    dev = lambda t, d=f32: t.to(d).to(DEV).contiguous()
+    y, wt, add, ag = rand((T * top + 3, D), 1), rand((T, top), 2), held(rand((T, D), 3), dt), rand((T,), 4)
+    y, wt, ag = y.float().double(), wt.float().double(), ag.float().double()
+    slot = torch.randperm(T * top + 3, generator=torch.Generator().manual_seed(5))[:T * top].int()
+    slot[1] = -1                                                              # a pair that has no row
+    s0, g, b, alpha = rand((T, D), 6).float(), (1.0 + 0.3 * rand((D,), 7)).float(), rand((D,), 8, 0.3).float(), torch.tensor([0.8])
+    rows = torch.where((slot >= 0)[:, None], y[slot.long().clamp(min=0)], torch.zeros(1, dtype=torch.float64)).reshape(T, top, D)
+    for weights, gate in ((wt, ag), (None, ag), (wt, None)):
+        total = ((rows * weights[..., None]) if weights is not None else rows).sum(1) + add * (gate[:, None] if gate is not None else 1.0)
+        args = (dev(y), slot.to(DEV), None if weights is None else dev(weights))
+        more = dict(add=dev(add, dt), add_gate=None if gate is None else dev(gate))
+        out = torch.empty((T, D), dtype=dt, device=DEV)
+        kernels.moe_combine(*args, out, T, top, **more)
+        assert_close(out, total, dt, "a row of its own", 3e-6 if dt == f32 else 0.01)
+        stream = dev(s0)
+        kernels.moe_combine(*args, out, T, top, stream=stream, norm=(dev(alpha), dev(g), dev(b)), **more)
+        assert_close(stream, s0.double() + total, f32, "stream", 3e-6)
+        assert_close(out, P.tanh_norm(s0.double() + total, alpha.double(), g.double(), b.double()), dt, "normed", 3e-6 if dt == f32 else 0.005)
+        stream = dev(s0)
+        kernels.moe_combine(*args, None, T, top, stream=stream, **more)
+        assert_close(stream, s0.double() + total, f32, "stream, no norm", 3e-6)

@@ -92,6 +92,36 @@ __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 32 floa
   return t;
 }
 
+// Four neighbouring elements of the model's type as floats, by one access.
+__device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
+  const float4 x = *reinterpret_cast<const float4*>(p);
+  v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+}
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+}
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
+  uint2 raw;
+  *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v[0], v[1]);
+  *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = raw;
+}
+
+// tanh(alpha * x) * w + b, the norm without statistics, for an output of type T: behind a 16-bit output the tanh is
+// 1 - 2 / (1 + e^(2z)) by the hardware's exponential and division (some 1e-7 absolute, below the output's own rounding); the
+// 32-bit path takes the accurate function.
+template <typename T>
+__device__ __forceinline__ float tanh_norm(float x, float alpha, float w, float b) {
+  const float z = alpha * x;
+  return fmaf(sizeof(T) == 2 ? 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(z, 15.f))) : tanhf(z), w, b);
+}
+
 // N neighbouring elements of the model's type by one 16-byte access (N = 8 bfloat16 or 4 floats), as floats.
 template <typename T> struct Wide16;
 template <> struct Wide16<float> {

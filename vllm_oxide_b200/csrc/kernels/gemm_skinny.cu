@@ -31,6 +31,10 @@
 //         at its start and scales by 1/rms in the epilogue: the same values as NORM 1 up to the order in which
 //         the squares are added.
 //
+//   * a FLOAT stream can take the product too (EPI_STREAM): out is the stream, the product is added to it unrounded, and where a
+//     norm without statistics follows (tanh(alpha x) * w + b) its bfloat16 output is written beside it: the step between two
+//     sublayers costs no kernel of its own.
+//
 // Every wait on an mbarrier is bounded: a wait that runs out sets an error bit and a block-wide
 // abort flag; the block then waits (bounded again) for the copies it still has in flight and returns.
 #define VOB_TIMEOUT_WHERE 0x100
@@ -44,7 +48,7 @@ constexpr int SK_SLICES = SK_KC / TMA_BOX_COLS;   // boxes of 64 columns per sta
 constexpr int SK_CONSUMERS = 4;
 constexpr int SK_THREADS = (SK_CONSUMERS + 1) * 32;
 
-enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_ADD = 3, EPI_GEGLU = 4 };
+enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_ADD = 3, EPI_GEGLU = 4, EPI_STREAM = 5 };
 
 __device__ __forceinline__ void sk_ldmatrix_x4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
@@ -75,7 +79,7 @@ __global__ void __launch_bounds__(SK_THREADS, 2)
 gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, void* out,
                    long ldo, int M, int N, int K, int num_tiles, const float* __restrict__ norm_w, float eps,
                    const float* ss_parts, int ss_count, const float* __restrict__ emit_w, __nv_bfloat16* emit_xn,
-                   float* emit_ss, int* err) {
+                   float* emit_ss, const float* __restrict__ emit_alpha, const float* __restrict__ emit_b, int* err) {
   constexpr int S = SkStages<R, MT>::N;
   constexpr int RT = R / 16, NT = MT / 8;
   constexpr int W_SLICE = R * 128, X_SLICE = MT * 128;
@@ -165,16 +169,18 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
     const int b_chunk = MT == 16 ? (mi & 1) : ((lane >> 3) & 1);
     long it = 0;
     for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x) {
-      // EPI_ADD: what the tile's outputs hold now, asked for before the products rather than at their end
+      // EPI_ADD, EPI_STREAM: what the tile's outputs hold now, asked for before the products rather than at their end
       constexpr int ADD_PER_THREAD = (R * MT + SK_CONSUMERS * 32 - 1) / (SK_CONSUMERS * 32);
       float prev[ADD_PER_THREAD];
-      if (EPI == EPI_ADD) {
+      if (EPI == EPI_ADD || EPI == EPI_STREAM) {
 #pragma unroll
         for (int i = 0; i < ADD_PER_THREAD; ++i) {
           const int idx = (int)threadIdx.x + i * SK_CONSUMERS * 32;
           const int tok = idx / R;
-          const long n = (long)tile * R + idx % R;
-          prev[i] = (idx < R * m_rows && n < N) ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(out)[(long)tok * ldo + n]) : 0.f;
+          const long n = (long)tile * R + idx % R, at = (long)tok * ldo + n;
+          prev[i] = 0.f;
+          if (idx < R * m_rows && n < N)
+            prev[i] = EPI == EPI_STREAM ? reinterpret_cast<const float*>(out)[at] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(out)[at]);
         }
       }
       float acc[RT][NT][4];
@@ -302,6 +308,12 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
             if (NORM == 2) v *= sumsq[tok];
             if (EPI == EPI_F32) {
               reinterpret_cast<float*>(out)[(long)tok * ldo + n] = bf16_round(v);
+            } else if (EPI == EPI_STREAM) {
+              const float sv = prev[i] + v;
+              reinterpret_cast<float*>(out)[(long)tok * ldo + n] = sv;
+              if (emit_xn)
+                emit_xn[(long)tok * N + n] =
+                    __float2bfloat16_rn(tanh_norm<__nv_bfloat16>(sv, __ldg(emit_alpha), __ldg(emit_w + n), emit_b ? __ldg(emit_b + n) : 0.f));
             } else if (EPI == EPI_ADD) {
               const float sv = bf16_round(bf16_round(v) + prev[i]);
               reinterpret_cast<__nv_bfloat16*>(out)[(long)tok * ldo + n] = __float2bfloat16_rn(sv);
@@ -334,6 +346,8 @@ struct SkExtra {        // what only some products use
   const float* emit_w = nullptr;     // EPI_ADD: weight [N] of the norm that follows,
   __nv_bfloat16* emit_xn = nullptr;  //          where bfloat16(stream * weight) goes, [M, N],
   float* emit_ss = nullptr;          //          and the sums of squares, [tiles][MT]
+  const float* emit_alpha = nullptr; // EPI_STREAM: the norm that follows, tanh(alpha x) * emit_w + emit_b, into emit_xn
+  const float* emit_b = nullptr;
 };
 
 template <int R, int MT, int EPI, int NORM>
@@ -351,7 +365,7 @@ static int skinny_launch(const CUtensorMap* tmW, const CUtensorMap* tmX, void* o
   const int resident = 2 * sm_count();   // two blocks of this kernel fit an SM
   const int grid = num_tiles < resident ? num_tiles : resident;
   return launch_kernel(gemm_skinny_kernel<R, MT, EPI, NORM>, grid, SK_THREADS, smem, stream, *tmW, *tmX, out, ldo, M, N, K,
-                       num_tiles, norm_w, eps, x.ss_parts, x.ss_count, x.emit_w, x.emit_xn, x.emit_ss, err);
+                       num_tiles, norm_w, eps, x.ss_parts, x.ss_count, x.emit_w, x.emit_xn, x.emit_ss, x.emit_alpha, x.emit_b, err);
 }
 
 template <int R, int MT>
@@ -372,6 +386,7 @@ static int skinny_dispatch(int epilogue, const CUtensorMap* tw, const CUtensorMa
   if (epilogue == EPI_SWIGLU) return skinny_launch<R, MT, EPI_SWIGLU, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
   if (epilogue == EPI_GEGLU) return skinny_launch<R, MT, EPI_GEGLU, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
   if (epilogue == EPI_ADD) return skinny_launch<R, MT, EPI_ADD, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
+  if (epilogue == EPI_STREAM) return skinny_launch<R, MT, EPI_STREAM, 0>(tw, tx, out, ldo, M, N, K, nullptr, 0.f, x, err, stream);
   return VOB_BAD_ARGUMENT;
 }
 
@@ -403,20 +418,27 @@ VOB_API int vob_gemm_skinny_token_box(int M) { return M <= 8 ? 8 : 16; }
 // norm's weight, and ss_parts [ss_count][8 or 16] (the token rows of a box for this M) holds sums of squares of the
 // unscaled tokens that add up to each token's; the product is scaled by 1/rms.  emit_w / emit_xn / emit_ss (all or none;
 // epilogue 3): beside the sum into `out`, bfloat16(out * emit_w) goes to emit_xn [M, N] and, per tile of
-// vob_gemm_skinny_weight_box(N) rows and token, the sum of the squares of the new values of `out` to emit_ss.  Needs M <= 16.
+// vob_gemm_skinny_weight_box(N) rows and token, the sum of the squares of the new values of `out` to emit_ss.  Epilogue 5: out
+// [M,N] float += the product (a float residual stream); with emit_w, emit_xn and emit_alpha (one float, on the device; emit_b float
+// [N] or null) also bfloat16(tanh(alpha * out) * emit_w + emit_b) to emit_xn [M, N].  Needs M <= 16.
 VOB_API int vob_gemm_skinny(const void* map_w, const void* map_x, void* out, long ldo, int M, int N, int K, int epilogue,
                             const float* norm_w, float eps, const float* ss_parts, int ss_count, const float* emit_w,
-                            void* emit_xn, float* emit_ss, int* err, cudaStream_t stream) {
+                            void* emit_xn, float* emit_ss, const float* emit_alpha, const float* emit_b, int* err,
+                            cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 16 || K <= 0 || K % 64 || !map_w || !map_x) return VOB_UNSUPPORTED;
   if ((epilogue == EPI_SWIGLU || epilogue == EPI_GEGLU) && N % 16) return VOB_BAD_ARGUMENT;
   if (norm_w && (uintptr_t)norm_w % 8) return VOB_BAD_ARGUMENT;
   if (ss_parts && (norm_w || ss_count <= 0)) return VOB_BAD_ARGUMENT;
-  if ((emit_w != nullptr) != (emit_xn != nullptr) || (emit_w != nullptr) != (emit_ss != nullptr)) return VOB_BAD_ARGUMENT;
-  if (emit_w && epilogue != EPI_ADD) return VOB_BAD_ARGUMENT;
+  const bool streams = epilogue == EPI_STREAM;
+  if ((emit_w != nullptr) != (emit_xn != nullptr) || (emit_w != nullptr) != ((streams ? (const void*)emit_alpha : emit_ss) != nullptr))
+    return VOB_BAD_ARGUMENT;
+  if (emit_w && epilogue != EPI_ADD && !streams) return VOB_BAD_ARGUMENT;
+  if (streams ? emit_ss != nullptr : (emit_alpha || emit_b)) return VOB_BAD_ARGUMENT;
   SkExtra x;
   x.ss_parts = ss_parts; x.ss_count = ss_count;
   x.emit_w = emit_w; x.emit_xn = (__nv_bfloat16*)emit_xn; x.emit_ss = emit_ss;
+  x.emit_alpha = emit_alpha; x.emit_b = emit_b;
   const CUtensorMap* tw = (const CUtensorMap*)map_w;
   const CUtensorMap* tx = (const CUtensorMap*)map_x;
   const bool tall = vob_gemm_skinny_weight_box(N) == 32;

@@ -21,7 +21,8 @@
 //                 (the float path's product, with a tile's expert in front of it).
 //   moe_combine   out[t] = sum_j weight[t, j] * y[row of (t, j)], j in order, in float; a row may be added to it (`add`: what
 //                 an expert that every token uses has made of the token), times a number a token (`add_gate`).  No weights:
-//                 all ones (the weights went into the experts).
+//                 all ones (the weights went into the experts).  The sum may go into a float residual stream, with the norm
+//                 tanh(alpha x) * w + b of the new stream as what leaves.
 //   relu_squared  out = max(x, 0)^2 (the dense feed-forward's activation).
 #include "common.cuh"
 
@@ -312,21 +313,65 @@ moe_gemm_kernel(const TA* A, long lda, const TA* __restrict__ W, TC* C, long ldc
   }
 }
 
+// A thread takes four neighbouring columns of a token (`wide`: every row starts on a 16-byte boundary), or one; a token's row
+// falls into grid.y blocks.  With a float stream the sum does not leave as a row: stream[t] += sum, and with `norm_w` the norm
+// tanh(alpha x) * norm_w + norm_b of the new stream goes to out.
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_combine_kernel(const float* y, const int* slot_of, const float* weights, const T* add, const float* add_gate, T* out, int D, int top) {
+moe_combine_kernel(const float* y, const int* slot_of, const float* weights, const T* add, const float* add_gate, T* out, float* stream,
+                   const float* __restrict__ alpha, const float* __restrict__ norm_w, const float* __restrict__ norm_b, int D, int top,
+                   int wide) {
   pdl_launch_dependents();
+  const float a = norm_w ? *alpha : 0.f;
   pdl_wait();
-  const int t = blockIdx.x;
+  const int t = blockIdx.x, step = wide ? 4 : 1;
   const float ag = add_gate ? add_gate[t] : 1.f;
-  for (int d = threadIdx.x; d < D; d += 256) {
-    float acc = 0.f;
+  for (int d = (blockIdx.y * 256 + threadIdx.x) * step; d < D; d += gridDim.y * 256 * step) {
+    const size_t at = (size_t)t * D + d;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f}, x[4] = {0.f, 0.f, 0.f, 0.f}, s[4] = {0.f, 0.f, 0.f, 0.f};
+    if (add) {
+      if (wide) load4(add + at, x);
+      else x[0] = to_f<T>(add[at]);
+    }
+    if (stream) {
+      if (wide) load4(stream + at, s);
+      else s[0] = stream[at];
+    }
+#pragma unroll 4
     for (int j = 0; j < top; ++j) {
       const int row = slot_of ? slot_of[(size_t)t * top + j] : t * top + j;
-      if (row >= 0) acc = fmaf(weights ? weights[(size_t)t * top + j] : 1.f, y[(size_t)row * D + d], acc);
+      const float w = row < 0 ? 0.f : (weights ? weights[(size_t)t * top + j] : 1.f);
+      float v[4] = {0.f, 0.f, 0.f, 0.f};
+      if (row >= 0) {
+        if (wide) load4(y + (size_t)row * D + d, v);
+        else v[0] = y[(size_t)row * D + d];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i] = fmaf(w, v[i], acc[i]);
     }
-    if (add) acc = fmaf(ag, to_f<T>(add[(size_t)t * D + d]), acc);
-    out[(size_t)t * D + d] = from_f<T>(acc);
+    if (add) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i] = fmaf(ag, x[i], acc[i]);
+    }
+    if (stream) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[i] += acc[i];
+      if (wide) store4(stream + at, s);
+      else stream[at] = s[0];
+      if (!norm_w) continue;
+      float g[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+      if (wide) {
+        load4(norm_w + d, g);
+        if (norm_b) load4(norm_b + d, b);
+      } else {
+        g[0] = norm_w[d];
+        if (norm_b) b[0] = norm_b[d];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i] = tanh_norm<T>(s[i], a, g[i], b[i]);
+    }
+    if (wide) store4(out + at, acc);
+    else out[at] = from_f<T>(acc[0]);
   }
 }
 
@@ -568,16 +613,22 @@ VOB_API int vob_moe_gemv(const void* A, long lda, const void* W, void* C, long l
   return VOB_UNSUPPORTED;
 }
 
-// add [T, D] of `dtype`, or null; add_gate [T], or null; weights [T, top], or null (ones).
+// add [T, D] of `dtype`, or null; add_gate [T], or null; weights [T, top], or null (ones); stream float [T, D], or null: the sum is
+// added to it, and out (then null without norm_w) is its norm tanh(alpha x) * norm_w + norm_b, alpha one float on the device.
 VOB_API int vob_moe_combine(const float* y, const int* slot_of, const float* weights, const void* add, const float* add_gate, void* out,
-                            int T, int D, int top, int dtype, cudaStream_t stream) {
+                            float* stream_, const float* alpha, const float* norm_w, const float* norm_b, int T, int D, int top, int dtype,
+                            cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (dtype == VOB_F32)
-    return launch_kernel(moe_combine_kernel<float>, dim3(T), 256, 0, stream, y, slot_of, weights, (const float*)add, add_gate,
-                         (float*)out, D, top);
-  if (dtype == VOB_BF16)
-    return launch_kernel(moe_combine_kernel<__nv_bfloat16>, dim3(T), 256, 0, stream, y, slot_of, weights, (const __nv_bfloat16*)add,
-                         add_gate, (__nv_bfloat16*)out, D, top);
+  if ((norm_w && (!stream_ || !alpha)) || (!out && (!stream_ || norm_w))) return VOB_BAD_ARGUMENT;
+  const int wide = D % 4 == 0 && (((uintptr_t)y | (uintptr_t)add | (uintptr_t)out | (uintptr_t)stream_ | (uintptr_t)norm_w | (uintptr_t)norm_b) & 15) == 0;
+  const int per = 256 * (wide ? 4 : 1);
+  const dim3 grid(T, std::min(64, (D + per - 1) / per));
+#define VOB_MC(TT)                                                                                                                \
+  return launch_kernel(moe_combine_kernel<TT>, grid, 256, 0, stream, y, slot_of, weights, (const TT*)add, add_gate, (TT*)out, stream_, \
+                       alpha, norm_w, norm_b, D, top, wide)
+  if (dtype == VOB_F32) { VOB_MC(float); }
+  if (dtype == VOB_BF16) { VOB_MC(__nv_bfloat16); }
+#undef VOB_MC
   return VOB_BAD_ARGUMENT;
 }
 

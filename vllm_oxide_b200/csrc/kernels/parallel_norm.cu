@@ -19,27 +19,6 @@ namespace vob {
 
 constexpr int PN_NT = 256;
 
-// Four neighbouring elements of the model's type as floats, by one access.
-__device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
-  const float4 x = *reinterpret_cast<const float4*>(p);
-  v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
-}
-__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&v)[4]) {
-  const uint2 raw = *reinterpret_cast<const uint2*>(p);
-  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-  v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
-}
-__device__ __forceinline__ void store4(float* p, const float (&v)[4]) {
-  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-}
-__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
-  uint2 raw;
-  *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v[0], v[1]);
-  *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v[2], v[3]);
-  *reinterpret_cast<uint2*>(p) = raw;
-}
-
 template <typename T>
 __global__ void __launch_bounds__(PN_NT)
 layer_norm_step_kernel(float* stream, const T* y1, const T* y2, const float* __restrict__ w, const float* __restrict__ b,
@@ -182,14 +161,7 @@ rms_norm_step_kernel(float* stream, const T* y1, const T* y2, const float* __res
 
 // The same pass with a norm that has no statistics: out = tanh(alpha * x) * w + b, alpha one learned number (Zhu, Chen, He, LeCun
 // and Liu, "Transformers without Normalization").  Every element stands for itself, so a row falls into as many blocks as fill
-// the device.  Behind 16-bit outputs the tanh is 1 - 2 / (1 + e^(2z)) by the hardware's exponential and division (some 1e-7
-// absolute, below the output's own rounding); the 32-bit path takes the accurate function.
-template <typename T>
-__device__ __forceinline__ float norm_tanh(float z) {
-  if (sizeof(T) == 2) return 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(z, 15.f)));
-  return tanhf(z);
-}
-
+// the device.
 template <typename T>
 __global__ void __launch_bounds__(PN_NT)
 tanh_norm_step_kernel(float* stream, const T* y1, const T* y2, const float* __restrict__ alpha, const float* __restrict__ w,
@@ -229,7 +201,7 @@ tanh_norm_step_kernel(float* stream, const T* y1, const T* y2, const float* __re
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       x[i] += u[i] + v[i];
-      o[i] = fmaf(norm_tanh<T>(a * x[i]), g[i], c[i]);
+      o[i] = tanh_norm<T>(x[i], a, g[i], c[i]);
     }
     if (wide) {
       if (store) store4(stream + base + d, x);

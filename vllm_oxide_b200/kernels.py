@@ -634,14 +634,23 @@ def moe_gemv(a, w, c, ids, order, n: int, top: int, relu_squared: bool, silu_pai
                               ctypes.c_float(glu_limit), _stream()), "moe_gemv")
 
 
-def moe_combine(y, slot_of, weights, out, num_tokens: int, top: int, add=None, add_gate=None) -> None:
+def moe_combine(y, slot_of, weights, out, num_tokens: int, top: int, add=None, add_gate=None, stream=None, norm=None) -> None:
     """out[t] = sum_j weights[t, j] * y[slot_of[t, j]] (float, j in order); slot_of None: pair (t, j) is row t * top + j.
-    `add` (like out): added to the sum before it is rounded, times `add_gate` (float [tokens]) if given.  `weights` None: ones."""
-    _cuda(y, slot_of, weights, out, add, add_gate)
+    `add` (like out): added to the sum before it is rounded, times `add_gate` (float [tokens]) if given.  `weights` None: ones.
+    `stream` (float [tokens, width]): the sum is added to it instead; with `norm=(alpha, weight, bias)` out is
+    tanh(alpha * stream) * weight + bias, without it out is None."""
+    _cuda(y, slot_of, weights, out, add, add_gate, stream)
+    alpha, norm_w, norm_b = norm or (None, None, None)
+    assert stream is None or (stream.dtype == torch.float32 and stream.is_contiguous() and stream.shape[1] == y.shape[1])
+    assert (out is None) == (stream is not None and norm is None) and (norm is None or stream is not None)
+    for t in (alpha, norm_w, norm_b):
+        assert t is None or (t.is_cuda and t.dtype == torch.float32 and t.is_contiguous())
     assert add_gate is None or (add is not None and add_gate.dtype == torch.float32 and add_gate.is_contiguous())
-    assert add is None or (add.dtype == out.dtype and add.shape == out.shape and add.is_contiguous())
-    assert y.dtype == torch.float32 and y.is_contiguous() and out.is_contiguous()
-    _check(lib().vob_moe_combine(_p(y), _p(slot_of), _p(weights), _p(add), _p(add_gate), _p(out), num_tokens, out.shape[1], top, _code(out.dtype),
+    act = out if out is not None else add
+    assert add is None or (add.dtype == act.dtype and add.shape[1] == y.shape[1] and add.is_contiguous())
+    assert y.dtype == torch.float32 and y.is_contiguous() and (out is None or (out.is_contiguous() and out.shape[1] == y.shape[1]))
+    _check(lib().vob_moe_combine(_p(y), _p(slot_of), _p(weights), _p(add), _p(add_gate), _p(out), _p(stream), _p(alpha),
+                                 _p(norm_w), _p(norm_b), num_tokens, y.shape[1], top, _code(act.dtype if act is not None else torch.float32),
                                  _stream()), "moe_combine")
 
 
@@ -1015,7 +1024,7 @@ def gemm_f32(a, w, out, bias=None) -> None:
                               ctypes.c_long(out.stride(0)), _p(bias), M, N, K, _stream()), "gemm_f32")
 
 
-EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_ADD, EPI_GEGLU = 0, 1, 2, 3, 4
+EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_ADD, EPI_GEGLU, EPI_STREAM = 0, 1, 2, 3, 4, 5
 _tensor_maps = {}
 
 
@@ -1121,7 +1130,7 @@ def gemm_skinny_weight_tiles(n_rows: int) -> int:
     return (n_rows + box - 1) // box
 
 
-def gemm_skinny(x, w, out, epilogue: int, err, norm_weight=None, eps: float = 0.0, emit=None, prenormed=None) -> None:
+def gemm_skinny(x, w, out, epilogue: int, err, norm_weight=None, eps: float = 0.0, emit=None, prenormed=None, emit_tanh=None) -> None:
     """out = x @ w^T for at most 16 rows of x (see gemm_skinny_supported); epilogue EPI_BF16 (out bfloat16 [M,N]),
     EPI_F32 (out float32 [M,N], rounded to bfloat16 first), EPI_SWIGLU (the rows of w alternate in groups of
     eight between gate and up; out bfloat16 [M,N/2] = SiLU(gate) * up) or EPI_ADD (out bfloat16 [M,N] += the
@@ -1132,7 +1141,10 @@ def gemm_skinny(x, w, out, epilogue: int, err, norm_weight=None, eps: float = 0.
     The same norm in two halves, for a chain of products: `emit=(weight, scaled, parts)` (EPI_ADD) makes the product
     leave bfloat16(out * weight) in `scaled` [M,N] and per-tile sums of the squares of the new `out` in `parts`
     (float, gemm_skinny_weight_tiles(N) * 16 entries are enough) for the norm that follows; `prenormed=parts` (EPI_BF16
-    and EPI_SWIGLU, with `eps`) takes x to be such a `scaled` buffer and scales the product by 1/rms from the parts."""
+    and EPI_SWIGLU, with `eps`) takes x to be such a `scaled` buffer and scales the product by 1/rms from the parts.
+
+    EPI_STREAM: out is a float residual stream and the product is added to it unrounded; `emit_tanh=(alpha, weight, bias,
+    normed)` also leaves bfloat16(tanh(alpha * out) * weight + bias) in `normed` [M,N] (bias may be None)."""
     _cuda(x, w, out, norm_weight)
     if not gemm_skinny_supported(x, w):
         raise KernelError("gemm_skinny: this product is not supported (bfloat16, at most 16 rows, K a multiple of 64, 16-byte aligned rows)")
@@ -1140,7 +1152,7 @@ def gemm_skinny(x, w, out, epilogue: int, err, norm_weight=None, eps: float = 0.
     N = w.shape[0]
     assert w.shape[1] == K and out.stride(1) == 1 and out.shape[0] == M
     assert out.shape[1] == (N // 2 if epilogue in (EPI_SWIGLU, EPI_GEGLU) else N)
-    assert out.dtype == (torch.float32 if epilogue == EPI_F32 else torch.bfloat16)
+    assert out.dtype == (torch.float32 if epilogue in (EPI_F32, EPI_STREAM) else torch.bfloat16)
     if norm_weight is not None:
         assert epilogue in (EPI_BF16, EPI_SWIGLU) and norm_weight.dtype == torch.float32 and norm_weight.numel() == K
     box_m = 8 if M <= 8 else 16
@@ -1149,7 +1161,14 @@ def gemm_skinny(x, w, out, epilogue: int, err, norm_weight=None, eps: float = 0.
         assert norm_weight is None and epilogue in (EPI_BF16, EPI_SWIGLU) and prenormed.dtype == torch.float32
         ss_parts, ss_count = prenormed, gemm_skinny_weight_tiles(K)      # the product before wrote K outputs a token
         assert prenormed.numel() >= ss_count * box_m
-    emit_w = emit_xn = emit_ss = None
+    emit_w = emit_xn = emit_ss = emit_alpha = emit_b = None
+    if emit_tanh is not None:
+        emit_alpha, emit_w, emit_b, emit_xn = emit_tanh
+        _cuda(emit_alpha, emit_w, emit_b, emit_xn)
+        assert epilogue == EPI_STREAM and emit is None and emit_alpha.numel() == 1
+        for t, n in ((emit_alpha, 1), (emit_w, N), (emit_b, N)):
+            assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n)
+        assert emit_xn.dtype == torch.bfloat16 and emit_xn.is_contiguous() and emit_xn.shape == (M, N)
     if emit is not None:
         emit_w, emit_xn, emit_ss = emit
         _cuda(emit_w, emit_xn, emit_ss)
@@ -1160,7 +1179,7 @@ def gemm_skinny(x, w, out, epilogue: int, err, norm_weight=None, eps: float = 0.
     map_x = tensor_map(x, box_m, 4)
     _check(lib().vob_gemm_skinny(map_w, map_x, _p(out), ctypes.c_long(out.stride(0)), M, N, K, epilogue, _p(norm_weight),
                                  ctypes.c_float(eps), _p(ss_parts), ss_count, _p(emit_w), _p(emit_xn), _p(emit_ss),
-                                 _p(err), _stream()), "gemm_skinny")
+                                 _p(emit_alpha), _p(emit_b), _p(err), _stream()), "gemm_skinny")
 
 
 def gemm_skinny_set_wait_limit(tries: int, withhold_copies: bool = False) -> None:

@@ -99,6 +99,20 @@ class Prenormed:
     parts: torch.Tensor
 
 
+@dataclass
+class StreamEnd:
+    """An offer to a sublayer of a block around a float stream: its last kernel may add its output into `stream` itself and
+    leave `normed` = `norm` of the new stream, a norm without row statistics (both None: nothing follows).  A part with
+    `takes_stream_end` gets it as `forward(..., end=)` and returns None where it took it."""
+    stream: torch.Tensor
+    norm: Optional["Norm"]
+    normed: Optional[torch.Tensor]
+
+    def tanh_norm(self):
+        """(alpha, weight, bias) of the norm that follows, or None."""
+        return None if self.norm is None else (self.norm.alpha, self.norm.weight, self.norm.bias)
+
+
 class Workspace:
     """Activation buffers with fixed addresses: allocated once for the largest step and handed out
     by name, so that a step captured in a CUDA graph finds them where they were."""
@@ -146,6 +160,8 @@ class Part:
     # True when forward() launches the same kernels, with the same arguments, whatever the step's batch
     # holds (everything that varies is read on the device): such a part can be captured in a CUDA graph.
     graph_safe = False
+    # True where forward() takes `end` (a StreamEnd): see there
+    takes_stream_end = False
 
     def tensor_specs(self) -> List[TensorSpec]:
         return []

@@ -38,7 +38,7 @@ from .. import kernels
 from ..weights.loader import TensorSpec
 from .attention import paged_attend
 from .base import NO_ROTATION, CacheSpec, Mixer, register_part
-from .linear import linear
+from .linear import linear, linear_end
 
 
 FAST_GROUP = 16     # query heads that the tensor-core attention kernels take for one key head
@@ -61,6 +61,7 @@ def head_product(x, x_width: int, x_used: int, w, y, y_width: int, T: int) -> No
 
 class LatentAttention(Mixer):
     graph_safe = True
+    takes_stream_end = True
 
     def __init__(self, hidden_size: int, num_heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int,
                  scale: float, eps: float, window: Optional[int], position: Optional[str], prefix: str, positions: dict,
@@ -129,7 +130,7 @@ class LatentAttention(Mixer):
         return None if self.borrow else CacheSpec(1, self.row, self.cache_window, tensors=1)
 
     # ---- one step
-    def forward(self, x, ctx, cache, state=None, write_cache: bool = True):
+    def forward(self, x, ctx, cache, state=None, write_cache: bool = True, end=None):
         if write_cache == self.borrow:
             raise ValueError("a latent-attention layer writes its own plane, or borrows one: the plan's order says otherwise")
         T, nh = x.shape[0], self.nh
@@ -159,7 +160,7 @@ class LatentAttention(Mixer):
             head_product(packed, w, self.kv_rank, self.wuv[h0:h0 + n], heads[:, h0 * self.dv:(h0 + n) * self.dv], self.dv, T)
         if self.gate and not self.head_gate:
             kernels.sigmoid_gate_mul(heads, down[:, self.gate_off:], nh * self.dv)
-        return linear(heads, self.wo, ctx.ws.get("mixer_proj", T, self.H, x.dtype), ctx)
+        return linear_end(heads, self.wo, ctx.ws.get("mixer_proj", T, self.H, x.dtype), ctx, end)
 
 
 register_part("mixer", "latent_attention", LatentAttention)

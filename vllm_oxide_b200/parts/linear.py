@@ -51,6 +51,16 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, ctx=None) -
     return out
 
 
+def linear_end(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, ctx, end=None):
+    """A sublayer's last product: `linear`, or, with a `StreamEnd` and a product that the weight-streaming kernel takes (bfloat16, up to
+    16 tokens), added into the float stream with the norm that follows in the same kernel; None is then returned."""
+    if end is None or not kernels.gemm_skinny_supported(x, weight):
+        return linear(x, weight, out, ctx)
+    norm = end.tanh_norm()
+    kernels.gemm_skinny(x, weight, end.stream, kernels.EPI_STREAM, ctx.err, emit_tanh=(*norm, end.normed) if norm else None)
+    return None
+
+
 def linear_into_stream(x: torch.Tensor, weight: torch.Tensor, stream: torch.Tensor) -> None:
     """stream += x @ weight^T by the library's product with the stream as its addend (bfloat16 steps of more than 16
     tokens): the sum is made in float inside the product and rounded once, as the weight-streaming kernel's adding

@@ -40,7 +40,7 @@ import torch
 from .. import kernels
 from ..weights.loader import TensorSpec
 from .base import Mixer, StateSpec, register_part
-from .linear import linear
+from .linear import linear, linear_end
 
 
 def _up8(n: int) -> int:
@@ -173,6 +173,8 @@ class LightningAttention(_MatrixState):
 
 
 class MLSTM(_MatrixState):
+    takes_stream_end = True
+
     def __init__(self, hidden_size: int, num_heads: int, dim: int, vdim: int, gate_cap: float, eps: float, prefix: str, dtype=None,
                  device=None, **_):
         super().__init__(hidden_size, num_heads, dim, vdim, eps, prefix)
@@ -200,7 +202,7 @@ class MLSTM(_MatrixState):
         n = self.nh * (self.dk * (self.dv + 1) + 1)
         return StateSpec(((n + 3) // 4 * 4,), torch.float32)      # rows stay 16-byte aligned
 
-    def forward(self, x, ctx, cache, state, write_cache: bool = True):
+    def forward(self, x, ctx, cache, state, write_cache: bool = True, end=None):
         T, B, nh, dk, dv = x.shape[0], ctx.launch_requests, self.nh, self.dk, self.dv
         row = linear(x, self.w_in, ctx.ws.get("mlstm_in", T, self.w_in.shape[0], x.dtype), ctx)
         out = ctx.ws.get("mlstm_out", T, nh * dv, x.dtype)
@@ -216,7 +218,7 @@ class MLSTM(_MatrixState):
             kernels.mlstm_scan(*common, gates=gates, raw=raw, nq=nq, chunks=chunks, scratch=scratch)
             kernels.delta_out_norm(raw, row[:, self.gate_off:], self.norm_weight, out, T, nh, dv, self.eps, gate_sigmoid=True, nq=nq,
                                    gates=gates)
-        return linear(out, self.wo, ctx.ws.get("mixer_proj", T, self.H, x.dtype), ctx)
+        return linear_end(out, self.wo, ctx.ws.get("mixer_proj", T, self.H, x.dtype), ctx, end)
 
 
 register_part("mixer", "mlstm", MLSTM)

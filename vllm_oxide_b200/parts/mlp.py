@@ -10,7 +10,7 @@ import torch
 from .. import kernels
 from ..weights.loader import TensorSpec
 from .base import FeedForward, register_part
-from .linear import linear, linear_into_stream, tc5_product
+from .linear import linear, linear_end, linear_into_stream, tc5_product
 
 
 class SwiGLU(FeedForward):
@@ -48,8 +48,9 @@ class SwiGLU(FeedForward):
         self.wdown = tensors[self.n_down].contiguous()
 
     adds_into_stream = True
+    takes_stream_end = True
 
-    def forward(self, x, ctx, add_into=None):
+    def forward(self, x, ctx, add_into=None, end=None):
         """`add_into`: the residual stream; the down product then adds its result there and nothing is returned."""
         T = x.shape[0]
         act = ctx.ws.get("act", T, self.I, x.dtype)
@@ -64,7 +65,7 @@ class SwiGLU(FeedForward):
         if add_into is not None:
             linear_into_stream(act, self.wdown, add_into)
             return None
-        return linear(act, self.wdown, ctx.ws.get(self.out_name, T, self.H, x.dtype), ctx)
+        return linear_end(act, self.wdown, ctx.ws.get(self.out_name, T, self.H, x.dtype), ctx, end)
 
     # ---- the same with the residual stream kept inside the products (decode-sized steps)
     def can_forward_on_stream(self, stream, ctx) -> bool:

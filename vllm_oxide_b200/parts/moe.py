@@ -66,6 +66,7 @@ class ReluSquaredMLP(FeedForward):
 
 class RoutedExperts(FeedForward):
     graph_safe = True
+    takes_stream_end = True
 
     def __init__(self, hidden_size: int, expert_size: int, experts: int, top: int, prefix: str, groups: int = 1, keep: int = 1,
                  names=("up", "down", "router", "correction"), activation: str = "relu2", gate_name: str = "gate",
@@ -137,7 +138,17 @@ class RoutedExperts(FeedForward):
                           weight_scale=self.weight_scale, router_bias=self.router_b, w_shared=self.w_shared,
                           shared_gate=shared_gate)
 
-    def forward(self, x, ctx):
+    def _combine(self, y, slot_of, weights, T: int, dtype, ctx, add, add_gate, end):
+        """The tokens' sums: a row each, or (`end`) into the float stream, with the norm that follows."""
+        if end is not None:
+            kernels.moe_combine(y, slot_of, weights, end.normed, T, self.top, add=add, add_gate=add_gate, stream=end.stream,
+                                norm=end.tanh_norm())
+            return None
+        out = ctx.ws.get("mlp_out", T, self.H, dtype)
+        kernels.moe_combine(y, slot_of, weights, out, T, self.top, add=add, add_gate=add_gate)
+        return out
+
+    def forward(self, x, ctx, end=None):
         T, top = x.shape[0], self.top
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         n = T * top
@@ -159,9 +170,7 @@ class RoutedExperts(FeedForward):
                              weights=in_w)
             y = ctx.ws.get_flat("moe_y", n * self.H, torch.float32).view(n, self.H)
             kernels.moe_gemv(act, self.wdown, y, ids, order, n, top, False)
-            out = ctx.ws.get("mlp_out", T, self.H, x.dtype)
-            kernels.moe_combine(y, None, out_w, out, T, top, add=shared, add_gate=sg)
-            return out
+            return self._combine(y, None, out_w, T, x.dtype, ctx, shared, sg, end)
         tile = kernels.moe_tc5_row_tile() if fast else kernels.moe_row_tile()
         # every expert's rows are padded to a row tile: at most tile - 1 rows for each expert that has any
         max_rows = (n + min(self.E, n) * (tile - 1) + tile - 1) // tile * tile
@@ -183,9 +192,7 @@ class RoutedExperts(FeedForward):
             kernels.moe_gemm(x, self.wup, act, row_token, tile_expert, relu_squared=not self.gated, gather=True,
                              silu_pairs=self.gated, glu_limit=self.limit, row_weight=row_weight)
             kernels.moe_gemm(act, self.wdown, y, row_token, tile_expert, relu_squared=False, gather=False)
-        out = ctx.ws.get("mlp_out", T, self.H, x.dtype)
-        kernels.moe_combine(y, slot_of, out_w, out, T, top, add=shared, add_gate=sg)
-        return out
+        return self._combine(y, slot_of, out_w, T, x.dtype, ctx, shared, sg, end)
 
 
 register_part("feed_forward", "relu2_mlp", ReluSquaredMLP)

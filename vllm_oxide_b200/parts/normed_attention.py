@@ -28,7 +28,7 @@ from ..weights.loader import TensorSpec
 from .attention import paged_attend
 from .base import NO_ROTATION, CacheSpec, Mixer, register_part
 from .capped_attention import _pad_heads
-from .linear import linear
+from .linear import linear, linear_end
 from .linear_attention import merged_rows
 
 
@@ -38,6 +38,7 @@ PAD_HEADS = True
 
 class NormedAttention(Mixer):
     graph_safe = True
+    takes_stream_end = True
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float, eps: float, prefix: str,
                  positions: dict, dtype, device, window: Optional[int] = None, position: Optional[str] = None, bias: bool = True,
@@ -100,7 +101,7 @@ class NormedAttention(Mixer):
     def cache_spec(self) -> CacheSpec:
         return CacheSpec(self.kvh, self.kp, self.window, value_dim=self.vp)
 
-    def forward(self, x, ctx, cache, state=None, write_cache: bool = True, defer_bias: bool = False):
+    def forward(self, x, ctx, cache, state=None, write_cache: bool = True, defer_bias: bool = False, end=None):
         T = x.shape[0]
         row = linear(x, self.w_in, ctx.ws.get("normed_attn_in", T, self.width, x.dtype), ctx)
         kernels.headnorm_rope_kv_write(row, self.b_in, ctx.positions, ctx.slot_mapping[cache.group], self.wq_norm, self.wk_norm,
@@ -111,7 +112,7 @@ class NormedAttention(Mixer):
                      self.scale, self._pairs, sink=self.sinks if self.sink else False, softcap=self.softcap)
         if self.gate:
             kernels.sigmoid_gate_mul(heads, row[:, self.gate_off:], self.nh * self.vp)
-        out = linear(heads, self.wo, ctx.ws.get("normed_attn_proj", T, self.H, x.dtype), ctx)
+        out = linear_end(heads, self.wo, ctx.ws.get("normed_attn_proj", T, self.H, x.dtype), ctx, end if self.out_bias is None else None)
         if self.out_bias is not None and not defer_bias:
             kernels.add_bias(out, self.out_bias)
         return out

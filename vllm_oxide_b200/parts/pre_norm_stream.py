@@ -10,6 +10,11 @@ sublayer's output, not yet in the stream; the stream).
 The block takes any norm that is fused with a float stream's update (`layernorm_stream`, `rmsnorm_parallel_stream` of
 parts/parallel.py, or the one below).
 
+A norm without row statistics can be made where the stream is written: in front of a `StreamTanhNorm` the block offers its
+sublayer a `StreamEnd`, and a part whose last kernel can (the weight-streaming product of steps of up to 16 tokens, the sum of the
+experts' rows at any size) adds into the stream and leaves the normed row behind itself.  (hidden None between blocks: nothing is
+pending; `ctx.prenormed`: the next block's normed rows.)
+
 `StreamTanhNorm`: tanh(alpha * x) * w + b with ONE learned number alpha (<weight>.alpha) and a bias (<weight>.b): no mean, no
 variance, every element for itself (Zhu, Chen, He, LeCun and Liu, "Transformers without Normalization").
 """
@@ -21,7 +26,7 @@ import torch
 
 from .. import kernels
 from ..weights.loader import TensorSpec
-from .base import Block, Norm, PartSpec, build_part, register_part
+from .base import Block, Norm, PartSpec, StreamEnd, build_part, register_part
 from .parallel import StreamLayerNorm, StreamRMSNorm
 
 
@@ -64,6 +69,10 @@ class StreamTanhNorm(Norm):
         return self.enter(x, residual, ctx, name, rows=rows, n_rows=n_rows)
 
 
+# Whether sublayers may end in the stream themselves (else the stream's step is always a kernel of its own).
+END_IN_STREAM = True
+
+
 class PreNormStreamBlock(Block):
     def __init__(self, mixer: PartSpec, feed_forward: Optional[PartSpec], input_norm: PartSpec, post_mixer_norm: Optional[PartSpec],
                  size: int, **common):
@@ -89,12 +98,34 @@ class PreNormStreamBlock(Block):
         for p in self._parts:
             p.load({s.name: tensors[s.name] for s in p.tensor_specs()})
 
+    def _offer(self, part, norm, normed, stream, ctx) -> dict:
+        """The `end` argument of a sublayer that reads `normed` and is followed by `norm` (None: by nothing)."""
+        if not END_IN_STREAM or not part.takes_stream_end or not (norm is None or isinstance(norm, StreamTanhNorm)):
+            return {}
+        out = None
+        if norm is not None:        # the other of the two buffers: the sublayer's own input is not written over
+            out = next(b for b in (ctx.ws.get(n, normed.shape[0], self.size, normed.dtype) for n in ("normed", "normed_ff"))
+                       if b.data_ptr() != normed.data_ptr())
+        return dict(end=StreamEnd(stream, norm, out))
+
     def forward(self, hidden, residual, ctx, cache, state, write_cache=True):
-        normed, stream = self.input_norm.enter(hidden, residual, ctx, "normed")
-        y = self.mixer.forward(normed, ctx, cache, state, write_cache)
+        ahead, ctx.prenormed = getattr(ctx, "prenormed", None), None
+        if hidden is None and isinstance(ahead, StreamEnd) and ahead.norm is self.input_norm:
+            normed, stream = ahead.normed, residual
+        else:
+            normed, stream = self.input_norm.enter(hidden, residual, ctx, "normed")
+        following = getattr(ctx, "next_norm", None)
+        offer = self._offer(self.mixer, following if self.feed_forward is None else self.post_mixer_norm, normed, stream, ctx)
+        y = self.mixer.forward(normed, ctx, cache, state, write_cache, **offer)
         if self.feed_forward is not None:
-            normed, stream = self.post_mixer_norm.enter(y, stream, ctx, "normed_ff")
-            y = self.feed_forward.forward(normed, ctx)
+            if y is None:
+                normed = offer["end"].normed
+            else:
+                normed, stream = self.post_mixer_norm.enter(y, stream, ctx, "normed_ff")
+            offer = self._offer(self.feed_forward, following, normed, stream, ctx)
+            y = self.feed_forward.forward(normed, ctx, **offer)
+        if y is None:
+            ctx.prenormed = offer["end"]
         return y, stream
 
 
@@ -102,6 +133,8 @@ def stream_value(hidden, stream, ctx) -> torch.Tensor:
     """The residual stream [tokens, width] (float, a new tensor) after the pending write of `hidden`: what the next norm would
     see.  For inspection; no step of the engine needs it."""
     x = stream.clone()
+    if hidden is None and getattr(ctx, "pending_second", None) is None:
+        return x
     kernels.tanh_norm_step(x, ctx.err, y1=hidden, y2=getattr(ctx, "pending_second", None))
     return x
 
