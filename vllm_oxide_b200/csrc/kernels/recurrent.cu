@@ -594,6 +594,9 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
   const int per = (q1 - q0 + chunks - 1) / chunks;
   const int t0 = min(q1, q0 + chunk * per), t1 = min(q1, t0 + per);
   const int tiles = (t1 - t0 + HG_TT - 1) / HG_TT;
+  // where the walk's matrices start and end: the slot, or the range's place
+  float* whole = mode == 0 ? state + (size_t)slot * state_stride
+                           : ends + ((size_t)b * chunks + chunk) * ((size_t)heads * dk * (dv + (SOURCE::NORMALISER ? 1 : 0)));
   if ((int)threadIdx.x >= walkers) {
     // ------------------------------------------------ loaders
     const int tid = threadIdx.x - walkers;
@@ -607,6 +610,16 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
         q[HG_TT * W] = 0.f;
         if (ROWS) q[2 * HG_TT * W] = 0.f;
       }
+    // the head's normaliser: the first loader warp walks it, a tile when its gates are there; a lane holds eight rows as a walker
+    // does (groups of PARTS lanes hold copies)
+    const bool norm_warp = SOURCE::NORMALISER && c0 == 0 && tid < 32;
+    float* norm = whole + (size_t)heads * dk * dv + (size_t)h * dk + tid % PARTS * MS_R;
+    f32x2 n2[MS_R / 2];
+    if constexpr (SOURCE::NORMALISER) {
+      const int live = OUT && norm_warp ? dk - tid % PARTS * MS_R : 0;
+#pragma unroll
+      for (int p = 0; p < MS_R / 2; ++p) n2[p] = pack2(2 * p < live ? norm[2 * p] : 0.f, 2 * p + 1 < live ? norm[2 * p + 1] : 0.f);
+    }
     for (int k = 0; k < tiles; ++k) {
       float* qs = sm + (k & 1) * buffer;       // [HG_TT][W] q
       float* ws = qs + HG_TT * W;              // [HG_TT][W] w
@@ -649,15 +662,56 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
             if (tb + e * v_step < n) vs[(tb + e * v_step) * cols + c] = v[e];
         }
       __threadfence_block();
+      // (the loaders meet, so that the first of their warps may read the tile; they cannot come back to this buffer before it has
+      // met them at the next tile)
+      if constexpr (SOURCE::NORMALISER) named_sync(5, MS_LOADERS);
       named_arrive(1 + (k & 1), threads);
+      if constexpr (SOURCE::NORMALISER) {
+        if (norm_warp) {
+#pragma unroll 4
+          for (int tt = 0; tt < n; ++tt) {
+            const float f = vs[HG_TT * cols + tt];
+            const f32x2 keep = pack2(f, f);
+            f32x2 s2 = 0ull;
+#pragma unroll
+            for (int p = 0; p < 2; ++p) {
+              const int at = tt * W + (p * PARTS + tid % PARTS) * 4;
+              const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(ws + at);
+              n2[2 * p] = fma2(keep, n2[2 * p], w.x);
+              n2[2 * p + 1] = fma2(keep, n2[2 * p + 1], w.y);
+              if (OUT) {
+                const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(qs + at);
+                s2 = fma2(n2[2 * p], q.x, s2);
+                s2 = fma2(n2[2 * p + 1], q.y, s2);
+              }
+            }
+            if (OUT) {
+              const float2 s = unpack2(s2);
+              float sum = s.x + s.y;
+#pragma unroll
+              for (int d = 1; d < PARTS; d <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+              if (tid == 0) src.nq[(size_t)(ts + tt) * heads + h] = sum;
+            }
+          }
+        }
+      }
+    }
+    if constexpr (SOURCE::NORMALISER) {
+      if (norm_warp && tid < PARTS && mode != 2) {
+        const int live = dk - tid * MS_R;
+#pragma unroll
+        for (int p = 0; p < MS_R / 2; ++p) {
+          const float2 x = unpack2(n2[p]);
+          if (2 * p < live) norm[2 * p] = x.x;
+          if (2 * p + 1 < live) norm[2 * p + 1] = x.y;
+        }
+      }
     }
     return;
   }
   // -------------------------------------------------- walkers
   const int part = threadIdx.x % PARTS, group = threadIdx.x / PARTS;
   const int j0 = c0 + group * MS_C, i0 = part * MS_R;
-  float* whole = mode == 0 ? state + (size_t)slot * state_stride
-                           : ends + ((size_t)b * chunks + chunk) * ((size_t)heads * dk * (dv + (SOURCE::NORMALISER ? 1 : 0)));
   float* mine = whole + (size_t)h * dk * dv;
   // (a head's matrix starts on a 16-byte boundary where the state's rows do)
   const bool wide = dv % 4 == 0 && (((uintptr_t)mine) & 15) == 0;
@@ -687,16 +741,6 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
     }
 #pragma unroll
     for (int c = 0; c < MS_C; ++c) M[c][r / 2] = pack2(a[0][c], a[1][c]);
-  }
-  // the head's normaliser waits in shared memory: the first walker warp walks it tile by tile, behind the tile's matrices
-  __shared__ __align__(16) float norms[SOURCE::NORMALISER ? W : 4];
-  const bool norm_warp = SOURCE::NORMALISER && c0 == 0 && threadIdx.x < 32;
-  float* norm = whole + (size_t)heads * dk * dv + (size_t)h * dk;
-  if constexpr (SOURCE::NORMALISER) {
-    if (norm_warp) {
-      for (int i = threadIdx.x; i < W; i += 32) norms[tile_index<PARTS>(i)] = OUT && i < dk ? norm[i] : 0.f;
-      __syncwarp();
-    }
   }
   f32x2 f2[ROWS ? MS_R / 2 : 1];
   if (SOURCE::DECAY == DECAY_FIXED) {
@@ -782,58 +826,9 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
         }
       }
     }
-    if constexpr (SOURCE::NORMALISER) {
-      if (norm_warp) {      // the same for every lane of the warp; its groups hold copies
-        f32x2 n2[MS_R / 2];
-#pragma unroll
-        for (int p = 0; p < 2; ++p) {
-          const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(norms + (p * PARTS + part) * 4);
-          n2[2 * p] = x.x; n2[2 * p + 1] = x.y;
-        }
-#pragma unroll 1
-        for (int tt = 0; tt < n; ++tt) {
-          const float f = vs[HG_TT * cols + tt];
-          const f32x2 keep = pack2(f, f);
-          f32x2 s2 = 0ull;
-#pragma unroll
-          for (int p = 0; p < 2; ++p) {
-            const int at = tt * W + (p * PARTS + part) * 4;
-            const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(ws + at);
-            n2[2 * p] = fma2(keep, n2[2 * p], w.x);
-            n2[2 * p + 1] = fma2(keep, n2[2 * p + 1], w.y);
-            if (OUT) {
-              const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(qs + at);
-              s2 = fma2(n2[2 * p], q.x, s2);
-              s2 = fma2(n2[2 * p + 1], q.y, s2);
-            }
-          }
-          if (OUT) {
-            const float2 s = unpack2(s2);
-            float sum = s.x + s.y;
-#pragma unroll
-            for (int d = 1; d < PARTS; d <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
-            if (threadIdx.x == 0) src.nq[(size_t)(ts + tt) * heads + h] = sum;
-          }
-        }
-        __syncwarp();
-        if (group == 0) {
-#pragma unroll
-          for (int p = 0; p < 2; ++p) {
-            ulonglong2 x;
-            x.x = n2[2 * p]; x.y = n2[2 * p + 1];
-            *reinterpret_cast<ulonglong2*>(norms + (p * PARTS + part) * 4) = x;
-          }
-        }
-        __syncwarp();
-      }
-    }
     if (k + 2 < tiles) named_arrive(3 + (k & 1), threads);
   }
   if (mode == 2) return;
-  if constexpr (SOURCE::NORMALISER) {
-    if (norm_warp)
-      for (int i = threadIdx.x; i < dk; i += 32) norm[i] = norms[tile_index<PARTS>(i)];
-  }
 #pragma unroll
   for (int r = 0; r < MS_R; r += 2) {
     float a[2][MS_C];
