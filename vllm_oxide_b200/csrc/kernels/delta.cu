@@ -402,7 +402,7 @@ __device__ __forceinline__ float head_unit(const float* nq, const float4* gates,
 template <typename T>
 __global__ void __launch_bounds__(128)
 delta_out_norm_kernel(const float* raw, const T* gate, long gate_stride, const float* __restrict__ w, int w_head, const float* nq,
-                      const float4* gates, T* out, int heads, int vdim, float eps, int total, int gate_sigmoid) {
+                      const float4* gates, T* out, int heads, int vdim, float eps, int total, int gate_sigmoid, int wide) {
   pdl_launch_dependents();
   pdl_wait();
   const int idx = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -410,6 +410,47 @@ delta_out_norm_kernel(const float* raw, const T* gate, long gate_stride, const f
   const int t = idx / heads, h = idx % heads;
   const float* o = raw + ((size_t)t * heads + h) * vdim;
   const float unit = head_unit(nq, gates, (size_t)idx);
+  if (wide) {
+    // heads of up to 512 elements that start on 16-byte boundaries: a lane holds its elements, four an access
+    const float* gain = w + (size_t)h * w_head;
+    const T* grow = gate + (size_t)t * gate_stride + (size_t)h * vdim;
+    T* orow = out + ((size_t)t * heads + h) * vdim;
+    float x[4][4], g[4][4], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int d = (k * 32 + lane) * 4;
+      if (d < vdim) {
+        load4(o + d, x[k]);
+        load4(grow + d, g[k]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if ((k * 32 + lane) * 4 < vdim) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          x[k][i] *= unit;
+          ss = fmaf(x[k][i], x[k][i], ss);
+        }
+      }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int d = (k * 32 + lane) * 4;
+      if (d < vdim) {
+        float wv[4], y[4];
+        load4(gain + d, wv);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          // behind a 16-bit output the hardware's exponential and division (far below its rounding)
+          const float e = sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-g[k][i])) : 1.f / (1.f + expf(-g[k][i]));
+          y[i] = x[k][i] * inv * wv[i] * (gate_sigmoid ? e : g[k][i] * e);
+        }
+        store4(orow + d, y);
+      }
+    }
+    return;
+  }
   float ss = 0.f;
   for (int d = lane; d < vdim; d += 32) { const float x = o[d] * unit; ss = fmaf(x, x, ss); }
   ss = warp_sum(ss);
@@ -569,12 +610,13 @@ VOB_API int vob_delta_out_norm(const float* raw, const void* gate, long gate_str
                            gate_stride, w, w_head, nq, gates, (__nv_bfloat16*)out, heads, vdim, eps, gate_sigmoid);
     return VOB_BAD_ARGUMENT;
   }
+  const int wide = vdim % 4 == 0 && gate_stride % 4 == 0 && (((uintptr_t)raw | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
   dim3 grid((total + 3) / 4);
   if (dtype == VOB_F32)
     return launch_kernel(delta_out_norm_kernel<float>, grid, 128, 0, stream, raw, (const float*)gate, gate_stride, w,
-                         w_head, nq, gates, (float*)out, heads, vdim, eps, total, gate_sigmoid);
+                         w_head, nq, gates, (float*)out, heads, vdim, eps, total, gate_sigmoid, wide);
   if (dtype == VOB_BF16)
     return launch_kernel(delta_out_norm_kernel<__nv_bfloat16>, grid, 128, 0, stream, raw, (const __nv_bfloat16*)gate,
-                         gate_stride, w, w_head, nq, gates, (__nv_bfloat16*)out, heads, vdim, eps, total, gate_sigmoid);
+                         gate_stride, w, w_head, nq, gates, (__nv_bfloat16*)out, heads, vdim, eps, total, gate_sigmoid, wide);
   return VOB_BAD_ARGUMENT;
 }

@@ -180,7 +180,10 @@ lru_scan_kernel(const T* u, const float* gates, const T* y, long y_stride, const
 //   MlstmSource      q * scale, w = put * k, f = keep: two numbers a head and token (exponential gates, mlstm_gates below)
 // A source with a NORMALISER carries one more column beside the head's dv, whose value is 1 at every token: n = diag(f) n + w.
 // Its read-out n . q divides the head's outputs.  The column lies behind all heads' matrices, [heads, dk].
-// Decoding (matrix_scan_fused): one block a (request, head) that also takes the head's norm and what the source puts behind it.
+// Decoding, one token a request (matrix_scan_step): one block a (request, head) streams the state through registers once, 16 bytes
+// an access; its first loads are in flight before the kernels ahead have finished, for only an earlier step can have written the
+// state.  Short portions (matrix_scan_fused): one block a (request, head) holds the state in registers over the tokens.  Both take
+// the head's norm and what the source puts behind it, and the first may leave the bare o instead.  In the second
 // Column j of a head's state M (dk floats) is shared by PARTS neighbouring lanes, R rows each, in registers.  The gates of
 // HG_TT tokens are made by the whole block at once and parked in shared memory (rows padded so that the PARTS lanes of a column
 // read different banks).
@@ -554,6 +557,135 @@ matrix_scan_fused_kernel(const SOURCE src, const float* __restrict__ nw, float* 
     if (threadIdx.x < 32)
       for (int i = threadIdx.x; i < dk; i += 32) norm[i] = norms[i];
     if (threadIdx.x == 0) *kept = run;
+  }
+}
+
+
+// ---- decoding: the state passes through registers once a token
+// A thread has VEC neighbouring columns and every `groups`-th row, U rows in flight; the groups' shares of o meet in shared memory.
+template <typename T, typename SOURCE, int VEC, int NT>
+__global__ void __launch_bounds__(NT, 1024 / NT)
+matrix_scan_step_kernel(const SOURCE src, const float* __restrict__ nw, float* state, long state_stride, const int* __restrict__ cu_q,
+                        const int* __restrict__ state_slots, T* out, float* raw, int heads, int dk, int dv, float eps, int num_slots,
+                        int* err) {
+  constexpr int U = 8;
+  extern __shared__ float4 sm4[];
+  __shared__ float red[NT / 32];
+  float* qs = reinterpret_cast<float*>(sm4);      // [dk] each
+  float* fs = qs + dk;
+  float* ws = fs + dk;
+  float* os = ws + dk;                            // [groups][dv]
+  pdl_launch_dependents();
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
+  const int t0 = cu_q[b], t1 = cu_q[b + 1], slot = state_slots[b];
+  const bool ok = t1 > t0 && slot >= 0 && slot < num_slots;
+  const int C = dv / VEC, groups = NT / C;
+  const int c = tid % C * VEC, g = tid / C;
+  const bool have = g < groups;
+  float* whole = ok ? state + (size_t)slot * state_stride : nullptr;
+  float* mine = ok ? whole + (size_t)h * dk * dv + c : nullptr;
+  float m[U][VEC];
+  auto load_rows = [&](int r0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int r = r0 + u * groups + g;
+      if (have && r < dk) {
+        if constexpr (VEC == 4) load4(mine + (size_t)r * dv, m[u]);
+        else m[u][0] = mine[(size_t)r * dv];
+      }
+    }
+  };
+  float n_row = 0.f, run = 0.f;                   // the normaliser's row tid, the running maximum
+  float* norm = nullptr;
+  float* kept = nullptr;
+  const typename SOURCE::Fixed fx = src.fixed(h, min(tid, dk - 1));
+  if (ok) {
+    load_rows(0);
+    if constexpr (SOURCE::NORMALISER) {
+      norm = whole + (size_t)heads * dk * dv + (size_t)h * dk + tid;
+      kept = whole + (size_t)heads * dk * (dv + 1) + h;
+      if (tid < dk) n_row = *norm;
+      run = *kept;
+    }
+  }
+  pdl_wait();
+  if (!ok) {
+    if (t1 > t0 && tid == 0) atomicOr(err, VOB_ERR_SLOT);
+    return;
+  }
+  for (int t = t0; t < t1; ++t) {
+    float floor = 0.f, share = 0.f;
+    float v[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = src.value((size_t)t, h, c + e);
+    ScanGates gate = {0.f, 0.f, 0.f};
+    if (tid < dk) gate = src.make(src.load((size_t)t, h, tid), fx);
+    if constexpr (SOURCE::HEAD_GATES) {
+      const LogGates lg = src.pre((size_t)t, h);
+      const float next = fmaxf(lg.f + run, lg.i);
+      gate.f = expf(lg.f + run - next);
+      gate.w *= expf(lg.i - next);
+      floor = expf(-next);
+      run = next;
+    }
+    if (tid < dk) {
+      qs[tid] = gate.q;
+      fs[tid] = gate.f;
+      ws[tid] = gate.w;
+      if constexpr (SOURCE::NORMALISER) {
+        n_row = fmaf(gate.f, n_row, gate.w);
+        share = n_row * gate.q;
+      }
+    }
+    __syncthreads();
+    float o[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) o[e] = 0.f;
+    for (int r0 = 0; r0 < dk; r0 += U * groups) {
+      if (r0 > 0 || t > t0) load_rows(r0);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int r = r0 + u * groups + g;
+        if (have && r < dk) {
+          const float f = fs[r], w = ws[r], q = qs[r];
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            m[u][e] = fmaf(f, m[u][e], w * v[e]);
+            o[e] = fmaf(m[u][e], q, o[e]);
+          }
+          if constexpr (VEC == 4) store4(mine + (size_t)r * dv, m[u]);
+          else mine[(size_t)r * dv] = m[u][0];
+        }
+      }
+    }
+    if (have) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) os[g * dv + c + e] = o[e];
+    }
+    float unit = 1.f;
+    if constexpr (SOURCE::NORMALISER) unit = 1.f / (fmaxf(fabsf(block_sum<NT>(share, red)), floor) + MLSTM_EPS);
+    else __syncthreads();
+    float ss = 0.f;
+    for (int j = tid; j < dv; j += NT) {
+      float s = os[j];
+      for (int k = 1; k < groups; ++k) s += os[k * dv + j];
+      s *= unit;
+      os[j] = s;
+      ss = fmaf(s, s, ss);
+    }
+    const size_t row = (size_t)t * heads * dv + (size_t)h * dv;
+    if (raw) {
+      for (int j = tid; j < dv; j += NT) raw[row + j] = os[j];
+    } else {
+      const float denom = sqrtf(block_sum<NT>(ss, red) / (float)dv + eps);
+      const float* gain = SOURCE::HEAD_GATES ? nw + (size_t)h * dv : nw;
+      for (int j = tid; j < dv; j += NT) out[row + j] = from_f<T>(src.finish(os[j] / denom * gain[j], (size_t)t, h, j));
+    }
+    if (t + 1 < t1) __syncthreads();
+  }
+  if constexpr (SOURCE::NORMALISER) {
+    if (tid < dk) *norm = n_row;
+    if (tid == 0) *kept = run;
   }
 }
 
@@ -951,6 +1083,26 @@ int launch_scan_fused(const SOURCE& src, const float* nw, float* state, long sta
                        heads, dk, dv, eps, num_slots, err);
 }
 
+// One token a request: threads by the size of a head, and columns a thread.  dk up to 256 (a gate a thread).
+template <typename T, typename SOURCE>
+int launch_scan_step(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
+                     void* out, float* raw, int B, int heads, int dk, int dv, float eps, int num_slots, int* err, cudaStream_t stream) {
+  const bool vec = dv % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
+  const int threads = dk * dv >= 16384 || dv > (vec ? 1024 : 256) ? 512 : 256;
+  if (dv > threads * (vec ? 4 : 1) || dk > 256) return VOB_UNSUPPORTED;
+  const int groups = threads / (vec ? dv / 4 : dv);
+  const size_t smem = ((size_t)3 * dk + (size_t)groups * dv) * sizeof(float);
+#define VOB_ST(VV, NN)                                                                                                             \
+  return launch_kernel(matrix_scan_step_kernel<T, SOURCE, VV, NN>, dim3(heads, B), dim3(NN), smem, stream, src, nw, state, state_stride, \
+                       cu_q, state_slots, (T*)out, raw, heads, dk, dv, eps, num_slots, err)
+  if (vec && threads == 512) VOB_ST(4, 512);
+  if (vec) VOB_ST(4, 256);
+  if (threads == 512) VOB_ST(1, 512);
+  VOB_ST(1, 256);
+#undef VOB_ST
+}
+inline bool scan_can_step(int dk, int dv) { return dk <= 256 && dv <= 512; }
+
 inline int tile_parts(int dk) {
   int p = 2;
   while (p * MS_R < dk) p <<= 1;
@@ -1002,14 +1154,17 @@ int dispatch_scan_tile(int mode, const SOURCE& src, float* state, long state_str
 template <typename T, typename SOURCE>
 int run_matrix_scan(const SOURCE& src, const float* nw, float* state, long state_stride, const int* cu_q, const int* state_slots,
                     void* out, float* raw, float* scratch, int Tn, int B, int chunks, int heads, int dk, int dv, float eps,
-                    int num_slots, int fuse, int norm, int* err, cudaStream_t stream) {
+                    int num_slots, int fuse, int single, int norm, int* err, cudaStream_t stream) {
   const long per = (long)heads * dk * (dv + (SOURCE::NORMALISER ? 1 : 0));
-  if (heads <= 0 || dk <= 0 || dv <= 0 || dk > 256 || B > 65535 || (!fuse && !raw) || (fuse && !scan_can_fuse(dk, dv)) ||
-      chunks < 1 || chunks > HG_MAX_CHUNKS || (chunks > 1 && (fuse || !scratch)) || state_stride < per + (SOURCE::NORMALISER ? heads : 0))
+  if (heads <= 0 || dk <= 0 || dv <= 0 || dk > 256 || B > 65535 || (!fuse && !raw) ||
+      (fuse && !(single ? scan_can_step(dk, dv) : scan_can_fuse(dk, dv))) || chunks < 1 || chunks > HG_MAX_CHUNKS || (chunks > 1 && (fuse || !scratch)) || state_stride < per + (SOURCE::NORMALISER ? heads : 0))
     return VOB_UNSUPPORTED;
   int code = 0;
   // (a source that makes its head gates itself walks fused only, one whose gates are ready never)
   if constexpr (SOURCE::HEAD_GATES || !SOURCE::NORMALISER) {
+    if (single && (fuse || !norm))
+      return launch_scan_step<T>(src, nw, state, state_stride, cu_q, state_slots, fuse ? out : nullptr, fuse ? nullptr : raw, B, heads, dk, dv,
+                                 eps, num_slots, err, stream);
     if (fuse) {
 #define VOB_SF(RR, PP) return launch_scan_fused<T, SOURCE, RR, PP>(src, nw, state, state_stride, cu_q, state_slots, out, B, heads, dk, dv, eps, num_slots, err, stream)
       if (dk <= 16) VOB_SF(16, 1);
@@ -1081,6 +1236,9 @@ VOB_API int vob_mingru_scan(const void* zxg, const void* bz, const void* bx, flo
 // B * chunks * heads * dk * (dv + 1) floats.
 VOB_API int vob_hgrn2_can_fuse(int dk, int dv) { return scan_can_fuse(dk, dv) ? 1 : 0; }
 
+// The same for steps of one token a request (`single` below: no request brings more).
+VOB_API int vob_matrix_scan_can_step(int dk, int dv) { return scan_can_step(dk, dv) ? 1 : 0; }
+
 // Ranges that a request's tokens of a step should be cut into (unfused walks): the fewest units of time by a count of float
 // instructions a state element (three a token in one walk, five over the two walks of a cut portion, and what the join and the
 // launches cost in tokens), given how many blocks fit the device at once.
@@ -1099,12 +1257,12 @@ VOB_API int vob_matrix_scan_chunks(int T, int B, int heads, int dk, int dv) {
 
 VOB_API int vob_hgrn2_scan(const void* qfv, const void* bf, const float* lower, const float* nw, float* state, const int* cu_q,
                            const int* state_slots, void* out, float* raw, float* scratch, int T, int B, int chunks, int heads,
-                           int dk, int dv, float eps, int num_slots, int fuse, int dtype, int* err, cudaStream_t stream) {
+                           int dk, int dv, float eps, int num_slots, int fuse, int single, int dtype, int* err, cudaStream_t stream) {
   if (B <= 0 || T <= 0) return 0;
   const long width = (long)heads * (2 * dk + dv), per = (long)heads * dk * dv;
 #define VOB_HS(TT)                                                                                                            \
   return run_matrix_scan<TT>(HgrnSource<TT>{(const TT*)qfv, width, (const TT*)bf, lower, heads, dk, dv}, nw, state, per, cu_q, \
-                             state_slots, out, raw, scratch, T, B, chunks, heads, dk, dv, eps, num_slots, fuse, 1, err, stream)
+                             state_slots, out, raw, scratch, T, B, chunks, heads, dk, dv, eps, num_slots, fuse, single, 1, err, stream)
   if (dtype == VOB_F32) { VOB_HS(float); }
   if (dtype == VOB_BF16) { VOB_HS(__nv_bfloat16); }
 #undef VOB_HS
@@ -1117,12 +1275,12 @@ VOB_API int vob_hgrn2_scan(const void* qfv, const void* bf, const float* lower, 
 VOB_API int vob_gla_scan(const void* rows, long width, int z_off, int gate_off, const float* bias, const float* nw, float* state,
                          long state_stride, const int* cu_q, const int* state_slots, void* out, float* raw, float* scratch, int T,
                          int B, int chunks, int heads, int dk, int dv, float scale, float inv_tau, float eps, int num_slots,
-                         int fuse, int dtype, int* err, cudaStream_t stream) {
+                         int fuse, int single, int dtype, int* err, cudaStream_t stream) {
   if (B <= 0 || T <= 0) return 0;
 #define VOB_GS(TT)                                                                                                             \
   return run_matrix_scan<TT>(GlaSource<TT>{(const TT*)rows, width, bias, heads, dk, dv, z_off, gate_off, scale, inv_tau}, nw,  \
                              state, state_stride, cu_q, state_slots, out, raw, scratch, T, B, chunks, heads, dk, dv, eps,      \
-                             num_slots, fuse, 0, err, stream)
+                             num_slots, fuse, single, 0, err, stream)
   if (dtype == VOB_F32) { VOB_GS(float); }
   if (dtype == VOB_BF16) { VOB_GS(__nv_bfloat16); }
 #undef VOB_GS
@@ -1132,12 +1290,12 @@ VOB_API int vob_gla_scan(const void* rows, long width, int z_off, int gate_off, 
 // rows: `width` elements a token, q | k | v first; decays float [heads]; raw float [T, heads*dv].
 VOB_API int vob_lightning_scan(const void* rows, long width, const float* decays, float* state, long state_stride, const int* cu_q,
                                const int* state_slots, float* raw, float* scratch, int T, int B, int chunks, int heads, int dk,
-                               int dv, int num_slots, int dtype, int* err, cudaStream_t stream) {
+                               int dv, int num_slots, int single, int dtype, int* err, cudaStream_t stream) {
   if (B <= 0 || T <= 0) return 0;
 #define VOB_LS(TT)                                                                                                          \
   return run_matrix_scan<TT>(LightningSource<TT>{(const TT*)rows, width, decays, heads, dk, dv}, (const float*)nullptr,     \
                              state, state_stride, cu_q, state_slots, nullptr, raw, scratch, T, B, chunks, heads, dk, dv, 0.f, \
-                             num_slots, 0, 0, err, stream)
+                             num_slots, 0, single, 0, err, stream)
   if (dtype == VOB_F32) { VOB_LS(float); }
   if (dtype == VOB_BF16) { VOB_LS(__nv_bfloat16); }
 #undef VOB_LS
@@ -1180,7 +1338,8 @@ VOB_API int vob_lru_scan(const void* u, const float* gates, const void* y, long 
 VOB_API int vob_mlstm_scan(const void* rows, long width, int i_off, int f_off, int gate_off, const float* bi, const float* bf,
                            const float* nw, float* gates, float* state, long state_stride, const int* cu_q, const int* state_slots,
                            void* out, float* raw, float* nq, float* scratch, int T, int B, int chunks, int heads, int dk, int dv,
-                           float scale, float cap, float eps, int num_slots, int fuse, int dtype, int* err, cudaStream_t stream) {
+                           float scale, float cap, float eps, int num_slots, int fuse, int single, int dtype, int* err,
+                           cudaStream_t stream) {
   if (B <= 0 || T <= 0) return 0;
   if (!(cap > 0.f) || (!fuse && (!nq || !gates || ((uintptr_t)gates & 15)))) return VOB_BAD_ARGUMENT;
   if (heads <= 0 || B > 65535) return VOB_UNSUPPORTED;
@@ -1193,7 +1352,7 @@ VOB_API int vob_mlstm_scan(const void* rows, long width, int i_off, int f_off, i
     if (code != 0) return code;                                                                                                 \
   }                                                                                                                             \
   return run_matrix_scan<TT>(src, nw, state, state_stride, cu_q, state_slots, out, raw, scratch, T, B, chunks, heads, dk, dv,   \
-                             eps, num_slots, fuse, 0, err, stream)
+                             eps, num_slots, fuse, single, 0, err, stream)
   if (dtype == VOB_F32) {
     if (fuse) { VOB_ML(float, false); }
     VOB_ML(float, true);

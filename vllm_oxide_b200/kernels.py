@@ -754,12 +754,14 @@ def _scan_scratch_ok(chunks: int, raw, scratch, num_requests: int, heads: int, d
 
 
 def gla_scan(rows, z_off: int, gate_off: int, bias, norm_weight, state, cu_q, state_slots, num_requests: int, heads: int, dk: int,
-             dv: int, scale: float, tau: float, eps: float, err, out=None, raw=None, chunks: int = 1, scratch=None) -> None:
+             dv: int, scale: float, tau: float, eps: float, err, out=None, raw=None, chunks: int = 1, scratch=None,
+             single: bool = False) -> None:
     """Gated linear attention, M = diag(f) M + k v^T, o = M^T (scale q), f = sigmoid(z + bias)^(1 / tau), over every request's
     tokens of this step, from and to its slot (state float [slots, n], the heads' [dk, dv] matrices first).  rows: q | k | v
     (heads * dk, heads * dk, heads * dv) first, z (heads * dk) at z_off, the output gate (heads * dv) at gate_off.  With `out`
     one block a (request, head) does it all, the head's RMS norm (norm_weight float [dv]) and the product with SiLU(gate)
-    included (hgrn2_can_fuse); with `raw` (float [tokens, heads * dv]) the bare o.  `chunks`, `scratch`: as hgrn2_scan."""
+    included (matrix_scan_fuses); with `raw` (float [tokens, heads * dv]) the bare o.  `chunks`, `scratch`, `single`: as
+    hgrn2_scan."""
     _cuda(rows, bias, norm_weight, state, cu_q, state_slots, out, raw)
     T = (raw if out is None else out).shape[0]
     assert rows.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * dk * dv
@@ -770,35 +772,35 @@ def gla_scan(rows, z_off: int, gate_off: int, bias, norm_weight, state, cu_q, st
     _check(lib().vob_gla_scan(_p(rows), ctypes.c_long(rows.stride(0)), z_off, gate_off, _p(bias), _p(norm_weight), _p(state),
                               ctypes.c_long(state.stride(0)), _p(cu_q), _p(state_slots), _p(out), _p(raw), _p(scratch), T,
                               num_requests, int(chunks), heads, dk, dv, ctypes.c_float(scale), ctypes.c_float(1.0 / tau),
-                              ctypes.c_float(eps), state.shape[0], int(out is not None), _code(rows.dtype), _p(err), _stream()),
-           "gla_scan")
+                              ctypes.c_float(eps), state.shape[0], int(out is not None), int(bool(single)), _code(rows.dtype), _p(err),
+                              _stream()), "gla_scan")
 
 
 def lightning_scan(rows, decays, state, cu_q, state_slots, raw, num_requests: int, heads: int, dk: int, dv: int, err,
-                   chunks: int = 1, scratch=None) -> None:
-    """M = decay_h M + silu(k) silu(v)^T, o = M^T silu(q) into `raw` (float [tokens, heads * dv]); rows, state, chunks and scratch
-    as gla_scan, decays float [heads]."""
+                   chunks: int = 1, scratch=None, single: bool = False) -> None:
+    """M = decay_h M + silu(k) silu(v)^T, o = M^T silu(q) into `raw` (float [tokens, heads * dv]); rows, state, chunks, scratch and
+    single as gla_scan, decays float [heads]."""
     _cuda(rows, decays, state, cu_q, state_slots, raw)
     assert rows.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * dk * dv
     assert decays.dtype == torch.float32 and decays.numel() == heads and raw.dtype == torch.float32 and raw.is_contiguous()
     assert _scan_scratch_ok(chunks, raw, scratch, num_requests, heads, dk, dv)
     _check(lib().vob_lightning_scan(_p(rows), ctypes.c_long(rows.stride(0)), _p(decays), _p(state), ctypes.c_long(state.stride(0)),
                                     _p(cu_q), _p(state_slots), _p(raw), _p(scratch), raw.shape[0], num_requests, int(chunks), heads,
-                                    dk, dv, state.shape[0], _code(rows.dtype), _p(err), _stream()), "lightning_scan")
+                                    dk, dv, state.shape[0], int(bool(single)), _code(rows.dtype), _p(err), _stream()), "lightning_scan")
 
 
 def mlstm_scan(rows, i_off: int, f_off: int, gate_off: int, bias_i, bias_f, norm_weight, state, cu_q, state_slots, num_requests: int,
                heads: int, dk: int, dv: int, scale: float, cap: float, eps: float, err, out=None, gates=None, raw=None, nq=None,
-               chunks: int = 1, scratch=None) -> None:
+               chunks: int = 1, scratch=None, single: bool = False) -> None:
     """A matrix memory with exponential gates over every request's tokens of this step, from and to its slot: log gates
     i = cap tanh((zi + bias_i) / cap), f = log sigmoid(cap tanh((zf + bias_f) / cap)), m = max(f + m', i) (m' the token before's),
     M = exp(f + m' - m) M + exp(i - m) k v^T, n likewise with k alone, o = M^T (scale q) / (max(|n . scale q|, exp(-m)) + 1e-6).
     rows: q | k | v (heads * dk, heads * dk, heads * dv) first, zi, zf (heads each) at i_off, f_off, the output gate (heads * dv) at
     gate_off.  state float [slots, >= heads * (dk * (dv + 1) + 1)]: matrices, n, m.  With `out` one block a (request, head) does it
     all, the head's RMS norm, the gain (norm_weight float [heads * dv]) and the product with sigmoid(gate) included
-    (hgrn2_can_fuse).  Else `gates` [tokens, heads, 4], `raw` [tokens, heads * dv] and `nq` [tokens, heads] (float) receive the
-    factors, M^T (scale q) and n . scale q, and delta_out_norm makes the rest of them.  `chunks`, `scratch`: as hgrn2_scan, with
-    dv + 2 in the place of dv + 1."""
+    (matrix_scan_fuses).  Else `gates` [tokens, heads, 4], `raw` [tokens, heads * dv] and `nq` [tokens, heads] (float) receive the
+    factors, M^T (scale q) and n . scale q, and delta_out_norm makes the rest of them.  `chunks`, `scratch`, `single`: as hgrn2_scan,
+    with dv + 2 in the place of dv + 1."""
     _cuda(rows, bias_i, bias_f, norm_weight, state, cu_q, state_slots, out, gates, raw, nq)
     T = (raw if out is None else out).shape[0]
     assert rows.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * (dk * (dv + 1) + 1)
@@ -811,8 +813,8 @@ def mlstm_scan(rows, i_off: int, f_off: int, gate_off: int, bias_i, bias_f, norm
     _check(lib().vob_mlstm_scan(_p(rows), ctypes.c_long(rows.stride(0)), i_off, f_off, gate_off, _p(bias_i), _p(bias_f), _p(norm_weight),
                                 _p(gates), _p(state), ctypes.c_long(state.stride(0)), _p(cu_q), _p(state_slots), _p(out), _p(raw),
                                 _p(nq), _p(scratch), T, num_requests, int(chunks), heads, dk, dv, ctypes.c_float(scale),
-                                ctypes.c_float(cap), ctypes.c_float(eps), state.shape[0], int(out is not None), _code(rows.dtype),
-                                _p(err), _stream()), "mlstm_scan")
+                                ctypes.c_float(cap), ctypes.c_float(eps), state.shape[0], int(out is not None), int(bool(single)),
+                                _code(rows.dtype), _p(err), _stream()), "mlstm_scan")
 
 
 def lru_scan(u, gates, y, bias_r, bias_i, lam, bias_y, state, cu_q, state_slots, out, num_requests: int, blocks: int, err,
@@ -859,13 +861,14 @@ def mingru_scan(zxg, bias_z, bias_x, state, cu_q, state_slots, out, num_requests
 
 
 def hgrn2_scan(qfv, bias_f, lower, norm_weight, state, cu_q, state_slots, out, num_requests: int, heads: int, dk: int,
-               dv: int, eps: float, err, raw=None, chunks: int = 1, scratch=None) -> None:
+               dv: int, eps: float, err, raw=None, chunks: int = 1, scratch=None, single: bool = False) -> None:
     """The matrix-state recurrence M = diag(f) M + (1 - f) v^T, o = M^T q, with the per-head norm of o, over every
     request's tokens of this step; state float [slots, heads, dk, dv]; qfv [tokens, heads * (2 dk + dv)].  Without `raw`
-    one block a (request, head) does it all (decoding; the head must fit: hgrn2_can_fuse); with `raw` (float [tokens,
+    one block a (request, head) does it all (decoding; the head must fit: matrix_scan_fuses); with `raw` (float [tokens,
     heads * dv]) a head's columns are spread over blocks and the norm is a second kernel (portions).  Same numbers.
     `chunks` > 1 (with `raw`): a request's tokens are cut into that many ranges that are walked side by side, twice,
-    with a join in between; `scratch`: float, num_requests * chunks * heads * dk * (dv + 1) elements."""
+    with a join in between; `scratch`: float, num_requests * chunks * heads * dk * (dv + 1) elements.  `single`: no request brings
+    more than one token (the state then passes through registers once)."""
     _cuda(qfv, bias_f, lower, norm_weight, state, cu_q, state_slots, out, raw)
     T = out.shape[0]
     assert qfv.is_contiguous() and out.is_contiguous() and qfv.shape[1] == heads * (2 * dk + dv) and out.shape[1] == heads * dv
@@ -875,11 +878,19 @@ def hgrn2_scan(qfv, bias_f, lower, norm_weight, state, cu_q, state_slots, out, n
                            and scratch.numel() >= num_requests * chunks * heads * dk * (dv + 1))
     _check(lib().vob_hgrn2_scan(_p(qfv), _p(bias_f), _p(lower), _p(norm_weight), _p(state), _p(cu_q), _p(state_slots),
                                 _p(out), _p(raw), _p(scratch), T, num_requests, int(chunks), heads, dk, dv, ctypes.c_float(eps),
-                                state.shape[0], int(raw is None), _code(out.dtype), _p(err), _stream()), "hgrn2_scan")
+                                state.shape[0], int(raw is None), int(bool(single)), _code(out.dtype), _p(err), _stream()), "hgrn2_scan")
 
 
 def hgrn2_can_fuse(dk: int, dv: int) -> bool:
     return bool(lib().vob_hgrn2_can_fuse(dk, dv))
+
+
+def matrix_scan_fuses(dk: int, dv: int, num_tokens: int, num_requests: int, single: bool) -> bool:
+    """Whether a matrix-state scan of this step takes a block a (request, head) that does it all: steps of one token a request
+    (`single`: no request brings more) and short portions, for the head sizes that the kernels hold."""
+    if single:
+        return bool(lib().vob_matrix_scan_can_step(dk, dv))
+    return num_tokens <= 16 * num_requests and hgrn2_can_fuse(dk, dv)
 
 
 def latent_prep(down, wq, wkv, rule, positions, slots, cq, cache, num_tokens: int, q_rank: int, kv_rank: int, rot: int,

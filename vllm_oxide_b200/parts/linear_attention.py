@@ -132,8 +132,9 @@ class GatedLinearAttention(_MatrixState):
         out = ctx.ws.get("gla_out", T, self.nh * self.dv, x.dtype)
         common = (row, self.z_off, self.gate_off, self.bias, self.norm_weight, state, ctx.cu_q, ctx.state_slots, B, self.nh, self.dk,
                   self.dv, self.dk ** -0.5, self.tau, self.eps, ctx.err)
-        if kernels.hgrn2_can_fuse(self.dk, self.dv) and T <= 16 * B:
-            kernels.gla_scan(*common, out=out)
+        single = ctx.max_q <= 1
+        if kernels.matrix_scan_fuses(self.dk, self.dv, T, B, single):
+            kernels.gla_scan(*common, out=out, single=single)
         else:
             raw = ctx.ws.get("matrix_scan_raw", T, self.nh * self.dv, torch.float32)
             chunks, scratch = self._chunks(T, ctx)
@@ -165,7 +166,7 @@ class LightningAttention(_MatrixState):
         raw = ctx.ws.get("matrix_scan_raw", T, self.nh * self.dv, torch.float32)
         chunks, scratch = self._chunks(T, ctx)
         kernels.lightning_scan(row, self.decays, state, ctx.cu_q, ctx.state_slots, raw, B, self.nh, self.dk, self.dv, ctx.err,
-                               chunks=chunks, scratch=scratch)
+                               chunks=chunks, scratch=scratch, single=ctx.max_q <= 1 and kernels.matrix_scan_fuses(self.dk, self.dv, T, B, True))
         out = ctx.ws.get("lightning_out", T, self.nh * self.dv, x.dtype)
         # one norm over all heads: a row is one "head" of heads * vdim elements
         kernels.delta_out_norm(raw, row[:, self.gate_off:], self.norm_weight, out, T, 1, self.nh * self.dv, self.eps, gate_sigmoid=True)
@@ -208,8 +209,9 @@ class MLSTM(_MatrixState):
         out = ctx.ws.get("mlstm_out", T, nh * dv, x.dtype)
         common = (row, self.i_off, self.f_off, self.gate_off, self.bias_i, self.bias_f, self.norm_weight, state, ctx.cu_q,
                   ctx.state_slots, B, nh, dk, dv, dk ** -0.5, self.cap, self.eps, ctx.err)
-        if kernels.hgrn2_can_fuse(dk, dv) and T <= 16 * B:
-            kernels.mlstm_scan(*common, out=out)
+        single = ctx.max_q <= 1
+        if kernels.matrix_scan_fuses(dk, dv, T, B, single):
+            kernels.mlstm_scan(*common, out=out, single=single)
         else:
             gates = ctx.ws.get("mlstm_gates", T, nh * 4, torch.float32)
             raw = ctx.ws.get("matrix_scan_raw", T, nh * dv, torch.float32)

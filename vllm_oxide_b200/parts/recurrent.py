@@ -102,7 +102,8 @@ class HGRN2(Mixer):
         qfv = linear(x, self.wqfv, ctx.ws.get("hgrn2_qfv", T, width, x.dtype), ctx)
         out = ctx.ws.get("hgrn2_out", T, self.nh * self.dv, x.dtype)
         # decoding: one block a (request, head), norm included; portions: a head's columns over several blocks
-        fuse = kernels.hgrn2_can_fuse(self.dk, self.dv) and T <= 16 * ctx.launch_requests
+        single = ctx.max_q <= 1
+        fuse = kernels.matrix_scan_fuses(self.dk, self.dv, T, ctx.launch_requests, single)
         raw = None if fuse else ctx.ws.get("hgrn2_raw", T, self.nh * self.dv, torch.float32)
         # longer portions are also cut along the tokens
         B = ctx.launch_requests
@@ -110,7 +111,7 @@ class HGRN2(Mixer):
         scratch = None if chunks == 1 else ctx.ws.get_flat("hgrn2_ranges", B * chunks * self.nh * self.dk * (self.dv + 1),
                                                            torch.float32)
         kernels.hgrn2_scan(qfv, self.bf, self.lower, self.norm_weight, state, ctx.cu_q, ctx.state_slots, out,
-                           B, self.nh, self.dk, self.dv, self.eps, ctx.err, raw=raw, chunks=chunks, scratch=scratch)
+                           B, self.nh, self.dk, self.dv, self.eps, ctx.err, raw=raw, chunks=chunks, scratch=scratch, single=single and fuse)
         return linear(out, self.wo, ctx.ws.get("mixer_proj", T, self.H, x.dtype), ctx)
 
 
