@@ -600,12 +600,17 @@ def nesezen_config(width: int, layers: int) -> dict:
 def nesezen_kernel_bytes(cfg: dict, T: int) -> dict:
     """Bytes that each of the design's own row-wise kernels must move in a step of T tokens, summed over the layers (weights
     aside): what its time is held against.  Attention, the scans and the experts' products are held against arithmetic."""
-    D = cfg["width"]
-    b = {"tanh_norm_step": T * D * (2 + 4 + 2) - T * D * (2 + 2 * 4 + 2)}         # the stream begins: it is not read, and one output is less
+    D, products_end_in_stream = cfg["width"], T <= 16
+    b = {"tanh_norm_step": T * D * (2 + 4 + 2)}                                   # the stream begins
     add = lambda k, v: b.__setitem__(k, b.get(k, 0) + v)
-    for l in cfg["layers"]:
+    for i, l in enumerate(cfg["layers"]):
         m, mlp = l["mixer"], l["mlp"]
-        add("tanh_norm_step", (2 if mlp else 1) * T * D * (2 + 2 * 4 + 2))
+        # a sublayer's output in, the stream read and written, the normed row out: a kernel of its own behind the library's
+        # products (behind the last layer's it only reads the rows whose logits are wanted)
+        if not products_end_in_stream:
+            add("tanh_norm_step", T * D * (2 + 2 * 4 + 2))
+            if mlp and mlp["kind"] == "dense" and i + 1 < len(cfg["layers"]):
+                add("tanh_norm_step", T * D * (2 + 2 * 4 + 2))
         if l["type"] == "mlstm":
             add("delta_out_norm", T * m["heads"] * m["vdim"] * (4 + 2 + 2))
         elif l["type"] == "attention":
@@ -619,7 +624,8 @@ def nesezen_kernel_bytes(cfg: dict, T: int) -> dict:
             top = mlp["router"]["top"]
             add("silu_mul", T * 3 * mlp["shared"]["ff"] * 2)
             add("moe_gather_rows", T * top * D * 2 * 2)
-            add("moe_combine", T * (top * D * 4 + 2 * D * 2))
+            # the experts' rows and the shared one's, the stream read and written, the normed row
+            add("moe_combine", T * (top * D * 4 + D * 2 + 2 * D * 4 + D * 2))
     return b
 
 

@@ -195,8 +195,8 @@ lru_scan_kernel(const T* u, const float* gates, const T* y, long y_stride, const
 // "full" when a buffer is ready, "empty" when its tokens have been walked).  o leaves in float and a norm kernel follows.
 //
 // A long portion is also cut along the tokens (`chunks` > 1, four launches): MODE 1 walks every range from a zero state
-// and leaves its end state L; matrix_scan_range_decay takes the product F of every range's decays; matrix_scan_join goes
-// through the ranges in order,
+// and leaves its end state L; matrix_scan_range_decay takes the product F of every range's decays (a source with a normaliser has
+// it made in MODE 1, by the warp that walks the normaliser); matrix_scan_join goes through the ranges in order,
 // M_start(c+1) = diag(F_c) M_start(c) + L_c, leaves every range's start where its L was and the last state in the
 // slot; MODE 2 walks the ranges again from their starts and writes the outputs.  Nearly twice the arithmetic, on as many more
 // blocks as there are ranges.  MODE 0 is the walk from the slot's state to the slot's state in one launch.
@@ -339,7 +339,6 @@ struct MlstmSource {
   __device__ __forceinline__ ScanGates make(const Raw& r, const Fixed&) const { return {r.q * scale, r.g.x, r.k * r.g.y}; }
   __device__ __forceinline__ float token_decay(size_t t, int h) const { return gates[t * heads + h].x; }
   __device__ __forceinline__ float value(size_t t, int h, int c) const { return to_f<T>(rows[t * width + (size_t)2 * heads * dk + h * dv + c]); }
-  __device__ __forceinline__ float decay(size_t t, int h, int, const Fixed&) const { return token_decay(t, h); }
   __device__ __forceinline__ LogGates pre(size_t t, int h) const {
     const T* row = rows + t * width;
     return log_gates(to_f<T>(row[i_off + h]) + bi[h], to_f<T>(row[f_off + h]) + bf[h], cap);
@@ -353,7 +352,8 @@ struct MlstmSource {
 // The gates of a step's portions, one block a (request, head).  m over a range of tokens is max(a + m, b) with a the sum of its f:
 // every thread folds its own range, the block scans the folds, and every thread walks its range again from its start.  A
 // range's last maximum is the next range's start by construction, so what a token keeps and writes refers to one and the same m.
-constexpr int MG_NT = 256;
+constexpr int MG_NT = 1024;
+constexpr int MG_HELD = 4;      // tokens of a thread whose log gates stay in registers between the two walks
 
 template <typename T>
 __global__ void __launch_bounds__(MG_NT)
@@ -374,8 +374,18 @@ mlstm_gates_kernel(const MlstmSource<T, true> src, float4* gates, float* state, 
   const int per = (t1 - t0 + MG_NT - 1) / MG_NT;
   const int lo = min(t1, t0 + (int)threadIdx.x * per), hi = min(t1, lo + per);
   float a = 0.f, m = -INFINITY;
-#pragma unroll 4
-  for (int t = lo; t < hi; ++t) {
+  LogGates held[MG_HELD];
+#pragma unroll
+  for (int k = 0; k < MG_HELD; ++k)
+    if (lo + k < hi) held[k] = src.pre((size_t)(lo + k), h);
+#pragma unroll
+  for (int k = 0; k < MG_HELD; ++k)
+    if (lo + k < hi) {
+      a += held[k].f;
+      m = fmaxf(held[k].f + m, held[k].i);
+    }
+#pragma unroll 2
+  for (int t = lo + MG_HELD; t < hi; ++t) {
     const LogGates g = src.pre((size_t)t, h);
     a += g.f;
     m = fmaxf(g.f + m, g.i);
@@ -398,13 +408,16 @@ mlstm_gates_kernel(const MlstmSource<T, true> src, float4* gates, float* state, 
   __syncthreads();
   m = starts[threadIdx.x];
   const float last = starts[threadIdx.x + 1];
-#pragma unroll 2
-  for (int t = lo; t < hi; ++t) {
-    const LogGates g = src.pre((size_t)t, h);
+  auto put = [&](int t, const LogGates& g) {
     const float next = t + 1 < hi ? fmaxf(g.f + m, g.i) : last;
     gates[(size_t)t * src.heads + h] = make_float4(expf(g.f + m - next), expf(g.i - next), expf(-next), 0.f);
     m = next;
-  }
+  };
+#pragma unroll
+  for (int k = 0; k < MG_HELD; ++k)
+    if (lo + k < hi) put(lo + k, held[k]);
+#pragma unroll 2
+  for (int t = lo + MG_HELD; t < hi; ++t) put(t, src.pre((size_t)t, h));
   if (hi == t1 && lo < hi) *kept = m;
 }
 
@@ -747,6 +760,7 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
     const bool norm_warp = SOURCE::NORMALISER && c0 == 0 && tid < 32;
     float* norm = whole + (size_t)heads * dk * dv + (size_t)h * dk + tid % PARTS * MS_R;
     f32x2 n2[MS_R / 2];
+    float kept = 1.f;            // the product of the range's decays (one number a head)
     if constexpr (SOURCE::NORMALISER) {
       const int live = OUT && norm_warp ? dk - tid % PARTS * MS_R : 0;
 #pragma unroll
@@ -805,6 +819,7 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
             const float f = vs[HG_TT * cols + tt];
             const f32x2 keep = pack2(f, f);
             f32x2 s2 = 0ull;
+            kept *= f;
 #pragma unroll
             for (int p = 0; p < 2; ++p) {
               const int at = tt * W + (p * PARTS + tid % PARTS) * 4;
@@ -836,6 +851,11 @@ matrix_scan_tile_kernel(const SOURCE src, float* state, long state_stride, const
           const float2 x = unpack2(n2[p]);
           if (2 * p < live) norm[2 * p] = x.x;
           if (2 * p + 1 < live) norm[2 * p + 1] = x.y;
+        }
+        // (where matrix_scan_range_decay would leave it)
+        if (mode == 1) {
+          float* F = ends + (size_t)gridDim.y * chunks * heads * dk * (dv + 1) + (((size_t)b * chunks + chunk) * heads + h) * dk;
+          for (int i = tid; i < dk; i += PARTS) F[i] = kept;
         }
       }
     }
@@ -1185,9 +1205,11 @@ int run_matrix_scan(const SOURCE& src, const float* nw, float* state, long state
     code = dispatch_scan_tile(1, src, state, state_stride, cu_q, state_slots, raw, ends, B, chunks, heads, dk, dv, num_slots, err,
                                          stream);
     if (code != 0) return code;
-    code = launch_kernel(matrix_scan_range_decay_kernel<SOURCE>, dim3((heads * dk + 31) / 32, B, chunks), dim3(256), 0, stream, src, gates,
-                         cu_q, heads, dk);
-    if (code != 0) return code;
+    if constexpr (!SOURCE::NORMALISER) {      // (a source with a normaliser leaves the decays beside it)
+      code = launch_kernel(matrix_scan_range_decay_kernel<SOURCE>, dim3((heads * dk + 31) / 32, B, chunks), dim3(256), 0, stream, src,
+                           gates, cu_q, heads, dk);
+      if (code != 0) return code;
+    }
     code = launch_kernel(matrix_scan_join_kernel, dim3((unsigned)((per + 255) / 256), B), dim3(256), 0, stream, state, state_stride, ends,
                          (const float*)gates, cu_q, state_slots, chunks, heads, dk, dv, per, num_slots);
     if (code != 0) return code;
