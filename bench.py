@@ -585,7 +585,7 @@ def nesezen_config(width: int, layers: int) -> dict:
     but for the first layer of each block, whose feed-forward is dense and three times the width."""
     heads = width // 128
     window = dict(heads=heads, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask={"size": 1024},
-                  rot={"dims": 128, "base": 10000.0, "scaling": {"factor": 8.0, "original": 2048, "low": 1.0, "high": 4.0}})
+                  rot={"dims": 128, "base": 500000.0, "scaling": {"factor": 4.0, "original": 4096, "low": 1.0, "high": 4.0}})
     memory = dict(heads=heads, dim=128, vdim=128, gate_cap=15.0)
     latent = dict(heads=heads, dim=128, vdim=128, q_rank=3 * width // 8, kv_rank=256, scale=128 ** -0.5)
     moe = {"kind": "moe", "expert": {"ff": 3 * width // 4}, "router": {"experts": 16, "top": 4}, "shared": {"ff": 3 * width // 4}}

@@ -391,7 +391,7 @@ def run_ff(part, x, dt):
     (48, 16, 6, 6, 8, 9),            # every expert chosen
     (40, 8, 5, 1, 24, 5),            # one expert: its weight is not one
     (128, 64, 8, 4, 64, 300),        # enough pairs for the tcgen05 products in bfloat16
-    (192, 64, 12, 1, 128, 700),      # the same with one choice a token
+    (160, 48, 9, 1, 96, 700),        # the same with one choice a token
     (72, 33, 4, 2, 17, 3),           # odd widths: the float-accumulating tile kernel
     (70, 12, 3, 2, 10, 400),         # the same with many tokens
     (64, 24, 1, 1, 40, 7),           # a single expert
