@@ -181,11 +181,11 @@ lru_scan_kernel(const T* u, const float* gates, const T* y, long y_stride, const
 // A source with a NORMALISER carries one more column beside the head's dv, whose value is 1 at every token: n = diag(f) n + w.
 // Its read-out n . q divides the head's outputs.  The column lies behind all heads' matrices, [heads, dk].
 // Decoding, one token a request (matrix_scan_step): one block a (request, head) streams the state through registers once, 16 bytes
-// an access; its first loads are in flight before the kernels ahead have finished, for only an earlier step can have written the
-// state.  Short portions (matrix_scan_fused): one block a (request, head) holds the state in registers over the tokens.  Both take
-// the head's norm and what the source puts behind it, and the first may leave the bare o instead.  In the second
-// Column j of a head's state M (dk floats) is shared by PARTS neighbouring lanes, R rows each, in registers.  The gates of
-// HG_TT tokens are made by the whole block at once and parked in shared memory (rows padded so that the PARTS lanes of a column
+// an access; its first loads are in flight before the kernels ahead have finished (only an earlier step can have written the
+// state, and a step begins with a copy of its index arrays, which lets nothing of the step before run on).  Short portions
+// (matrix_scan_fused): one block a (request, head) holds the state in registers over the tokens: column j of a head's state M (dk
+// floats) is shared by PARTS neighbouring lanes, R rows each.  Both take the head's norm and what the source puts behind it; the
+// first may leave the bare o instead.  The fused walk's gates of HG_TT tokens are made by the whole block at once and parked in shared memory (rows padded so that the PARTS lanes of a column
 // read different banks).
 //
 // Portions (matrix_scan_tile): a walker thread holds a tile of 8 rows x 8 columns of M in registers, as pairs of rows, so that
